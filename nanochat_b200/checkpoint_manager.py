@@ -153,6 +153,16 @@ def find_last_step(checkpoint_dir):
     return max(steps)
 
 
+def load_model_folder(path, device, dtype=None, **serving):
+    """(model, tokenizer, meta) of a folder with config.json and model.safetensors; the tokenizer is None (such a folder
+    has none: prompts are token ids). The architecture comes from config.json, see models/registry.py."""
+    from nanochat_b200.models.registry import load_model_folder as load
+    log0(f"Loading model folder {path}")
+    with open(os.path.join(path, "config.json"), "r", encoding="utf-8") as f:
+        meta = {"step": 0, "model_config": json.load(f)}
+    return load(path, device, dtype, **serving), None, meta
+
+
 _SOURCE_DIRS = {"base": "base_checkpoints", "sft": "chatsft_checkpoints", "rl": "chatrl_checkpoints"}
 
 

@@ -141,15 +141,15 @@ PAGE_TOKENS = 64
 
 
 class _PromptView:
-    """The shared prompt pages of a PagedKVCache seen as a batch-1 contiguous cache: what the prefill writes into.
-    Has the KVCache surface the model's forward uses."""
+    """The shared prompt pages of a paged cache seen as a batch-1 cache: what the prefill writes into. `layer_cache(i)`
+    serves KVCache's surface; a latent cache's kernels use `pools` and `table` instead."""
 
     def __init__(self, owner, capacity):
         self.owner = owner
         self.batch_size = 1
         self.max_seq_len = capacity
         self.n_layers = owner.n_layers
-        self.cache_seqlens = torch.zeros(1, dtype=torch.int32, device=owner.k_pool.device)
+        self.cache_seqlens = torch.zeros(1, dtype=torch.int32, device=owner.device)
         self.prev_embedding = None
         self._pos = 0
 
@@ -161,48 +161,63 @@ class _PromptView:
         shape = (1, self.max_seq_len, o.n_heads, o.head_dim)
         return o.k_pool[layer_idx, :n].view(shape), o.v_pool[layer_idx, :n].view(shape)
 
+    @property
+    def pools(self):
+        return self.owner.pools
+
+    @property
+    def table(self):
+        return self.owner.identity_table[:, :self.max_seq_len // self.owner.page_tokens].contiguous()
+
     def advance(self, num_tokens):
         self.cache_seqlens += num_tokens
         self._pos += num_tokens
 
 
-class PagedKVCache:
-    """K/V store of `batch_size` sample rows as pages of PAGE_TOKENS tokens plus a per-row page table
-    (reference behaviour: nanochat/engine.py:82-137, a contiguous cache per row and a copy at the fork).
+class PagedCache:
+    """Pages of PAGE_TOKENS tokens plus a per-row page table for `batch_size` sample rows; what a page holds is up to the
+    subclass (`_allocate`, `_copy_tokens`).
 
     Pool pages [0, shared_pages) hold the prompt, written once by the batch-1 prefill through `begin_prompt()`;
     `fork()` points every row's table at the prompt's full pages and gives each row private pages for the prompt's
     partial last page (copied: rows append into it) and for what it decodes. The decode kernels address tokens
-    through the table (`ops/csrc/decode.cu`: KvPages). The pool grows when a request needs more pages than any before
-    it; `pool_version` then moves so that a captured decode graph is rebuilt on the new addresses.
+    through the table. The pool grows when a request needs more pages than any before it; `pool_version` then moves so
+    that a captured decode graph is rebuilt on the new addresses.
     """
 
     paged = True
 
-    def __init__(self, batch_size, num_heads, seq_len, head_dim, num_layers, device, dtype, page_tokens=PAGE_TOKENS):
+    def __init__(self, batch_size, num_layers, seq_len, device, dtype, page_tokens):
         assert page_tokens & (page_tokens - 1) == 0, "page size must be a power of two"
         self.batch_size = batch_size
         self.max_seq_len = seq_len                  # per-row capacity in tokens (what the page table can address)
-        self.n_layers, self.n_heads, self.head_dim = num_layers, num_heads, head_dim
+        self.n_layers = num_layers
         self.page_tokens = page_tokens
         self.max_pages = -(-seq_len // page_tokens)
         self.device, self.dtype = device, dtype
         self.table = torch.zeros(batch_size, self.max_pages, dtype=torch.int32, device=device)
         self.cache_seqlens = torch.zeros(batch_size, dtype=torch.int32, device=device)
-        self.k_pool = self.v_pool = None
         self.shared_pages = self.private_pages = 0
         self.pool_version = 0
         self.prev_embedding = None
         self._pos = 0
+        self._row_end = 0
 
     # ----------------------------------------------------------------------------- pool
     def reserve(self, prompt_tokens, new_tokens):
         """Make room for a prompt of `prompt_tokens` and `new_tokens` decoded tokens per row."""
         P = self.page_tokens
         assert prompt_tokens + new_tokens <= self.max_seq_len
-        shared = -(-prompt_tokens // P)
-        private = -(-(prompt_tokens % P + new_tokens) // P)
-        if self.k_pool is not None and shared <= self.shared_pages and private <= self.private_pages:
+        self._reserve_pages(-(-prompt_tokens // P), -(-(prompt_tokens % P + new_tokens) // P))
+
+    def reserve_any_prompt(self, tokens):
+        """Make room for `tokens` tokens per row, however many of them the prompt turns out to be."""
+        P = self.page_tokens
+        assert tokens <= self.max_seq_len
+        self._reserve_pages(-(-tokens // P), -(-tokens // P))
+
+    def _reserve_pages(self, shared, private):
+        if self.pool_version and shared <= self.shared_pages and private <= self.private_pages:
             return
         self.shared_pages = max(shared, self.shared_pages)
         self.private_pages = max(private, self.private_pages)
@@ -210,14 +225,9 @@ class PagedKVCache:
         # pages lands there instead of in a page that holds someone's keys
         total = self.shared_pages + self.batch_size * self.private_pages + 1
         self.spare_page = total - 1
-        shape = (self.n_layers, total, P, self.n_heads, self.head_dim)
-        self.k_pool = self.v_pool = None            # release before allocating the larger pool
-        self.k_pool = torch.zeros(shape, device=self.device, dtype=self.dtype)
-        self.v_pool = torch.zeros(shape, device=self.device, dtype=self.dtype)
+        self._allocate(total)
+        self.identity_table = torch.arange(total, dtype=torch.int32, device=self.device)[None]
         self.pool_version += 1
-
-    def pool_bytes(self):
-        return 0 if self.k_pool is None else 2 * self.k_pool.numel() * self.k_pool.element_size()
 
     def reset(self):
         self.cache_seqlens.zero_()
@@ -227,37 +237,42 @@ class PagedKVCache:
     def get_pos(self):
         return self._pos
 
-    def get_layer_cache(self, layer_idx):
-        """One layer's pools, (pages, PAGE_TOKENS, H, D): the paged decode kernels take them with `table`."""
-        return self.k_pool[layer_idx], self.v_pool[layer_idx]
-
     def advance(self, num_tokens):
         self.cache_seqlens += num_tokens
         self._pos += num_tokens
 
     # --------------------------------------------------------------------- prompt, fork
     def begin_prompt(self, prompt_tokens):
-        """A batch-1 contiguous view of the shared pages for the prefill of a `prompt_tokens`-token prompt."""
-        assert self.k_pool is not None and -(-prompt_tokens // self.page_tokens) <= self.shared_pages
+        """A batch-1 view of the shared pages for the prefill of a `prompt_tokens`-token prompt."""
+        assert self.pool_version and -(-prompt_tokens // self.page_tokens) <= self.shared_pages
         self.reset()
         return _PromptView(self, -(-prompt_tokens // self.page_tokens) * self.page_tokens)
+
+    def begin_rows(self):
+        """Every row starts empty on its private pages."""
+        self.reset()
+        self._point_rows(0)
+
+    def _point_rows(self, full):
+        """Tables: the first `full` prompt pages, then each row's private pages, then the spare page."""
+        first_private = self.shared_pages + torch.arange(self.batch_size, dtype=torch.int32, device=self.device) * self.private_pages
+        table = torch.full((self.batch_size, self.max_pages), self.spare_page, dtype=torch.int32, device=self.device)
+        if full:
+            table[:, :full] = torch.arange(full, dtype=torch.int32, device=self.device)
+        own = min(self.private_pages, self.max_pages - full)
+        table[:, full:full + own] = first_private[:, None] + torch.arange(own, dtype=torch.int32, device=self.device)
+        self.table.copy_(table)
+        self._row_end = min(self.max_seq_len, (full + own) * self.page_tokens)
+        return first_private
 
     def fork(self, view):
         """Every row continues the prompt in `view`: full prompt pages are shared, the partial last one is copied."""
         P, B = self.page_tokens, self.batch_size
         n = view.get_pos()
         full, rem = n // P, n % P
-        first_private = self.shared_pages + torch.arange(B, dtype=torch.int32, device=self.device) * self.private_pages
-        table = torch.full((B, self.max_pages), self.spare_page, dtype=torch.int32, device=self.device)
-        if full:
-            table[:, :full] = torch.arange(full, dtype=torch.int32, device=self.device)
-        own = min(self.private_pages, self.max_pages - full)
-        table[:, full:full + own] = first_private[:, None] + torch.arange(own, dtype=torch.int32, device=self.device)
-        self.table.copy_(table)
+        first_private = self._point_rows(full)
         if rem:
-            idx = first_private.long()
-            self.k_pool[:, idx, :rem] = self.k_pool[:, full:full + 1, :rem]
-            self.v_pool[:, idx, :rem] = self.v_pool[:, full:full + 1, :rem]
+            self._copy_tokens(first_private.long(), full, rem)
         self.cache_seqlens.fill_(n)
         self._pos = n
         self.prev_embedding = None
@@ -266,15 +281,69 @@ class PagedKVCache:
 
     def row_capacity(self):
         """Tokens a row can hold with the pages it has now."""
-        return min(self.max_seq_len, (self._pos // self.page_tokens + self.private_pages) * self.page_tokens)
+        return self._row_end
+
+    def _row_pages(self, row):
+        return self.table[row, :-(-self._pos // self.page_tokens)].long()
+
+
+class PagedKVCache(PagedCache):
+    """Keys and values of every head (reference behaviour: nanochat/engine.py:82-137, a contiguous cache per row and a
+    copy at the fork)."""
+
+    def __init__(self, batch_size, num_heads, seq_len, head_dim, num_layers, device, dtype, page_tokens=PAGE_TOKENS):
+        super().__init__(batch_size, num_layers, seq_len, device, dtype, page_tokens)
+        self.n_heads, self.head_dim = num_heads, head_dim
+        self.k_pool = self.v_pool = None
+
+    def _allocate(self, total):
+        shape = (self.n_layers, total, self.page_tokens, self.n_heads, self.head_dim)
+        self.k_pool = self.v_pool = None            # release before allocating the larger pool
+        self.k_pool = torch.zeros(shape, device=self.device, dtype=self.dtype)
+        self.v_pool = torch.zeros(shape, device=self.device, dtype=self.dtype)
+
+    def _copy_tokens(self, pages, source, n):
+        self.k_pool[:, pages, :n] = self.k_pool[:, source:source + 1, :n]
+        self.v_pool[:, pages, :n] = self.v_pool[:, source:source + 1, :n]
+
+    def pool_bytes(self):
+        return 0 if self.k_pool is None else 2 * self.k_pool.numel() * self.k_pool.element_size()
+
+    def get_layer_cache(self, layer_idx):
+        """One layer's pools, (pages, PAGE_TOKENS, H, D): the paged decode kernels take them with `table`."""
+        return self.k_pool[layer_idx], self.v_pool[layer_idx]
 
     def gather_row(self, layer_idx, row):
         """(T, H, D) keys and values of one row in position order (tests and debugging; copies)."""
-        n = self._pos
-        pages = self.table[row, :-(-n // self.page_tokens)].long()
+        n, pages = self._pos, self._row_pages(row)
         k = self.k_pool[layer_idx, pages].reshape(-1, self.n_heads, self.head_dim)[:n]
         v = self.v_pool[layer_idx, pages].reshape(-1, self.n_heads, self.head_dim)[:n]
         return k, v
+
+
+class PagedLatentCache(PagedCache):
+    """One vector per token and layer run, `widths[run]` elements (latent attention: the latent and the shared rotated key
+    part). Layers of a loop have one pool per pass."""
+
+    def __init__(self, batch_size, widths, seq_len, device, dtype, page_tokens=PAGE_TOKENS):
+        super().__init__(batch_size, len(widths), seq_len, device, dtype, page_tokens)
+        self.widths = list(widths)
+        self.pools = None
+
+    def _allocate(self, total):
+        self.pools = None
+        self.pools = [torch.zeros(total, self.page_tokens, w, device=self.device, dtype=self.dtype) for w in self.widths]
+
+    def _copy_tokens(self, pages, source, n):
+        for pool in self.pools:
+            pool[pages, :n] = pool[source:source + 1, :n]
+
+    def pool_bytes(self):
+        return 0 if self.pools is None else sum(p.numel() * p.element_size() for p in self.pools)
+
+    def gather_row(self, run, row):
+        """(T, width) entries of one row in position order (tests and debugging; copies)."""
+        return self.pools[run][self._row_pages(row)].reshape(-1, self.widths[run])[:self._pos]
 
 
 @torch.inference_mode()
@@ -300,12 +369,83 @@ def ids_on_cuda(device):
     return torch.device(device).type == "cuda"
 
 
+class Sequence:
+    """One request fed in portions of any size: `extend` runs a portion's tokens on top of what earlier ones left and
+    returns logits where asked. The first portion, and later ones of several tokens where the model can continue a
+    sequence that way, take the prefill path, single tokens the decode step, as in `Engine.generate`. `close()` gives
+    the pages back."""
+
+    def __init__(self, engine, max_tokens):
+        self.engine, self.max_tokens, self.length = engine, max_tokens, 0
+        self.cache = engine._row_cache(1) if engine.latent or engine._graph_applies(1, max_tokens) else None
+        if self.cache is None:                      # no captured decode here: a contiguous cache of its own
+            self.cache = KVCache(batch_size=1, seq_len=max_tokens, **engine._kv_geometry())
+        else:
+            self.cache.reset()
+            self.cache.reserve_any_prompt(max_tokens)
+
+    @torch.inference_mode()
+    def extend(self, tokens, want=()):
+        """(len(want), V) float logits at the places `want` among `tokens`, or None when nothing is wanted."""
+        n, want = len(tokens), list(want)
+        if n == 0:
+            return None
+        if self.length + n > self.max_tokens:
+            raise ValueError(f"sequence of {self.length + n} tokens, room for {self.max_tokens}")
+        engine, paged = self.engine, getattr(self.cache, "paged", False)
+        ids = torch.tensor([tokens], dtype=torch.long, device=engine.model.get_device())
+        if self.length == 0:
+            view = self.cache.begin_prompt(n) if paged else self.cache
+            logits = engine._prompt_logits(ids, view, want)
+            if paged:
+                self.cache.fork(view)
+            engine._begin_decode(self.cache)
+        elif n > 1 and engine.latent:
+            logits = engine._prompt_logits(ids, self.cache, want)
+        else:
+            rows = {}
+            for i in range(n):
+                step = engine._decode_step(ids[:, i:i + 1], self.cache)
+                if i in want:
+                    rows[i] = step.float().clone()
+            logits = torch.cat([rows[i] for i in want]) if want else None
+        self.length += n
+        return logits
+
+    def close(self):
+        self.cache.reset()
+        self.cache.in_use = False
+
+
 class Engine:
+    """`tokenizer` may be None (models without one): prompts and results are token ids and no token is special."""
+
     def __init__(self, model, tokenizer):
         self.model = model
         self.tokenizer = tokenizer
         self._decode_graphs = {}
-        self._cache_pool = {}      # rows -> full-length KVCache reused across generations (keeps its decode graph)
+        self._cache_pool = {}      # rows -> full-length cache reused across generations (keeps its decode graph)
+        self.latent = hasattr(model, "make_cache")      # the model brings its own paged store
+
+    def open_sequence(self, max_tokens):
+        """A request of up to `max_tokens` tokens to be fed in portions; see Sequence."""
+        return Sequence(self, max_tokens)
+
+    def _prompt_logits(self, ids, cache, want):
+        """Run a portion of tokens; (len(want), V) logits at the places `want`, None when there are none."""
+        if self.latent:
+            logits = self.model.forward(ids, kv_cache=cache, want=list(want))
+            return logits if len(want) else None
+        logits = self.model.forward(ids, kv_cache=cache)[0]
+        return logits[list(want)].float() if len(want) else None
+
+    def _begin_decode(self, cache):
+        """The cache has been filled by a prompt: let its captured decode step take over what the prompt left."""
+        if ids_on_cuda(self.model.get_device()) and ops.get_kernel_mode() == "native":
+            from nanochat_b200.runtime import decode_graph_for
+            runner = decode_graph_for(self, cache)
+            if runner is not None:
+                runner.begin()
 
     def _decode_step(self, ids, kv_cache):
         """One lock-step decode forward; returns (B, V) logits for the new position."""
@@ -315,6 +455,8 @@ class Engine:
             runner = decode_graph_for(self, kv_cache)
         if runner is not None:
             return runner.step(ids)
+        if getattr(kv_cache, "paged", False) and kv_cache.get_pos() >= kv_cache.row_capacity():
+            raise ValueError(f"no room for token {kv_cache.get_pos()}: the rows' pages hold {kv_cache.row_capacity()}")
         return self.model.forward(ids, kv_cache=kv_cache)[:, -1, :]
 
     @torch.inference_mode()
@@ -324,58 +466,85 @@ class Engine:
         rng = torch.Generator(device=device)
         rng.manual_seed(seed)
 
-        tok = self.tokenizer
-        python_start = tok.encode_special("<|python_start|>")
-        python_end = tok.encode_special("<|python_end|>")
-        output_start = tok.encode_special("<|output_start|>")
-        output_end = tok.encode_special("<|output_end|>")
-        assistant_end = tok.encode_special("<|assistant_end|>")
-        bos = tok.get_bos_token_id()
-
         cfg = self.model.config
-        geometry = dict(num_heads=cfg.n_kv_head, head_dim=cfg.n_embd // cfg.n_head,
-                        num_layers=cfg.n_layer, device=device, dtype=common.COMPUTE_DTYPE)
         ids = torch.tensor([tokens], dtype=torch.long, device=device)
         capacity = (len(tokens) + max_tokens) if max_tokens is not None else cfg.sequence_len
-        cache = self._pooled_cache(num_samples, len(tokens), capacity, geometry)
+        cache = self._pooled_cache(num_samples, len(tokens), capacity)
         pooled = cache is not None
         if pooled:
             # 1) batch-1 prefill straight into the pages every row will share  2) fork = page tables + one partial page
             view = cache.begin_prompt(len(tokens))
-            logits = self.model.forward(ids, kv_cache=view)
+            logits = self._prompt_logits(ids, view, [len(tokens) - 1])
             cache.fork(view)
+            logits = logits.expand(num_samples, -1)
         else:
             # 1) batch-1 prefill of the prompt  2) fork: copy it into every sample row of a contiguous cache
+            geometry = self._kv_geometry()
             prompt_cache = KVCache(batch_size=1, seq_len=len(tokens), **geometry)
             logits = self.model.forward(ids, kv_cache=prompt_cache)
             cache = KVCache(batch_size=num_samples, seq_len=capacity, **geometry)
             cache.prefill(prompt_cache)
             del prompt_cache
-        logits = logits[:, -1, :].expand(num_samples, -1)
+            logits = logits[:, -1, :].expand(num_samples, -1)
         try:
             yield from self._decode_loop(tokens, num_samples, max_tokens, temperature, top_k, rng, logits, cache,
-                                         (python_start, python_end, output_start, output_end, assistant_end, bos))
+                                         self._special_tokens())
         finally:
             if pooled:
                 cache.in_use = False
 
-    def _pooled_cache(self, rows, prompt_tokens, capacity, geometry):
-        """The paged cache of this row count. It lives as long as the engine, so its captured decode graph is reused;
-        its page pool grows to the largest request seen. None when the graph path does not apply or the cache is
-        busy (nested generations)."""
-        from nanochat_b200.runtime import graph_path_applies
+    def _kv_geometry(self):
         cfg = self.model.config
-        if capacity > cfg.sequence_len or not graph_path_applies(self.model, rows):
-            return None
+        return dict(num_heads=cfg.n_kv_head, head_dim=cfg.n_embd // cfg.n_head, num_layers=cfg.n_layer,
+                    device=self.model.get_device(), dtype=common.COMPUTE_DTYPE)
+
+    def _graph_applies(self, rows, capacity):
+        from nanochat_b200.runtime import graph_path_applies
+        return capacity <= self.model.config.sequence_len and graph_path_applies(self.model, rows)
+
+    def check(self):
+        """Raise if a kernel behind this engine recorded an error (a failed wait, a token without a page)."""
+        if ids_on_cuda(self.model.get_device()) and ops.get_kernel_mode() == "native":
+            (ops.serving_module() if self.latent else ops.native_module()).check_status()
+
+    def _special_tokens(self):
+        tok = self.tokenizer
+        if tok is None:
+            return (None,) * 6
+        names = ("<|python_start|>", "<|python_end|>", "<|output_start|>", "<|output_end|>", "<|assistant_end|>")
+        return (*(tok.encode_special(n) for n in names), tok.get_bos_token_id())
+
+    def _row_cache(self, rows):
+        """The paged cache of this row count, marked in use. It lives as long as the engine, so its captured decode graph
+        is reused; its page pool grows to the largest request seen. A model with its own store gets a second, unpooled
+        cache when the pooled one is busy (nested generations); for the others None then."""
         cache = self._cache_pool.get(rows)
         if cache is None:
-            cache = PagedKVCache(batch_size=rows, seq_len=cfg.sequence_len, **geometry)
+            if self.latent:
+                cache = self.model.make_cache(rows)
+            else:
+                cache = PagedKVCache(batch_size=rows, seq_len=self.model.config.sequence_len, **self._kv_geometry())
             cache.pooled = True
             cache.in_use = False
             self._cache_pool[rows] = cache
         if cache.in_use:
-            return None
+            if not self.latent:
+                return None
+            cache = self.model.make_cache(rows)
         cache.in_use = True
+        return cache
+
+    def _pooled_cache(self, rows, prompt_tokens, capacity):
+        """A paged cache with room for the request, or None when the model decodes without one here (no captured graph
+        for it, or its cache is busy)."""
+        if self.latent:
+            if capacity > self.model.config.sequence_len:
+                raise ValueError(f"request of {capacity} tokens; this server holds {self.model.config.sequence_len} per row")
+        elif not self._graph_applies(rows, capacity):
+            return None
+        cache = self._row_cache(rows)
+        if cache is None:
+            return None
         cache.reset()
         cache.reserve(prompt_tokens, capacity - prompt_tokens)
         return cache
@@ -384,11 +553,7 @@ class Engine:
         python_start, python_end, output_start, output_end, assistant_end, bos = specials
         tok = self.tokenizer
         device = self.model.get_device()
-        if ids_on_cuda(device) and ops.get_kernel_mode() == "native":
-            from nanochat_b200.runtime import decode_graph_for
-            runner = decode_graph_for(self, cache)
-            if runner is not None:
-                runner.begin()
+        self._begin_decode(cache)
         # 3) lock-step decode with the per-row state machine
         rows = [RowState(tokens.copy()) for _ in range(num_samples)]
         produced = 0
@@ -428,8 +593,7 @@ class Engine:
 
     def generate_batch(self, tokens, num_samples=1, **kwargs):
         """Non-streaming: returns (sequences, masks) without the terminal token; prompt mask is 0."""
-        assistant_end = self.tokenizer.encode_special("<|assistant_end|>")
-        bos = self.tokenizer.get_bos_token_id()
+        *_, assistant_end, bos = self._special_tokens()
         results = [tokens.copy() for _ in range(num_samples)]
         masks = [[0] * len(tokens) for _ in range(num_samples)]
         done = [False] * num_samples

@@ -28,6 +28,7 @@ from nanochat_b200 import common
 from nanochat_b200 import ops
 from nanochat_b200.common import print0
 from nanochat_b200.flash_attention import flash_attn
+from nanochat_b200.models.sampling import NaiveSampler
 from nanochat_b200.ops import reference as ref_ops
 
 
@@ -133,7 +134,7 @@ class Block(nn.Module):
         return x + self.mlp(xn)
 
 
-class GPT(nn.Module):
+class GPT(nn.Module, NaiveSampler):
     def __init__(self, config, pad_vocab_size_to=64):
         """Shapes only: construction may happen under `torch.device('meta')`; values come from
         `init_weights()` (reference: gpt.py:157-201)."""
@@ -417,27 +418,3 @@ class GPT(nn.Module):
         kv_cache.advance(T)
         x = ops.backout_norm(x, x_backout, self.backout_lambda)
         return nat.softcap_logits(x, self.lm_head.weight, self.config.vocab_size)
-
-    @torch.inference_mode()
-    def generate(self, tokens, max_tokens, temperature=1.0, top_k=None, seed=42):
-        """Naive batch-1 streaming sampler that recomputes the whole prefix per token; the
-        Engine must agree with it token for token at temperature 0 (reference: gpt.py:526-555)."""
-        assert isinstance(tokens, list)
-        device = self.get_device()
-        rng = None
-        if temperature > 0:
-            rng = torch.Generator(device=device)
-            rng.manual_seed(seed)
-        ids = torch.tensor([tokens], dtype=torch.long, device=device)
-        for _ in range(max_tokens):
-            logits = self.forward(ids)[:, -1, :]
-            if top_k is not None and top_k > 0:
-                kth, _ = torch.topk(logits, min(top_k, logits.size(-1)))
-                logits[logits < kth[:, [-1]]] = -float("inf")
-            if temperature > 0:
-                probs = F.softmax(logits / temperature, dim=-1)
-                nxt = torch.multinomial(probs, num_samples=1, generator=rng)
-            else:
-                nxt = torch.argmax(logits, dim=-1, keepdim=True)
-            ids = torch.cat((ids, nxt), dim=1)
-            yield nxt.item()

@@ -7,6 +7,9 @@ Every op has two bodies with one meaning:
                      `csrc/` (tcgen05/TMEM GEMMs, flash attention, fused
                      norm/rope/loss/optimizer kernels).
 
+A third module, `serving.py`, holds the native bodies of the inference-only mechanisms (latent attention, mixtures of
+experts, gated residuals), whose kernels are a library of their own and also run in float32.
+
 `use_native(t)` decides per call: CUDA bf16 tensors go to the kernels, everything
 else to the reference body. On a CUDA device a missing extension is an error, not
 a silent fallback, unless NANOCHAT_KERNELS=torch is set explicitly.
@@ -21,6 +24,7 @@ from . import reference
 _MODE = os.environ.get("NANOCHAT_KERNELS", "native")  # native | torch
 _native = None
 _native_err = None
+_serving = None
 
 
 def set_kernel_mode(mode: str):
@@ -121,3 +125,44 @@ def sample_next_token(logits, rng, temperature=1.0, top_k=None):
             and _MODE == "native"):
         return native_module().sample_next_token(logits, rng, temperature, top_k)
     return reference.sample_next_token(logits, rng, temperature, top_k)
+
+
+# ------------------------------------------------------------------- inference mechanisms
+# Used by models that are served only. Their kernels run in bf16 and in float32; on a CUDA device nothing else does
+# unless NANOCHAT_KERNELS=torch is set.
+
+def serving_module():
+    """Import the native bodies of the inference mechanisms (loads, and if need be builds, their library) once."""
+    global _serving
+    if _serving is None:
+        from . import serving
+        _serving = serving
+    return _serving
+
+
+def _serve(name, probe):
+    return getattr(serving_module() if _MODE == "native" and probe.is_cuda else reference, name)
+
+
+def linear_rows(h, w, out_dtype=None):
+    return _serve("linear_rows", h)(h, w, out_dtype)
+
+
+def embed_norm(ids, table, vocab, w, eps, n, keep_x0=False):
+    return _serve("embed_norm", table)(ids, table, vocab, w, eps, n, keep_x0)
+
+
+def gated_residual_norm(x, terms, mult, extra, w, eps, n, dtype):
+    return _serve("gated_residual_norm", x)(x, terms, mult, extra, w, eps, n, dtype)
+
+
+def poly_norm(z, coef, eps, n):
+    return _serve("poly_norm", z)(z, coef, eps, n)
+
+
+def latent_attention(p, z, cache, run, T):
+    return _serve("latent_attention", z)(p, z, cache, run, T)
+
+
+def mixture(h, p):
+    return _serve("mixture", h)(h, p)

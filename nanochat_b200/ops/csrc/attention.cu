@@ -1,4 +1,5 @@
-// Flash attention forward for sm_100a (head dim 128, bf16, causal with optional left window).
+// Flash attention forward for sm_100a (bf16, causal with optional left window): head dim 128, or query / key vectors in
+// two parts (per-head part up to 128, part shared by all key heads up to 64) with values of their own size up to 128.
 //
 // One CTA per (256-query block, head, batch): two 128-query tiles share every K/V block that is
 // loaded, and their softmax phases are staggered so the tensor core always has the other tile's
@@ -27,16 +28,27 @@ namespace nc {
 namespace attn {
 constexpr int BQ = 128;                          // rows of one query tile
 constexpr int TILES = 2;                         // query tiles per CTA
-constexpr int BKV = 128, D = 128;
+constexpr int BKV = 128;
 constexpr int THREADS = 320;
 constexpr int HALF_TILE = 128 * 64 * 2;          // one TMA box: 128 rows x 64 bf16 = 16 KB
-constexpr int TILE = 2 * HALF_TILE;              // 128 x 128 bf16 = 32 KB
-constexpr int KV_STAGES = 2;
-constexpr int SMEM_BYTES = TILES * TILE /*Q*/ + KV_STAGES * 2 * TILE + 1024 + 256;
+constexpr int K_STAGES = 2;
 constexpr int TMEM_COLS = 512;
 constexpr int COL_S = 0, COL_O = 256;            // + 128 * tile
 constexpr float NEG_BIG = -1.0e30f;
 constexpr float RESCALE_STEP = 8.f;              // log2 units the row maximum may outgrow the exponent base
+// Tile shapes of one kernel: query / key tiles are QU boxes of the per-head part and QR boxes of the shared part (64
+// columns each, zero-filled past the part's size), value tiles DV columns. The values are double buffered where
+// everything fits into shared memory.
+template <int QU, int QR, int DV_>
+struct Shape {
+  static constexpr int QB = QU + QR;
+  static constexpr int DV = DV_;
+  static constexpr int K_TILE = QB * HALF_TILE;
+  static constexpr int V_TILE = DV / 64 * HALF_TILE;
+  static constexpr int V_STAGES = QB > 2 && DV > 64 ? 1 : 2;
+  static constexpr int SMEM_BYTES = TILES * K_TILE /*Q*/ + K_STAGES * K_TILE + V_STAGES * V_TILE + 1024 + 256;
+  static_assert(SMEM_BYTES <= 227 * 1024, "tiles must fit shared memory");
+};
 }  // namespace attn
 
 struct AttnKernelArgs {
@@ -45,6 +57,7 @@ struct AttnKernelArgs {
   float* amax_o;        // optional max |o|
   long long o_bat, o_tok, o_head;
   int Tq, Tk, H, Hkv;
+  int dv;               // value columns stored (QR > 0 only)
   int window;           // < 0: unlimited
   float scale_log2;     // softmax scale * log2(e)
   int* status;
@@ -67,16 +80,19 @@ __device__ __forceinline__ BlockRange tile_blocks(int q0x, const AttnKernelArgs&
   return r;
 }
 
+template <int QU, int QR, int DV>
 __global__ void __launch_bounds__(attn::THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                const __grid_constant__ CUtensorMap tmV, const AttnKernelArgs args) {
+                const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQ2,
+                const __grid_constant__ CUtensorMap tmK2, const AttnKernelArgs args) {
   using namespace attn;
+  using S = Shape<QU, QR, DV>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;                            // TILES tiles
-  uint8_t* sK = sQ + TILES * TILE;               // KV_STAGES tiles
-  uint8_t* sV = sK + KV_STAGES * TILE;           // KV_STAGES tiles
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + KV_STAGES * TILE);
+  uint8_t* sK = sQ + TILES * S::K_TILE;          // K_STAGES tiles
+  uint8_t* sV = sK + K_STAGES * S::K_TILE;       // V_STAGES tiles
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + S::V_STAGES * S::V_TILE);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;                   // [2]
   uint64_t* v_full = bars + 3;                   // [2]
@@ -101,7 +117,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < KV_STAGES; ++s) {
+    for (int s = 0; s < 2; ++s) {
       mbar_init(&k_full[s], 1); mbar_init(&v_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_empty[s], 1);
     }
     for (int x = 0; x < TILES; ++x) { mbar_init(&s_full[x], 1); mbar_init(&p_ready[x], 4); mbar_init(&pv_done[x], 1); }
@@ -118,39 +134,50 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     // ---------------------------------------------------------------- producer
     if (lane == 0) {
       tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
+      if (QR > 0) { tma_prefetch_desc(&tmQ2); tma_prefetch_desc(&tmK2); }
       // rows past the end of the sequence (second tile of a ragged block) are zero-filled by TMA
-      mbar_arrive_expect_tx(q_full, TILES * TILE);
+      mbar_arrive_expect_tx(q_full, TILES * S::K_TILE);
 #pragma unroll
       for (int x = 0; x < TILES; ++x) {
-        tma_load_4d(sQ + x * TILE, &tmQ, q_full, 0, q0 + x * BQ, h, b);
-        tma_load_4d(sQ + x * TILE + HALF_TILE, &tmQ, q_full, 64, q0 + x * BQ, h, b);
+#pragma unroll
+        for (int u = 0; u < QU; ++u)
+          tma_load_4d(sQ + x * S::K_TILE + u * HALF_TILE, &tmQ, q_full, u * 64, q0 + x * BQ, h, b);
+#pragma unroll
+        for (int u = 0; u < QR; ++u)
+          tma_load_4d(sQ + x * S::K_TILE + (QU + u) * HALF_TILE, &tmQ2, q_full, u * 64, q0 + x * BQ, h, b);
       }
       bool ok = true;
       for (int it = 0; it < n_blocks && ok; ++it) {
         const int s = it & 1; const uint32_t ph = (it >> 1) & 1;
+        const int sv = S::V_STAGES == 2 ? s : 0; const uint32_t pv = S::V_STAGES == 2 ? ph : it & 1;
         const int k0 = (j_first + it) * BKV;
         if (!mbar_wait(&k_empty[s], ph ^ 1, abort_flag, args.status, ST_WAIT_EMPTY, it)) { ok = false; break; }
-        mbar_arrive_expect_tx(&k_full[s], TILE);
-        tma_load_4d(sK + s * TILE, &tmK, &k_full[s], 0, k0, hkv, b);
-        tma_load_4d(sK + s * TILE + HALF_TILE, &tmK, &k_full[s], 64, k0, hkv, b);
-        if (!mbar_wait(&v_empty[s], ph ^ 1, abort_flag, args.status, ST_WAIT_EMPTY, it)) { ok = false; break; }
-        mbar_arrive_expect_tx(&v_full[s], TILE);
-        tma_load_4d(sV + s * TILE, &tmV, &v_full[s], 0, k0, hkv, b);
-        tma_load_4d(sV + s * TILE + HALF_TILE, &tmV, &v_full[s], 64, k0, hkv, b);
+        mbar_arrive_expect_tx(&k_full[s], S::K_TILE);
+#pragma unroll
+        for (int u = 0; u < QU; ++u)
+          tma_load_4d(sK + s * S::K_TILE + u * HALF_TILE, &tmK, &k_full[s], u * 64, k0, hkv, b);
+#pragma unroll
+        for (int u = 0; u < QR; ++u)
+          tma_load_4d(sK + s * S::K_TILE + (QU + u) * HALF_TILE, &tmK2, &k_full[s], u * 64, k0, 0, b);
+        if (!mbar_wait(&v_empty[sv], pv ^ 1, abort_flag, args.status, ST_WAIT_EMPTY, it)) { ok = false; break; }
+        mbar_arrive_expect_tx(&v_full[sv], S::V_TILE);
+#pragma unroll
+        for (int u = 0; u < DV / 64; ++u)
+          tma_load_4d(sV + sv * S::V_TILE + u * HALF_TILE, &tmV, &v_full[sv], u * 64, k0, hkv, b);
       }
     }
   } else if (warp == 1) {
     // -------------------------------------------------------------- MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(BQ, BKV, false, false);   // Q (K-major) x K (K-major)
-      constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, D, false, true);     // P (TMEM)    x V (MN-major)
+      constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, DV, false, true);    // P (TMEM)    x V (MN-major)
       bool ok = mbar_wait(q_full, 0, abort_flag, args.status, ST_WAIT_FULL, 0xff);
       // Descriptors are built once; a byte offset inside the tile adds offset/16 to the address field
       // (shared memory is smaller than the field's range, so the add never carries out of it).
-      const uint64_t dq[2] = {umma_desc_sw128(smem_u32(sQ), 16, 1024), umma_desc_sw128(smem_u32(sQ + TILE), 16, 1024)};
-      const uint64_t dk[2] = {umma_desc_sw128(smem_u32(sK), 16, 1024), umma_desc_sw128(smem_u32(sK + TILE), 16, 1024)};
+      const uint64_t dq[2] = {umma_desc_sw128(smem_u32(sQ), 16, 1024), umma_desc_sw128(smem_u32(sQ + S::K_TILE), 16, 1024)};
+      const uint64_t dk[2] = {umma_desc_sw128(smem_u32(sK), 16, 1024), umma_desc_sw128(smem_u32(sK + S::K_TILE), 16, 1024)};
       const uint64_t dv[2] = {umma_desc_sw128(smem_u32(sV), HALF_TILE, 1024),
-                              umma_desc_sw128(smem_u32(sV + TILE), HALF_TILE, 1024)};
+                              umma_desc_sw128(smem_u32(sV + (S::V_STAGES - 1) * S::V_TILE), HALF_TILE, 1024)};
       int n_pv[2] = {0, 0};                        // products issued per tile (barrier parities are per tile)
       auto active = [&](int x, int j) { return j >= rng[x].lo && j <= rng[x].hi; };
       auto issue_s = [&](int x, int it) -> bool {
@@ -158,7 +185,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         if (!mbar_wait(&k_full[s], ph, abort_flag, args.status, ST_WAIT_FULL, it)) return false;
         tc_fence_after();
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < S::QB * 4; ++kk) {
           const uint64_t o = static_cast<uint64_t>(((kk >> 2) * HALF_TILE + (kk & 3) * 32) >> 4);
           mma_f16(tmem_base + COL_S + x * 128, dq[x] + o, dk[s] + o, idesc_s, kk != 0);
         }
@@ -166,7 +193,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         return true;
       };
       auto issue_pv = [&](int x, int it) -> bool {
-        const int s = it & 1; const uint32_t ph = (it >> 1) & 1;
+        const int s = S::V_STAGES == 2 ? it & 1 : 0; const uint32_t ph = S::V_STAGES == 2 ? (it >> 1) & 1 : it & 1;
         const int n = n_pv[x]++;
         if (!mbar_wait(&p_ready[x], n & 1, abort_flag, args.status, ST_WAIT_PEER, it)) return false;
         if (!mbar_wait(&v_full[s], ph, abort_flag, args.status, ST_WAIT_FULL, 0x100 + it)) return false;
@@ -192,7 +219,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         if (ok && more && active(0, j + 1)) ok = issue_s(0, it + 1);     // overwrites P_A(j): issued after PV_A(j)
         if (ok && active(1, j)) ok = issue_pv(1, it);
         if (!ok) break;
-        mma_commit(&v_empty[it & 1]);
+        mma_commit(&v_empty[S::V_STAGES == 2 ? it & 1 : 0]);
         if (more) {
           if (active(1, j + 1)) ok = issue_s(1, it + 1);
           mma_commit(&k_empty[(it + 1) & 1]);
@@ -249,7 +276,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           if (!mbar_wait(&pv_done[x], (n - 1) & 1, abort_flag, args.status, ST_WAIT_TMEM_FULL, 0x200 + j)) { ok = false; break; }
           tc_fence_after();
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t v[32];
             tmem_ld32(t_o + c * 32, v);
             tmem_wait_ld();
@@ -292,7 +319,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(args.o) + (long long)b * args.o_bat +
                             (long long)qi * args.o_tok + (long long)h * args.o_head;
 #pragma unroll 1
-      for (int c = 0; c < D / 32; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         uint32_t v[32];
         tmem_ld32(t_o + c * 32, v);
         tmem_wait_ld();
@@ -303,7 +330,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           w.y = pack_bf16(__uint_as_float(v[e + 2]) * inv_l, __uint_as_float(v[e + 3]) * inv_l);
           w.z = pack_bf16(__uint_as_float(v[e + 4]) * inv_l, __uint_as_float(v[e + 5]) * inv_l);
           w.w = pack_bf16(__uint_as_float(v[e + 6]) * inv_l, __uint_as_float(v[e + 7]) * inv_l);
-          if (row_ok) *reinterpret_cast<uint4*>(orow + c * 32 + e) = w;
+          if (row_ok && (QR == 0 || c * 32 + e < args.dv)) *reinterpret_cast<uint4*>(orow + c * 32 + e) = w;
         }
         if (args.amax_o && row_ok) {
 #pragma unroll
@@ -333,35 +360,66 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-static bool make_qkv_map(CUtensorMap* m, const void* base, int T, int Hn, int B, long long tok, long long head,
-                         long long bat) {
-  // dims innermost-first: (d, t, h, b)
-  uint64_t dims[4] = {128, (uint64_t)T, (uint64_t)Hn, (uint64_t)B};
+static bool make_part_map(CUtensorMap* m, const void* base, int D, int T, int Hn, int B, long long tok, long long head,
+                          long long bat) {
+  // dims innermost-first: (d, t, h, b); boxes of 64 columns, zero-filled past D
+  uint64_t dims[4] = {(uint64_t)D, (uint64_t)T, (uint64_t)Hn, (uint64_t)B};
   uint64_t str[3] = {(uint64_t)tok * 2, (uint64_t)head * 2, (uint64_t)bat * 2};
   uint32_t box[4] = {64, 128, 1, 1};
   return make_tmap(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, str, box);
 }
 
-cudaError_t attention_fwd(const AttnDesc& d, int* status, cudaStream_t stream) {
-  if (d.D != 128 || d.H % d.Hkv != 0 || d.Tq > d.Tk) return cudaErrorInvalidValue;
+template <int QU, int QR, int DV>
+static cudaError_t launch_attn(const SplitAttnDesc& sd, int* status, cudaStream_t stream) {
+  using S = attn::Shape<QU, QR, DV>;
+  const AttnDesc& d = sd.a;
   static PerDeviceOnce configured;
-  cudaError_t ce = configured.once([] {
-    return cudaFuncSetAttribute(attn_fwd_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, attn::SMEM_BYTES);
+  auto kern = attn_fwd_kernel<QU, QR, DV>;
+  cudaError_t ce = configured.once([&] {
+    return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::SMEM_BYTES);
   });
   if (ce != cudaSuccess) return ce;
   CUtensorMap tmQ, tmK, tmV;
-  if (!make_qkv_map(&tmQ, d.q, d.Tq, d.H, d.B, d.q_tok, d.q_head, d.q_bat)) return cudaErrorInvalidValue;
-  if (!make_qkv_map(&tmK, d.k, d.Tk, d.Hkv, d.B, d.k_tok, d.k_head, d.k_bat)) return cudaErrorInvalidValue;
-  if (!make_qkv_map(&tmV, d.v, d.Tk, d.Hkv, d.B, d.v_tok, d.v_head, d.v_bat)) return cudaErrorInvalidValue;
+  if (!make_part_map(&tmQ, d.q, d.D, d.Tq, d.H, d.B, d.q_tok, d.q_head, d.q_bat)) return cudaErrorInvalidValue;
+  if (!make_part_map(&tmK, d.k, d.D, d.Tk, d.Hkv, d.B, d.k_tok, d.k_head, d.k_bat)) return cudaErrorInvalidValue;
+  if (!make_part_map(&tmV, d.v, sd.Dv, d.Tk, d.Hkv, d.B, d.v_tok, d.v_head, d.v_bat)) return cudaErrorInvalidValue;
+  CUtensorMap tmQ2 = tmQ, tmK2 = tmK;
+  if (QR > 0) {
+    if (!make_part_map(&tmQ2, sd.q2, sd.D2, d.Tq, d.H, d.B, sd.q2_tok, sd.q2_head, sd.q2_bat)) return cudaErrorInvalidValue;
+    if (!make_part_map(&tmK2, sd.k2, sd.D2, d.Tk, 1, d.B, sd.k2_tok, sd.k2_tok, sd.k2_bat)) return cudaErrorInvalidValue;
+  }
   AttnKernelArgs a;
   a.o = d.o; a.lse = d.lse; a.amax_o = d.amax_o; a.o_bat = d.o_bat; a.o_tok = d.o_tok; a.o_head = d.o_head;
   a.Tq = d.Tq; a.Tk = d.Tk; a.H = d.H; a.Hkv = d.Hkv;
+  a.dv = sd.Dv;
   a.window = d.window;
   a.scale_log2 = d.scale * 1.4426950408889634f;
   a.status = status;
   dim3 grid((d.Tq + attn::TILES * attn::BQ - 1) / (attn::TILES * attn::BQ), d.H, d.B);
-  attn_fwd_kernel<<<grid, attn::THREADS, attn::SMEM_BYTES, stream>>>(tmQ, tmK, tmV, a);
+  kern<<<grid, attn::THREADS, S::SMEM_BYTES, stream>>>(tmQ, tmK, tmV, tmQ2, tmK2, a);
   return cudaGetLastError();
 }
+
+#ifndef NC_SERVING
+cudaError_t attention_fwd(const AttnDesc& d, int* status, cudaStream_t stream) {
+  if (d.D != 128 || d.H % d.Hkv != 0 || d.Tq > d.Tk) return cudaErrorInvalidValue;
+  SplitAttnDesc sd{};
+  sd.a = d;
+  sd.Dv = 128;
+  return launch_attn<2, 0, 128>(sd, status, stream);
+}
+#endif
+
+bool attention_split_supported(int D, int D2, int Dv) {
+  return D > 0 && D <= 128 && D2 > 0 && D2 <= 64 && Dv > 0 && Dv <= 128 && !((D | D2 | Dv) & 7);
+}
+
+#ifdef NC_SERVING
+cudaError_t attention_split_fwd(const SplitAttnDesc& d, int* status, cudaStream_t stream) {
+  if (!attention_split_supported(d.a.D, d.D2, d.Dv) || d.a.H % d.a.Hkv != 0 || d.a.Tq > d.a.Tk) return cudaErrorInvalidValue;
+  if (d.a.D <= 64) return d.Dv <= 64 ? launch_attn<1, 1, 64>(d, status, stream) : launch_attn<1, 1, 128>(d, status, stream);
+  return d.Dv <= 64 ? launch_attn<2, 1, 64>(d, status, stream) : launch_attn<2, 1, 128>(d, status, stream);
+}
+#endif
 
 }  // namespace nc

@@ -19,6 +19,18 @@ struct AttnDesc {
   float* amax_o = nullptr;   // optional: receives max |o| (atomic max on the fp32 bits; zero it first)
 };
 
+// Keys and queries in two parts: scores are q . k + q2 . k2, with k2 (B, Tk, D2) shared by all heads, and values of their
+// own size. D, D2, Dv multiples of 8 (16-byte pitches), D <= 128, D2 <= 64, Dv <= 128. Otherwise as AttnDesc; AttnDesc::D
+// is the size of q and k, its lse and amax_o may be null.
+struct SplitAttnDesc {
+  AttnDesc a;
+  const void *q2, *k2;
+  long long q2_bat, q2_tok, q2_head, k2_bat, k2_tok;
+  int D2, Dv;
+};
+bool attention_split_supported(int D, int D2, int Dv);
+cudaError_t attention_split_fwd(const SplitAttnDesc& d, int* status, cudaStream_t stream);
+
 cudaError_t attention_fwd(const AttnDesc& d, int* status, cudaStream_t stream);
 
 // Backward: fwd holds q,k,v,o,lse and the problem geometry of the forward call. d_o like o; dq like q;

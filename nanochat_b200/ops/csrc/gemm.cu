@@ -50,6 +50,7 @@ struct GemmKernelArgs {
   int symmetric;            // C = C^T by construction (X X^T, A A): tiles below the diagonal are skipped, the caller mirrors
   uint32_t idesc;
   int* status;
+  const int* m_group;       // matrix of B per 128-row block (grouped product), or null
 };
 
 constexpr int next_pow2_cols(int n) { return n <= 32 ? 32 : n <= 64 ? 64 : n <= 128 ? 128 : 256; }
@@ -97,6 +98,12 @@ __device__ __forceinline__ void tile_coords(int t, const GemmKernelArgs& a, int&
   int in_g = r - g * group_tiles;
   mb = first_m + in_g % gm;
   nb = in_g / gm;
+}
+
+// Grouped product: the matrix of B a tile multiplies by, < 0 when the tile holds no rows. Every role of the CTA reads
+// the same entries, so all of them skip the same tiles.
+__device__ __forceinline__ int tile_group(const GemmKernelArgs& a, int mb, int b) {
+  return a.m_group ? __ldg(a.m_group + mb) : b;
 }
 
 // Epilogue of one accumulator tile for one thread: its row of 128 x BN fp32 values comes out of tensor memory
@@ -450,6 +457,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
       int stage = 0; uint32_t phase = 0; bool ok = true;
       for (int t = blockIdx.x; t < total_tiles && ok; t += gridDim.x) {
         int b, mb, nb; tile_coords(t, args, b, mb, nb);
+        const int group = tile_group(args, mb, b);
+        if (group < 0) continue;
         const int m0 = mb * BM, n0 = nb * BN;
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait(&empty[stage], phase ^ 1, abort_flag, args.status, ST_WAIT_EMPTY, t)) { ok = false; break; }
@@ -467,9 +476,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
           if constexpr (B_MN) {
 #pragma unroll
             for (int j = 0; j < C::B_CHUNKS; ++j)
-              tma_load_3d(sB + j * C::CHUNK_BYTES, &tmB, &full[stage], n0 + C::MN_CHUNK * j, k0, b);
+              tma_load_3d(sB + j * C::CHUNK_BYTES, &tmB, &full[stage], n0 + C::MN_CHUNK * j, k0, group);
           } else {
-            tma_load_3d(sB, &tmB, &full[stage], k0, n0, b);
+            tma_load_3d(sB, &tmB, &full[stage], k0, n0, group);
           }
           if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
         }
@@ -482,6 +491,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
       int stage = 0; uint32_t phase = 0; bool ok = true;
       int acc = 0; uint32_t acc_phase = 0;
       for (int t = blockIdx.x; t < total_tiles && ok; t += gridDim.x) {
+        if (args.m_group) {
+          int b, mb, nb; tile_coords(t, args, b, mb, nb);
+          if (tile_group(args, mb, b) < 0) continue;
+        }
         if (!mbar_wait(&acc_empty[acc], acc_phase ^ 1, abort_flag, args.status, ST_WAIT_TMEM_EMPTY, t)) { ok = false; break; }
         tc_fence_after();
         const uint32_t d_tmem = tmem_base + acc * C::ACC_STRIDE;
@@ -534,6 +547,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
     if (use_aux && blockIdx.x < total_tiles) aux_request(args, ahead, tile_at(blockIdx.x), c_begin, c_end, lane);
     for (int t = blockIdx.x; t < total_tiles && ok; t += gridDim.x) {
       int b, mb, nb; tile_coords(t, args, b, mb, nb);
+      if (tile_group(args, mb, b) < 0) continue;
       const TileAt next = use_aux ? tile_at(t + gridDim.x) : TileAt{0, 0, 0, false};
       if (use_aux) aux_prefetch_l2(args, next, c_begin, c_end, lane);
       if (!mbar_wait(&acc_full[acc], acc_phase, abort_flag, args.status, ST_WAIT_TMEM_FULL, t)) { ok = false; break; }
@@ -999,6 +1013,12 @@ static bool make_c_tmap(const GemmDesc& d, const CUtensorMap& placeholder, CUten
 }
 
 // bf16 output with an auxiliary operand that the epilogue combines with the product (not relu^2, which needs none)
+static constexpr bool kAuxAhead =
+#ifdef NC_SERVING
+    false;
+#else
+    true;
+#endif
 static bool aux_ahead_wanted(const GemmDesc& d) {
   return d.aux != nullptr && !d.c_f32 && d.epi != EPI_RELU2 && d.epi != EPI_RELU;
 }
@@ -1029,9 +1049,9 @@ static cudaError_t launch_cfg(const GemmDesc& d, int* status, cudaStream_t strea
     uint64_t dims[3], str[2]; uint32_t box[3];
     if (B_MN) { dims[0] = d.N; dims[1] = d.K; box[0] = C::MN_CHUNK; box[1] = BK; }
     else      { dims[0] = d.K; dims[1] = d.N; box[0] = BK; box[1] = BN; }
-    dims[2] = batch; box[2] = 1;
+    dims[2] = d.m_group ? static_cast<uint64_t>(d.groups) : batch; box[2] = 1;
     str[0] = static_cast<uint64_t>(d.ldb) * ELT;
-    str[1] = d.batch > 1 ? static_cast<uint64_t>(d.bsb) * ELT : str[0] * dims[1];
+    str[1] = dims[2] > 1 ? static_cast<uint64_t>(d.bsb) * ELT : str[0] * dims[1];
     if (!make_tmap(&tmB, dt, 3, d.B, dims, str, box)) return cudaErrorInvalidValue;
   }
   GemmKernelArgs a;
@@ -1049,6 +1069,7 @@ static cudaError_t launch_cfg(const GemmDesc& d, int* status, cudaStream_t strea
   a.tiles_per_batch = a.symmetric ? a.n_blocks * (a.n_blocks + 1) / 2 : a.m_blocks * a.n_blocks;
   a.idesc = FP8 ? umma_idesc_f8(BM, BN, A_MN, B_MN, d.a_e5m2, d.b_e5m2) : umma_idesc_bf16(BM, BN, A_MN, B_MN);
   a.status = status;
+  a.m_group = d.m_group;
   const long long tiles = 1ll * a.tiles_per_batch * d.batch;
   const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
   kern<<<grid, GEMM_THREADS, C::SMEM_BYTES, stream>>>(tmA, tmB, tmC, a);
@@ -1059,7 +1080,7 @@ template <bool A_MN, bool B_MN, bool FP8>
 static cudaError_t launch_bn(int bn, const GemmDesc& d, int* status, cudaStream_t s) {
   // forward and activation-gradient layouts with a bf16 auxiliary operand (residual add, the MLP's relu^2 derivative)
   // have kernels of their own, which request that operand ahead of its use
-  if constexpr (!A_MN) {
+  if constexpr (!A_MN && kAuxAhead) {
     if (aux_ahead_wanted(d) && bn == 256) return launch_cfg<256, A_MN, B_MN, FP8, true>(d, status, s);
     if (aux_ahead_wanted(d) && bn == 208) return launch_cfg<208, A_MN, B_MN, FP8, true>(d, status, s);
     if (aux_ahead_wanted(d) && bn == 128) return launch_cfg<128, A_MN, B_MN, FP8, true>(d, status, s);
@@ -1120,6 +1141,7 @@ static cudaError_t launch_pair_cfg(const GemmDesc& d, int* status, cudaStream_t 
   a.tiles_per_batch = a.symmetric ? a.n_blocks * (a.n_blocks + 1) / 2 : a.m_blocks * a.n_blocks;
   a.idesc = FP8 ? umma_idesc_f8(2 * BM, BN, A_MN, B_MN, d.a_e5m2, d.b_e5m2) : umma_idesc_bf16(2 * BM, BN, A_MN, B_MN);
   a.status = status;
+  a.m_group = nullptr;
   const long long tiles = 1ll * a.tiles_per_batch * d.batch;
   const int max_pairs = sm_count() / 2;
   const int pairs = static_cast<int>(tiles < max_pairs ? tiles : max_pairs);
@@ -1138,7 +1160,7 @@ static cudaError_t launch_pair_cfg(const GemmDesc& d, int* status, cudaStream_t 
 
 template <bool A_MN, bool B_MN, bool FP8>
 static cudaError_t launch_pair_bn(int bn, const GemmDesc& d, int* status, cudaStream_t s) {
-  if constexpr (!A_MN) {
+  if constexpr (!A_MN && kAuxAhead) {
     if (aux_ahead_wanted(d) && bn == 256) return launch_pair_cfg<256, A_MN, B_MN, FP8, true>(d, status, s);
     if (aux_ahead_wanted(d) && bn == 208) return launch_pair_cfg<208, A_MN, B_MN, FP8, true>(d, status, s);
     if (aux_ahead_wanted(d) && bn == 128) return launch_pair_cfg<128, A_MN, B_MN, FP8, true>(d, status, s);
@@ -1153,6 +1175,10 @@ static cudaError_t launch_pair_bn(int bn, const GemmDesc& d, int* status, cudaSt
 
 template <bool FP8>
 static cudaError_t launch_major(int bn, bool pair, const GemmDesc& d, int* status, cudaStream_t stream) {
+#ifdef NC_SERVING      // inference library: y = x W^T without an auxiliary operand is the only layout it uses
+  if (d.a_mn || d.b_mn || FP8) return cudaErrorInvalidValue;
+  return pair ? launch_pair_bn<false, false, false>(bn, d, status, stream) : launch_bn<false, false, false>(bn, d, status, stream);
+#else
   if (pair) {
     if (d.a_mn && d.b_mn) return launch_pair_bn<true, true, FP8>(bn, d, status, stream);
     if (!d.a_mn && d.b_mn) return launch_pair_bn<false, true, FP8>(bn, d, status, stream);
@@ -1163,6 +1189,7 @@ static cudaError_t launch_major(int bn, bool pair, const GemmDesc& d, int* statu
   if (!d.a_mn && d.b_mn) return launch_bn<false, true, FP8>(bn, d, status, stream);
   if (!d.a_mn && !d.b_mn) return launch_bn<false, false, FP8>(bn, d, status, stream);
   return launch_bn<true, false, FP8>(bn, d, status, stream);
+#endif
 }
 
 int gemm_pick_bn(int M, int N, int batch) {
@@ -1205,7 +1232,7 @@ static GemmPlan gemm_plan(const GemmDesc& d, bool fp8) {
   };
   GemmPlan best{128, false};
   double best_score = -1;
-  const bool pair_ok = d.pair > 0 || (d.pair < 0 && env_pair > 0 && d.M > 2 * BM);
+  const bool pair_ok = d.m_group == nullptr && (d.pair > 0 || (d.pair < 0 && env_pair > 0 && d.M > 2 * BM));
   const bool single_ok = d.pair <= 0;
   if (d.symmetric && d.M == d.N && d.bn == 0) return pair_ok ? GemmPlan{256, true} : GemmPlan{128, false};   // square tiles
   static const int cand[5] = {256, 208, 128, 64, 32};
@@ -1262,11 +1289,14 @@ cudaError_t symmetrize_bf16(void* C, int n, long long ld, long long bs, int batc
 cudaError_t gemm_bf16(const GemmDesc& d, int* status, cudaStream_t stream) {
   if (d.M <= 0 || d.N <= 0 || d.K <= 0 || d.batch <= 0) return cudaErrorInvalidValue;
   if ((d.N & 7) || (d.lda & 7) || (d.ldb & 7) || (d.ldc & 3)) return cudaErrorInvalidValue;
+  if (d.m_group && (d.groups <= 0 || d.batch != 1 || d.a_mn || d.b_mn || d.symmetric || (d.bsb & 7) || d.pair > 0 || d.aux))
+    return cudaErrorInvalidValue;
   const GemmPlan p = gemm_plan(d, false);
   if (best_is_invalid(p, d)) return cudaErrorInvalidValue;
   return launch_major<false>(p.bn, p.pair, d, status, stream);
 }
 
+#ifndef NC_SERVING
 cudaError_t gemm_fp8(const GemmDesc& d, int* status, cudaStream_t stream) {
   if (d.M <= 0 || d.N <= 0 || d.K <= 0 || d.batch <= 0) return cudaErrorInvalidValue;
   // TMA strides are multiples of 16 bytes; output rows as for the bf16 kernel
@@ -1315,6 +1345,7 @@ static cudaError_t launch_mx(const GemmDesc& d, const MxScales& sf, int* status,
   a.tiles_per_batch = a.m_blocks * a.n_blocks;
   a.idesc = umma_idesc_mxf8(BM, BN, d.a_e5m2, d.b_e5m2, 0, 0);
   a.status = status;
+  a.m_group = nullptr;
   MxKernelScales ks;
   ks.sfa = sf.sfa; ks.sfb = sf.sfb; ks.k_blocks = d.K / 128; ks.sfb_row_blocks = (d.N + 127) / 128;
   const long long tiles = 1ll * a.m_blocks * a.n_blocks;
@@ -1334,5 +1365,7 @@ cudaError_t gemm_mxfp8(const GemmDesc& d, const MxScales& sf, int* status, cudaS
   if (bn == 128) return launch_mx<128>(d, sf, status, stream);
   return cudaErrorInvalidValue;
 }
+
+#endif  // NC_SERVING
 
 }  // namespace nc

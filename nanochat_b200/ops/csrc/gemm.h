@@ -42,6 +42,11 @@ struct GemmDesc {
   // above the diagonal are computed (57 % of them at 1664 / 256) and the part of C below those tiles is left untouched;
   // `symmetrize_bf16` then copies the upper triangle over the lower one.
   int symmetric = 0;
+  // Grouped product (gemm_bf16, batch == 1, both operands K-major): the rows of A come in groups that start at multiples
+  // of 128; the 128-row block i multiplies by matrix m_group[i] of B (groups matrices, bsb apart), and is left out when
+  // m_group[i] < 0. m_group holds ceil(M / 128) entries in device memory.
+  const int* m_group = nullptr;
+  int groups = 0;
 };
 
 // C[b][j][i] = C[b][i][j] for j > i: bf16 (batch, n, n) with row pitch ld and batch stride bs (elements).

@@ -1,0 +1,466 @@
+// Python bindings of the serving library: unpack torch tensors into pointers and pitches, check shapes and bounds that
+// the kernels rely on, call the launchers. No math, and no allocation except the one status word per device.
+#include <torch/extension.h>
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+
+#include <atomic>
+
+#include "../attention.h"
+#include "../gemm.h"
+#include "serve.h"
+
+namespace {
+
+using at::Tensor;
+using c10::optional;
+using namespace nc::serve;
+
+std::atomic<long long> g_launches{0};
+
+#define NC_CHECK(expr)                                                                                \
+  do {                                                                                                \
+    ++g_launches;                                                                                     \
+    cudaError_t _e = (expr);                                                                          \
+    TORCH_CHECK(_e == cudaSuccess, "nanochat_b200 kernel launch failed: ", cudaGetErrorString(_e), " at " #expr); \
+  } while (0)
+
+cudaStream_t stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+
+Tensor& status_tensor(const at::Device& dev) {
+  static std::vector<Tensor> per_dev(64);
+  Tensor& t = per_dev[dev.index()];
+  if (!t.defined()) t = torch::zeros({4}, torch::dtype(torch::kInt32).device(dev));
+  return t;
+}
+int* status_ptr(const Tensor& like) { return status_tensor(like.device()).data_ptr<int>(); }
+
+bool is_f32(const Tensor& t) { return t.scalar_type() == at::kFloat; }
+// A row matrix the kernels read 8 elements at a time: (rows, n) with dense rows, aligned pitch and base.
+void check_rows(const Tensor& t, const char* name) {
+  TORCH_CHECK(t.is_cuda() && t.dim() == 2 && t.stride(1) == 1 && (t.scalar_type() == at::kBFloat16 || is_f32(t)), name,
+              ": CUDA bf16 or float rows");
+  TORCH_CHECK((t.size(0) == 1 || t.stride(0) % 8 == 0) && t.size(1) % 8 == 0 && (reinterpret_cast<uintptr_t>(t.data_ptr()) & 15) == 0, name,
+              ": rows must be multiples of 8 elements and 16-byte aligned");
+}
+void check_vec(const Tensor& t, int64_t n, const char* name) {
+  TORCH_CHECK(t.is_cuda() && is_f32(t) && t.is_contiguous() && t.numel() >= n && (reinterpret_cast<uintptr_t>(t.data_ptr()) & 15) == 0, name,
+              ": float vector of at least ", n);
+}
+long long pitch(const Tensor& t) { return t.size(0) == 1 ? (t.size(1) + 7) / 8 * 8 : t.stride(0); }
+void same_type(const Tensor& a, const Tensor& b, const char* name) {
+  TORCH_CHECK(a.scalar_type() == b.scalar_type() && a.device() == b.device(), name, ": type or device differs");
+}
+bool has(const optional<Tensor>& t) { return t.has_value() && t->defined(); }
+
+// pool: (pages, page tokens, width); table: int32 (sequences, max pages); lens: int32 (sequences)
+Pages pages_of(const Tensor& pool, const Tensor& table) {
+  TORCH_CHECK(pool.is_cuda() && pool.dim() == 3 && pool.is_contiguous() && pool.size(2) % 8 == 0, "pool: dense (pages, tokens, width)");
+  TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.dim() == 2 && table.is_contiguous(), "page table: int32 (sequences, pages)");
+  const int64_t tokens = pool.size(1);
+  TORCH_CHECK(tokens > 0 && (tokens & (tokens - 1)) == 0, "page size must be a power of two");
+  int shift = 0;
+  while ((int64_t(1) << shift) < tokens) ++shift;
+  return Pages{pool.data_ptr(), table.data_ptr<int>(), (int)table.size(1), shift, (int)pool.size(0), (int)pool.size(2)};
+}
+RowPos positions(const Tensor& lens, const Tensor& table, int64_t per_seq, int64_t rows) {
+  TORCH_CHECK(lens.is_cuda() && lens.scalar_type() == at::kInt && lens.is_contiguous() && per_seq > 0 && rows % per_seq == 0 &&
+              rows / per_seq <= lens.numel() && rows / per_seq <= table.size(0), "sequence lengths: int32, one per sequence");
+  return RowPos{lens.data_ptr<int>(), (int)per_seq};
+}
+NextWeights next_weights(const optional<Tensor>& t) {
+  if (!has(t) || !t->is_contiguous() || (reinterpret_cast<uintptr_t>(t->data_ptr()) & 15)) return {nullptr, 0};
+  return {t->data_ptr(), (long long)t->numel() * (long long)t->element_size()};
+}
+
+// ------------------------------------------------------------------------------------------------- GEMM, attention
+// out (M, N) = A (M, K) B (N, K)^T; grouped: B (groups, N, K), m_group int32, one per 128 rows of A
+void gemm(const Tensor& A, const Tensor& B, Tensor& C, const optional<Tensor>& m_group) {
+  check_rows(A, "A"); check_rows(C, "C");
+  const bool grouped = has(m_group);
+  TORCH_CHECK(A.scalar_type() == at::kBFloat16 && B.scalar_type() == at::kBFloat16 && B.is_cuda() && B.dim() == (grouped ? 3 : 2) &&
+              B.stride(-1) == 1 && B.size(-1) == A.size(1) && B.size(-2) == C.size(1) && A.size(0) == C.size(0), "gemm operands");
+  const c10::cuda::CUDAGuard guard(A.device());
+  nc::GemmDesc d{};
+  d.A = A.data_ptr(); d.lda = pitch(A);
+  d.B = B.data_ptr(); d.ldb = B.stride(-2);
+  d.C = C.data_ptr(); d.ldc = pitch(C); d.c_f32 = is_f32(C);
+  d.M = (int)A.size(0); d.N = (int)C.size(1); d.K = (int)A.size(1); d.batch = 1; d.alpha = 1.f;
+  if (grouped) {
+    TORCH_CHECK(m_group->is_cuda() && m_group->scalar_type() == at::kInt && m_group->is_contiguous() && A.size(0) % 128 == 0 &&
+                m_group->numel() * 128 >= A.size(0), "m_group: int32, one per 128 rows");
+    d.m_group = m_group->data_ptr<int>(); d.groups = (int)B.size(0); d.bsb = B.stride(0);
+  }
+  NC_CHECK(nc::gemm_bf16(d, status_ptr(A), stream()));
+}
+
+// q (T, H, D), q2 (T, H, D2), k (S, H, D), k2 (S, D2), v (S, H, Dv), o (T, H, Dv): views with dense innermost dims
+void attention_split(const Tensor& q, const Tensor& q2, const Tensor& k, const Tensor& k2, const Tensor& v, Tensor& o,
+                     int64_t window_left, double scale) {
+  for (const Tensor* t : {&q, &q2, &k, &k2, &v, (const Tensor*)&o}) {
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kBFloat16 && t->stride(-1) == 1 && (reinterpret_cast<uintptr_t>(t->data_ptr()) & 15) == 0,
+                "attention operands: bf16, dense innermost, 16-byte aligned");
+    for (int64_t i = 0; i + 1 < t->dim(); ++i) TORCH_CHECK(t->stride(i) % 8 == 0, "attention operands: pitches must be multiples of 8");
+  }
+  const int64_t T = q.size(0), H = q.size(1), S = k.size(0);
+  TORCH_CHECK(q2.size(0) == T && q2.size(1) == H && k.size(1) == H && k.size(2) == q.size(2) && k2.dim() == 2 && k2.size(0) == S &&
+              k2.size(1) == q2.size(2) && v.size(0) == S && v.size(1) == H && o.size(0) == T && o.size(1) == H && o.size(2) == v.size(2),
+              "attention shapes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  nc::SplitAttnDesc d{};
+  d.a.q = q.data_ptr(); d.a.q_tok = q.stride(0); d.a.q_head = q.stride(1); d.a.q_bat = q.stride(0) * T;
+  d.a.k = k.data_ptr(); d.a.k_tok = k.stride(0); d.a.k_head = k.stride(1); d.a.k_bat = k.stride(0) * S;
+  d.a.v = v.data_ptr(); d.a.v_tok = v.stride(0); d.a.v_head = v.stride(1); d.a.v_bat = v.stride(0) * S;
+  d.a.o = o.data_ptr(); d.a.o_tok = o.stride(0); d.a.o_head = o.stride(1); d.a.o_bat = o.stride(0) * T;
+  d.q2 = q2.data_ptr(); d.q2_tok = q2.stride(0); d.q2_head = q2.stride(1); d.q2_bat = q2.stride(0) * T;
+  d.k2 = k2.data_ptr(); d.k2_tok = k2.stride(0); d.k2_bat = k2.stride(0) * S;
+  d.a.B = 1; d.a.Tq = (int)T; d.a.Tk = (int)S; d.a.H = (int)H; d.a.Hkv = (int)H; d.a.D = (int)q.size(2);
+  d.D2 = (int)q2.size(2); d.Dv = (int)v.size(2);
+  d.a.window = (int)window_left; d.a.scale = (float)scale;
+  NC_CHECK(nc::attention_split_fwd(d, status_ptr(q), stream()));
+}
+
+// ------------------------------------------------------------------------------------------------------------ rows
+void embed_norm_(const Tensor& ids, const Tensor& table, int64_t vocab, const Tensor& w, double eps, int64_t n, Tensor& x,
+                 const optional<Tensor>& x0, const optional<Tensor>& h) {
+  check_rows(table, "table"); check_rows(x, "x");
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && ids.numel() == x.size(0), "ids: int64, one per row");
+  TORCH_CHECK(is_f32(x) && x.is_contiguous() && x.size(1) <= table.size(1) && n <= x.size(1) && vocab <= table.size(0), "embedding shapes");
+  if (has(x0)) TORCH_CHECK(is_f32(*x0) && x0->is_contiguous() && x0->sizes() == x.sizes(), "x0 like x");
+  if (has(h)) { same_type(*h, table, "h"); TORCH_CHECK(h->is_contiguous() && h->sizes() == x.sizes(), "h shaped like x"); check_vec(w, x.size(1), "w"); }
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(embed_norm(is_f32(table), reinterpret_cast<const long long*>(ids.data_ptr<int64_t>()), table.data_ptr(), table.stride(0),
+                      (int)vocab, w.data_ptr<float>(), (float)eps, (int)x.size(0), (int)n, (int)x.size(1), x.data_ptr<float>(),
+                      has(x0) ? x0->data_ptr<float>() : nullptr, has(h) ? h->data_ptr() : nullptr, stream()));
+}
+
+// terms: (gate logits, bias, y) or (gate logits, bias, expert rows, slot, wt)
+void gated_residual_norm_(Tensor& x, const std::vector<std::vector<Tensor>>& terms, double mult, const optional<Tensor>& extra,
+                          const Tensor& w, double eps, int64_t n, Tensor& h) {
+  check_rows(x, "x"); check_rows(h, "h"); check_vec(w, x.size(1), "w");
+  TORCH_CHECK(is_f32(x) && x.is_contiguous() && h.is_contiguous() && h.sizes() == x.sizes() && terms.size() <= 2 && n <= x.size(1), "residual shapes");
+  if (has(extra)) TORCH_CHECK(is_f32(*extra) && extra->is_contiguous() && extra->sizes() == x.sizes(), "extra like x");
+  GatedTerm t[2] = {};
+  for (size_t i = 0; i < terms.size(); ++i) {
+    const auto& v = terms[i];
+    TORCH_CHECK(v.size() == 3 || v.size() == 5, "a term has 3 or 5 tensors");
+    check_rows(v[0], "gate"); same_type(v[0], h, "gate"); check_vec(v[1], x.size(1), "bias"); check_rows(v[2], "y"); same_type(v[2], h, "y");
+    TORCH_CHECK(v[0].size(0) == x.size(0) && v[0].size(1) == x.size(1) && v[2].size(1) == x.size(1), "term shapes");
+    t[i] = {v[0].data_ptr(), pitch(v[0]), v[1].data_ptr<float>(), v[2].data_ptr(), pitch(v[2]), nullptr, nullptr, 0};
+    if (v.size() == 5) {
+      TORCH_CHECK(v[3].scalar_type() == at::kInt && v[3].is_contiguous() && v[4].sizes() == v[3].sizes() && is_f32(v[4]) && v[4].is_contiguous() &&
+                  v[3].dim() == 2 && v[3].size(0) == x.size(0), "slot / wt: (rows, top)");
+      t[i].slot = v[3].data_ptr<int>(); t[i].wt = v[4].data_ptr<float>(); t[i].top = (int)v[3].size(1);
+    } else {
+      TORCH_CHECK(v[2].size(0) == x.size(0), "term rows");
+    }
+  }
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(gated_residual_norm(is_f32(h), x.data_ptr<float>(), t, (int)terms.size(), (float)mult,
+                               has(extra) ? extra->data_ptr<float>() : nullptr, w.data_ptr<float>(), (float)eps, (int)x.size(0), (int)n,
+                               (int)x.size(1), h.data_ptr(), stream()));
+}
+
+void poly_norm_(const Tensor& z, const Tensor& coef, double eps, int64_t n, Tensor& out) {
+  check_rows(z, "z"); check_rows(out, "out"); same_type(z, out, "out");
+  TORCH_CHECK(coef.is_cuda() && is_f32(coef) && coef.is_contiguous() && coef.numel() == 4, "poly_norm: four float coefficients");
+  TORCH_CHECK(z.sizes() == out.sizes() && n <= z.size(1), "poly_norm shapes");
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(poly_norm(is_f32(z), z.data_ptr(), pitch(z), coef.data_ptr<float>(), (float)eps, (int)z.size(0), (int)n, (int)z.size(1),
+                     out.data_ptr(), pitch(out), stream()));
+}
+
+// ---------------------------------------------------------------------------------------------------------- latent
+void check_latent(const Tensor& z, int64_t off, int64_t n) { TORCH_CHECK(off >= 0 && off + n <= z.size(1), "latent segments out of range"); }
+
+void latent_post_(const Tensor& z, int64_t q_rank, const optional<Tensor>& q_w, const optional<Tensor>& cq, int64_t c_off, int64_t kv_rank,
+                  int64_t kvp, const Tensor& kv_w, double eps, int64_t rot_off, int64_t rot_dim, const Tensor& freq, const Tensor& pool,
+                  const Tensor& table, const Tensor& lens, int64_t per_seq, const optional<Tensor>& kv_out) {
+  check_rows(z, "z");
+  LatentPost d{};
+  d.f32 = is_f32(pool); d.z_f32 = is_f32(z);
+  d.z = z.data_ptr(); d.ldz = pitch(z); d.rows = (int)z.size(0);
+  if (has(cq)) {
+    check_rows(*cq, "cq"); same_type(*cq, pool, "cq"); check_vec(*q_w, q_rank, "q_w");
+    TORCH_CHECK(cq->size(0) == z.size(0) && q_rank <= cq->size(1) && q_rank <= z.size(1), "cq shape");
+    d.q_rank = (int)q_rank; d.qp = (int)cq->size(1); d.q_w = q_w->data_ptr<float>(); d.cq = cq->data_ptr(); d.ldcq = pitch(*cq);
+  }
+  check_latent(z, c_off, kv_rank); check_latent(z, rot_off, rot_dim);
+  check_vec(kv_w, kv_rank, "kv_w");
+  TORCH_CHECK(is_f32(freq) && freq.is_contiguous() && freq.is_cuda(), "freq");
+  d.c_off = (int)c_off; d.kv_rank = (int)kv_rank; d.kvp = (int)kvp; d.kv_w = kv_w.data_ptr<float>(); d.eps = (float)eps;
+  d.rot_off = (int)rot_off; d.rot_dim = (int)rot_dim; d.rp = (int)(pool.size(2) - kvp); d.dims = (int)freq.numel() * 2; d.freq = freq.data_ptr<float>();
+  d.pg = pages_of(pool, table); d.pos = positions(lens, table, per_seq, z.size(0));
+  if (has(kv_out)) {
+    check_rows(*kv_out, "kv_out"); same_type(*kv_out, pool, "kv_out");
+    TORCH_CHECK(kv_out->size(0) == z.size(0) && kv_out->size(1) == pool.size(2), "kv_out shape");
+    d.kv_out = kv_out->data_ptr(); d.ldkv = pitch(*kv_out);
+  }
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(latent_post(d, status_ptr(z), stream()));
+}
+
+void latent_gather_(const Tensor& pool, const Tensor& table, int64_t seq, int64_t first, Tensor& out) {
+  check_rows(out, "out"); same_type(out, pool, "out");
+  TORCH_CHECK(seq >= 0 && seq < table.size(0) && out.size(1) == pool.size(2), "gather shape");
+  const c10::cuda::CUDAGuard guard(out.device());
+  NC_CHECK(latent_gather(is_f32(out), pages_of(pool, table), (int)seq, (int)first, (int)out.size(0), out.data_ptr(), pitch(out),
+                         status_ptr(out), stream()));
+}
+
+void rotate_heads_(Tensor& q, int64_t heads, int64_t off, const Tensor& freq, const Tensor& table, const Tensor& lens, int64_t per_seq) {
+  check_rows(q, "q");
+  TORCH_CHECK(q.size(1) % heads == 0 && is_f32(freq) && freq.is_contiguous(), "rotate_heads shapes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  NC_CHECK(rotate_heads(is_f32(q), q.data_ptr(), pitch(q), (int)q.size(0), (int)heads, (int)(q.size(1) / heads), (int)off,
+                        (int)freq.numel() * 2, freq.data_ptr<float>(), positions(lens, table, per_seq, q.size(0)), stream()));
+}
+
+void absorb_query_(const Tensor& q, int64_t heads, const Tensor& Wuk, Tensor& qa, bool pdl) {
+  check_rows(q, "q"); check_rows(Wuk, "Wuk"); same_type(q, Wuk, "Wuk"); same_type(q, qa, "qa");
+  TORCH_CHECK(q.size(1) % heads == 0 && Wuk.is_contiguous() && Wuk.size(0) % heads == 0 && qa.is_contiguous() &&
+              qa.numel() == q.size(0) * heads * Wuk.size(1), "absorb_query shapes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  NC_CHECK(absorb_query(is_f32(q), q.data_ptr(), pitch(q), (int)q.size(0), (int)heads, (int)(q.size(1) / heads), (int)(Wuk.size(0) / heads),
+                        Wuk.data_ptr(), (int)Wuk.size(1), qa.data_ptr(), pdl, stream()));
+}
+
+void latent_attention_(const Tensor& qa, const Tensor& q, int64_t heads, int64_t dp, int64_t rot_dim, const Tensor& freq, int64_t kvp,
+                       const Tensor& pool, const Tensor& table, const Tensor& lens, int64_t per_seq, int64_t window, double scale,
+                       int64_t splits, Tensor& ml, Tensor& acc, bool pdl) {
+  check_rows(q, "q"); same_type(q, pool, "pool"); same_type(q, qa, "qa");
+  const int64_t rows = q.size(0);
+  TORCH_CHECK(q.size(1) % heads == 0 && qa.is_contiguous() && qa.numel() == rows * heads * kvp && is_f32(ml) && is_f32(acc) &&
+              ml.is_contiguous() && acc.is_contiguous() && splits > 0 && ml.numel() >= rows * heads * splits * 2 &&
+              acc.numel() >= rows * heads * splits * kvp && is_f32(freq) && freq.is_contiguous() && pool.size(2) > kvp, "latent_attention shapes");
+  LatentAttn d{};
+  d.f32 = is_f32(q); d.qa = qa.data_ptr(); d.q = q.data_ptr(); d.ldq = pitch(q); d.head_pitch = (int)(q.size(1) / heads); d.dp = (int)dp;
+  d.rot_dim = (int)rot_dim; d.rp = (int)(pool.size(2) - kvp); d.dims = (int)freq.numel() * 2; d.freq = freq.data_ptr<float>();
+  d.rows = (int)rows; d.heads = (int)heads; d.kvp = (int)kvp;
+  d.pg = pages_of(pool, table); d.pos = positions(lens, table, per_seq, rows);
+  d.window = (int)window; d.scale = (float)scale; d.splits = (int)splits; d.ml = ml.data_ptr<float>(); d.acc = acc.data_ptr<float>(); d.pdl = pdl;
+  const c10::cuda::CUDAGuard guard(q.device());
+  NC_CHECK(latent_attention(d, stream()));
+}
+
+void latent_values_(const Tensor& ml, const Tensor& acc, int64_t rows, int64_t heads, int64_t splits, const Tensor& Wuv, Tensor& y, bool pdl,
+                    const optional<Tensor>& next) {
+  check_rows(Wuv, "Wuv"); check_rows(y, "y"); same_type(Wuv, y, "y");
+  const int64_t kvp = Wuv.size(1), vp = Wuv.size(0) / heads;
+  TORCH_CHECK(Wuv.is_contiguous() && Wuv.size(0) % heads == 0 && y.size(0) == rows && y.size(1) == heads * vp &&
+              ml.numel() >= rows * heads * splits * 2 && acc.numel() >= rows * heads * splits * kvp, "latent_values shapes");
+  const c10::cuda::CUDAGuard guard(y.device());
+  NC_CHECK(latent_values(is_f32(y), ml.data_ptr<float>(), acc.data_ptr<float>(), (int)rows, (int)heads, (int)splits, (int)kvp,
+                         Wuv.data_ptr(), (int)vp, y.data_ptr(), pitch(y), pdl, next_weights(next), stream()));
+}
+
+// --------------------------------------------------------------------------------------------------------- experts
+void route_topk_(const Tensor& logits, int64_t experts, Tensor& idx, Tensor& wt, const optional<Tensor>& counts, const optional<Tensor>& rank) {
+  TORCH_CHECK(logits.is_cuda() && is_f32(logits) && logits.dim() == 2 && logits.stride(1) == 1 && experts <= logits.size(1), "router logits");
+  TORCH_CHECK(idx.scalar_type() == at::kInt && idx.is_contiguous() && idx.dim() == 2 && idx.size(0) == logits.size(0) && is_f32(wt) &&
+              wt.is_contiguous() && wt.sizes() == idx.sizes(), "idx / wt: (rows, top)");
+  if (has(counts)) TORCH_CHECK(counts->scalar_type() == at::kInt && counts->numel() >= experts && has(rank) && rank->sizes() == idx.sizes() &&
+                               rank->scalar_type() == at::kInt && rank->is_contiguous(), "counts / rank");
+  const c10::cuda::CUDAGuard guard(logits.device());
+  NC_CHECK(route_topk(logits.data_ptr<float>(), logits.size(0) == 1 ? logits.size(1) : logits.stride(0), (int)logits.size(0), (int)experts,
+                      (int)idx.size(1), idx.data_ptr<int>(), wt.data_ptr<float>(), has(counts) ? counts->data_ptr<int>() : nullptr,
+                      has(rank) ? rank->data_ptr<int>() : nullptr, stream()));
+}
+
+void group_rows(const Tensor& h, const Tensor& idx, const Tensor& rank, const Tensor& counts, Tensor& offsets, Tensor& tile_group,
+                Tensor& slot, Tensor& xg) {
+  check_rows(h, "h"); check_rows(xg, "xg");
+  const int64_t rows = h.size(0), top = idx.size(1), experts = counts.numel();
+  for (const Tensor* t : {&idx, &rank, &counts, (const Tensor*)&offsets, (const Tensor*)&tile_group, (const Tensor*)&slot})
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kInt && t->is_contiguous(), "group_rows: int32 indices");
+  TORCH_CHECK(h.scalar_type() == at::kBFloat16 && xg.scalar_type() == at::kBFloat16 && xg.is_contiguous() && xg.size(1) == h.size(1) &&
+              xg.size(0) == tile_group.numel() * 128 && xg.size(0) >= rows * top + experts * 127 && offsets.numel() >= experts &&
+              slot.numel() == rows * top && rank.numel() == rows * top && idx.size(0) == rows, "group_rows shapes");
+  const c10::cuda::CUDAGuard guard(h.device());
+  NC_CHECK(plan_groups(counts.data_ptr<int>(), (int)experts, offsets.data_ptr<int>(), tile_group.data_ptr<int>(), (int)tile_group.numel(), stream()));
+  NC_CHECK(gather_groups(h.data_ptr(), pitch(h), (int)rows, (int)top, (int)h.size(1), idx.data_ptr<int>(), rank.data_ptr<int>(),
+                         offsets.data_ptr<int>(), slot.data_ptr<int>(), xg.data_ptr(), stream()));
+}
+
+void silu_mul_(const Tensor& gu, const Tensor& tile_group, Tensor& act) {
+  check_rows(gu, "gu"); check_rows(act, "act");
+  TORCH_CHECK(gu.scalar_type() == at::kBFloat16 && act.scalar_type() == at::kBFloat16 && gu.is_contiguous() && act.is_contiguous() &&
+              gu.size(0) == act.size(0) && gu.size(1) == 2 * act.size(1) && tile_group.scalar_type() == at::kInt &&
+              tile_group.numel() * 128 >= gu.size(0), "silu_mul shapes");
+  const c10::cuda::CUDAGuard guard(gu.device());
+  NC_CHECK(silu_mul(gu.data_ptr(), (int)gu.size(0), (int)act.size(1), tile_group.data_ptr<int>(), act.data_ptr(), stream()));
+}
+
+Routing routing_of(const optional<Tensor>& idx, const optional<Tensor>& wt, const optional<Tensor>& logits, int64_t rows, int64_t experts, int64_t top) {
+  Routing r{};
+  r.experts = (int)experts; r.top = (int)top;
+  if (has(idx)) {
+    TORCH_CHECK(idx->scalar_type() == at::kInt && idx->is_contiguous() && idx->numel() == rows * top && has(wt) && is_f32(*wt) &&
+                wt->is_contiguous() && wt->numel() == rows * top, "routing: (rows, top)");
+    r.idx = idx->data_ptr<int>(); r.wt = wt->data_ptr<float>();
+  } else {
+    TORCH_CHECK(has(logits) && is_f32(*logits) && logits->dim() == 2 && logits->stride(1) == 1 && logits->size(0) == rows && logits->size(1) >= experts,
+                "router logits");
+    r.logits = logits->data_ptr<float>(); r.ld = logits->stride(0);
+  }
+  return r;
+}
+
+void expert_gate_up_(const Tensor& h, const Tensor& Wgu, int64_t top, const optional<Tensor>& idx, const optional<Tensor>& wt,
+                     const optional<Tensor>& logits, Tensor& act, bool pdl, const optional<Tensor>& next) {
+  check_rows(h, "h"); check_rows(act, "act"); same_type(h, Wgu, "Wgu"); same_type(h, act, "act");
+  TORCH_CHECK(Wgu.dim() == 3 && Wgu.is_contiguous() && Wgu.size(2) == h.size(1) && Wgu.size(1) == 2 * act.size(1) && act.is_contiguous() &&
+              act.size(0) == h.size(0) * top, "expert_gate_up shapes");
+  const c10::cuda::CUDAGuard guard(h.device());
+  NC_CHECK(expert_gate_up(is_f32(h), h.data_ptr(), pitch(h), (int)h.size(0), (int)h.size(1), Wgu.data_ptr(), (int)act.size(1),
+                          routing_of(idx, wt, logits, h.size(0), Wgu.size(0), top), act.data_ptr(), pdl, next_weights(next), stream()));
+}
+
+ExpertDown expert_down_of(const Tensor& act, const Tensor& Wdown, int64_t rows, int64_t top, const optional<Tensor>& idx, const optional<Tensor>& wt,
+                          const optional<Tensor>& logits) {
+  check_rows(act, "act"); same_type(act, Wdown, "Wdown");
+  TORCH_CHECK(act.is_contiguous() && act.size(0) == rows * top && Wdown.dim() == 3 && Wdown.is_contiguous() && Wdown.size(2) == act.size(1),
+              "expert_down shapes");
+  ExpertDown d{};
+  d.f32 = is_f32(act); d.act = act.data_ptr(); d.rows = (int)rows; d.fp = (int)act.size(1); d.Wdown = Wdown.data_ptr(); d.N = (int)Wdown.size(1);
+  d.rt = routing_of(idx, wt, logits, rows, Wdown.size(0), top);
+  return d;
+}
+void expert_down_(const Tensor& act, const Tensor& Wdown, const Tensor& idx, const Tensor& wt, Tensor& y) {
+  check_rows(y, "y"); same_type(y, act, "y");
+  ExpertDown d = expert_down_of(act, Wdown, y.size(0), idx.size(1), idx, wt, c10::nullopt);
+  TORCH_CHECK(y.size(1) == Wdown.size(1), "expert_down shapes");
+  d.y = y.data_ptr(); d.ldy = pitch(y);
+  const c10::cuda::CUDAGuard guard(y.device());
+  NC_CHECK(expert_down(d, stream()));
+}
+void check_gate(const Tensor& x, const Tensor& g, const Tensor& bias, const optional<Tensor>& extra, int64_t rows, int64_t n) {
+  TORCH_CHECK(is_f32(x) && x.is_cuda() && x.is_contiguous() && x.dim() == 2 && x.size(0) == rows && x.size(1) == n, "residual: float (rows, n)");
+  TORCH_CHECK(is_f32(g) && g.dim() == 2 && g.stride(1) == 1 && g.size(0) == rows && g.size(1) == n && is_f32(bias) && bias.is_contiguous() &&
+              bias.numel() >= n, "gate logits / bias: float");
+  if (has(extra)) TORCH_CHECK(is_f32(*extra) && extra->is_contiguous() && extra->sizes() == x.sizes(), "extra like the residual");
+}
+void expert_down_residual(const Tensor& act, const Tensor& Wdown, int64_t top, const Tensor& logits, Tensor& x, const Tensor& g,
+                          const Tensor& bias, double mult, const optional<Tensor>& extra, const optional<Tensor>& next) {
+  ExpertDown d = expert_down_of(act, Wdown, x.size(0), top, c10::nullopt, c10::nullopt, logits);
+  check_gate(x, g, bias, extra, x.size(0), Wdown.size(1));
+  d.resid = x.data_ptr<float>(); d.ldr = x.stride(0); d.g = g.data_ptr<float>(); d.ldg = g.stride(0); d.bias = bias.data_ptr<float>();
+  d.mult = (float)mult; d.extra = has(extra) ? extra->data_ptr<float>() : nullptr; d.pdl = true; d.next = next_weights(next);
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(expert_down(d, stream()));
+}
+
+// ------------------------------------------------------------------------------------------------------------ gemv
+GemvDesc gemv_of(const Tensor& x, const Tensor& W, const optional<Tensor>& next) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1 && W.is_cuda() && W.scalar_type() == at::kBFloat16, "gemv operands");
+  check_rows(x, "x"); check_rows(W, "W");
+  TORCH_CHECK(x.size(1) == W.size(1) && x.size(0) <= 8, "gemv shapes");
+  GemvDesc d{};
+  d.x = x.data_ptr(); d.ldx = pitch(x); d.W = W.data_ptr(); d.ldw = pitch(W); d.rows = (int)x.size(0); d.N = (int)W.size(0); d.K = (int)x.size(1);
+  d.next = next_weights(next);
+  return d;
+}
+int store_kind(GemvDesc& d, Tensor& out) {
+  TORCH_CHECK(out.is_cuda() && out.dim() == 2 && out.stride(1) == 1 && out.size(0) == d.rows && out.size(1) == d.N &&
+              (is_f32(out) || out.scalar_type() == at::kBFloat16), "gemv output");
+  d.out = out.data_ptr(); d.ldo = out.stride(0);
+  return is_f32(out) ? GEMV_STORE_F32 : GEMV_STORE_BF16;
+}
+// out = (x / rms(x) * w) W^T; h: the normed rows as bf16. `store`: see latent_store_args.
+void gemv_norm(const Tensor& x, const Tensor& w, double eps, int64_t n, const Tensor& W, Tensor& out, const optional<Tensor>& h,
+               const optional<Tensor>& next) {
+  GemvDesc d = gemv_of(x, W, next);
+  TORCH_CHECK(is_f32(x), "gemv_norm: float rows"); check_vec(w, x.size(1), "w");
+  d.w = w.data_ptr<float>(); d.eps = (float)eps; d.n_real = (int)n;
+  if (has(h)) {
+    TORCH_CHECK(h->scalar_type() == at::kBFloat16 && h->is_contiguous() && h->sizes() == x.sizes(), "h: bf16 like x");
+    d.h_out = h->data_ptr(); d.ldh = x.size(1);
+  }
+  const int epi = store_kind(d, out);
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(gemv(d, PRE_NORM, epi, stream()));
+}
+// The query half of a latent layer's decode step: q = (norm of z[:, :q_rank]) Wq^T, and the step's store entries.
+void gemv_query_store(const Tensor& z, int64_t q_rank, const Tensor& q_w, double eps, const Tensor& Wq, Tensor& q, int64_t c_off, int64_t kv_rank,
+                      int64_t kvp, const Tensor& kv_w, int64_t rot_off, int64_t rot_dim, const Tensor& freq, const Tensor& pool,
+                      const Tensor& table, const Tensor& lens, const optional<Tensor>& next) {
+  TORCH_CHECK(is_f32(z) && z.dim() == 2 && z.stride(1) == 1 && Wq.size(1) <= z.size(1), "z: float rows");
+  const Tensor x = z.narrow(1, 0, Wq.size(1));
+  GemvDesc d = gemv_of(x, Wq, next);
+  d.ldx = z.size(0) == 1 ? d.ldx : z.stride(0);
+  check_vec(q_w, Wq.size(1), "q_w"); check_vec(kv_w, kv_rank, "kv_w");
+  d.w = q_w.data_ptr<float>(); d.eps = (float)eps; d.n_real = (int)q_rank;
+  check_latent(z, c_off, kv_rank); check_latent(z, rot_off, rot_dim);
+  TORCH_CHECK(pool.scalar_type() == at::kBFloat16 && pool.size(2) > kvp && kv_rank <= kvp && is_f32(freq) && freq.is_contiguous() && freq.numel() * 2 <= rot_dim &&
+              rot_dim <= pool.size(2) - kvp && rot_off >= c_off, "store shapes");
+  LatentStore s{};
+  s.z = z.data_ptr<float>() + c_off; s.ldz = z.stride(0); s.kv_rank = (int)kv_rank; s.kvp = (int)kvp; s.kv_w = kv_w.data_ptr<float>(); s.eps = (float)eps;
+  s.rot_off = (int)(rot_off - c_off); s.rot_dim = (int)rot_dim; s.rp = (int)(pool.size(2) - kvp); s.dims = (int)freq.numel() * 2; s.freq = freq.data_ptr<float>();
+  s.pg = pages_of(pool, table); s.pos = positions(lens, table, 1, z.size(0)); s.status = status_ptr(z);
+  d.store = &s;
+  const int epi = store_kind(d, q);
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(gemv(d, PRE_NORM, epi, stream()));
+}
+// x[b] += mult * sigmoid(g + bias) * (y W^T) (+ extra); y: bf16 rows, or float rows z put through poly_norm (coef given)
+void gemv_residual(const Tensor& y, const optional<Tensor>& coef, double eps, int64_t n, const Tensor& W, Tensor& x, const Tensor& g,
+                   const Tensor& bias, double mult, const optional<Tensor>& extra, const optional<Tensor>& next) {
+  GemvDesc d = gemv_of(y, W, next);
+  d.ldx = y.size(0) == 1 ? d.ldx : y.stride(0);
+  int pre = PRE_PLAIN;
+  if (has(coef)) {
+    TORCH_CHECK(is_f32(y) && coef->is_cuda() && is_f32(*coef) && coef->is_contiguous() && coef->numel() == 4, "poly_norm rows: float, four coefficients");
+    pre = PRE_POLY; d.w = coef->data_ptr<float>(); d.eps = (float)eps; d.n_real = (int)n;
+  } else {
+    TORCH_CHECK(y.scalar_type() == at::kBFloat16, "y: bf16 rows");
+  }
+  check_gate(x, g, bias, extra, y.size(0), W.size(0));
+  d.resid = x.data_ptr<float>(); d.ldr = x.stride(0); d.g = g.data_ptr<float>(); d.ldg = g.stride(0); d.bias = bias.data_ptr<float>();
+  d.mult = (float)mult; d.extra = has(extra) ? extra->data_ptr<float>() : nullptr;
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(gemv(d, pre, GEMV_RESIDUAL, stream()));
+}
+
+std::vector<int64_t> read_status(const Tensor& like) {
+  Tensor& t = status_tensor(like.device());
+  const Tensor h = t.cpu();
+  t.zero_();
+  const int* p = h.data_ptr<int>();
+  return {p[0], p[1], p[2], p[3]};
+}
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+  m.def("gemm", &gemm, py::arg("A"), py::arg("B"), py::arg("C"), py::arg("m_group") = py::none());
+  m.def("attention_split", &attention_split);
+  m.def("attention_split_supported", &nc::attention_split_supported);
+  m.def("embed_norm", &embed_norm_);
+  m.def("gated_residual_norm", &gated_residual_norm_);
+  m.def("poly_norm", &poly_norm_);
+  m.def("latent_post", &latent_post_);
+  m.def("latent_gather", &latent_gather_);
+  m.def("rotate_heads", &rotate_heads_);
+  m.def("absorb_query", &absorb_query_);
+  m.def("latent_attention", &latent_attention_);
+  m.def("latent_values", &latent_values_, py::arg("ml"), py::arg("acc"), py::arg("rows"), py::arg("heads"), py::arg("splits"), py::arg("Wuv"),
+        py::arg("y"), py::arg("pdl"), py::arg("next") = py::none());
+  m.def("route_topk", &route_topk_, py::arg("logits"), py::arg("experts"), py::arg("idx"), py::arg("wt"), py::arg("counts") = py::none(),
+        py::arg("rank") = py::none());
+  m.def("group_rows", &group_rows);
+  m.def("silu_mul", &silu_mul_);
+  m.def("expert_gate_up", &expert_gate_up_, py::arg("h"), py::arg("Wgu"), py::arg("top"), py::arg("idx"), py::arg("wt"), py::arg("logits"),
+        py::arg("act"), py::arg("pdl"), py::arg("next") = py::none());
+  m.def("expert_down", &expert_down_);
+  m.def("expert_down_residual", &expert_down_residual, py::arg("act"), py::arg("Wdown"), py::arg("top"), py::arg("logits"), py::arg("x"),
+        py::arg("g"), py::arg("bias"), py::arg("mult"), py::arg("extra") = py::none(), py::arg("next") = py::none());
+  m.def("gemv_norm", &gemv_norm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("n"), py::arg("W"), py::arg("out"),
+        py::arg("h") = py::none(), py::arg("next") = py::none());
+  m.def("gemv_query_store", &gemv_query_store, py::arg("z"), py::arg("q_rank"), py::arg("q_w"), py::arg("eps"), py::arg("Wq"), py::arg("q"),
+        py::arg("c_off"), py::arg("kv_rank"), py::arg("kvp"), py::arg("kv_w"), py::arg("rot_off"), py::arg("rot_dim"), py::arg("freq"),
+        py::arg("pool"), py::arg("table"), py::arg("lens"), py::arg("next") = py::none());
+  m.def("gemv_residual", &gemv_residual, py::arg("y"), py::arg("coef"), py::arg("eps"), py::arg("n"), py::arg("W"), py::arg("x"), py::arg("g"),
+        py::arg("bias"), py::arg("mult"), py::arg("extra") = py::none(), py::arg("next") = py::none());
+  m.def("read_status", &read_status);
+  m.def("launch_count", [] { return g_launches.load(); });
+}

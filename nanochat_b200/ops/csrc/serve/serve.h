@@ -1,0 +1,162 @@
+// Host interface of the serving kernels: rows.cu (norms, gated residual, activations, matrix-vector products),
+// latent.cu (latent attention over a paged store) and experts.cu (mixture of experts).
+//
+// Conventions. "f32" selects float or bf16 for the typed pointers (weights and activations share one type). The
+// residual stream, gates' biases, norm weights, router logits and attention partials are always float. Row sizes and
+// pitches are multiples of 8 elements, pointers 16-byte aligned; entries past a row's real size are zero.
+#pragma once
+
+#include <cuda_runtime.h>
+#include <stddef.h>
+
+namespace nc {
+namespace serve {
+
+// One layer's paged store: n_pages pages of 2^shift tokens, each token `width` elements; `table` (sequences x
+// max_pages) names the page of every 2^shift tokens of a sequence.
+struct Pages {
+  void* pool;
+  const int* table;
+  int max_pages, shift, n_pages, width;
+};
+
+// Rows of a step: row r belongs to sequence r / per_seq and sits at position lens[r / per_seq] + r % per_seq.
+struct RowPos {
+  const int* lens;
+  int per_seq;
+};
+
+struct NextWeights {      // memory a later kernel will stream; ptr = nullptr: none
+  const void* ptr;
+  long long bytes;
+};
+
+// ------------------------------------------------------------------------------ rows.cu
+// x[r] = table[ids[r]] (float), x0[r] the same when x0 is given, h[r] = x / rms(x) * w. Ids are clamped to [0, vocab).
+cudaError_t embed_norm(bool f32, const long long* ids, const void* table, long long ld, int vocab, const float* w,
+                       float eps, int rows, int n, int np, float* x, float* x0, void* h, cudaStream_t s);
+
+// One term of the residual update: sigmoid(g + bias) * y, y a row or the weighted sum of the rows a token's experts
+// wrote (slot / wt: rows x top).
+struct GatedTerm {
+  const void* g; long long ldg;
+  const float* bias;
+  const void* y; long long ldy;
+  const int* slot; const float* wt; int top;
+};
+// x[r] += mult * sum of terms (+ extra[r]); h[r] = x / rms(x) * w.
+cudaError_t gated_residual_norm(bool f32, float* x, const GatedTerm* terms, int n_terms, float mult, const float* extra,
+                                const float* w, float eps, int rows, int n, int np, void* h, cudaStream_t s);
+
+// out[r] = c[0] N(z) + c[1] N(z^2) + c[2] N(z^3) + c[3], N(v) = v / rms(v) over the row's n entries.
+cudaError_t poly_norm(bool f32, const void* z, long long ldz, const float* coef, float eps, int rows, int n, int np,
+                      void* out, long long ldo, cudaStream_t s);
+
+// Matrix-vector products of a decode step, bf16 weights, rows <= 8: out[b, j] = epilogue(sum_k pre(x)[b, k] W[j, k]).
+enum GemvPre : int {
+  PRE_NORM = 0,     // x float, x / rms(x) * w
+  PRE_PLAIN = 1,    // x bf16
+  PRE_POLY = 2,     // x float, the poly_norm activation with coefficients `w` (4)
+};
+enum GemvEpi : int {
+  GEMV_STORE_F32 = 0,
+  GEMV_STORE_BF16 = 1,
+  GEMV_RESIDUAL = 2,     // resid[b, j] += mult * sigmoid(g[b, j] + bias[j]) * value (+ extra[b, j])
+};
+struct LatentStore {     // see latent_store below; used by the extra CTAs of a product that also appends to the store
+  const void* z; long long ldz;
+  int kv_rank, kvp; const float* kv_w; float eps;
+  int rot_off, rot_dim, rp, dims; const float* freq;
+  Pages pg; RowPos pos; int* status;
+};
+struct GemvDesc {
+  const void* x; long long ldx;
+  const float* w; float eps; int n_real;            // norm weight / coefficients, entries of the row that count
+  const void* W; long long ldw;
+  int rows, N, K;
+  void* out; long long ldo;
+  float* resid; long long ldr; const float* g; long long ldg; const float* bias; float mult; const float* extra;
+  void* h_out; long long ldh;                       // PRE_NORM: the normed row as bf16, when wanted
+  NextWeights next;
+  const LatentStore* store;                         // PRE_NORM only
+};
+cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s);
+
+// ---------------------------------------------------------------------------- latent.cu
+// Per row: cq = norm(z[:q_rank]) (when asked), and the entry [norm(z[c_off:c_off+kv_rank]) | rotated z[rot_off:]]
+// into the store and (kv_out) a dense row. TZ of z: float when z_f32.
+struct LatentPost {
+  bool f32, z_f32;
+  const void* z; long long ldz; int rows;
+  int q_rank, qp; const float* q_w; void* cq; long long ldcq;
+  int c_off, kv_rank, kvp; const float* kv_w; float eps;
+  int rot_off, rot_dim, rp, dims; const float* freq;
+  Pages pg; RowPos pos;
+  void* kv_out; long long ldkv;
+};
+cudaError_t latent_post(const LatentPost& d, int* status, cudaStream_t s);
+// out[j] = the store's entry of token first + j of sequence `seq`, j < count.
+cudaError_t latent_gather(bool f32, const Pages& pg, int seq, int first, int count, void* out, long long ldo,
+                          int* status, cudaStream_t s);
+// q[r, h, off : off + dims] rotated in place (rows x heads x head_pitch).
+cudaError_t rotate_heads(bool f32, void* q, long long ldq, int rows, int heads, int head_pitch, int off, int dims,
+                         const float* freq, const RowPos& pos, cudaStream_t s);
+// qa[r, h, :] = sum_d q[r, h, d] Wuk[h * dp + d, :]     (d < dp)
+cudaError_t absorb_query(bool f32, const void* q, long long ldq, int rows, int heads, int head_pitch, int dp,
+                         const void* Wuk, int kvp, void* qa, bool pdl, cudaStream_t s);
+// Attention of absorbed queries over stored entries; per (row, head, split) an unnormalised partial
+// [max, sum] in ml and sum of exp weights times latents in acc (kvp floats). The query's last part is rotated here.
+struct LatentAttn {
+  bool f32;
+  const void* qa; const void* q; long long ldq; int head_pitch, dp, rot_dim, rp, dims; const float* freq;
+  int rows, heads, kvp;
+  Pages pg; RowPos pos;
+  int window;            // keys a query sees, itself included; <= 0: all
+  float scale;
+  int splits;
+  float* ml; float* acc;
+  bool pdl;
+};
+cudaError_t latent_attention(const LatentAttn& d, cudaStream_t s);
+bool latent_attention_tensor_cores(const LatentAttn& d);
+// y[r, h * vp + j] = sum_k merged(r, h)[k] Wuv[h * vp + j, k], merged = the splits' partials combined and normalised.
+cudaError_t latent_values(bool f32, const float* ml, const float* acc, int rows, int heads, int splits, int kvp,
+                          const void* Wuv, int vp, void* y, long long ldy, bool pdl, const NextWeights& next,
+                          cudaStream_t s);
+
+// --------------------------------------------------------------------------- experts.cu
+// The `top` largest logits of every row (ties: lower index first) and the softmax over them. counts / rank (optional):
+// how many rows chose an expert, and a row's place among them.
+cudaError_t route_topk(const float* logits, long long ld, int rows, int experts, int top, int* idx, float* wt,
+                       int* counts, int* rank, cudaStream_t s);
+// Rows grouped by expert, every group starting at a multiple of 128: offsets (experts), tile_group (tiles, -1 = unused).
+cudaError_t plan_groups(const int* counts, int experts, int* offsets, int* tile_group, int tiles, cudaStream_t s);
+// xg[slot] = h[r], slot[r, k] = offsets[idx[r, k]] + rank[r, k]
+cudaError_t gather_groups(const void* h, long long ldh, int rows, int top, int np, const int* idx, const int* rank,
+                          const int* offsets, int* slot, void* xg, cudaStream_t s);
+// act[i, :fp] = silu(gu[i, :fp]) * gu[i, fp:2fp] for the rows of used tiles (bf16)
+cudaError_t silu_mul(const void* gu, int rows, int fp, const int* tile_group, void* act, cudaStream_t s);
+
+// Experts as matrix-vector products, one per (row, chosen expert). Wgu: experts x [gate fp rows | up fp rows] x K.
+// Either idx / wt hold the routing, or `logits` is given and it is worked out here.
+struct Routing {
+  const int* idx; const float* wt;
+  const float* logits; long long ld;
+  int experts, top;
+};
+cudaError_t expert_gate_up(bool f32, const void* h, long long ldh, int rows, int K, const void* Wgu, int fp,
+                           const Routing& rt, void* act, bool pdl, const NextWeights& next, cudaStream_t s);
+// y[r] = sum_k wt[r, k] Wdown[idx[r, k]] act[r * top + k]; with resid: resid[r] += mult * sigmoid(g + bias) * that (+ extra).
+struct ExpertDown {
+  bool f32;
+  const void* act; int rows, fp;
+  const void* Wdown; int N;
+  Routing rt;
+  void* y; long long ldy;
+  float* resid; long long ldr; const float* g; long long ldg; const float* bias; float mult; const float* extra;
+  bool pdl; NextWeights next;
+};
+cudaError_t expert_down(const ExpertDown& d, cudaStream_t s);
+
+}  // namespace serve
+}  // namespace nc

@@ -224,3 +224,109 @@ def muon_update(grads, params, momentum_buf, second_buf, momentum, lr, wd, beta2
     g = g * (step_size * (v_norm / v_norm_new.clamp_min(1e-10))).to(g.dtype)
     mask = (g * params) >= 0
     params.sub_(lr * g + lr * wd * params * mask)
+
+
+# ------------------------------------------------------------------- inference mechanisms
+# Plain bodies of `ops/serving.py`: latent attention over a paged store, gated residual update, normed-powers
+# activation, mixture of experts. Weight holders are the modules of `nanochat_b200.models.lupodra` (sizes padded with
+# zeros). Products run in the weights' type, everything else in float32.
+
+def linear_rows(h, w, out_dtype=None):
+    if out_dtype is not None and out_dtype != h.dtype:
+        return h.to(out_dtype) @ w.to(out_dtype).t()
+    return h @ w.t()
+
+
+def _rms(x, eps, n):
+    return torch.rsqrt(x.square().sum(-1, keepdim=True) / n + eps)
+
+
+def embed_norm(ids, table, vocab, w, eps, n, keep_x0=False):
+    x = table[ids.clamp(0, vocab - 1)].float()
+    return x, x.clone() if keep_x0 else None, (x * _rms(x, eps, n) * w).to(table.dtype)
+
+
+def gated_residual_norm(x, terms, mult, extra, w, eps, n, dtype):
+    total = torch.zeros_like(x)
+    for gate, bias, y, *chosen in terms:
+        y = y.float()
+        if chosen:
+            slot, wt = chosen
+            y = (y[slot.long()] * wt[..., None]).sum(1)
+        total += torch.sigmoid(gate.float() + bias) * y
+    x += mult * total
+    if extra is not None:
+        x += extra
+    return (x * _rms(x, eps, n) * w).to(dtype)
+
+
+def poly_norm(z, coef, eps, n):
+    a, b, c, e = coef.tolist()
+    v = z[:, :n].float()
+    out = torch.zeros(z.shape, dtype=z.dtype, device=z.device)
+    v2, v3 = v * v, v * v * v
+    out[:, :n] = (a * v * _rms(v, eps, n) + b * v2 * _rms(v2, eps, n) + c * v3 * _rms(v3, eps, n) + e).to(z.dtype)
+    return out
+
+
+def rotate_pairs(x, positions, freq):
+    """x (R, ..., n): entry i and entry i + len(freq) of the first 2 len(freq) turn by positions * freq[i]."""
+    half = freq.numel()
+    angle = (positions.float()[:, None] * freq).reshape(-1, *([1] * (x.dim() - 2)), half)
+    c, s, u, v = angle.cos(), angle.sin(), x[..., :half].float(), x[..., half:2 * half].float()
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:].float()], -1).to(x.dtype)
+
+
+def latent_attention(p, z, cache, run, T):
+    R, pool = z.shape[0], cache.pools[run]
+    P, flat = pool.shape[1], pool.view(-1, pool.shape[2])
+    table = cache.table.long()
+    start = cache.cache_seqlens.long()
+    pos = (start[:, None] + torch.arange(T, device=z.device)).reshape(R)
+    seq = torch.arange(R, device=z.device) // T
+    f = lambda t: t.float()
+    zq = f(z[:, :p.q_rank])
+    cq = torch.zeros(R, p.qp, device=z.device)
+    cq[:, :p.q_rank] = zq * _rms(zq, p.eps, p.q_rank) * p.q_norm[:p.q_rank]
+    q = (cq.to(p.w_q.dtype) @ p.w_q.t()).view(R, p.heads, p.dp + p.rp)
+    q_turn = rotate_pairs(q[..., p.dp:], pos, p.freq)
+    zc = f(z[:, p.c_off:p.c_off + p.kv_rank])
+    entry = torch.zeros(R, p.kvp + p.rp, device=z.device)
+    entry[:, :p.kv_rank] = zc * _rms(zc, p.eps, p.kv_rank) * p.kv_norm[:p.kv_rank]
+    entry[:, p.kvp:p.kvp + p.rot_dim] = f(rotate_pairs(z[:, p.rot_off:p.rot_off + p.rot_dim], pos, p.freq))
+    flat[table[seq, pos // P] * P + pos % P] = entry.to(pool.dtype)
+    wuk, wuv = f(p.w_uk).view(p.heads, p.dp, p.kvp), f(p.w_uv).view(p.heads, p.vp, p.kvp)
+    qa = torch.einsum("rhd,hdk->rhk", f(q[..., :p.dp]), wuk)
+    y = torch.empty(R, p.heads, p.vp, device=z.device)
+    for b in range(R // T):
+        rows = slice(b * T, (b + 1) * T)
+        end = int(start[b]) + T
+        j = torch.arange(end, device=z.device)
+        keys = f(flat[table[b, j // P] * P + j % P])
+        score = (torch.einsum("rhk,jk->hrj", qa[rows], keys[:, :p.kvp]) +
+                 torch.einsum("rhk,jk->hrj", f(q_turn[rows]), keys[:, p.kvp:])) * p.scale
+        gap = pos[rows, None] - j
+        hidden = gap < 0
+        if p.window is not None:
+            hidden = hidden | (gap >= p.window)
+        w = torch.softmax(score.masked_fill(hidden, -float("inf")), -1)
+        y[rows] = torch.einsum("hrk,hvk->rhv", torch.einsum("hrj,jk->hrk", w, keys[:, :p.kvp]), wuv)
+    return y.view(R, -1).to(p.w_o.dtype) @ p.w_o.t()
+
+
+def route(h, p):
+    z = (h.float() @ p.router.float().t())[:, :p.experts]
+    best, idx = torch.topk(z, p.top, dim=-1)
+    return idx.int(), torch.softmax(best, -1)
+
+
+def mixture(h, p):
+    idx, wt = route(h, p)
+    y = torch.zeros(h.shape, device=h.device)
+    for e in range(p.experts):
+        row, k = (idx == e).nonzero(as_tuple=True)
+        if row.numel():
+            g, u = (h[row] @ p.w_gate_up[e].t()).float().chunk(2, -1)
+            out = (g * torch.sigmoid(g) * u).to(h.dtype) @ p.w_down[e].t()
+            y.index_add_(0, row, out.float() * wt[row, k, None])
+    return (y.to(h.dtype),)

@@ -9,8 +9,11 @@ QK-norm + value-embedding gate + cache append, split-key attention) over static 
 position-dependent quantity is read from device memory (`KVCache.cache_seqlens`), so the whole
 step is captured once per (engine, cache) and replayed with a single launch per token.
 
-`decode_graph_for(engine, kv_cache)` returns the `DecodeGraph` of a cache, or None when the
-fast path does not apply (CPU, kernels disabled, more than 64 rows, head dim != 128).
+`StepGraph` is the capture-and-replay shell; `DecodeGraph` is GPT's step, `LatentDecodeGraph` that of models over a
+paged latent store.
+
+`decode_graph_for(engine, kv_cache)` returns the graph of a cache, or None when the
+fast path does not apply (CPU, kernels disabled, more than 64 rows, GPT with a head dim != 128).
 """
 
 import os
@@ -32,22 +35,65 @@ FOLD_MIX_ROWS = int(os.environ.get("NANOCHAT_DECODE_FOLD_ROWS", "2"))
 PREFETCH_NEXT = os.environ.get("NANOCHAT_DECODE_PREFETCH", "1") != "0"
 
 
-class DecodeGraph:
+class StepGraph:
+    """A decode step over static buffers, run eagerly once (kernels get configured outside a capture), captured at the
+    second call and replayed from then on. Subclasses define `_forward` (reads `self.ids`, leaves `self.logits`) and may
+    refresh what it reads in `_prepare`."""
+
     def __init__(self, model, kv_cache):
-        nat = ops.native_module()
-        self.nat, self.C_ = nat, nat._C
         self.model, self.cache = model, kv_cache
-        cfg = model.config
-        dev = kv_cache.cache_seqlens.device
         self.paged = getattr(kv_cache, "paged", False)
         self.pool_version = getattr(kv_cache, "pool_version", 0)
+        self.B = kv_cache.batch_size
+        self.ids = torch.zeros(self.B, 1, dtype=torch.long, device=kv_cache.cache_seqlens.device)
+        self.graph = None
+        self.warm = False
+
+    def begin(self):
+        """Start of a generation: the cache has just been filled by a prompt."""
+
+    def _prepare(self):
+        pass
+
+    @torch.inference_mode()
+    def step(self, ids):
+        """ids: (B, 1) token ids of the new position; returns (B, V) fp32 logits (a static buffer, valid until
+        the next step)."""
+        if self.paged and self.cache.get_pos() >= self.cache.row_capacity():
+            raise ValueError(f"no room for token {self.cache.get_pos()}: the rows' pages hold {self.cache.row_capacity()}")
+        self.ids.copy_(ids)
+        self._prepare()
+        if self.graph is not None:
+            self.graph.replay()
+        elif not self.warm:
+            self._forward()                      # first step runs eagerly: kernels get configured outside capture
+            self.warm = True
+        else:
+            torch.cuda.synchronize()
+            g = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(g):
+                self._forward()
+            self.graph = g
+            g.replay()
+        self.cache._pos += 1
+        return self.logits
+
+
+class DecodeGraph(StepGraph):
+    """GPT's decode step."""
+
+    def __init__(self, model, kv_cache):
+        super().__init__(model, kv_cache)
+        nat = ops.native_module()
+        self.nat, self.C_ = nat, nat._C
+        cfg = model.config
+        dev = kv_cache.cache_seqlens.device
         B, C = kv_cache.batch_size, cfg.n_embd
-        self.B, self.C = B, C
+        self.C = C
         self.H, self.Hkv = cfg.n_head, cfg.n_kv_head
         nq, nkv = self.H * 128, self.Hkv * 128
         bf16 = torch.bfloat16
         e = lambda *shape, dtype=bf16: torch.empty(*shape, dtype=dtype, device=dev)
-        self.ids = torch.zeros(B, 1, dtype=torch.long, device=dev)
         self.prev = torch.zeros(B, C, dtype=bf16, device=dev)
         self.xm, self.xn, self.xa, self.xn2 = e(B, C), e(B, C), e(B, C), e(B, C)
         self.xs = [e(B, C), e(B, C)]                       # residual stream ping-pong
@@ -62,8 +108,6 @@ class DecodeGraph:
         self.use_gemv = B <= GEMV_ROWS     # more rows: the tcgen05 GEMM (rows padded to a 128-row tile) inside the graph
         self.weights_epoch = None
         self.w = None
-        self.graph = None
-        self.warm = False
 
     # ------------------------------------------------------------------ weights
     def _refresh_weights(self):
@@ -175,33 +219,102 @@ class DecodeGraph:
             self.prev.copy_(prev.reshape(self.B, self.C))
         self._refresh_weights()
 
-    @torch.inference_mode()
-    def step(self, ids):
-        """ids: (B, 1) token ids of the new position; returns (B, V) fp32 logits (a static buffer, valid until
-        the next step)."""
-        self.ids.copy_(ids)
+    def _prepare(self):
         if self.weights_epoch != self.nat._weights_epoch or self.w is None:
             self._refresh_weights()
-        if self.graph is not None:
-            self.graph.replay()
-        elif not self.warm:
-            self._forward()                      # first step runs eagerly: kernels get configured outside capture
-            self.warm = True
+
+
+class LatentDecodeGraph(StepGraph):
+    """Decode step of models over a paged latent store (`make_cache`).
+
+    Up to GEMV_ROWS bf16 rows: a fixed chain of serving kernels, 7 per layer with a dense feed-forward and 8 with experts,
+    launched so that each may start while the one before it ends:
+        norm + everything that reads it (down-projections, gates, up-projection, router)  ->  query latent's norm + query
+        projection, extra CTAs append to the store  ->  absorbed queries  ->  attention, split over keys  ->  splits merged
+        + value projection  ->  output projection + gated residual  ->  [experts' gate and up, routing worked out on the
+        spot ->] activation + down projection + gated residual
+    Otherwise (more rows, or float32): the model's forward over the rows, captured as it is."""
+
+    def __init__(self, model, kv_cache):
+        super().__init__(model, kv_cache)
+        S = ops.serving_module()
+        self.S = S
+        cfg, B, dev = model.config, self.B, kv_cache.cache_seqlens.device
+        self.logits = torch.empty(B, model.embed.shape[0], dtype=torch.float32, device=dev)[:, :cfg.vocab_size]
+        self.fused = B <= GEMV_ROWS and model.dtype == torch.bfloat16
+        if not self.fused:
+            return
+        f32 = lambda *shape: torch.empty(*shape, dtype=torch.float32, device=dev)
+        b16 = lambda *shape: torch.empty(*shape, dtype=torch.bfloat16, device=dev)
+        self.x, self.h = f32(B, model.width), b16(B, model.width)
+        self.x0 = f32(B, model.width) if model.keep_x0 else None
+        self.all_logits = f32(B, model.embed.shape[0])
+        self.logits = self.all_logits[:, :cfg.vocab_size]
+        layers = [layer for layer, _ in model.runs]
+        most = lambda size: max((size(layer) for layer in layers), default=8)
+        self.z = f32(B * most(lambda l: l.w_all.shape[0]))
+        self.q = b16(B * most(lambda l: l.attn.w_q.shape[0]))
+        self.qa = b16(B * most(lambda l: l.attn.heads * l.attn.kvp))
+        self.y = b16(B * most(lambda l: l.attn.heads * l.attn.vp))
+        self.act = b16(B * most(lambda l: l.mlp.top * l.mlp.fp if hasattr(l.mlp, "top") else 8))
+        self.splits = [S.attention_splits(l.attn, B, min(kv_cache.max_seq_len, l.attn.window or kv_cache.max_seq_len), True)
+                       for l in layers]
+        self.ml = f32(max([B * l.attn.heads * s * 2 for l, s in zip(layers, self.splits)] + [2]))
+        self.acc = f32(max([B * l.attn.heads * s * l.attn.kvp for l, s in zip(layers, self.splits)] + [8]))
+
+    def _forward(self):
+        if self.fused:
+            self._fused_step()
+            self.cache.cache_seqlens.add_(1)
         else:
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                self._forward()
-            self.graph = g
-            g.replay()
-        self.cache._pos += 1
-        return self.logits
+            pos = self.cache._pos
+            self.logits.copy_(self.model.forward(self.ids, kv_cache=self.cache)[:, 0])
+            self.cache._pos = pos                # step() moves the host's mirror, replayed or not
+
+    def _fused_step(self):
+        m, K, B, cache, cfg = self.model, self.S._S, self.B, self.cache, self.model.config
+        C, eps, mult = cfg.n_embd, cfg.eps, cfg.residual_mult
+        table, lens, x = cache.table, cache.cache_seqlens, self.x
+        ahead = lambda w: w if PREFETCH_NEXT else None
+        view = lambda buf, n: buf[:B * n].view(B, n)
+        K.embed_norm(self.ids, m.embed, cfg.vocab_size, m.final_norm, eps, C, x, self.x0, None)
+        for run, (layer, _) in enumerate(m.runs):
+            a, mlp = layer.attn, layer.mlp
+            again = run + 1 < len(m.runs) and m.runs[run + 1][1]
+            extra = self.x0 if again else None
+            moe = hasattr(mlp, "top")
+            z = view(self.z, layer.w_all.shape[0])
+            q, qa, y = view(self.q, a.w_q.shape[0]), view(self.qa, a.heads * a.kvp), view(self.y, a.heads * a.vp)
+            K.gemv_norm(x, layer.norm, eps, C, layer.w_all, z, self.h if moe else None, ahead(a.w_q))
+            K.gemv_query_store(z, a.q_rank, a.q_norm, eps, a.w_q, q, a.c_off, a.kv_rank, a.kvp, a.kv_norm, a.rot_off,
+                               a.rot_dim, a.freq, cache.pools[run], table, lens, ahead(a.w_kv))
+            K.absorb_query(q, a.heads, a.w_uk, qa, True)
+            splits = self.splits[run]
+            K.latent_attention(qa, q, a.heads, a.dp, a.rot_dim, a.freq, a.kvp, cache.pools[run], table, lens, 1,
+                               a.window or 0, a.scale, splits, self.ml, self.acc, True)
+            K.latent_values(self.ml, self.acc, B, a.heads, splits, a.w_uv, y, True, ahead(a.w_o))
+            gate = lambda k: z[:, layer.gates[k]:layer.gates[k] + m.width]
+            K.gemv_residual(y, None, eps, 0, a.w_o, x, gate(0), layer.rg1_bias, mult, None if mlp is not None else extra,
+                            ahead(mlp.w_down if mlp is not None and not moe else None))
+            if moe:
+                act = self.act[:B * mlp.top * mlp.fp].view(B * mlp.top, mlp.fp)
+                logits = z[:, layer.n_in:]
+                K.expert_gate_up(self.h, mlp.w_gate_up, mlp.top, None, None, logits, act, True)
+                K.expert_down_residual(act, mlp.w_down, mlp.top, logits, x, gate(1), layer.rg2_bias, mult, extra)
+            elif mlp is not None:
+                K.gemv_residual(z[:, layer.up_off:layer.n_in], mlp.act, eps, mlp.ff, mlp.w_down, x, gate(1), layer.rg2_bias,
+                                mult, extra)
+        K.gemv_norm(x, m.final_norm, eps, C, m.embed, self.all_logits)
 
 
 def graph_path_applies(model, rows):
     """True when `rows` sample rows of this model decode through the captured-graph kernels."""
+    if ops.get_kernel_mode() != "native":
+        return False
+    if hasattr(model, "make_cache"):
+        return model.get_device().type == "cuda" and rows <= MAX_ROWS
     from nanochat_b200.models.gpt import GPT
-    if not isinstance(model, GPT) or ops.get_kernel_mode() != "native":
+    if not isinstance(model, GPT):
         return False
     cfg = model.config
     wte = model.transformer.wte.weight
@@ -218,6 +331,7 @@ def decode_graph_for(engine, kv_cache):
     graphs = engine._decode_graphs
     g = graphs.get(id(kv_cache))
     if g is None or g.cache is not kv_cache or g.pool_version != getattr(kv_cache, "pool_version", 0):
-        g = DecodeGraph(model, kv_cache)       # first use, or the page pool moved: capture on the new addresses
+        kind = LatentDecodeGraph if hasattr(model, "make_cache") else DecodeGraph
+        g = kind(model, kv_cache)              # first use, or the page pool moved: capture on the new addresses
         graphs[id(kv_cache)] = g
     return g

@@ -2,6 +2,9 @@
 In-tree build of the native extensions with explicit compiler commands.
 
   nanochat_b200/_C*.so    CUDA kernels (nvcc, sm_100a only) + torch bindings
+  nanochat_b200/_S*.so    the serving kernels (latent attention, experts, decode steps) with the forward GEMM and
+                          attention: what inference of those models needs, built on its own so that a first call
+                          does not wait for the training kernels
   nanochat_b200/_tok*.so  C++ tokenizer (BPE trainer / encoder) + best-fit packer
 
 The shared objects are written next to the package so they are found wherever the
@@ -23,6 +26,7 @@ from concurrent.futures import ThreadPoolExecutor
 
 PKG_DIR = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CSRC = os.path.join(PKG_DIR, "ops", "csrc")
+SERVE_CSRC = os.path.join(CSRC, "serve")
 TOK_SRC = os.path.join(PKG_DIR, "csrc", "tokenizer")
 BUILD_DIR = os.path.join(PKG_DIR, "_build")
 EXT_SUFFIX = sysconfig.get_config_var("EXT_SUFFIX") or ".so"
@@ -84,7 +88,8 @@ def _write_stamp(so_path, digest):
 
 # Optimizer and collective kernels keep IEEE division / square root and denormals: their state (second moments,
 # running norms) lives for the whole run, and approximate math there shows up as drift, not as noise.
-PRECISE_SOURCES = ("optim.cu", "comm.cu")
+# The serving kernels also run in float, where angles, exponentials and statistics are held to float accuracy.
+PRECISE_SOURCES = ("optim.cu", "comm.cu", "rows.cu", "latent.cu", "experts.cu")
 
 
 def _load(name, so_path):
@@ -101,14 +106,26 @@ def cuda_sources():
     return sorted(glob.glob(os.path.join(CSRC, "*.cu"))), sorted(glob.glob(os.path.join(CSRC, "*.cpp")))
 
 
+def serving_sources():
+    shared = [os.path.join(CSRC, f) for f in ("attention.cu", "gemm.cu")]
+    return (sorted(glob.glob(os.path.join(SERVE_CSRC, "*.cu"))) + shared, sorted(glob.glob(os.path.join(SERVE_CSRC, "*.cpp"))))
+
+
 def build_cuda_extension(verbose=False, force=False):
     """Compile every .cu for sm_100a and link `_C`. Returns the path of the shared object."""
+    return _build_cuda("_C", *cuda_sources(), [], verbose, force)
+
+
+def build_serving_extension(verbose=False, force=False):
+    """The serving library `_S`: its own kernels plus the forward GEMM and attention (compiled with NC_SERVING)."""
+    return _build_cuda("_S", *serving_sources(), ["-DNC_SERVING"], verbose, force)
+
+
+def _build_cuda(name, cus, cpps, defines, verbose, force):
     import torch
-    name = "_C"
     so_path = os.path.join(PKG_DIR, name + EXT_SUFFIX)
-    cus, cpps = cuda_sources()
-    headers = glob.glob(os.path.join(CSRC, "*.h")) + glob.glob(os.path.join(CSRC, "*.cuh"))
-    extra_flags = os.environ.get("NANOCHAT_NVCC_FLAGS", "").split()     # e.g. -DNC_ATTN_TRACE for kernel timelines
+    headers = [h for d in {os.path.dirname(s) for s in cus} | {CSRC} for e in ("*.h", "*.cuh") for h in glob.glob(os.path.join(d, e))]
+    extra_flags = defines + os.environ.get("NANOCHAT_NVCC_FLAGS", "").split()     # e.g. -DNC_ATTN_TRACE for kernel timelines
     digest = _hash_files(cus + cpps + headers, extra=torch.__version__ + " ".join(extra_flags) + " precise:" + ",".join(PRECISE_SOURCES))
     if not force and not _stale(so_path, digest):
         return so_path
@@ -131,14 +148,15 @@ def _build_cuda_locked(name, so_path, cus, cpps, extra_flags, digest, verbose):
     nvcc = _nvcc()
     jobs = []
     for src in cus:
-        obj = os.path.join(BUILD_DIR, os.path.basename(src) + ".o")
+        obj = os.path.join(BUILD_DIR, name + "." + os.path.basename(src) + ".o")
         fast = [] if os.path.basename(src) in PRECISE_SOURCES else ["--use_fast_math"]
-        cmd = [nvcc, *NVCC_ARCH, "-lineinfo", "-O3", "-std=c++17", *fast, "-Xcompiler", "-fPIC",
+        # -fno-gnu-unique: statics of templates stay private to each library (both hold instances of the same kernels)
+        cmd = [nvcc, *NVCC_ARCH, "-lineinfo", "-O3", "-std=c++17", *fast, "-Xcompiler", "-fPIC,-fno-gnu-unique",
                "-Xptxas", "-v" if verbose else "-O3", *extra_flags, "-I", CSRC, "-c", src, "-o", obj]
         jobs.append((cmd, obj))
     for src in cpps:
-        obj = os.path.join(BUILD_DIR, os.path.basename(src) + ".o")
-        cmd = ["g++", "-O2", "-std=c++17", "-fPIC", *common_defs, *incs, "-c", src, "-o", obj]
+        obj = os.path.join(BUILD_DIR, name + "." + os.path.basename(src) + ".o")
+        cmd = ["g++", "-O2", "-std=c++17", "-fPIC", "-fno-gnu-unique", *common_defs, *incs, "-c", src, "-o", obj]
         jobs.append((cmd, obj))
     with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as pool:
         logs = list(pool.map(lambda j: _run(j[0]), jobs))
@@ -159,6 +177,16 @@ def _build_cuda_locked(name, so_path, cus, cpps, extra_flags, digest, verbose):
 
 
 _cuda_ext = None
+_serving_ext = None
+
+
+def load_serving_extension():
+    """Import `_S`, building it first if it is missing or out of date."""
+    global _serving_ext
+    if _serving_ext is None:
+        import torch  # noqa: F401
+        _serving_ext = _load("nanochat_b200._S", build_serving_extension())
+    return _serving_ext
 
 
 def load_cuda_extension():
@@ -226,7 +254,7 @@ def sanitizer_runtime_libs():
 
 
 def build_all(verbose=False, force=False):
-    out = [build_cuda_extension(verbose=verbose, force=force)]
+    out = [build_cuda_extension(verbose=verbose, force=force), build_serving_extension(verbose=verbose, force=force)]
     try:
         out.append(build_tokenizer_extension(force=force))
     except FileNotFoundError:
