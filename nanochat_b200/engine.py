@@ -434,8 +434,7 @@ class Engine:
     def _prompt_logits(self, ids, cache, want):
         """Run a portion of tokens; (len(want), V) logits at the places `want`, None when there are none."""
         if self.latent:
-            logits = self.model.forward(ids, kv_cache=cache, want=list(want))
-            return logits if len(want) else None
+            return self.model.forward(ids, kv_cache=cache, want=list(want))
         logits = self.model.forward(ids, kv_cache=cache)[0]
         return logits[list(want)].float() if len(want) else None
 

@@ -357,7 +357,7 @@ class Lupodra(nn.Module, NaiveSampler):
     # ------------------------------------------------------------------------- forward
     @torch.inference_mode()
     def forward(self, idx, targets=None, kv_cache=None, want=None, residuals=None):
-        """Logits (B, T, vocab), or (len(want), vocab) for `want`ed rows of the flattened (B * T). The tokens continue
+        """Logits (B, T, vocab), or (len(want), vocab) for the `want`ed rows of the flattened (B * T), None for none. The tokens continue
         what `kv_cache` holds and are appended to it. `residuals`, a list, collects the stream after every layer run."""
         if targets is not None:
             raise NotImplementedError("Lupodra is served, not trained: no loss")
@@ -383,6 +383,8 @@ class Lupodra(nn.Module, NaiveSampler):
                 residuals.append((x if extra is None else x - extra)[:, :C].clone())
         kv_cache.advance(T)
         if want is not None:
+            if len(want) == 0:
+                return None
             h = h[torch.as_tensor(want, dtype=torch.long, device=h.device)]
         logits = ops.linear_rows(h, self.embed, torch.float32)[:, :cfg.vocab_size]
         return logits if want is not None else logits.reshape(B, T, -1)
