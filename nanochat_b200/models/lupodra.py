@@ -143,7 +143,9 @@ def _up(n, m=8):
 
 def _fit(w, *shape):
     """w at the origin of a zero tensor of `shape`."""
-    out = torch.zeros(shape, dtype=w.dtype)
+    if tuple(w.shape) == shape:
+        return w
+    out = w.new_zeros(shape)
     out[tuple(slice(0, s) for s in w.shape)] = w
     return out
 
@@ -289,7 +291,7 @@ class Lupodra(nn.Module, NaiveSampler):
     # ------------------------------------------------------------------------- weights
     @torch.no_grad()
     def load_tensors(self, tensors, device):
-        """Take the named tensors (CPU, any float type) into the layouts of the kernels."""
+        """Take the named tensors (any float type) into the layouts of the kernels."""
         C, left = self.config.n_embd, set(tensors)
 
         def take(name, *shape):
@@ -332,15 +334,15 @@ class Lupodra(nn.Module, NaiveSampler):
 
     def init_weights(self, device, seed=0):
         """Random weights of a plausible scale (benchmarks, demonstrations)."""
-        g = torch.Generator().manual_seed(seed)
+        g = torch.Generator(device=device).manual_seed(seed)
         tensors = {}
         for name, shape in self.tensor_shapes().items():
             if len(shape) == 2:
-                t = torch.randn(shape, generator=g) * (1.0 if name == "embed" else shape[1] ** -0.5)
+                t = torch.randn(shape, generator=g, device=device) * (1.0 if name == "embed" else shape[1] ** -0.5)
             else:
-                t = torch.ones(shape) if name.endswith((".dq.norm", ".dkv.norm")) else torch.zeros(shape)
+                t = (torch.ones if name.endswith((".dq.norm", ".dkv.norm")) else torch.zeros)(shape, device=device)
                 if name.endswith(".act"):
-                    t = torch.tensor([0.7, 0.3, 0.1, 0.0])
+                    t = torch.tensor([0.7, 0.3, 0.1, 0.0], device=device)
             tensors[name] = t.to(torch.bfloat16)
         return self.load_tensors(tensors, device)
 

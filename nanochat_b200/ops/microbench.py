@@ -5,6 +5,7 @@ Micro-benchmarks of the hand-written kernels, one operation per invocation:
     python -m nanochat_b200.ops.microbench attn_fwd --batch 16 --seq 2048 --heads 13 --window -1
     python -m nanochat_b200.ops.microbench attn_bwd --batch 2 --iters 1 --warmup 1      # small: profiler runs
     python -m nanochat_b200.ops.microbench sweep --m 32768     # the memory-bound kernels against their algorithmic bytes
+    python -m nanochat_b200.ops.microbench serve               # serving kernels beside the like kernels of GPT
 
 Timing follows the usual hygiene: warm-up launches, a write larger than L2 between timed launches,
 CUDA events on the launching stream, median of the timed launches. Prints one JSON line with the
@@ -227,9 +228,153 @@ def bench_sweep(args, nat):
     return dict(op="sweep", rows_m=M, kernels=rows, measured_hbm_gbs=peak)
 
 
+def _time_chain(calls, iters=10):
+    """Microseconds per call of a captured chain of calls (their launch cost is the graph's, as in a decode step)."""
+    for c in calls:
+        c()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for c in calls:
+            c()
+    return 1e3 * _time(g.replay, iters, 3) / len(calls)
+
+
+def bench_serve(T=2048, C=1664, window=512, ctx=1024):
+    """Every kernel of the latent-attention model at the d26 width beside the like kernel of GPT: time, roofline (the
+    slower of its FLOPs at the measured GEMM rate and its bytes at the measured copy rate) and the ratio of the two
+    distances. Prompt kernels: T tokens. Decode kernels: chains over several layers' weights (more than L2)."""
+    from nanochat_b200.ops import native as nat
+    from nanochat_b200.ops import serving as sv
+    K, N = sv._S, nat._C
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    if os.path.exists("MEASURED_PEAKS.json"):
+        with open("MEASURED_PEAKS.json") as f:
+            peaks.update({k: v for k, v in json.load(f).items() if k in peaks})
+    dev, bf16, f32 = "cuda", torch.bfloat16, torch.float32
+    r = lambda *s, dtype=bf16: torch.randn(*s, device=dev).to(dtype)
+    e = lambda *s, dtype=bf16: torch.empty(*s, device=dev, dtype=dtype)
+    H, D, D2, DV, KV = C // 128, 128, 64, 128, 512
+    E, TOP, FF = 16, 4, C
+    rows, base = [], {}
+
+    def add(name, us, flops=0.0, nbytes=0.0, like=None, key=None):
+        roof = max(flops / peaks["bf16_tflops"] / 1e6, nbytes / peaks["hbm_gbs"] / 1e3)
+        row = {"kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "distance": round(us / roof, 2)}
+        if like is not None:
+            row["like"] = like
+            row["relative_distance"] = round(us / roof / base[like], 2)
+        if key is not None:
+            base[key] = us / roof
+        rows.append(row)
+
+    us = lambda fn: 1e3 * _time(fn, 10, 3)
+    # ------------------------------------------------------------------ prompts
+    x, w, y = r(T, C), r(4 * C, C), e(T, 4 * C)
+    add("gpt gemm (MLP up)", us(lambda: nat.gemm(x, w, y)), 2.0 * T * C * 4 * C, key="gemm")
+    n_in = 1280 + 576 + 2 * C + 4 * C
+    w_in, z = r(n_in, C), e(T, n_in)
+    add("gemm (fused input projection)", us(lambda: K.gemm(x, w_in, z)), 2.0 * T * C * n_in, like="gemm")
+    idx, wt = torch.empty(T, TOP, dtype=torch.int32, device=dev), e(T, TOP, dtype=f32)
+    rank, slot, off = torch.empty_like(idx), torch.empty_like(idx), torch.empty(E, dtype=torch.int32, device=dev)
+    counts, logits = torch.zeros(E, dtype=torch.int32, device=dev), r(T, E, dtype=f32)
+    tiles = -(-(T * TOP + E * 127) // 128)
+    tg = torch.empty(tiles, dtype=torch.int32, device=dev)
+    xg, wgu, gu, act, wd, yg = e(tiles * 128, C), r(E, 2 * FF, C), e(tiles * 128, 2 * FF), e(tiles * 128, FF), r(E, C, FF), e(tiles * 128, C)
+
+    def regroup():
+        counts.zero_()
+        K.route_topk(logits, E, idx, wt, counts, rank)
+        K.group_rows(x, idx, rank, counts, off, tg, slot, xg)
+    regroup()
+    add("grouped gemm (experts' gate and up)", us(lambda: K.gemm(xg, wgu, gu, tg)), 2.0 * T * TOP * C * 2 * FF, like="gemm")
+    add("grouped gemm (experts' down)", us(lambda: K.gemm(act, wd, yg, tg)), 2.0 * T * TOP * C * FF, like="gemm")
+    for win, tag in ((-1, "all keys"), (window, f"window {window}")):
+        q, k, v, o = (r(1, T, H, 128) for _ in range(4))
+        lse = e(1, H, T, dtype=f32)
+        pairs = _attn_pairs(T, win)
+        add(f"gpt attention, {tag}", us(lambda: N.attn_fwd(q, k, v, o, lse, win, 0.088)), 4.0 * H * 128 * pairs, key=f"attn{win}")
+        q4, k3, k2, v3, o3 = r(T, H, D + D2), r(T, H, D), r(T, D2), r(T, H, DV), e(T, H, DV)
+        add(f"split attention, {tag}", us(lambda: K.attention_split(q4[..., :D], q4[..., D:], k3, k2, v3, o3, win, 0.07)),
+            2.0 * H * (D + D2 + DV) * pairs, like=f"attn{win}")
+    xr, lam = r(T, C), torch.ones(1, device=dev)
+    xm, xn = e(T, C), e(T, C)
+    add("gpt mix + norm", us(lambda: N.mixnorm_fwd(xr, x, lam, lam, 0, xm, xn, None)), nbytes=2.0 * T * C * 4, key="rows")
+    xf, bias, wn = r(T, C, dtype=f32), r(C, dtype=f32), r(C, dtype=f32)
+    g1, g2, y1, h = z[:, :C], z[:, C:2 * C], r(T, C), e(T, C)
+    add("gated residual + norm, dense", us(lambda: K.gated_residual_norm(xf, [[g1, bias, y1], [g2, bias, y1]], 0.7, None, wn, 1e-6, C, h)),
+        nbytes=T * C * (8 + 2 * 4 + 2.0), like="rows")
+    add("gated residual + norm, experts", us(lambda: K.gated_residual_norm(xf, [[g1, bias, y1], [g2, bias, yg, slot, wt]], 0.7, None, wn, 1e-6, C, h)),
+        nbytes=T * C * (8 + 2 * 3 + 2.0 * TOP + 2.0), like="rows")
+    coef, zu, au = torch.tensor([0.7, 0.3, 0.1, 0.0], device=dev), z[:, :4 * C], e(T, 4 * C)
+    add("normed-powers activation", us(lambda: K.poly_norm(zu, coef, 1e-6, 4 * C, au)), nbytes=2.0 * T * 4 * C * 2, like="rows")
+    add("gather rows by expert", us(lambda: K.group_rows(x, idx, rank, counts, off, tg, slot, xg)), nbytes=2.0 * (1 + TOP) * T * C, like="rows")
+    add("silu * up", us(lambda: K.silu_mul(gu, tg, act)), nbytes=2.0 * T * TOP * FF * 3, like="rows")
+    P = 64
+    pages = -(-(T + 1) // P)
+    pool = torch.zeros(pages, P, KV + D2, dtype=bf16, device=dev)
+    table = torch.arange(pages, dtype=torch.int32, device=dev)[None].contiguous()
+    lens, freq = torch.zeros(1, dtype=torch.int32, device=dev), 10000.0 ** (-torch.arange(D2 // 2, device=dev, dtype=f32) * 2 / D2)
+    qkv, cs = r(1, T, 3 * H * 128), e(1, T, 64)
+    qw, kw, cq, kv = r(1280, dtype=f32), r(KV, dtype=f32), e(T, 1280), e(T, KV + D2)
+    cs.fill_(0.7)
+    rstd = e(T, 2 * H, dtype=f32)
+    add("gpt rotary + QK norm", us(lambda: N.qkv_post_fwd(qkv, H, H, cs.view(T, 64), cs.view(T, 64), T, rstd, None, None, None, None)),
+        nbytes=2.0 * T * 2 * H * 128 * 2, key="post")
+    add("latent norms + store", us(lambda: K.latent_post(z, 1280, qw, cq, 1280, KV, KV, kw, 1e-6, 1280 + KV, D2, freq, pool, table, lens, T, kv)),
+        nbytes=2.0 * T * (2 * 1280 + 3 * (KV + D2)), like="post")
+    q5 = r(T, H * (D + D2))
+    add("rotate query heads", us(lambda: K.rotate_heads(q5, H, D, freq, table, lens, T)), nbytes=4.0 * T * H * D2, like="post")
+    # ------------------------------------------------------------------- decode
+    L = 12                                          # chain length: weights of several layers, more than L2 holds
+    for B in (1, 8):
+        lens = torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
+        xb, wq, ob = r(B, C), [r(3 * C, C) for _ in range(L)], e(B, 3 * C)
+        add(f"gpt gemv (QKV), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, ob, None, 0, True, None) for a in wq]), nbytes=2.0 * 3 * C * C, key=f"gemv{B}")
+        n_all = n_in
+        wa, zb, xf = [r(n_all, C) for _ in range(L)], e(B, n_all, dtype=f32), r(B, C, dtype=f32)
+        add(f"norm + input projection, {B} rows", _time_chain([lambda a=a: K.gemv_norm(xf, wn, 1e-6, C, a, zb) for a in wa]), nbytes=2.0 * n_all * C, like=f"gemv{B}")
+        zb.normal_()
+        pg = -(-ctx // P)
+        pools = [torch.randn(B * pg, P, KV + D2, device=dev).to(bf16) for _ in range(L)]
+        table = torch.arange(B * pg, dtype=torch.int32, device=dev).view(B, pg).contiguous()
+        wqs, qb = [r(H * (D + D2), 1280) for _ in range(L)], e(B, H * (D + D2))
+        add(f"query projection + store, {B} rows", _time_chain([lambda a=a, p=p: K.gemv_query_store(zb, 1280, qw, 1e-6, a, qb, 1280, KV, KV, kw, 1280 + KV, D2, freq, p, table, lens)
+                                                                 for a, p in zip(wqs, pools)]), nbytes=2.0 * 1280 * H * (D + D2), like=f"gemv{B}")
+        wkv, qa, yb = [r(H * (D + DV), KV) for _ in range(L)], e(B, H, KV), e(B, H * DV)
+        add(f"absorb queries, {B} rows", _time_chain([lambda a=a: K.absorb_query(qb, H, a[:H * D], qa, True) for a in wkv]), nbytes=2.0 * H * D * KV, like=f"gemv{B}")
+        k4 = [torch.randn(B * pg, P, H, 128, device=dev).to(bf16) for _ in range(L)]
+        scratch, yg4, qg = torch.zeros(N.decode_attn_scratch(B, H), device=dev), e(B, H * 128), r(B, H * 128)
+        add(f"gpt decode attention, {window} keys, {B} rows", _time_chain([lambda a=a: N.decode_attn(qg, a, a, lens, H, H, window - 1, 0.088, scratch, yg4, table) for a in k4]),
+            nbytes=2.0 * B * window * H * 256, flops=4.0 * B * window * H * 128, key=f"dattn{B}")
+
+        class P_:                                   # what attention_splits asks for
+            heads, window = H, None
+        splits = sv.attention_splits(P_, B, window, True)
+        ml, acc = e(B, H, splits, 2, dtype=f32), e(B, H, splits, KV, dtype=f32)
+        add(f"latent attention, {window} keys, {B} rows", _time_chain([lambda p=p: K.latent_attention(qa, qb, H, D, D2, freq, KV, p, table, lens, 1, window, 0.07, splits, ml, acc, True) for p in pools]),
+            nbytes=2.0 * B * window * (KV + D2), flops=2.0 * B * window * H * (2 * KV + D2), like=f"dattn{B}")
+        add(f"merge splits + values, {B} rows", _time_chain([lambda a=a: K.latent_values(ml, acc, B, H, splits, a[H * D:], yb, True) for a in wkv]), nbytes=2.0 * H * DV * KV, like=f"gemv{B}")
+        wo, gb = [r(C, H * DV) for _ in range(L)], zb[:, :C]
+        wp, op, aux = [r(C, C) for _ in range(L)], e(B, C), r(B, C)
+        add(f"gpt gemv (attention out), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, op, aux, 0, False, None) for a in wp]), nbytes=2.0 * C * C, key=f"gemvo{B}")
+        add(f"output projection + gated residual, {B} rows", _time_chain([lambda a=a: K.gemv_residual(yb, None, 1e-6, 0, a, xf, gb, bias, 0.7) for a in wo]), nbytes=2.0 * C * H * DV, like=f"gemvo{B}")
+        wdn, zz = [r(C, 4 * C) for _ in range(L)], zb[:, :4 * C]
+        hb = r(B, 4 * C)
+        add(f"gpt gemv (MLP down), {B} rows", _time_chain([lambda a=a: N.gemv_rows(hb, a, op, aux, 0, False, None) for a in wdn]), nbytes=2.0 * 4 * C * C, key=f"gemvd{B}")
+        add(f"activation + down + gated residual, {B} rows", _time_chain([lambda a=a: K.gemv_residual(zz, coef, 1e-6, 4 * C, a, xf, gb, bias, 0.7) for a in wdn]), nbytes=2.0 * 4 * C * C, like=f"gemvd{B}")
+        lbs, hb, ab = [r(B, E, dtype=f32) for _ in range(L)], r(B, C), e(B * TOP, FF)       # other experts in every call
+        used = min(B * TOP, E * (1 - (1 - TOP / E) ** B))      # experts a step reads, on average
+        add(f"experts' gate and up, {B} rows", _time_chain([lambda l=l: K.expert_gate_up(hb, wgu, TOP, None, None, l, ab, True) for l in lbs]), nbytes=2.0 * used * 2 * FF * C, like=f"gemvd{B}")
+        add(f"experts' down + gated residual, {B} rows", _time_chain([lambda l=l: K.expert_down_residual(ab, wd, TOP, l, xf, gb, bias, 0.7) for l in lbs]), nbytes=2.0 * used * FF * C, like=f"gemvd{B}")
+    sv.check_status()
+    nat.check_status()
+    return rows
+
+
 def main():
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("op", choices=["gemm", "attn_fwd", "attn_bwd", "sweep"])
+    ap.add_argument("op", choices=["gemm", "attn_fwd", "attn_bwd", "sweep", "serve"])
     ap.add_argument("--m", type=int, default=32768)
     ap.add_argument("--n", type=int, default=4992)
     ap.add_argument("--k", type=int, default=1664)
@@ -248,6 +393,10 @@ def main():
     args = ap.parse_args()
     from nanochat_b200.ops import native as nat
     torch.manual_seed(0)
+    if args.op == "serve":
+        for row in bench_serve():
+            print(json.dumps(row))
+        return
     res = {"gemm": bench_gemm, "attn_fwd": bench_attn_fwd, "attn_bwd": bench_attn_bwd, "sweep": bench_sweep}[args.op](args, nat)
     nat.check_status()
     if os.path.exists("MEASURED_PEAKS.json"):

@@ -3,6 +3,7 @@ Inference benchmark: time to first token, time per output token, tokens/sec, mem
 and compute utilisation over a sweep of decode batch sizes, through `Engine.generate`.
 
     python -m scripts.infer_bench -i base --batch-sizes 1,8,32,64
+    python -m scripts.infer_bench --model-dir DIR --batch-sizes 1,8       # config.json + model.safetensors
     python -m scripts.infer_bench --random-init --depth 26 --prompt-tokens 512 --decode-tokens 256 \
         --batch-sizes 1,8,32,64 -t 1.0 -k 50          # no checkpoint needed
 
@@ -26,6 +27,8 @@ from nanochat_b200.engine import Engine
 def weight_bytes(model):
     """Bytes a decode step has to read for the parameters, as they are consumed (bf16 shadows of the
     fp32 masters on the native path, the stored dtype otherwise)."""
+    if hasattr(model, "decode_weight_bytes"):
+        return model.decode_weight_bytes()
     if hasattr(model, "transformer") and next(model.parameters()).is_cuda:
         # bf16 operand copies of the block matrices and lm_head; embedding tables are only touched by row
         dense = list(model.transformer.h.parameters()) + [model.lm_head.weight]
@@ -155,6 +158,7 @@ def main():
     ap.add_argument("--batch-sizes", type=str, default="1,8,32,128")
     ap.add_argument("-t", "--temperature", type=float, default=0.0)
     ap.add_argument("-k", "--top-k", type=int, default=None)
+    ap.add_argument("--model-dir", type=str, default=None, help="model folder (any registered architecture) instead of a checkpoint")
     ap.add_argument("--random-init", action="store_true", help="random weights of --depth instead of a checkpoint")
     ap.add_argument("--depth", type=int, default=26)
     args = ap.parse_args()
@@ -180,6 +184,11 @@ def main():
         meta = {"step": 0, "model_config": vars(cfg).copy()}
         g = torch.Generator().manual_seed(0)
         prompt_source = lambda n: torch.randint(0, cfg.vocab_size - 9, (n,), generator=g).tolist()
+    elif args.model_dir is not None:
+        from nanochat_b200.checkpoint_manager import load_model_folder
+        model, tokenizer, meta = load_model_folder(args.model_dir, device)
+        g = torch.Generator().manual_seed(0)
+        prompt_source = lambda n: torch.randint(0, model.config.vocab_size, (n,), generator=g).tolist()
     else:
         from nanochat_b200.checkpoint_manager import load_model
         model, tokenizer, meta = load_model(args.source, device, phase="eval", model_tag=args.model_tag,
@@ -203,13 +212,13 @@ def main():
     ceiling = peak_bw / (w_bytes + kv_read)
     max_rows = int((vram - w_bytes) / (kv_store * cfg.sequence_len))
     print("=" * 100)
-    print(f"Model: {args.source} (step {meta['step']}) | depth {cfg.n_layer}, dim {cfg.n_embd}, heads {cfg.n_head}, "
-          f"kv heads {cfg.n_kv_head}")
+    heads = f", heads {cfg.n_head}, kv heads {cfg.n_kv_head}" if hasattr(cfg, "n_head") else ""
+    print(f"Model: {args.model_dir or args.source} (step {meta['step']}) | depth {cfg.n_layer}, dim {cfg.n_embd}{heads}")
     print(f"GPU: {name} | peak bandwidth {peak_bw/1e12:.2f} TB/s | peak compute {peak_flops/1e12:.0f} TFLOPS | "
           f"VRAM {vram/2**30:.0f} GiB")
     print(f"Parameters: {n_params:,} | weight bytes as stored: {w_bytes/2**20:.0f} MiB")
     print(f"KV cache: {kv_store:,} bytes/token stored | {kv_read:,} bytes read/step at context {ctx_mid} "
-          f"(window pattern {cfg.window_pattern})")
+          f"(window pattern {getattr(cfg, 'window_pattern', 'per layer')})")
     print(f"Theoretical decode ceiling at batch 1: {ceiling:,.0f} tok/s | max ~{max_rows:,} full-context rows in VRAM")
     print("=" * 100)
     finite = lambda v: v if v != float("inf") else None
