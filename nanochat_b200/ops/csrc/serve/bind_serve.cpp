@@ -162,11 +162,12 @@ void gated_residual_norm_(Tensor& x, const std::vector<std::vector<Tensor>>& ter
 }
 
 void poly_norm_(const Tensor& z, const Tensor& coef, double eps, int64_t n, Tensor& out) {
-  check_rows(z, "z"); check_rows(out, "out"); same_type(z, out, "out");
+  check_rows(z, "z"); check_rows(out, "out");
+  TORCH_CHECK(is_f32(z) || !is_f32(out), "poly_norm: float output needs float input");
   TORCH_CHECK(coef.is_cuda() && is_f32(coef) && coef.is_contiguous() && coef.numel() == 4, "poly_norm: four float coefficients");
   TORCH_CHECK(z.sizes() == out.sizes() && n <= z.size(1), "poly_norm shapes");
   const c10::cuda::CUDAGuard guard(z.device());
-  NC_CHECK(poly_norm(is_f32(z), z.data_ptr(), pitch(z), coef.data_ptr<float>(), (float)eps, (int)z.size(0), (int)n, (int)z.size(1),
+  NC_CHECK(poly_norm(is_f32(out), is_f32(z), z.data_ptr(), pitch(z), coef.data_ptr<float>(), (float)eps, (int)z.size(0), (int)n, (int)z.size(1),
                      out.data_ptr(), pitch(out), stream()));
 }
 
@@ -181,8 +182,8 @@ void latent_post_(const Tensor& z, int64_t q_rank, const optional<Tensor>& q_w, 
   d.f32 = is_f32(pool); d.z_f32 = is_f32(z);
   d.z = z.data_ptr(); d.ldz = pitch(z); d.rows = (int)z.size(0);
   if (has(cq)) {
-    check_rows(*cq, "cq"); same_type(*cq, pool, "cq"); check_vec(*q_w, q_rank, "q_w");
-    TORCH_CHECK(cq->size(0) == z.size(0) && q_rank <= cq->size(1) && q_rank <= z.size(1), "cq shape");
+    check_rows(*cq, "cq"); same_type(*cq, pool, "cq"); check_vec(*q_w, cq->size(1), "q_w");
+    TORCH_CHECK(cq->size(0) == z.size(0) && q_rank <= cq->size(1) && cq->size(1) <= z.size(1), "cq shape");
     d.q_rank = (int)q_rank; d.qp = (int)cq->size(1); d.q_w = q_w->data_ptr<float>(); d.cq = cq->data_ptr(); d.ldcq = pitch(*cq);
   }
   check_latent(z, c_off, kv_rank); check_latent(z, rot_off, rot_dim);
@@ -291,45 +292,28 @@ void silu_mul_(const Tensor& gu, const Tensor& tile_group, Tensor& act) {
   NC_CHECK(silu_mul(gu.data_ptr(), (int)gu.size(0), (int)act.size(1), tile_group.data_ptr<int>(), act.data_ptr(), stream()));
 }
 
-Routing routing_of(const optional<Tensor>& idx, const optional<Tensor>& wt, const optional<Tensor>& logits, int64_t rows, int64_t experts, int64_t top) {
-  Routing r{};
-  r.experts = (int)experts; r.top = (int)top;
-  if (has(idx)) {
-    TORCH_CHECK(idx->scalar_type() == at::kInt && idx->is_contiguous() && idx->numel() == rows * top && has(wt) && is_f32(*wt) &&
-                wt->is_contiguous() && wt->numel() == rows * top, "routing: (rows, top)");
-    r.idx = idx->data_ptr<int>(); r.wt = wt->data_ptr<float>();
-  } else {
-    TORCH_CHECK(has(logits) && is_f32(*logits) && logits->dim() == 2 && logits->stride(1) == 1 && logits->size(0) == rows && logits->size(1) >= experts,
-                "router logits");
-    r.logits = logits->data_ptr<float>(); r.ld = logits->stride(0);
-  }
-  return r;
+Routing routing_of(const Tensor& idx, const Tensor& wt, int64_t rows, int64_t experts) {
+  TORCH_CHECK(idx.scalar_type() == at::kInt && idx.is_contiguous() && idx.dim() == 2 && idx.size(0) == rows && is_f32(wt) && wt.is_contiguous() &&
+              wt.sizes() == idx.sizes(), "routing: (rows, top)");
+  return Routing{idx.data_ptr<int>(), wt.data_ptr<float>(), (int)experts, (int)idx.size(1)};
 }
 
-void expert_gate_up_(const Tensor& h, const Tensor& Wgu, int64_t top, const optional<Tensor>& idx, const optional<Tensor>& wt,
-                     const optional<Tensor>& logits, Tensor& act, bool pdl, const optional<Tensor>& next) {
+void expert_gate_up_(const Tensor& h, const Tensor& Wgu, const Tensor& idx, const Tensor& wt, Tensor& act) {
   check_rows(h, "h"); check_rows(act, "act"); same_type(h, Wgu, "Wgu"); same_type(h, act, "act");
   TORCH_CHECK(Wgu.dim() == 3 && Wgu.is_contiguous() && Wgu.size(2) == h.size(1) && Wgu.size(1) == 2 * act.size(1) && act.is_contiguous() &&
-              act.size(0) == h.size(0) * top, "expert_gate_up shapes");
+              act.size(0) == idx.numel(), "expert_gate_up shapes");
   const c10::cuda::CUDAGuard guard(h.device());
   NC_CHECK(expert_gate_up(is_f32(h), h.data_ptr(), pitch(h), (int)h.size(0), (int)h.size(1), Wgu.data_ptr(), (int)act.size(1),
-                          routing_of(idx, wt, logits, h.size(0), Wgu.size(0), top), act.data_ptr(), pdl, next_weights(next), stream()));
+                          routing_of(idx, wt, h.size(0), Wgu.size(0)), act.data_ptr(), stream()));
 }
 
-ExpertDown expert_down_of(const Tensor& act, const Tensor& Wdown, int64_t rows, int64_t top, const optional<Tensor>& idx, const optional<Tensor>& wt,
-                          const optional<Tensor>& logits) {
-  check_rows(act, "act"); same_type(act, Wdown, "Wdown");
-  TORCH_CHECK(act.is_contiguous() && act.size(0) == rows * top && Wdown.dim() == 3 && Wdown.is_contiguous() && Wdown.size(2) == act.size(1),
-              "expert_down shapes");
-  ExpertDown d{};
-  d.f32 = is_f32(act); d.act = act.data_ptr(); d.rows = (int)rows; d.fp = (int)act.size(1); d.Wdown = Wdown.data_ptr(); d.N = (int)Wdown.size(1);
-  d.rt = routing_of(idx, wt, logits, rows, Wdown.size(0), top);
-  return d;
-}
 void expert_down_(const Tensor& act, const Tensor& Wdown, const Tensor& idx, const Tensor& wt, Tensor& y) {
-  check_rows(y, "y"); same_type(y, act, "y");
-  ExpertDown d = expert_down_of(act, Wdown, y.size(0), idx.size(1), idx, wt, c10::nullopt);
-  TORCH_CHECK(y.size(1) == Wdown.size(1), "expert_down shapes");
+  check_rows(act, "act"); same_type(act, Wdown, "Wdown"); check_rows(y, "y"); same_type(y, act, "y");
+  TORCH_CHECK(act.is_contiguous() && act.size(0) == idx.numel() && Wdown.dim() == 3 && Wdown.is_contiguous() && Wdown.size(2) == act.size(1) &&
+              y.size(1) == Wdown.size(1), "expert_down shapes");
+  ExpertDown d{};
+  d.f32 = is_f32(act); d.act = act.data_ptr(); d.rows = (int)y.size(0); d.fp = (int)act.size(1); d.Wdown = Wdown.data_ptr(); d.N = (int)Wdown.size(1);
+  d.rt = routing_of(idx, wt, y.size(0), Wdown.size(0));
   d.y = y.data_ptr(); d.ldy = pitch(y);
   const c10::cuda::CUDAGuard guard(y.device());
   NC_CHECK(expert_down(d, stream()));
@@ -340,14 +324,23 @@ void check_gate(const Tensor& x, const Tensor& g, const Tensor& bias, const opti
               bias.numel() >= n, "gate logits / bias: float");
   if (has(extra)) TORCH_CHECK(is_f32(*extra) && extra->is_contiguous() && extra->sizes() == x.sizes(), "extra like the residual");
 }
-void expert_down_residual(const Tensor& act, const Tensor& Wdown, int64_t top, const Tensor& logits, Tensor& x, const Tensor& g,
-                          const Tensor& bias, double mult, const optional<Tensor>& extra, const optional<Tensor>& next) {
-  ExpertDown d = expert_down_of(act, Wdown, x.size(0), top, c10::nullopt, c10::nullopt, logits);
-  check_gate(x, g, bias, extra, x.size(0), Wdown.size(1));
-  d.resid = x.data_ptr<float>(); d.ldr = x.stride(0); d.g = g.data_ptr<float>(); d.ldg = g.stride(0); d.bias = bias.data_ptr<float>();
-  d.mult = (float)mult; d.extra = has(extra) ? extra->data_ptr<float>() : nullptr; d.pdl = true; d.next = next_weights(next);
-  const c10::cuda::CUDAGuard guard(x.device());
-  NC_CHECK(expert_down(d, stream()));
+// out[b] = mult * sigmoid(g + bias) * (the row's weighted experts on h) (+ extra), float (rows, n), rows <= 8
+void expert_rows_(const Tensor& h, const Tensor& Wgu, const Tensor& Wdown, const Tensor& idx, const Tensor& wt, Tensor& act, Tensor& out,
+                  const Tensor& g, const Tensor& bias, double mult, const optional<Tensor>& extra) {
+  check_rows(h, "h"); check_rows(act, "act");
+  for (const Tensor* t : {&h, &Wgu, &Wdown, (const Tensor*)&act}) TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kBFloat16, "expert_rows: bf16");
+  TORCH_CHECK(Wgu.dim() == 3 && Wgu.is_contiguous() && Wgu.size(2) == h.size(1) && Wgu.size(1) == 2 * act.size(1) && Wdown.dim() == 3 && Wdown.is_contiguous() &&
+              Wdown.size(0) == Wgu.size(0) && Wdown.size(2) == act.size(1) && act.is_contiguous() && act.size(0) == idx.numel(), "expert_rows shapes");
+  check_gate(out, g, bias, extra, h.size(0), Wdown.size(1));
+  const Routing rt = routing_of(idx, wt, h.size(0), Wgu.size(0));
+  ExpertRows d{};
+  d.h = h.data_ptr(); d.ldh = pitch(h); d.rows = (int)h.size(0); d.top = rt.top; d.experts = rt.experts; d.K = (int)h.size(1); d.fp = (int)act.size(1);
+  d.N = (int)Wdown.size(1); d.Wgu = Wgu.data_ptr(); d.Wdown = Wdown.data_ptr(); d.idx = rt.idx; d.wt = rt.wt; d.act = act.data_ptr();
+  d.out = out.data_ptr<float>(); d.ldo = out.stride(0); d.g = g.data_ptr<float>(); d.ldg = g.stride(0); d.bias = bias.data_ptr<float>(); d.mult = (float)mult;
+  d.extra = has(extra) ? extra->data_ptr<float>() : nullptr;
+  const c10::cuda::CUDAGuard guard(h.device());
+  ++g_launches;
+  NC_CHECK(expert_rows(d, stream()));
 }
 
 // ------------------------------------------------------------------------------------------------------------ gemv
@@ -357,7 +350,7 @@ GemvDesc gemv_of(const Tensor& x, const Tensor& W, const optional<Tensor>& next)
   TORCH_CHECK(x.size(1) == W.size(1) && x.size(0) <= 8, "gemv shapes");
   GemvDesc d{};
   d.x = x.data_ptr(); d.ldx = pitch(x); d.W = W.data_ptr(); d.ldw = pitch(W); d.rows = (int)x.size(0); d.N = (int)W.size(0); d.K = (int)x.size(1);
-  d.next = next_weights(next);
+  d.next = next_weights(next); d.pdl = true; d.accumulate = true;
   return d;
 }
 int store_kind(GemvDesc& d, Tensor& out) {
@@ -402,23 +395,17 @@ void gemv_query_store(const Tensor& z, int64_t q_rank, const Tensor& q_w, double
   const c10::cuda::CUDAGuard guard(z.device());
   NC_CHECK(gemv(d, PRE_NORM, epi, stream()));
 }
-// x[b] += mult * sigmoid(g + bias) * (y W^T) (+ extra); y: bf16 rows, or float rows z put through poly_norm (coef given)
-void gemv_residual(const Tensor& y, const optional<Tensor>& coef, double eps, int64_t n, const Tensor& W, Tensor& x, const Tensor& g,
-                   const Tensor& bias, double mult, const optional<Tensor>& extra, const optional<Tensor>& next) {
+// x[b] (+)= mult * sigmoid(g + bias) * (y W^T) (+ extra); y: bf16 rows. pdl: false where the kernel before is not the only
+// one this waits for
+void gemv_residual(const Tensor& y, const Tensor& W, Tensor& x, const Tensor& g, const Tensor& bias, double mult, const optional<Tensor>& extra,
+                   const optional<Tensor>& next, bool accumulate, bool pdl) {
   GemvDesc d = gemv_of(y, W, next);
-  d.ldx = y.size(0) == 1 ? d.ldx : y.stride(0);
-  int pre = PRE_PLAIN;
-  if (has(coef)) {
-    TORCH_CHECK(is_f32(y) && coef->is_cuda() && is_f32(*coef) && coef->is_contiguous() && coef->numel() == 4, "poly_norm rows: float, four coefficients");
-    pre = PRE_POLY; d.w = coef->data_ptr<float>(); d.eps = (float)eps; d.n_real = (int)n;
-  } else {
-    TORCH_CHECK(y.scalar_type() == at::kBFloat16, "y: bf16 rows");
-  }
+  TORCH_CHECK(y.scalar_type() == at::kBFloat16, "y: bf16 rows");
   check_gate(x, g, bias, extra, y.size(0), W.size(0));
   d.resid = x.data_ptr<float>(); d.ldr = x.stride(0); d.g = g.data_ptr<float>(); d.ldg = g.stride(0); d.bias = bias.data_ptr<float>();
-  d.mult = (float)mult; d.extra = has(extra) ? extra->data_ptr<float>() : nullptr;
+  d.mult = (float)mult; d.extra = has(extra) ? extra->data_ptr<float>() : nullptr; d.accumulate = accumulate; d.pdl = pdl;
   const c10::cuda::CUDAGuard guard(x.device());
-  NC_CHECK(gemv(d, pre, GEMV_RESIDUAL, stream()));
+  NC_CHECK(gemv(d, PRE_PLAIN, GEMV_RESIDUAL, stream()));
 }
 
 std::vector<int64_t> read_status(const Tensor& like) {
@@ -449,18 +436,18 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("rank") = py::none());
   m.def("group_rows", &group_rows);
   m.def("silu_mul", &silu_mul_);
-  m.def("expert_gate_up", &expert_gate_up_, py::arg("h"), py::arg("Wgu"), py::arg("top"), py::arg("idx"), py::arg("wt"), py::arg("logits"),
-        py::arg("act"), py::arg("pdl"), py::arg("next") = py::none());
+  m.def("expert_gate_up", &expert_gate_up_);
   m.def("expert_down", &expert_down_);
-  m.def("expert_down_residual", &expert_down_residual, py::arg("act"), py::arg("Wdown"), py::arg("top"), py::arg("logits"), py::arg("x"),
-        py::arg("g"), py::arg("bias"), py::arg("mult"), py::arg("extra") = py::none(), py::arg("next") = py::none());
+  m.def("expert_rows", &expert_rows_, py::arg("h"), py::arg("Wgu"), py::arg("Wdown"), py::arg("idx"), py::arg("wt"), py::arg("act"), py::arg("out"),
+        py::arg("g"), py::arg("bias"), py::arg("mult"), py::arg("extra") = py::none());
+  m.def("expert_rows_supported", &expert_rows_supported);
   m.def("gemv_norm", &gemv_norm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("n"), py::arg("W"), py::arg("out"),
         py::arg("h") = py::none(), py::arg("next") = py::none());
   m.def("gemv_query_store", &gemv_query_store, py::arg("z"), py::arg("q_rank"), py::arg("q_w"), py::arg("eps"), py::arg("Wq"), py::arg("q"),
         py::arg("c_off"), py::arg("kv_rank"), py::arg("kvp"), py::arg("kv_w"), py::arg("rot_off"), py::arg("rot_dim"), py::arg("freq"),
         py::arg("pool"), py::arg("table"), py::arg("lens"), py::arg("next") = py::none());
-  m.def("gemv_residual", &gemv_residual, py::arg("y"), py::arg("coef"), py::arg("eps"), py::arg("n"), py::arg("W"), py::arg("x"), py::arg("g"),
-        py::arg("bias"), py::arg("mult"), py::arg("extra") = py::none(), py::arg("next") = py::none());
+  m.def("gemv_residual", &gemv_residual, py::arg("y"), py::arg("W"), py::arg("x"), py::arg("g"), py::arg("bias"), py::arg("mult"),
+        py::arg("extra") = py::none(), py::arg("next") = py::none(), py::arg("accumulate") = true, py::arg("pdl") = true);
   m.def("read_status", &read_status);
   m.def("launch_count", [] { return g_launches.load(); });
 }

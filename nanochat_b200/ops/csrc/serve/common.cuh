@@ -113,6 +113,9 @@ __device__ __forceinline__ float warp_sum_many(float (&v)[NV], int lane) {
 
 // -------------------------------------------------------------------------- small math
 __device__ __forceinline__ float sigmoidf(float v) { return 1.f / (1.f + expf(-v)); }
+// next to bf16 values: a few units in the last place of a float do not matter
+__device__ __forceinline__ float fast_sigmoidf(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <typename T> __device__ __forceinline__ float sigmoid_of(float v) { return sizeof(T) == 4 ? sigmoidf(v) : fast_sigmoidf(v); }
 __device__ __forceinline__ float inv_rms(float sumsq, int n, float eps) { return 1.f / sqrtf(sumsq / n + eps); }
 
 // ------------------------------------------------------------------------- paged store
@@ -156,6 +159,14 @@ cudaError_t launch_pdl(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t sme
   at[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = at; cfg.numAttrs = 1;
   return cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
+}
+
+// plain launch, or one that may overlap the end of the kernel before it
+template <typename... KArgs, typename... Args>
+cudaError_t launch(bool pdl, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args... args) {
+  if (pdl) return launch_pdl(kern, grid, block, smem, s, args...);
+  kern<<<grid, block, smem, s>>>(static_cast<KArgs>(args)...);
+  return cudaGetLastError();
 }
 
 // This CTA's slice of the weights a later kernel will stream, requested into L2.

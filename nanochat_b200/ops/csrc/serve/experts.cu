@@ -5,8 +5,8 @@
 //   route_topk -> plan_groups -> gather_groups -> grouped GEMM -> silu_mul -> grouped GEMM
 // A row's place inside its group comes from an atomic counter, so it varies; its values do not depend on it.
 //
-// Decode (and float): one matrix-vector product per (row, chosen expert), a CTA per four outputs with K split over its
-// threads. Given the logits, every CTA works its row's routing out itself, which costs less than a kernel of its own.
+// Few rows, and float: one matrix-vector product per (row, chosen expert), a CTA per four outputs with K split over its
+// threads. (bf16 decode steps read each expert once for all their rows instead, see gemv.cu.)
 #include "common.cuh"
 
 namespace nc {
@@ -19,6 +19,8 @@ route_topk_kernel(const float* __restrict__ logits, long long ld, int rows, int 
                   float* __restrict__ wt, int* __restrict__ counts, int* __restrict__ rank) {
   const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= rows) return;
+  pdl_wait();
+  pdl_trigger();
   const float* z = logits + row * ld;
   float v = INFINITY, best = 0.f, sum = 0.f;
   int i = -1;
@@ -89,7 +91,7 @@ silu_mul_kernel(const bf16* __restrict__ gu, int fp, const int* __restrict__ til
     load8(gu + row * 2 * fp + c, g);
     load8(gu + row * 2 * fp + fp + c, u);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) g[j] = g[j] * sigmoidf(g[j]) * u[j];
+    for (int j = 0; j < 8; ++j) g[j] = g[j] * fast_sigmoidf(g[j]) * u[j];
     store8(act + row * fp + c, g);
   }
 }
@@ -114,26 +116,12 @@ __device__ __forceinline__ float block_cols(float (&v)[COLS], float (*smem)[COLS
 template <typename T>
 __global__ void __launch_bounds__(256)
 expert_gate_up_kernel(const T* __restrict__ h, long long ldh, int K, const T* __restrict__ Wgu, int fp, Routing rt,
-                      T* __restrict__ act, NextWeights next) {
+                      T* __restrict__ act) {
   __shared__ float s_g[8][COLS], s_u[8][COLS];
-  __shared__ int s_expert;
   const int row = blockIdx.x / rt.top, k = blockIdx.x - row * rt.top, n0 = blockIdx.y * COLS;
-  prefetch_l2_slice(next, blockIdx.x + (long long)gridDim.x * blockIdx.y, (long long)gridDim.x * gridDim.y);
   pdl_wait();
   pdl_trigger();
-  if (rt.idx == nullptr) {
-    if (threadIdx.x < 32) {
-      float v = INFINITY; int i = -1;
-      for (int t = 0; t <= k; ++t) {
-        float nv; int ni;
-        next_best(rt.logits + row * rt.ld, rt.experts, v, i, threadIdx.x, nv, ni);
-        v = nv; i = ni;
-      }
-      if (threadIdx.x == 0) s_expert = i;
-    }
-    __syncthreads();
-  }
-  const long long e = rt.idx ? rt.idx[(long long)row * rt.top + k] : s_expert;
+  const long long e = rt.idx[(long long)row * rt.top + k];
   const T* wg = Wgu + e * 2 * fp * K;
   const T* wu = wg + (long long)fp * K;
   float g[COLS] = {0.f, 0.f, 0.f, 0.f}, u[COLS] = {0.f, 0.f, 0.f, 0.f};
@@ -162,45 +150,19 @@ expert_gate_up_kernel(const T* __restrict__ h, long long ldh, int K, const T* __
     act[(long long)blockIdx.x * fp + n0 + threadIdx.x] = from_f<T>(gs * sigmoidf(gs) * us);
 }
 
-// grid (rows, ceil(N / 4)); dynamic shared memory: top ints, top floats
+// grid (rows, ceil(N / 4))
 template <typename T>
 __global__ void __launch_bounds__(256)
 expert_down_kernel(const ExpertDown d) {
-  extern __shared__ float s_route[];
   __shared__ float s_acc[8][COLS];
-  float* s_wt = s_route;
-  int* s_idx = reinterpret_cast<int*>(s_route + d.rt.top);
   const int row = blockIdx.x, n0 = blockIdx.y * COLS, top = d.rt.top;
-  prefetch_l2_slice(d.next, blockIdx.x + (long long)gridDim.x * blockIdx.y, (long long)gridDim.x * gridDim.y);
   pdl_wait();
   pdl_trigger();
-  if (d.rt.idx == nullptr) {
-    if (threadIdx.x < 32) {
-      float v = INFINITY, best = 0.f, sum = 0.f; int i = -1;
-      for (int t = 0; t < top; ++t) {
-        float nv; int ni;
-        next_best(d.rt.logits + row * d.rt.ld, d.rt.experts, v, i, threadIdx.x, nv, ni);
-        v = nv; i = ni;
-        if (t == 0) best = v;
-        const float e = expf(v - best);
-        sum += e;
-        if (threadIdx.x == 0) { s_idx[t] = i; s_wt[t] = e; }
-      }
-      __syncwarp();
-      for (int t = threadIdx.x; t < top; t += 32) s_wt[t] /= sum;
-    }
-  } else {
-    for (int t = threadIdx.x; t < top; t += 256) {
-      s_idx[t] = d.rt.idx[(long long)row * top + t];
-      s_wt[t] = d.rt.wt[(long long)row * top + t];
-    }
-  }
-  __syncthreads();
   float acc[COLS] = {0.f, 0.f, 0.f, 0.f};
   for (int t = 0; t < top; ++t) {
-    const T* w = (const T*)d.Wdown + (long long)s_idx[t] * d.N * d.fp;
+    const T* w = (const T*)d.Wdown + (long long)d.rt.idx[(long long)row * top + t] * d.N * d.fp;
     const T* a = (const T*)d.act + ((long long)row * top + t) * d.fp;
-    const float wt = s_wt[t];
+    const float wt = d.rt.wt[(long long)row * top + t];
     for (int c = threadIdx.x * 8; c < d.fp; c += 2048) {
       Raw8<T> rw[COLS];
 #pragma unroll
@@ -219,26 +181,11 @@ expert_down_kernel(const ExpertDown d) {
   }
   const float v = block_cols(acc, s_acc);
   const int n = n0 + threadIdx.x;
-  if (threadIdx.x < COLS && n < d.N) {
-    if (d.resid) {
-      float x = d.resid[row * d.ldr + n] + d.mult * sigmoidf(d.g[row * d.ldg + n] + d.bias[n]) * v;
-      if (d.extra) x += d.extra[row * d.ldr + n];
-      d.resid[row * d.ldr + n] = x;
-    } else {
-      ((T*)d.y)[row * d.ldy + n] = from_f<T>(v);
-    }
-  }
+  if (threadIdx.x < COLS && n < d.N) ((T*)d.y)[row * d.ldy + n] = from_f<T>(v);
 }
 
 bool routing_ok(const Routing& r) {
-  return r.experts > 0 && r.top > 0 && r.top <= r.experts && (r.idx != nullptr || r.logits != nullptr);
-}
-
-template <typename... KArgs, typename... Args>
-cudaError_t launch(bool pdl, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args... args) {
-  if (pdl) return launch_pdl(kern, grid, block, smem, s, args...);
-  kern<<<grid, block, smem, s>>>(static_cast<KArgs>(args)...);
-  return cudaGetLastError();
+  return r.experts > 0 && r.top > 0 && r.top <= r.experts && r.idx != nullptr && r.wt != nullptr;
 }
 
 }  // namespace
@@ -247,8 +194,7 @@ cudaError_t route_topk(const float* logits, long long ld, int rows, int experts,
                        int* counts, int* rank, cudaStream_t s) {
   if (rows <= 0 || experts <= 0 || top <= 0 || top > experts || ld < experts || (counts != nullptr) != (rank != nullptr))
     return cudaErrorInvalidValue;
-  route_topk_kernel<<<(rows + 3) / 4, 128, 0, s>>>(logits, ld, rows, experts, top, idx, wt, counts, rank);
-  return cudaGetLastError();
+  return launch_pdl(route_topk_kernel, dim3((rows + 3) / 4), dim3(128), 0, s, logits, ld, rows, experts, top, idx, wt, counts, rank);
 }
 
 cudaError_t plan_groups(const int* counts, int experts, int* offsets, int* tile_group, int tiles, cudaStream_t s) {
@@ -271,21 +217,19 @@ cudaError_t silu_mul(const void* gu, int rows, int fp, const int* tile_group, vo
 }
 
 cudaError_t expert_gate_up(bool f32, const void* h, long long ldh, int rows, int K, const void* Wgu, int fp,
-                           const Routing& rt, void* act, bool pdl, const NextWeights& next, cudaStream_t s) {
+                           const Routing& rt, void* act, cudaStream_t s) {
   if (rows <= 0 || K <= 0 || (K & 7) || (ldh & 7) || fp <= 0 || (fp & 7) || fp / COLS > 65535 || !routing_ok(rt)) return cudaErrorInvalidValue;
   const dim3 grid(rows * rt.top, (fp + COLS - 1) / COLS);
-  if (f32) return launch(pdl, expert_gate_up_kernel<float>, grid, dim3(256), 0, s, (const float*)h, ldh, K, (const float*)Wgu, fp, rt, (float*)act, next);
-  return launch(pdl, expert_gate_up_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)h, ldh, K, (const bf16*)Wgu, fp, rt, (bf16*)act, next);
+  if (f32) return launch(true, expert_gate_up_kernel<float>, grid, dim3(256), 0, s, (const float*)h, ldh, K, (const float*)Wgu, fp, rt, (float*)act);
+  return launch(true, expert_gate_up_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)h, ldh, K, (const bf16*)Wgu, fp, rt, (bf16*)act);
 }
 
 cudaError_t expert_down(const ExpertDown& d, cudaStream_t s) {
-  if (d.rows <= 0 || d.fp <= 0 || (d.fp & 7) || d.N <= 0 || d.N / COLS > 65534 || !routing_ok(d.rt) || (d.rt.idx && !d.rt.wt) ||
-      d.rt.top > 2048 || (d.resid ? (!d.g || !d.bias) : !d.y))
+  if (d.rows <= 0 || d.fp <= 0 || (d.fp & 7) || d.N <= 0 || d.N / COLS > 65534 || !routing_ok(d.rt) || !d.y)
     return cudaErrorInvalidValue;
   const dim3 grid(d.rows, (d.N + COLS - 1) / COLS);
-  const size_t smem = (size_t)d.rt.top * 8;
-  if (d.f32) return launch(d.pdl, expert_down_kernel<float>, grid, dim3(256), smem, s, d);
-  return launch(d.pdl, expert_down_kernel<bf16>, grid, dim3(256), smem, s, d);
+  if (d.f32) return launch(true, expert_down_kernel<float>, grid, dim3(256), 0, s, d);
+  return launch(true, expert_down_kernel<bf16>, grid, dim3(256), 0, s, d);
 }
 
 }  // namespace serve

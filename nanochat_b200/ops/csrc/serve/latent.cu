@@ -18,6 +18,7 @@ namespace serve {
 namespace {
 
 constexpr float NEG_BIG = -1.0e30f;
+constexpr int MAX_SPLITS = 32;
 
 __device__ __forceinline__ int row_position(const RowPos& p, int row, int& seq) {
   seq = row / p.per_seq;
@@ -25,19 +26,33 @@ __device__ __forceinline__ int row_position(const RowPos& p, int row, int& seq) 
 }
 
 // ---------------------------------------------------------------------- post / gather
+// grid (rows, 1 or 2): y = 0 the store entry, y = 1 the query latent. The norm weights' padding is zero.
 template <typename T, typename TZ>
 __global__ void __launch_bounds__(128)
 latent_post_kernel(const LatentPost d, int* status) {
   __shared__ float red[32];
   const int row = blockIdx.x;
   const TZ* z = (const TZ*)d.z + (long long)row * d.ldz;
-  if (d.cq) {
+  if (blockIdx.y == 1) {
     float ss[1] = {0.f};
-    for (int c = threadIdx.x; c < d.q_rank; c += blockDim.x) { const float v = to_f(z[c]); ss[0] += v * v; }
+    for (int c = threadIdx.x * 8; c < d.qp; c += 1024) {
+      float v[8];
+      load8(z + c, v);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss[0] += v[j] * v[j];
+    }
     block_sum<1>(ss, red);
     const float r = inv_rms(ss[0], d.q_rank, d.eps);
     T* cq = (T*)d.cq + (long long)row * d.ldcq;
-    for (int c = threadIdx.x; c < d.qp; c += blockDim.x) cq[c] = from_f<T>(c < d.q_rank ? to_f(z[c]) * r * d.q_w[c] : 0.f);
+    for (int c = threadIdx.x * 8; c < d.qp; c += 1024) {
+      float v[8], w[8];
+      load8(z + c, v);
+      load8(d.q_w + c, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= r * w[j];
+      store8(cq + c, v);
+    }
+    return;
   }
   int seq;
   const int pos = row_position(d.pos, row, seq);
@@ -61,23 +76,38 @@ latent_gather_kernel(const Pages pg, int seq, int first, T* out, long long ldo, 
   }
 }
 
-// one thread per (row, pair): the angle is shared by all heads
-template <typename T>
+// one thread per (row, head, V pairs)
+template <typename T, int V>
 __global__ void __launch_bounds__(128)
 rotate_heads_kernel(T* __restrict__ q, long long ldq, int rows, int heads, int head_pitch, int off, int half,
                     const float* __restrict__ freq, RowPos rp) {
+  const int chunks = half / V;
   const long long t = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  const int row = (int)(t / half), i = (int)(t - (long long)row * half);
+  const int i = (int)(t % chunks) * V, h = (int)(t / chunks % heads), row = (int)(t / ((long long)chunks * heads));
   if (row >= rows) return;
   int seq;
   const int pos = row_position(rp, row, seq);
-  float sn, cs;
-  sincosf((float)pos * freq[i], &sn, &cs);
-  T* p = q + row * ldq + off + i;
-  for (int h = 0; h < heads; ++h, p += head_pitch) {
-    const float a = to_f(p[0]), b = to_f(p[half]);
-    p[0] = from_f<T>(a * cs - b * sn);
-    p[half] = from_f<T>(b * cs + a * sn);
+  T* p = q + row * ldq + (long long)h * head_pitch + off + i;
+  float a[V], b[V];
+  if constexpr (V == 8) {
+    load8(p, a);
+    load8(p + half, b);
+  } else {
+    a[0] = to_f(p[0]); b[0] = to_f(p[half]);
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    float sn, cs;
+    sincosf((float)pos * freq[i + j], &sn, &cs);
+    const float u = a[j], v = b[j];
+    a[j] = u * cs - v * sn;
+    b[j] = v * cs + u * sn;
+  }
+  if constexpr (V == 8) {
+    store8(p, a);
+    store8(p + half, b);
+  } else {
+    p[0] = from_f<T>(a[0]); p[half] = from_f<T>(b[0]);
   }
 }
 
@@ -221,8 +251,10 @@ latent_attention_kernel(const LatentAttn d) {
   for (int c = tid; c < d.kvp; c += 128) d.acc[slot * d.kvp + c] = so[c];
 }
 
-// Tensor-core form: grid (splits, ceil(heads / 16), rows), 128 threads.
+// Tensor-core form: grid (splits, ceil(heads / 16), rows), 256 threads. Each of the eight warps scores eight of a tile's
+// keys, then owns every eighth 16-column unit of the weighted latents.
 constexpr int KT = 64;                       // keys per tile
+constexpr int AW = 8;                        // warps
 __device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
@@ -240,28 +272,30 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-inline size_t mma_smem_bytes(int W, int rp) {
-  return (size_t)(16 + KT) * (W + 8) * 2 + (size_t)16 * (KT + 8) * 2 + (size_t)rp * 4;
-}
+__host__ __device__ constexpr int padded_width(int W) { return (W + 31) / 32 * 32; }      // scores step through 32 columns
+inline size_t mma_smem_bytes(int W) { return (size_t)(16 + KT) * (padded_width(W) + 8) * 2 + (size_t)16 * (KT + 8) * 2; }
 
-// NU: 16-column units of the latent per warp (kvp <= 64 * NU)
+// NU: 16-column units of the latent per warp (kvp <= 128 * NU)
 template <int NU>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(AW * 32)
 latent_attention_mma_kernel(const LatentAttn d) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  __shared__ float s_max[4][16];
-  __shared__ float s_sum[4][16];
+  __shared__ float s_max[AW][16];
+  __shared__ float s_sum[AW][16];
   const int split = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int W = d.kvp + d.rp, LD = W + 8, LP = KT + 8;
+  const int W = d.kvp + d.rp, WP = padded_width(W), LD = WP + 8, LP = KT + 8;
   bf16* sQ = reinterpret_cast<bf16*>(smem_raw);
   bf16* sK = sQ + 16 * LD;
   bf16* sP = sK + KT * LD;
-  float* s_cs = reinterpret_cast<float*>(sP + 16 * LP);        // cos | sin of this position
-  int seq;
   const int half = d.dims >> 1;
+  if (WP > W) {                                                 // columns that only fill up the last step
+    for (int i = tid; i < (16 + KT) * 2; i += AW * 32)
+      *reinterpret_cast<uint4*>(sQ + (i >> 1) * LD + W + (i & 1) * 8) = make_uint4(0, 0, 0, 0);
+  }
   pdl_wait();
   pdl_trigger();
+  int seq;
   const int pos = row_position(d.pos, row, seq);
   const KeyRange kr = split_keys(pos, d.window, d.splits, split, KT);
   if (kr.begin >= kr.end) {
@@ -272,9 +306,12 @@ latent_attention_mma_kernel(const LatentAttn d) {
     return;
   }
   auto load_tile = [&](int tile) {
-    for (int k = warp; k < KT; k += 4) {
-      const long long off = tile + k < kr.end ? token_offset(d.pg, seq, tile + k) : -1;
-      bf16* dst = sK + k * LD;
+    const int mine = tile + warp * 8 + (lane & 7);              // the warp's eight keys: addresses first, then the copies
+    const long long my_off = mine < kr.end ? token_offset(d.pg, seq, mine) : -1;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const long long off = __shfl_sync(0xffffffffu, my_off, k);
+      bf16* dst = sK + (warp * 8 + k) * LD;
       if (off >= 0) {
         const bf16* src = (const bf16*)d.pg.pool + off;
         for (int c = lane * 8; c < W; c += 256) cp_async16(dst + c, src + c);
@@ -285,30 +322,21 @@ latent_attention_mma_kernel(const LatentAttn d) {
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   load_tile(kr.begin);
-  for (int i = tid; i < half; i += 128) sincosf((float)pos * d.freq[i], &s_cs[half + i], &s_cs[i]);
-  for (int h = warp; h < 16; h += 4) {
+  for (int h = warp; h < 16; h += AW) {
     const bool on = h0 + h < d.heads;
     const bf16* qa = (const bf16*)d.qa + ((long long)row * d.heads + h0 + h) * d.kvp;
     for (int c = lane * 8; c < d.kvp; c += 256)
       *reinterpret_cast<uint4*>(sQ + h * LD + c) = on ? *reinterpret_cast<const uint4*>(qa + c) : make_uint4(0, 0, 0, 0);
-  }
-  __syncthreads();                                              // s_cs
-  for (int h = warp; h < 16; h += 4) {
-    const bool on = h0 + h < d.heads;
     const bf16* qr = (const bf16*)d.q + row * d.ldq + (long long)(h0 + h) * d.head_pitch + d.dp;
-    for (int i = lane; i < d.rp; i += 32) {
-      float v = 0.f;
-      if (on) {
-        if (i < d.dims) {
-          const int p = i < half ? i : i - half;
-          const float a = to_f(qr[p]), b = to_f(qr[p + half]), cs = s_cs[p], sn = s_cs[half + p];
-          v = i < half ? a * cs - b * sn : b * cs + a * sn;
-        } else if (i < d.rot_dim) {
-          v = to_f(qr[i]);
-        }
-      }
-      sQ[h * LD + d.kvp + i] = __float2bfloat16_rn(v);
+    bf16* dst = sQ + h * LD + d.kvp;
+    for (int i = lane; i < half; i += 32) {
+      float sn, cs;
+      sincosf((float)pos * d.freq[i], &sn, &cs);
+      const float a = on ? to_f(qr[i]) : 0.f, b = on ? to_f(qr[i + half]) : 0.f;
+      dst[i] = __float2bfloat16_rn(a * cs - b * sn);
+      dst[i + half] = __float2bfloat16_rn(b * cs + a * sn);
     }
+    for (int i = d.dims + lane; i < d.rp; i += 32) dst[i] = on && i < d.rot_dim ? qr[i] : __float2bfloat16_rn(0.f);
   }
   const float sc = d.scale * 1.4426950408889634f;
   float m_run[2] = {NEG_BIG, NEG_BIG}, l_run[2] = {0.f, 0.f};
@@ -323,29 +351,26 @@ latent_attention_mma_kernel(const LatentAttn d) {
   for (int tile = kr.begin; tile < kr.end; tile += KT) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    // scores of 16 heads x this warp's 16 keys
+    // scores of 16 heads x this warp's 8 keys, even and odd steps in accumulators of their own
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     const bf16* qp = sQ + (lane & 15) * LD + (lane >> 4) * 8;
-    const bf16* kp = sK + (warp * 16 + (lane >> 4) * 8 + (lane & 7)) * LD + ((lane >> 3) & 1) * 8;
+    const bf16* kp = sK + (warp * 8 + (lane & 7)) * LD + (lane >> 3) * 8;
 #pragma unroll 4
-    for (int k = 0; k < W; k += 16) {
-      uint32_t a[4], b[4];
-      ldmatrix4(a, qp + k);
+    for (int k = 0; k < WP; k += 32) {
+      uint32_t a0[4], a1[4], b[4];
+      ldmatrix4(a0, qp + k);
+      ldmatrix4(a1, qp + k + 16);
       ldmatrix4(b, kp + k);
-      mma_16816(s[0], a, b[0], b[1]);
-      mma_16816(s[1], a, b[2], b[3]);
+      mma_16816(s[0], a0, b[0], b[1]);
+      mma_16816(s[1], a1, b[2], b[3]);
     }
-    float mx[2] = {NEG_BIG, NEG_BIG};
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int j = tile + warp * 16 + t * 8 + (lane & 3) * 2 + (e & 1);
-        s[t][e] = j < kr.end ? s[t][e] * sc : NEG_BIG;
-        mx[e >> 1] = fmaxf(mx[e >> 1], s[t][e]);
-      }
+    const int j = tile + warp * 8 + (lane & 3) * 2;             // this lane's keys: j, j + 1
+    float mx[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) s[0][r * 2 + e] = j + e < kr.end ? (s[0][r * 2 + e] + s[1][r * 2 + e]) * sc : NEG_BIG;
+      mx[r] = fmaxf(s[0][r * 2], s[0][r * 2 + 1]);
       mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
       mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
       if ((lane & 3) == 0) s_max[warp][(lane >> 2) + r * 8] = mx[r];
@@ -355,40 +380,31 @@ latent_attention_mma_kernel(const LatentAttn d) {
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int hr = (lane >> 2) + r * 8;
-      const float m_new = fmaxf(m_run[r], fmaxf(fmaxf(s_max[0][hr], s_max[1][hr]), fmaxf(s_max[2][hr], s_max[3][hr])));
+      float m_new = m_run[r];
+#pragma unroll
+      for (int w = 0; w < AW; ++w) m_new = fmaxf(m_new, s_max[w][hr]);
       alpha[r] = exp2f(m_run[r] - m_new);
       m_run[r] = m_new;
-      l_run[r] *= alpha[r];
+      const float p0 = j < kr.end ? exp2f(s[0][r * 2] - m_new) : 0.f;
+      const float p1 = j + 1 < kr.end ? exp2f(s[0][r * 2 + 1] - m_new) : 0.f;
+      l_run[r] = l_run[r] * alpha[r] + p0 + p1;
+      *reinterpret_cast<uint32_t*>(sP + hr * LP + warp * 8 + (lane & 3) * 2) = pack_bf16(p0, p1);
     }
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int j = tile + warp * 16 + t * 8 + (lane & 3) * 2;
-        const float p0 = j < kr.end ? exp2f(s[t][r * 2] - m_run[r]) : 0.f;
-        const float p1 = j + 1 < kr.end ? exp2f(s[t][r * 2 + 1] - m_run[r]) : 0.f;
-        l_run[r] += p0 + p1;
-        *reinterpret_cast<uint32_t*>(sP + ((lane >> 2) + r * 8) * LP + warp * 16 + t * 8 + (lane & 3) * 2) = pack_bf16(p0, p1);
-      }
     __syncthreads();
     // weighted latents: this warp's column units
 #pragma unroll
-    for (int u = 0; u < NU; ++u) {
-      const int unit = warp + u * 4;
-      if (unit < units) {
+    for (int u = 0; u < NU; ++u)
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
+      for (int t = 0; t < 2; ++t)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) o[u][t][e] *= alpha[e >> 1];
-      }
-    }
+        for (int e = 0; e < 4; ++e) o[u][t][e] *= alpha[e >> 1];
 #pragma unroll
     for (int k = 0; k < KT; k += 16) {
       uint32_t a[4];
       ldmatrix4(a, sP + (lane & 15) * LP + k + (lane >> 4) * 8);
 #pragma unroll
       for (int u = 0; u < NU; ++u) {
-        const int unit = warp + u * 4;
+        const int unit = warp + u * AW;
         if (unit < units) {
           uint32_t b[4];
           ldmatrix4_trans(b, sK + (k + (lane & 15)) * LD + unit * 16 + (lane >> 4) * 8);
@@ -397,37 +413,36 @@ latent_attention_mma_kernel(const LatentAttn d) {
         }
       }
     }
-    __syncthreads();                                            // the tile's keys and weights have been read
-    if (tile + KT < kr.end) load_tile(tile + KT);
+    if (tile + KT < kr.end) {
+      __syncthreads();                                          // the tile's keys and weights have been read
+      load_tile(tile + KT);
+    }
   }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
-    if ((lane & 3) == 0) {
-      s_sum[warp][(lane >> 2) + r * 8] = l_run[r];
-      if (warp == 0) s_max[0][(lane >> 2) + r * 8] = m_run[r];
-    }
-  }
-  __syncthreads();
-  if (tid < 16 && h0 + tid < d.heads) {
-    const long long slot = ((long long)row * d.heads + h0 + tid) * d.splits + split;
-    d.ml[slot * 2] = s_max[0][tid];
-    d.ml[slot * 2 + 1] = s_sum[0][tid] + s_sum[1][tid] + s_sum[2][tid] + s_sum[3][tid];
-  }
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
+    if ((lane & 3) == 0) s_sum[warp][(lane >> 2) + r * 8] = l_run[r];
     const int h = h0 + (lane >> 2) + r * 8;
     if (h >= d.heads) continue;
-    float* dst = d.acc + (((long long)row * d.heads + h) * d.splits + split) * d.kvp;
+    const long long slot = ((long long)row * d.heads + h) * d.splits + split;
+    if (warp == 0 && (lane & 3) == 0) d.ml[slot * 2] = m_run[r];
+    float* dst = d.acc + slot * d.kvp;
 #pragma unroll
     for (int u = 0; u < NU; ++u) {
-      const int unit = warp + u * 4;
+      const int unit = warp + u * AW;
       if (unit >= units) continue;
 #pragma unroll
       for (int t = 0; t < 2; ++t)
         *reinterpret_cast<float2*>(dst + unit * 16 + t * 8 + (lane & 3) * 2) = make_float2(o[u][t][r * 2], o[u][t][r * 2 + 1]);
     }
+  }
+  __syncthreads();
+  if (tid < 16 && h0 + tid < d.heads) {
+    float l = 0.f;
+#pragma unroll
+    for (int w = 0; w < AW; ++w) l += s_sum[w][tid];
+    d.ml[(((long long)row * d.heads + h0 + tid) * d.splits + split) * 2 + 1] = l;
   }
 }
 
@@ -437,6 +452,7 @@ __global__ void __launch_bounds__(256)
 latent_values_kernel(const float* __restrict__ ml, const float* __restrict__ acc, int heads, int splits, int kvp,
                      const T* __restrict__ Wuv, int vp, T* __restrict__ y, long long ldy, NextWeights next) {
   extern __shared__ float lat[];
+  __shared__ float s_w[MAX_SPLITS];
   const int h = blockIdx.y, row = blockIdx.z;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int j0 = blockIdx.x * 32 + warp * 4;
@@ -449,20 +465,23 @@ latent_values_kernel(const float* __restrict__ ml, const float* __restrict__ acc
   pdl_wait();
   pdl_trigger();
   const long long slot = ((long long)row * heads + h) * splits;
-  float M = NEG_BIG;
-  for (int s = 0; s < splits; ++s)
-    if (ml[(slot + s) * 2 + 1] > 0.f) M = fmaxf(M, ml[(slot + s) * 2]);
-  float L = 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float l = ml[(slot + s) * 2 + 1];
-    if (l > 0.f) L += l * exp2f(ml[(slot + s) * 2] - M);
+  if (warp == 0) {                                  // a lane per split: its weight in the combination
+    const float m = lane < splits ? ml[(slot + lane) * 2] : NEG_BIG, l = lane < splits ? ml[(slot + lane) * 2 + 1] : 0.f;
+    const float M = warp_max(l > 0.f ? m : NEG_BIG);
+    const float f = l > 0.f ? exp2f(m - M) : 0.f;
+    const float L = warp_sum(l * f);
+    s_w[lane] = L > 0.f ? f / L : 0.f;
   }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  __syncthreads();
   for (int c = threadIdx.x; c < kvp; c += 256) {
     float v = 0.f;
-    for (int s = 0; s < splits; ++s)
-      if (ml[(slot + s) * 2 + 1] > 0.f) v += acc[(slot + s) * kvp + c] * exp2f(ml[(slot + s) * 2] - M);
-    lat[c] = v * inv;
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) {
+      const float f = s_w[s];                       // an empty split leaves its sums unwritten
+      const float t = f > 0.f ? acc[(slot + s) * kvp + c] : 0.f;
+      v += f * t;
+    }
+    lat[c] = v;
   }
   __syncthreads();
   float sum[4] = {0.f, 0.f, 0.f, 0.f};
@@ -489,23 +508,16 @@ bool pages_ok(const Pages& p) {
 }
 bool rows_ok(const RowPos& p) { return p.lens && p.per_seq > 0; }
 
-// plain launch or one that may overlap the end of the kernel before it
-template <typename... KArgs, typename... Args>
-cudaError_t launch(bool pdl, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args... args) {
-  if (pdl) return launch_pdl(kern, grid, block, smem, s, args...);
-  kern<<<grid, block, smem, s>>>(static_cast<KArgs>(args)...);
-  return cudaGetLastError();
-}
-
 }  // namespace
 
 cudaError_t latent_post(const LatentPost& d, int* status, cudaStream_t s) {
   if (d.rows <= 0 || !pages_ok(d.pg) || !rows_ok(d.pos) || d.pg.width != d.kvp + d.rp || d.kv_rank > d.kvp || d.kv_rank <= 0 ||
       d.dims > d.rot_dim || d.rot_dim > d.rp || (d.dims & 1) || d.q_rank > d.qp || (d.f32 && !d.z_f32))
     return cudaErrorInvalidValue;
-  if (d.f32) latent_post_kernel<float, float><<<d.rows, 128, 0, s>>>(d, status);
-  else if (d.z_f32) latent_post_kernel<bf16, float><<<d.rows, 128, 0, s>>>(d, status);
-  else latent_post_kernel<bf16, bf16><<<d.rows, 128, 0, s>>>(d, status);
+  const dim3 grid(d.rows, d.cq ? 2 : 1);
+  if (d.f32) latent_post_kernel<float, float><<<grid, 128, 0, s>>>(d, status);
+  else if (d.z_f32) latent_post_kernel<bf16, float><<<grid, 128, 0, s>>>(d, status);
+  else latent_post_kernel<bf16, bf16><<<grid, 128, 0, s>>>(d, status);
   return cudaGetLastError();
 }
 
@@ -522,10 +534,17 @@ cudaError_t rotate_heads(bool f32, void* q, long long ldq, int rows, int heads, 
   if (rows <= 0 || heads <= 0 || dims < 0 || (dims & 1) || off + dims > head_pitch || (long long)heads * head_pitch > ldq || !rows_ok(pos))
     return cudaErrorInvalidValue;
   if (dims == 0) return cudaSuccess;
-  const long long n = (long long)rows * (dims / 2);
+  const int half = dims / 2;
+  const bool vec = half % 8 == 0 && off % 8 == 0 && head_pitch % 8 == 0 && ldq % 8 == 0;
+  const long long n = (long long)rows * heads * (half / (vec ? 8 : 1));
   const dim3 grid((unsigned)((n + 127) / 128));
-  if (f32) rotate_heads_kernel<float><<<grid, 128, 0, s>>>((float*)q, ldq, rows, heads, head_pitch, off, dims / 2, freq, pos);
-  else rotate_heads_kernel<bf16><<<grid, 128, 0, s>>>((bf16*)q, ldq, rows, heads, head_pitch, off, dims / 2, freq, pos);
+  if (f32) {
+    auto k = vec ? rotate_heads_kernel<float, 8> : rotate_heads_kernel<float, 1>;
+    k<<<grid, 128, 0, s>>>((float*)q, ldq, rows, heads, head_pitch, off, half, freq, pos);
+  } else {
+    auto k = vec ? rotate_heads_kernel<bf16, 8> : rotate_heads_kernel<bf16, 1>;
+    k<<<grid, 128, 0, s>>>((bf16*)q, ldq, rows, heads, head_pitch, off, half, freq, pos);
+  }
   return cudaGetLastError();
 }
 
@@ -539,7 +558,7 @@ cudaError_t absorb_query(bool f32, const void* q, long long ldq, int rows, int h
 }
 
 bool latent_attention_tensor_cores(const LatentAttn& d) {
-  return !d.f32 && !(d.kvp & 15) && !(d.rp & 15) && d.kvp <= 512 && mma_smem_bytes(d.kvp + d.rp, d.rp) <= 200 * 1024;
+  return !d.f32 && !(d.kvp & 15) && !(d.rp & 15) && d.kvp <= 512 && mma_smem_bytes(d.kvp + d.rp) <= 200 * 1024;
 }
 
 template <int NU>
@@ -549,19 +568,19 @@ static cudaError_t launch_mma(const LatentAttn& d, cudaStream_t s) {
     return cudaFuncSetAttribute(latent_attention_mma_kernel<NU>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   });
   if (ce != cudaSuccess) return ce;
-  return launch(d.pdl, latent_attention_mma_kernel<NU>, dim3(d.splits, (d.heads + 15) / 16, d.rows), dim3(128),
-                mma_smem_bytes(d.kvp + d.rp, d.rp), s, d);
+  return launch(d.pdl, latent_attention_mma_kernel<NU>, dim3(d.splits, (d.heads + 15) / 16, d.rows), dim3(AW * 32),
+                mma_smem_bytes(d.kvp + d.rp), s, d);
 }
 
 cudaError_t latent_attention(const LatentAttn& d, cudaStream_t s) {
-  if (d.rows <= 0 || d.rows > 65535 || d.heads <= 0 || d.heads > 65535 || d.splits <= 0 || !pages_ok(d.pg) || !rows_ok(d.pos) ||
+  if (d.rows <= 0 || d.rows > 65535 || d.heads <= 0 || d.heads > 65535 || d.splits <= 0 || d.splits > MAX_SPLITS || !pages_ok(d.pg) || !rows_ok(d.pos) ||
       d.pg.width != d.kvp + d.rp || (d.kvp & 7) || (d.rp & 7) || d.dims > d.rot_dim || d.rot_dim > d.rp || (d.dims & 1) ||
       d.dp + d.rot_dim > d.head_pitch)
     return cudaErrorInvalidValue;
   if (latent_attention_tensor_cores(d)) {
-    if (d.kvp <= 128) return launch_mma<2>(d, s);
-    if (d.kvp <= 256) return launch_mma<4>(d, s);
-    return launch_mma<8>(d, s);
+    if (d.kvp <= 128) return launch_mma<1>(d, s);
+    if (d.kvp <= 256) return launch_mma<2>(d, s);
+    return launch_mma<4>(d, s);
   }
   const size_t smem = (size_t)(2 * d.kvp + d.rp) * sizeof(float);
   if (smem > 40 * 1024) return cudaErrorInvalidValue;
@@ -573,7 +592,7 @@ cudaError_t latent_attention(const LatentAttn& d, cudaStream_t s) {
 cudaError_t latent_values(bool f32, const float* ml, const float* acc, int rows, int heads, int splits, int kvp,
                           const void* Wuv, int vp, void* y, long long ldy, bool pdl, const NextWeights& next,
                           cudaStream_t s) {
-  if (rows <= 0 || rows > 65535 || heads <= 0 || heads > 65535 || splits <= 0 || kvp <= 0 || (kvp & 7) || vp <= 0 || kvp > 10240)
+  if (rows <= 0 || rows > 65535 || heads <= 0 || heads > 65535 || splits <= 0 || splits > MAX_SPLITS || kvp <= 0 || (kvp & 7) || vp <= 0 || kvp > 10240)
     return cudaErrorInvalidValue;
   const dim3 grid((vp + 31) / 32, heads, rows);
   const size_t smem = (size_t)kvp * sizeof(float);

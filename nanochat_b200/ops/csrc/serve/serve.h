@@ -1,5 +1,5 @@
-// Host interface of the serving kernels: rows.cu (norms, gated residual, activations, matrix-vector products),
-// latent.cu (latent attention over a paged store) and experts.cu (mixture of experts).
+// Host interface of the serving kernels: rows.cu (norms, gated residual, activations), gemv.cu (matrix-vector products of
+// a decode step), latent.cu (latent attention over a paged store) and experts.cu (mixture of experts).
 //
 // Conventions. "f32" selects float or bf16 for the typed pointers (weights and activations share one type). The
 // residual stream, gates' biases, norm weights, router logits and attention partials are always float. Row sizes and
@@ -49,19 +49,19 @@ cudaError_t gated_residual_norm(bool f32, float* x, const GatedTerm* terms, int 
                                 const float* w, float eps, int rows, int n, int np, void* h, cudaStream_t s);
 
 // out[r] = c[0] N(z) + c[1] N(z^2) + c[2] N(z^3) + c[3], N(v) = v / rms(v) over the row's n entries.
-cudaError_t poly_norm(bool f32, const void* z, long long ldz, const float* coef, float eps, int rows, int n, int np,
+cudaError_t poly_norm(bool f32, bool z_f32, const void* z, long long ldz, const float* coef, float eps, int rows, int n, int np,
                       void* out, long long ldo, cudaStream_t s);
 
+// ------------------------------------------------------------------------------ gemv.cu
 // Matrix-vector products of a decode step, bf16 weights, rows <= 8: out[b, j] = epilogue(sum_k pre(x)[b, k] W[j, k]).
 enum GemvPre : int {
   PRE_NORM = 0,     // x float, x / rms(x) * w
   PRE_PLAIN = 1,    // x bf16
-  PRE_POLY = 2,     // x float, the poly_norm activation with coefficients `w` (4)
 };
 enum GemvEpi : int {
   GEMV_STORE_F32 = 0,
   GEMV_STORE_BF16 = 1,
-  GEMV_RESIDUAL = 2,     // resid[b, j] += mult * sigmoid(g[b, j] + bias[j]) * value (+ extra[b, j])
+  GEMV_RESIDUAL = 2,     // resid[b, j] (+)= mult * sigmoid(g[b, j] + bias[j]) * value (+ extra[b, j])
 };
 struct LatentStore {     // see latent_store below; used by the extra CTAs of a product that also appends to the store
   const void* z; long long ldz;
@@ -71,16 +71,29 @@ struct LatentStore {     // see latent_store below; used by the extra CTAs of a 
 };
 struct GemvDesc {
   const void* x; long long ldx;
-  const float* w; float eps; int n_real;            // norm weight / coefficients, entries of the row that count
+  const float* w; float eps; int n_real;            // norm weight, entries of the row that count
   const void* W; long long ldw;
   int rows, N, K;
   void* out; long long ldo;
   float* resid; long long ldr; const float* g; long long ldg; const float* bias; float mult; const float* extra;
+  bool accumulate;                                  // GEMV_RESIDUAL: add to resid, or overwrite it
   void* h_out; long long ldh;                       // PRE_NORM: the normed row as bf16, when wanted
   NextWeights next;
   const LatentStore* store;                         // PRE_NORM only
+  bool pdl;
 };
 cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s);
+// The experts of a decode step, rows <= 8: out[b] = mult * sigmoid(g + bias) * sum_k wt[b, k] expert(idx[b, k])(h[b]) (+ extra).
+// act: rows * top x fp scratch.
+struct ExpertRows {
+  const void* h; long long ldh; int rows, top, experts, K, fp, N;
+  const void* Wgu; const void* Wdown;
+  const int* idx; const float* wt;
+  void* act;
+  float* out; long long ldo; const float* g; long long ldg; const float* bias; float mult; const float* extra;
+};
+bool expert_rows_supported(int rows, int top);
+cudaError_t expert_rows(const ExpertRows& d, cudaStream_t s);
 
 // ---------------------------------------------------------------------------- latent.cu
 // Per row: cq = norm(z[:q_rank]) (when asked), and the entry [norm(z[c_off:c_off+kv_rank]) | rotated z[rot_off:]]
@@ -138,23 +151,19 @@ cudaError_t gather_groups(const void* h, long long ldh, int rows, int top, int n
 cudaError_t silu_mul(const void* gu, int rows, int fp, const int* tile_group, void* act, cudaStream_t s);
 
 // Experts as matrix-vector products, one per (row, chosen expert). Wgu: experts x [gate fp rows | up fp rows] x K.
-// Either idx / wt hold the routing, or `logits` is given and it is worked out here.
 struct Routing {
-  const int* idx; const float* wt;
-  const float* logits; long long ld;
+  const int* idx; const float* wt;      // rows x top
   int experts, top;
 };
 cudaError_t expert_gate_up(bool f32, const void* h, long long ldh, int rows, int K, const void* Wgu, int fp,
-                           const Routing& rt, void* act, bool pdl, const NextWeights& next, cudaStream_t s);
-// y[r] = sum_k wt[r, k] Wdown[idx[r, k]] act[r * top + k]; with resid: resid[r] += mult * sigmoid(g + bias) * that (+ extra).
+                           const Routing& rt, void* act, cudaStream_t s);
+// y[r] = sum_k wt[r, k] Wdown[idx[r, k]] act[r * top + k]
 struct ExpertDown {
   bool f32;
   const void* act; int rows, fp;
   const void* Wdown; int N;
   Routing rt;
   void* y; long long ldy;
-  float* resid; long long ldr; const float* g; long long ldg; const float* bias; float mult; const float* extra;
-  bool pdl; NextWeights next;
 };
 cudaError_t expert_down(const ExpertDown& d, cudaStream_t s);
 

@@ -331,6 +331,8 @@ def bench_serve(T=2048, C=1664, window=512, ctx=1024):
         lens = torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
         xb, wq, ob = r(B, C), [r(3 * C, C) for _ in range(L)], e(B, 3 * C)
         add(f"gpt gemv (QKV), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, ob, None, 0, True, None) for a in wq]), nbytes=2.0 * 3 * C * C, key=f"gemv{B}")
+        wp, op, aux = [r(C, C) for _ in range(L)], e(B, C), r(B, C)
+        add(f"gpt gemv (attention out), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, op, aux, 0, False, None) for a in wp]), nbytes=2.0 * C * C, key=f"gemvo{B}")
         n_all = n_in
         wa, zb, xf = [r(n_all, C) for _ in range(L)], e(B, n_all, dtype=f32), r(B, C, dtype=f32)
         add(f"norm + input projection, {B} rows", _time_chain([lambda a=a: K.gemv_norm(xf, wn, 1e-6, C, a, zb) for a in wa]), nbytes=2.0 * n_all * C, like=f"gemv{B}")
@@ -340,9 +342,9 @@ def bench_serve(T=2048, C=1664, window=512, ctx=1024):
         table = torch.arange(B * pg, dtype=torch.int32, device=dev).view(B, pg).contiguous()
         wqs, qb = [r(H * (D + D2), 1280) for _ in range(L)], e(B, H * (D + D2))
         add(f"query projection + store, {B} rows", _time_chain([lambda a=a, p=p: K.gemv_query_store(zb, 1280, qw, 1e-6, a, qb, 1280, KV, KV, kw, 1280 + KV, D2, freq, p, table, lens)
-                                                                 for a, p in zip(wqs, pools)]), nbytes=2.0 * 1280 * H * (D + D2), like=f"gemv{B}")
+                                                                 for a, p in zip(wqs, pools)]), nbytes=2.0 * 1280 * H * (D + D2), like=f"gemvo{B}")
         wkv, qa, yb = [r(H * (D + DV), KV) for _ in range(L)], e(B, H, KV), e(B, H * DV)
-        add(f"absorb queries, {B} rows", _time_chain([lambda a=a: K.absorb_query(qb, H, a[:H * D], qa, True) for a in wkv]), nbytes=2.0 * H * D * KV, like=f"gemv{B}")
+        add(f"absorb queries, {B} rows", _time_chain([lambda a=a: K.absorb_query(qb, H, a[:H * D], qa, True) for a in wkv]), nbytes=2.0 * H * D * KV, like=f"gemvo{B}")
         k4 = [torch.randn(B * pg, P, H, 128, device=dev).to(bf16) for _ in range(L)]
         scratch, yg4, qg = torch.zeros(N.decode_attn_scratch(B, H), device=dev), e(B, H * 128), r(B, H * 128)
         add(f"gpt decode attention, {window} keys, {B} rows", _time_chain([lambda a=a: N.decode_attn(qg, a, a, lens, H, H, window - 1, 0.088, scratch, yg4, table) for a in k4]),
@@ -354,19 +356,19 @@ def bench_serve(T=2048, C=1664, window=512, ctx=1024):
         ml, acc = e(B, H, splits, 2, dtype=f32), e(B, H, splits, KV, dtype=f32)
         add(f"latent attention, {window} keys, {B} rows", _time_chain([lambda p=p: K.latent_attention(qa, qb, H, D, D2, freq, KV, p, table, lens, 1, window, 0.07, splits, ml, acc, True) for p in pools]),
             nbytes=2.0 * B * window * (KV + D2), flops=2.0 * B * window * H * (2 * KV + D2), like=f"dattn{B}")
-        add(f"merge splits + values, {B} rows", _time_chain([lambda a=a: K.latent_values(ml, acc, B, H, splits, a[H * D:], yb, True) for a in wkv]), nbytes=2.0 * H * DV * KV, like=f"gemv{B}")
+        add(f"merge splits + values, {B} rows", _time_chain([lambda a=a: K.latent_values(ml, acc, B, H, splits, a[H * D:], yb, True) for a in wkv]), nbytes=2.0 * H * DV * KV, like=f"gemvo{B}")
         wo, gb = [r(C, H * DV) for _ in range(L)], zb[:, :C]
-        wp, op, aux = [r(C, C) for _ in range(L)], e(B, C), r(B, C)
-        add(f"gpt gemv (attention out), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, op, aux, 0, False, None) for a in wp]), nbytes=2.0 * C * C, key=f"gemvo{B}")
-        add(f"output projection + gated residual, {B} rows", _time_chain([lambda a=a: K.gemv_residual(yb, None, 1e-6, 0, a, xf, gb, bias, 0.7) for a in wo]), nbytes=2.0 * C * H * DV, like=f"gemvo{B}")
-        wdn, zz = [r(C, 4 * C) for _ in range(L)], zb[:, :4 * C]
-        hb = r(B, 4 * C)
+        add(f"output projection + gated residual, {B} rows", _time_chain([lambda a=a: K.gemv_residual(yb, a, xf, gb, bias, 0.7) for a in wo]), nbytes=2.0 * C * H * DV, like=f"gemvo{B}")
+        wdn, zz, az = [r(C, 4 * C) for _ in range(L)], zb[:, :4 * C], e(B, 4 * C)
+        hb, ff = r(B, 4 * C), e(B, C, dtype=f32)
         add(f"gpt gemv (MLP down), {B} rows", _time_chain([lambda a=a: N.gemv_rows(hb, a, op, aux, 0, False, None) for a in wdn]), nbytes=2.0 * 4 * C * C, key=f"gemvd{B}")
-        add(f"activation + down + gated residual, {B} rows", _time_chain([lambda a=a: K.gemv_residual(zz, coef, 1e-6, 4 * C, a, xf, gb, bias, 0.7) for a in wdn]), nbytes=2.0 * 4 * C * C, like=f"gemvd{B}")
+        add(f"activation, then down + gate, {B} rows", _time_chain([lambda a=a: (K.poly_norm(zz, coef, 1e-6, 4 * C, az), K.gemv_residual(az, a, ff, gb, bias, 0.7, accumulate=False)) for a in wdn]),
+            nbytes=2.0 * 4 * C * C, like=f"gemvd{B}")
         lbs, hb, ab = [r(B, E, dtype=f32) for _ in range(L)], r(B, C), e(B * TOP, FF)       # other experts in every call
+        ids, wts = torch.empty(B, TOP, dtype=torch.int32, device=dev), e(B, TOP, dtype=f32)
         used = min(B * TOP, E * (1 - (1 - TOP / E) ** B))      # experts a step reads, on average
-        add(f"experts' gate and up, {B} rows", _time_chain([lambda l=l: K.expert_gate_up(hb, wgu, TOP, None, None, l, ab, True) for l in lbs]), nbytes=2.0 * used * 2 * FF * C, like=f"gemvd{B}")
-        add(f"experts' down + gated residual, {B} rows", _time_chain([lambda l=l: K.expert_down_residual(ab, wd, TOP, l, xf, gb, bias, 0.7) for l in lbs]), nbytes=2.0 * used * FF * C, like=f"gemvd{B}")
+        add(f"routing + experts, {B} rows", _time_chain([lambda l=l: (K.route_topk(l, E, ids, wts), K.expert_rows(hb, wgu, wd, ids, wts, ab, ff, gb, bias, 0.7)) for l in lbs]),
+            nbytes=2.0 * used * 3 * FF * C, like=f"gemvd{B}")
     sv.check_status()
     nat.check_status()
     return rows

@@ -150,7 +150,7 @@ def mixture(h, p):
         idx, wt = route(h, p)
         act = torch.empty(R * p.top, p.fp, dtype=h.dtype, device=h.device)
         y = torch.empty(R, h.shape[1], dtype=h.dtype, device=h.device)
-        _S.expert_gate_up(h, p.w_gate_up, p.top, idx, wt, None, act, False)
+        _S.expert_gate_up(h, p.w_gate_up, idx, wt, act)
         _S.expert_down(act, p.w_down, idx, wt, y)
         return (y,)
     logits = linear_rows(h, p.router, torch.float32)

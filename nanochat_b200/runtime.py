@@ -227,12 +227,14 @@ class DecodeGraph(StepGraph):
 class LatentDecodeGraph(StepGraph):
     """Decode step of models over a paged latent store (`make_cache`).
 
-    Up to GEMV_ROWS bf16 rows: a fixed chain of serving kernels, 7 per layer with a dense feed-forward and 8 with experts,
+    Up to GEMV_ROWS bf16 rows: a fixed set of serving kernels per layer. Both sublayers read the same normed rows, so after
+    the product that reads them the feed-forward runs beside the attention on a second stream; kernels of one stream are
     launched so that each may start while the one before it ends:
-        norm + everything that reads it (down-projections, gates, up-projection, router)  ->  query latent's norm + query
-        projection, extra CTAs append to the store  ->  absorbed queries  ->  attention, split over keys  ->  splits merged
-        + value projection  ->  output projection + gated residual  ->  [experts' gate and up, routing worked out on the
-        spot ->] activation + down projection + gated residual
+        norm + everything that reads it (down-projections, gates, up-projection, router)
+        main: query latent's norm + query projection, extra CTAs append to the store  ->  absorbed queries  ->  attention,
+              split over keys  ->  splits merged + value projection
+        side: activation  ->  down projection + gate;   or routing  ->  experts' gate and up  ->  experts' down + gate
+        join: output projection + gated residual, the side's result added
     Otherwise (more rows, or float32): the model's forward over the rows, captured as it is."""
 
     def __init__(self, model, kv_cache):
@@ -241,7 +243,8 @@ class LatentDecodeGraph(StepGraph):
         self.S = S
         cfg, B, dev = model.config, self.B, kv_cache.cache_seqlens.device
         self.logits = torch.empty(B, model.embed.shape[0], dtype=torch.float32, device=dev)[:, :cfg.vocab_size]
-        self.fused = B <= GEMV_ROWS and model.dtype == torch.bfloat16
+        self.fused = (B <= GEMV_ROWS and model.dtype == torch.bfloat16 and
+                      all(S._S.expert_rows_supported(B, getattr(layer.mlp, "top", 1)) for layer in model.layers))
         if not self.fused:
             return
         f32 = lambda *shape: torch.empty(*shape, dtype=torch.float32, device=dev)
@@ -256,7 +259,12 @@ class LatentDecodeGraph(StepGraph):
         self.q = b16(B * most(lambda l: l.attn.w_q.shape[0]))
         self.qa = b16(B * most(lambda l: l.attn.heads * l.attn.kvp))
         self.y = b16(B * most(lambda l: l.attn.heads * l.attn.vp))
-        self.act = b16(B * most(lambda l: l.mlp.top * l.mlp.fp if hasattr(l.mlp, "top") else 8))
+        self.act = b16(B * most(lambda l: 8 if l.mlp is None else l.mlp.fp * getattr(l.mlp, "top", 1)))
+        self.ff = f32(B, model.width)                      # the feed-forward's gated contribution to the stream
+        tops = [getattr(l.mlp, "top", 1) for l in layers] + [1]
+        self.idx = torch.empty(B * max(tops), dtype=torch.int32, device=dev)
+        self.wt = f32(B * max(tops))
+        self.side = torch.cuda.Stream(device=dev)
         self.splits = [S.attention_splits(l.attn, B, min(kv_cache.max_seq_len, l.attn.window or kv_cache.max_seq_len), True)
                        for l in layers]
         self.ml = f32(max([B * l.attn.heads * s * 2 for l, s in zip(layers, self.splits)] + [2]))
@@ -285,7 +293,21 @@ class LatentDecodeGraph(StepGraph):
             moe = hasattr(mlp, "top")
             z = view(self.z, layer.w_all.shape[0])
             q, qa, y = view(self.q, a.w_q.shape[0]), view(self.qa, a.heads * a.kvp), view(self.y, a.heads * a.vp)
+            gate = lambda k: z[:, layer.gates[k]:layer.gates[k] + m.width]
             K.gemv_norm(x, layer.norm, eps, C, layer.w_all, z, self.h if moe else None, ahead(a.w_q))
+            if mlp is not None:
+                main = torch.cuda.current_stream()
+                self.side.wait_stream(main)
+                with torch.cuda.stream(self.side):
+                    if moe:
+                        idx, wt = (view(t, mlp.top) for t in (self.idx, self.wt))
+                        K.route_topk(z[:, layer.n_in:], mlp.experts, idx, wt)
+                        act = self.act[:B * mlp.top * mlp.fp].view(B * mlp.top, mlp.fp)
+                        K.expert_rows(self.h, mlp.w_gate_up, mlp.w_down, idx, wt, act, self.ff, gate(1), layer.rg2_bias, mult, extra)
+                    else:
+                        act = view(self.act, mlp.fp)
+                        K.poly_norm(z[:, layer.up_off:layer.n_in], mlp.act, eps, mlp.ff, act)
+                        K.gemv_residual(act, mlp.w_down, self.ff, gate(1), layer.rg2_bias, mult, extra, accumulate=False)
             K.gemv_query_store(z, a.q_rank, a.q_norm, eps, a.w_q, q, a.c_off, a.kv_rank, a.kvp, a.kv_norm, a.rot_off,
                                a.rot_dim, a.freq, cache.pools[run], table, lens, ahead(a.w_kv))
             K.absorb_query(q, a.heads, a.w_uk, qa, True)
@@ -293,17 +315,11 @@ class LatentDecodeGraph(StepGraph):
             K.latent_attention(qa, q, a.heads, a.dp, a.rot_dim, a.freq, a.kvp, cache.pools[run], table, lens, 1,
                                a.window or 0, a.scale, splits, self.ml, self.acc, True)
             K.latent_values(self.ml, self.acc, B, a.heads, splits, a.w_uv, y, True, ahead(a.w_o))
-            gate = lambda k: z[:, layer.gates[k]:layer.gates[k] + m.width]
-            K.gemv_residual(y, None, eps, 0, a.w_o, x, gate(0), layer.rg1_bias, mult, None if mlp is not None else extra,
-                            ahead(mlp.w_down if mlp is not None and not moe else None))
-            if moe:
-                act = self.act[:B * mlp.top * mlp.fp].view(B * mlp.top, mlp.fp)
-                logits = z[:, layer.n_in:]
-                K.expert_gate_up(self.h, mlp.w_gate_up, mlp.top, None, None, logits, act, True)
-                K.expert_down_residual(act, mlp.w_down, mlp.top, logits, x, gate(1), layer.rg2_bias, mult, extra)
-            elif mlp is not None:
-                K.gemv_residual(z[:, layer.up_off:layer.n_in], mlp.act, eps, mlp.ff, mlp.w_down, x, gate(1), layer.rg2_bias,
-                                mult, extra)
+            if mlp is not None:
+                main.wait_stream(self.side)
+            after = m.runs[run + 1][0].w_all if run + 1 < len(m.runs) else m.embed[:LM_HEAD_PREFETCH_ROWS]
+            K.gemv_residual(y, a.w_o, x, gate(0), layer.rg1_bias, mult, extra if mlp is None else self.ff, ahead(after),
+                            pdl=mlp is None)
         K.gemv_norm(x, m.final_norm, eps, C, m.embed, self.all_logits)
 
 
