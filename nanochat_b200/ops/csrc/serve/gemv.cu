@@ -262,10 +262,12 @@ expert_gate_up_rows_kernel(const ExpertArgs a) {
   float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
   const bf16* h = a.in + (long long)(lane >> 2) * a.ldin;
   auto x = [&](int k) -> uint4 { return choice >= 0 ? *reinterpret_cast<const uint4*>(h + k) : make_uint4(0, 0, 0, 0); };
-  Frag<2, U> f;
+  Frag<2, U> cur, nxt;
+  load_frag(cur, w, warp * 32, q8, a.K);
   for (int k0 = warp * 32; k0 < a.K; k0 += U * WARPS * 32) {
-    load_frag(f, w, k0, q8, a.K);
-    mma_frag(acc, f, k0, q8, a.K, x);
+    if (k0 + U * WARPS * 32 < a.K) load_frag(nxt, w, k0 + U * WARPS * 32, q8, a.K);
+    mma_frag(acc, cur, k0, q8, a.K, x);
+    cur = nxt;
   }
   spill_tiles<2>(acc, s_acc, warp, lane);
   __syncthreads();
@@ -283,7 +285,7 @@ expert_gate_up_rows_kernel(const ExpertArgs a) {
 // grid (ceil(N / 16)): out[b] = mult * sigmoid(g + bias) * sum over the row's experts (+ extra)
 __global__ void __launch_bounds__(THREADS)
 expert_down_rows_kernel(const ExpertArgs a) {
-  constexpr int U = 2;
+  constexpr int U = 4;
   __shared__ Choices c;
   __shared__ float s_acc[WARPS][16][ROWS + 1];
   __shared__ short s_list[MAX_CHOICES];                 // first mentions, in order

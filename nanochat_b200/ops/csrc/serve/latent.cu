@@ -76,38 +76,49 @@ latent_gather_kernel(const Pages pg, int seq, int first, T* out, long long ldo, 
   }
 }
 
-// one thread per (row, head, V pairs)
-template <typename T, int V>
+// one thread per (row, V pairs, G heads): the angles are worked out once for its heads
+template <typename T, int V, int G>
 __global__ void __launch_bounds__(128)
 rotate_heads_kernel(T* __restrict__ q, long long ldq, int rows, int heads, int head_pitch, int off, int half,
                     const float* __restrict__ freq, RowPos rp) {
-  const int chunks = half / V;
+  const int chunks = half / V, groups = (heads + G - 1) / G;
   const long long t = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  const int i = (int)(t % chunks) * V, h = (int)(t / chunks % heads), row = (int)(t / ((long long)chunks * heads));
+  const int i = (int)(t % chunks) * V, h0 = (int)(t / chunks % groups) * G, row = (int)(t / ((long long)chunks * groups));
   if (row >= rows) return;
   int seq;
   const int pos = row_position(rp, row, seq);
-  T* p = q + row * ldq + (long long)h * head_pitch + off + i;
-  float a[V], b[V];
-  if constexpr (V == 8) {
-    load8(p, a);
-    load8(p + half, b);
-  } else {
-    a[0] = to_f(p[0]); b[0] = to_f(p[half]);
+  T* p = q + row * ldq + (long long)h0 * head_pitch + off + i;
+  float a[G][V], b[G][V];
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    if (h0 + g >= heads) continue;
+    if constexpr (V == 8) {
+      load8(p + g * head_pitch, a[g]);
+      load8(p + g * head_pitch + half, b[g]);
+    } else {
+      a[g][0] = to_f(p[g * head_pitch]); b[g][0] = to_f(p[g * head_pitch + half]);
+    }
   }
 #pragma unroll
   for (int j = 0; j < V; ++j) {
     float sn, cs;
     sincosf((float)pos * freq[i + j], &sn, &cs);
-    const float u = a[j], v = b[j];
-    a[j] = u * cs - v * sn;
-    b[j] = v * cs + u * sn;
+#pragma unroll
+    for (int g = 0; g < G; ++g) {
+      const float u = a[g][j], v = b[g][j];
+      a[g][j] = u * cs - v * sn;
+      b[g][j] = v * cs + u * sn;
+    }
   }
-  if constexpr (V == 8) {
-    store8(p, a);
-    store8(p + half, b);
-  } else {
-    p[0] = from_f<T>(a[0]); p[half] = from_f<T>(b[0]);
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    if (h0 + g >= heads) continue;
+    if constexpr (V == 8) {
+      store8(p + g * head_pitch, a[g]);
+      store8(p + g * head_pitch + half, b[g]);
+    } else {
+      p[g * head_pitch] = from_f<T>(a[g][0]); p[g * head_pitch + half] = from_f<T>(b[g][0]);
+    }
   }
 }
 
@@ -446,22 +457,25 @@ latent_attention_mma_kernel(const LatentAttn d) {
   }
 }
 
-// grid (ceil(vp / 32), heads, rows), 256 threads; dynamic shared memory: kvp floats
+// grid (ceil(vp / 16), heads, rows), 256 threads, two outputs per warp; dynamic shared memory: kvp floats
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_values_kernel(const float* __restrict__ ml, const float* __restrict__ acc, int heads, int splits, int kvp,
                      const T* __restrict__ Wuv, int vp, T* __restrict__ y, long long ldy, NextWeights next) {
+  constexpr int OUT = 2, AHEAD = 2;                 // outputs per warp, 256-column chunks requested before the wait
   extern __shared__ float lat[];
   __shared__ float s_w[MAX_SPLITS];
   const int h = blockIdx.y, row = blockIdx.z;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int j0 = blockIdx.x * 32 + warp * 4;
+  const int j0 = blockIdx.x * (8 * OUT) + warp * OUT;
   prefetch_l2_slice(next, blockIdx.x + (long long)gridDim.x * blockIdx.y, (long long)gridDim.x * gridDim.y);
-  const T* w = Wuv + ((long long)h * vp + j0) * kvp;
-  Raw8<T> first[4];
+  const T* w = Wuv + ((long long)h * vp + j0) * kvp + lane * 8;
+  Raw8<T> first[AHEAD][OUT];
 #pragma unroll
-  for (int r = 0; r < 4; ++r)
-    if (j0 + r < vp && lane * 8 < kvp) first[r] = raw8(w + (long long)r * kvp + lane * 8);
+  for (int i = 0; i < AHEAD; ++i)
+#pragma unroll
+    for (int r = 0; r < OUT; ++r)
+      if (j0 + r < vp && i * 256 + lane * 8 < kvp) first[i][r] = raw8(w + (long long)r * kvp + i * 256);
   pdl_wait();
   pdl_trigger();
   const long long slot = ((long long)row * heads + h) * splits;
@@ -484,20 +498,25 @@ latent_values_kernel(const float* __restrict__ ml, const float* __restrict__ acc
     lat[c] = v;
   }
   __syncthreads();
-  float sum[4] = {0.f, 0.f, 0.f, 0.f};
-  for (int c = lane * 8; c < kvp; c += 256) {
+  float sum[OUT] = {0.f, 0.f};
+  auto dot = [&](const Raw8<T>& raw, int r, int c) {
+    float f[8];
+    unraw8(raw, f);
 #pragma unroll
-    for (int r = 0; r < 4; ++r) {
-      if (j0 + r < vp) {
-        float f[8];
-        unraw8(c < 256 ? first[r] : raw8(w + (long long)r * kvp + c), f);
+    for (int i = 0; i < 8; ++i) sum[r] += f[i] * lat[c + lane * 8 + i];
+  };
 #pragma unroll
-        for (int i = 0; i < 8; ++i) sum[r] += f[i] * lat[c + i];
-      }
-    }
+  for (int i = 0; i < AHEAD; ++i)
+#pragma unroll
+    for (int r = 0; r < OUT; ++r)
+      if (j0 + r < vp && i * 256 + lane * 8 < kvp) dot(first[i][r], r, i * 256);
+  for (int c = AHEAD * 256; c + lane * 8 < kvp; c += 256) {
+#pragma unroll
+    for (int r = 0; r < OUT; ++r)
+      if (j0 + r < vp) dot(raw8(w + (long long)r * kvp + c), r, c);
   }
 #pragma unroll
-  for (int r = 0; r < 4; ++r) {
+  for (int r = 0; r < OUT; ++r) {
     const float v = warp_sum(sum[r]);
     if (lane == 0 && j0 + r < vp) y[row * ldy + (long long)h * vp + j0 + r] = from_f<T>(v);
   }
@@ -536,13 +555,14 @@ cudaError_t rotate_heads(bool f32, void* q, long long ldq, int rows, int heads, 
   if (dims == 0) return cudaSuccess;
   const int half = dims / 2;
   const bool vec = half % 8 == 0 && off % 8 == 0 && head_pitch % 8 == 0 && ldq % 8 == 0;
-  const long long n = (long long)rows * heads * (half / (vec ? 8 : 1));
+  constexpr int G = 4;
+  const long long n = (long long)rows * ((heads + G - 1) / G) * (half / (vec ? 8 : 1));
   const dim3 grid((unsigned)((n + 127) / 128));
   if (f32) {
-    auto k = vec ? rotate_heads_kernel<float, 8> : rotate_heads_kernel<float, 1>;
+    auto k = vec ? rotate_heads_kernel<float, 8, G> : rotate_heads_kernel<float, 1, G>;
     k<<<grid, 128, 0, s>>>((float*)q, ldq, rows, heads, head_pitch, off, half, freq, pos);
   } else {
-    auto k = vec ? rotate_heads_kernel<bf16, 8> : rotate_heads_kernel<bf16, 1>;
+    auto k = vec ? rotate_heads_kernel<bf16, 8, G> : rotate_heads_kernel<bf16, 1, G>;
     k<<<grid, 128, 0, s>>>((bf16*)q, ldq, rows, heads, head_pitch, off, half, freq, pos);
   }
   return cudaGetLastError();
@@ -594,7 +614,7 @@ cudaError_t latent_values(bool f32, const float* ml, const float* acc, int rows,
                           cudaStream_t s) {
   if (rows <= 0 || rows > 65535 || heads <= 0 || heads > 65535 || splits <= 0 || splits > MAX_SPLITS || kvp <= 0 || (kvp & 7) || vp <= 0 || kvp > 10240)
     return cudaErrorInvalidValue;
-  const dim3 grid((vp + 31) / 32, heads, rows);
+  const dim3 grid((vp + 15) / 16, heads, rows);
   const size_t smem = (size_t)kvp * sizeof(float);
   if (f32) return launch(pdl, latent_values_kernel<float>, grid, dim3(256), smem, s, ml, acc, heads, splits, kvp, (const float*)Wuv, vp, (float*)y, ldy, next);
   return launch(pdl, latent_values_kernel<bf16>, grid, dim3(256), smem, s, ml, acc, heads, splits, kvp, (const bf16*)Wuv, vp, (bf16*)y, ldy, next);
