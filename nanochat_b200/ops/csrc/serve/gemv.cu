@@ -8,7 +8,11 @@
 //
 //   gemv            one product; input norm (linear once the row statistic is known: the statistic rides along), gated
 //                   residual update of the output, extra CTAs that append the step's entries to the latent store
-//   expert_*_rows   a step's experts: every chosen expert's weights are read once for all rows that chose it
+//                   Few outputs and a long K: four CTAs of a cluster share K and add up over distributed shared memory
+//   expert_*_rows   a step's experts: every chosen expert's weights are read once for all rows that chose it (down: the
+//                   four CTAs of a cluster take every fourth expert)
+#include <cooperative_groups.h>
+
 #include "latent_store.cuh"
 
 namespace nc {
@@ -89,6 +93,29 @@ __device__ __forceinline__ void spill_tiles(const float (&acc)[MT][4], float (*s
   }
 }
 
+constexpr int CLUSTER = 4;
+
+// The CTA's tile (outputs x rows), summed over its warps, then over the cluster; the result is valid in the cluster's first
+// CTA. All threads of all CTAs of the cluster call this.
+template <int M>
+__device__ __forceinline__ float cluster_total(float (*s_acc)[M][ROWS + 1], float (*s_part)[ROWS], bool mine, int m, int b) {
+  namespace cg = cooperative_groups;
+  cg::cluster_group cluster = cg::this_cluster();
+  float v = 0.f;
+  if (mine) {
+#pragma unroll
+    for (int i = 0; i < WARPS; ++i) v += s_acc[i][m][b];
+    s_part[m][b] = v;
+  }
+  cluster.sync();
+  if (mine && cluster.block_rank() == 0) {
+#pragma unroll
+    for (int r = 1; r < CLUSTER; ++r) v += cluster.map_shared_rank(&s_part[0][0], r)[m * ROWS + b];
+  }
+  cluster.sync();                       // the others' shared memory stays until it has been read
+  return v;
+}
+
 struct GemvArgs {
   const void* x; long long ldx;
   const float* w; float eps; int n_real;
@@ -102,10 +129,13 @@ struct GemvArgs {
   int n_blocks;
 };
 
-template <bool NORM, int MT>
-__global__ void __launch_bounds__(THREADS)
-gemv_kernel(const GemvArgs a) {
+// SPLIT: CTAs of a cluster (grid y) that share K; 1 or CLUSTER
+template <bool NORM, int MT, int SPLIT>
+__device__ __forceinline__ void gemv_body(const GemvArgs& a) {
+  static_assert(SPLIT == 1 || (!NORM && SPLIT == CLUSTER), "only plain products share K");
   constexpr int U = MT == 1 ? 4 : 2;
+  constexpr int STEP = U * WARPS * 32;
+  __shared__ float s_part[SPLIT > 1 ? MT * 16 : 1][ROWS];
   __shared__ float s_acc[WARPS][MT * 16][ROWS + 1];
   __shared__ float s_ss[WARPS][ROWS];
   __shared__ float s_red[32];
@@ -127,10 +157,11 @@ gemv_kernel(const GemvArgs a) {
     return;
   }
   const int n0 = blockIdx.x * (MT * 16), q8 = (lane & 3) * 8, row = lane >> 2;
-  prefetch_l2_slice(a.next, blockIdx.x, a.n_blocks);
+  if (SPLIT == 1 || blockIdx.y == 0) prefetch_l2_slice(a.next, blockIdx.x, a.n_blocks);
   const TileRows<MT> w = tile_rows<MT>(a.W, a.ldw, n0, a.N, lane);
   Frag<MT, U> f;
-  load_frag(f, w, warp * 32, q8, a.K);             // weights do not depend on the kernel before
+  const int k_first = warp * 32 + (SPLIT > 1 ? (int)blockIdx.y * STEP : 0);
+  load_frag(f, w, k_first, q8, a.K);               // weights do not depend on the kernel before
   pdl_wait();
   pdl_trigger();
   float acc[MT][4], ss = 0.f;
@@ -150,9 +181,9 @@ gemv_kernel(const GemvArgs a) {
     for (int j = 0; j < 8; ++j) { ss += v[j] * v[j]; v[j] *= nw[j]; }
     return make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
   };
-  for (int k0 = warp * 32; k0 < a.K;) {
+  for (int k0 = k_first; k0 < a.K;) {
     mma_frag(acc, f, k0, q8, a.K, x);
-    k0 += U * WARPS * 32;
+    k0 += SPLIT * STEP;
     if (k0 < a.K) load_frag(f, w, k0, q8, a.K);
   }
   spill_tiles<MT>(acc, s_acc, warp, lane);
@@ -181,12 +212,18 @@ gemv_kernel(const GemvArgs a) {
       }
     }
   }
+  const int m = tid & (MT * 16 - 1), b = tid / (MT * 16), n = n0 + m;
+  float v = 0.f;
+  if constexpr (SPLIT > 1) {
+    v = cluster_total<MT * 16>(s_acc, s_part, tid < MT * 16 * ROWS, m, b);
+    if (blockIdx.y != 0) return;
+  }
   if (tid < MT * 16 * ROWS) {
-    const int m = tid & (MT * 16 - 1), b = tid / (MT * 16), n = n0 + m;
     if (b < a.B && n < a.N) {
-      float v = 0.f;
+      if constexpr (SPLIT == 1) {
 #pragma unroll
-      for (int i = 0; i < WARPS; ++i) v += s_acc[i][m][b];
+        for (int i = 0; i < WARPS; ++i) v += s_acc[i][m][b];
+      }
       if (NORM) v *= scale(b);
       if (a.epi == GEMV_STORE_F32) {
         ((float*)a.out)[b * a.ldo + n] = v;
@@ -200,6 +237,12 @@ gemv_kernel(const GemvArgs a) {
       }
     }
   }
+}
+
+template <bool NORM, int MT>
+__global__ void __launch_bounds__(THREADS) gemv_kernel(const GemvArgs a) { gemv_body<NORM, MT, 1>(a); }
+__global__ void __cluster_dims__(1, CLUSTER, 1) __launch_bounds__(THREADS) gemv_cluster_kernel(const GemvArgs a) {
+  gemv_body<false, 1, CLUSTER>(a);
 }
 
 // ----------------------------------------------------------------------------- experts
@@ -282,12 +325,13 @@ expert_gate_up_rows_kernel(const ExpertArgs a) {
   }
 }
 
-// grid (ceil(N / 16)): out[b] = mult * sigmoid(g + bias) * sum over the row's experts (+ extra)
-__global__ void __launch_bounds__(THREADS)
+// grid (ceil(N / 16), CLUSTER), one cluster per 16 outputs: out[b] = mult * sigmoid(g + bias) * sum over the row's experts (+ extra)
+__global__ void __cluster_dims__(1, CLUSTER, 1) __launch_bounds__(THREADS)
 expert_down_rows_kernel(const ExpertArgs a) {
   constexpr int U = 4;
   __shared__ Choices c;
   __shared__ float s_acc[WARPS][16][ROWS + 1];
+  __shared__ float s_part[16][ROWS];
   __shared__ short s_list[MAX_CHOICES];                 // first mentions, in order
   __shared__ short s_pick[ROWS][MAX_CHOICES];           // the row's choice of that expert, or -1
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = a.B * a.top;
@@ -305,16 +349,17 @@ expert_down_rows_kernel(const ExpertArgs a) {
   const int n0 = blockIdx.x * 16, q8 = (lane & 3) * 8, row = lane >> 2;
   float acc[1][4] = {{0.f, 0.f, 0.f, 0.f}};
   // (expert, k) as one loop, the next fragment on its way while the current one is used
-  const int per = (a.K + U * WARPS * 32 - 1) / (U * WARPS * 32), steps = per * c.distinct;
+  const int per = (a.K + U * WARPS * 32 - 1) / (U * WARPS * 32), rank = blockIdx.y;
+  const int steps = per * ((c.distinct - rank + CLUSTER - 1) / CLUSTER);      // experts rank, rank + CLUSTER, ...
   auto fetch = [&](Frag<1, U>& f, int s) {
-    const int e = s / per, k0 = (s - e * per) * (U * WARPS * 32) + warp * 32;
+    const int t = s / per, e = rank + t * CLUSTER, k0 = (s - t * per) * (U * WARPS * 32) + warp * 32;
     load_frag(f, tile_rows<1>(a.W + (long long)c.idx[s_list[e]] * a.N * a.K, a.K, n0, a.N, lane), k0, q8, a.K);
   };
   Frag<1, U> cur, nxt;
   if (steps > 0) fetch(cur, 0);
   for (int s = 0; s < steps; ++s) {
     if (s + 1 < steps) fetch(nxt, s + 1);
-    const int e = s / per, k0 = (s - e * per) * (U * WARPS * 32) + warp * 32;
+    const int t = s / per, e = rank + t * CLUSTER, k0 = (s - t * per) * (U * WARPS * 32) + warp * 32;
     const int choice = row < a.B ? s_pick[row][e] : -1;
     const float wt = choice >= 0 ? a.wt[choice] : 0.f;
     const bf16* in = a.in + (long long)max(choice, 0) * a.K;
@@ -329,12 +374,10 @@ expert_down_rows_kernel(const ExpertArgs a) {
   }
   spill_tiles<1>(acc, s_acc, warp, lane);
   __syncthreads();
-  if (tid < 16 * ROWS) {
-    const int m = tid & 15, b = tid >> 4, j = n0 + m;
+  const int m = tid & 15, b = tid >> 4, j = n0 + m;
+  const float v = cluster_total<16>(s_acc, s_part, tid < 16 * ROWS, m, b);
+  if (rank == 0 && tid < 16 * ROWS) {
     if (b < a.B && j < a.N) {
-      float v = 0.f;
-#pragma unroll
-      for (int i = 0; i < WARPS; ++i) v += s_acc[i][m][b];
       float r = a.mult * sigmoidf(a.g[b * a.ldg + j] + a.bias[j]) * v;
       if (a.extra) r += a.extra[b * a.ldo + j];
       a.out[b * a.ldo + j] = r;
@@ -359,6 +402,7 @@ cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s) {
   a.n_blocks = (d.N + (wide ? 31 : 15)) / (wide ? 32 : 16);
   int grid = a.n_blocks;
   if (d.store) { a.store = *d.store; grid += d.rows; }
+  if (pre == PRE_PLAIN && !wide && a.n_blocks < 148 && d.K >= 3072) return launch(d.pdl, gemv_cluster_kernel, dim3(grid, CLUSTER), dim3(THREADS), 0, s, a);
   auto kern = pre == PRE_NORM ? (wide ? gemv_kernel<true, 2> : gemv_kernel<true, 1>) : (wide ? gemv_kernel<false, 2> : gemv_kernel<false, 1>);
   return launch(d.pdl, kern, dim3(grid), dim3(THREADS), 0, s, a);
 }
@@ -377,7 +421,7 @@ cudaError_t expert_rows(const ExpertRows& d, cudaStream_t s) {
   if (e != cudaSuccess) return e;
   a.in = (const bf16*)d.act; a.K = d.fp; a.N = d.N; a.W = (const bf16*)d.Wdown;
   a.out = d.out; a.ldo = d.ldo; a.g = d.g; a.ldg = d.ldg; a.bias = d.bias; a.mult = d.mult; a.extra = d.extra;
-  return launch(true, expert_down_rows_kernel, dim3((d.N + 15) / 16), dim3(THREADS), 0, s, a);
+  return launch(true, expert_down_rows_kernel, dim3((d.N + 15) / 16, CLUSTER), dim3(THREADS), 0, s, a);
 }
 
 }  // namespace serve
