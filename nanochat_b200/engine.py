@@ -141,7 +141,7 @@ PAGE_TOKENS = 64
 
 
 class _PromptView:
-    """The shared prompt pages of a paged cache seen as a batch-1 cache: what the prefill writes into. `layer_cache(i)`
+    """The shared prompt pages of a paged cache seen as a batch-1 cache: what the prefill writes into. `get_layer_cache`
     serves KVCache's surface; a latent cache's kernels use `pools` and `table` instead."""
 
     def __init__(self, owner, capacity):

@@ -359,7 +359,7 @@ int store_kind(GemvDesc& d, Tensor& out) {
   d.out = out.data_ptr(); d.ldo = out.stride(0);
   return is_f32(out) ? GEMV_STORE_F32 : GEMV_STORE_BF16;
 }
-// out = (x / rms(x) * w) W^T; h: the normed rows as bf16. `store`: see latent_store_args.
+// out = (x / rms(x) * w) W^T; h: the normed rows as bf16.
 void gemv_norm(const Tensor& x, const Tensor& w, double eps, int64_t n, const Tensor& W, Tensor& out, const optional<Tensor>& h,
                const optional<Tensor>& next) {
   GemvDesc d = gemv_of(x, W, next);
