@@ -23,6 +23,7 @@ row's page table points at, so forking N samples copies at most one partial page
 per row instead of the whole prompt, and N samples hold the prompt once.
 """
 
+import math
 import signal
 import warnings
 from collections import deque
@@ -336,7 +337,8 @@ class PagedLatentCache(PagedCache):
 
     def _copy_tokens(self, pages, source, n):
         for pool in self.pools:
-            pool[pages, :n] = pool[source:source + 1, :n]
+            if pool.shape[2]:
+                pool[pages, :n] = pool[source:source + 1, :n]
 
     def pool_bytes(self):
         return 0 if self.pools is None else sum(p.numel() * p.element_size() for p in self.pools)
@@ -344,6 +346,43 @@ class PagedLatentCache(PagedCache):
     def gather_row(self, run, row):
         """(T, width) entries of one row in position order (tests and debugging; copies)."""
         return self.pools[run][self._row_pages(row)].reshape(-1, self.widths[run])[:self._pos]
+
+
+class RecurrentCache(PagedLatentCache):
+    """A paged store for the layers that attend (`widths[run]` elements a token, 0: none) and, beside it, fixed-size float
+    states for the layers with a recurrence: `shapes[run]` names a layer's states and their shapes. All states of one
+    sequence are one row of memory; row `batch_size` belongs to the prompt, and `fork()` copies it to the others.
+
+    Nothing is cleared: kernels start a sequence at position 0 from zeros whatever its row holds."""
+
+    ALIGN = 32                                       # floats
+
+    def __init__(self, batch_size, widths, shapes, seq_len, device, dtype, page_tokens=PAGE_TOKENS):
+        super().__init__(batch_size, widths, seq_len, device, dtype, page_tokens)
+        places, total = [], 0
+        for names in shapes:
+            places.append({})
+            for name, shape in names.items():
+                n = math.prod(shape)
+                places[-1][name] = (total, n, shape)
+                total += -(-n // self.ALIGN) * self.ALIGN
+        self.memory = torch.zeros(batch_size + 1, max(total, self.ALIGN), device=device)
+        self.all_states = [{name: self.memory[:, at:at + n].unflatten(1, shape) for name, (at, n, shape) in p.items()} for p in places]
+        self.states = [{name: t[:batch_size] for name, t in p.items()} for p in self.all_states]
+        self.prompt_states = [{name: t[batch_size:] for name, t in p.items()} for p in self.all_states]
+        self.done = torch.zeros(batch_size, dtype=torch.int32, device=device)     # counters of the step kernels, zero between steps
+
+    def begin_prompt(self, prompt_tokens):
+        view = super().begin_prompt(prompt_tokens)
+        view.states, view.done = self.prompt_states, self.done[:1]
+        return view
+
+    def fork(self, view):
+        super().fork(view)
+        self.memory[:-1] = self.memory[-1]
+
+    def state_bytes(self):
+        return self.memory.numel() * self.memory.element_size()
 
 
 @torch.inference_mode()
@@ -377,7 +416,7 @@ class Sequence:
 
     def __init__(self, engine, max_tokens):
         self.engine, self.max_tokens, self.length = engine, max_tokens, 0
-        self.cache = engine._row_cache(1) if engine.latent or engine._graph_applies(1, max_tokens) else None
+        self.cache = engine._row_cache(1) if engine.own_cache or engine._graph_applies(1, max_tokens) else None
         if self.cache is None:                      # no captured decode here: a contiguous cache of its own
             self.cache = KVCache(batch_size=1, seq_len=max_tokens, **engine._kv_geometry())
         else:
@@ -400,7 +439,7 @@ class Sequence:
             if paged:
                 self.cache.fork(view)
             engine._begin_decode(self.cache)
-        elif n > 1 and engine.latent:
+        elif n > 1 and engine.own_cache:
             logits = engine._prompt_logits(ids, self.cache, want)
         else:
             rows = {}
@@ -425,7 +464,7 @@ class Engine:
         self.tokenizer = tokenizer
         self._decode_graphs = {}
         self._cache_pool = {}      # rows -> full-length cache reused across generations (keeps its decode graph)
-        self.latent = hasattr(model, "make_cache")      # the model brings its own paged store
+        self.own_cache = hasattr(model, "make_cache")      # the model brings its own paged store
 
     def open_sequence(self, max_tokens):
         """A request of up to `max_tokens` tokens to be fed in portions; see Sequence."""
@@ -433,7 +472,7 @@ class Engine:
 
     def _prompt_logits(self, ids, cache, want):
         """Run a portion of tokens; (len(want), V) logits at the places `want`, None when there are none."""
-        if self.latent:
+        if self.own_cache:
             return self.model.forward(ids, kv_cache=cache, want=list(want))
         logits = self.model.forward(ids, kv_cache=cache)[0]
         return logits[list(want)].float() if len(want) else None
@@ -504,7 +543,7 @@ class Engine:
     def check(self):
         """Raise if a kernel behind this engine recorded an error (a failed wait, a token without a page)."""
         if ids_on_cuda(self.model.get_device()) and ops.get_kernel_mode() == "native":
-            (ops.serving_module() if self.latent else ops.native_module()).check_status()
+            (ops.serving_module() if self.own_cache else ops.native_module()).check_status()
 
     def _special_tokens(self):
         tok = self.tokenizer
@@ -519,7 +558,7 @@ class Engine:
         cache when the pooled one is busy (nested generations); for the others None then."""
         cache = self._cache_pool.get(rows)
         if cache is None:
-            if self.latent:
+            if self.own_cache:
                 cache = self.model.make_cache(rows)
             else:
                 cache = PagedKVCache(batch_size=rows, seq_len=self.model.config.sequence_len, **self._kv_geometry())
@@ -527,7 +566,7 @@ class Engine:
             cache.in_use = False
             self._cache_pool[rows] = cache
         if cache.in_use:
-            if not self.latent:
+            if not self.own_cache:
                 return None
             cache = self.model.make_cache(rows)
         cache.in_use = True
@@ -536,7 +575,7 @@ class Engine:
     def _pooled_cache(self, rows, prompt_tokens, capacity):
         """A paged cache with room for the request, or None when the model decodes without one here (no captured graph
         for it, or its cache is busy)."""
-        if self.latent:
+        if self.own_cache:
             if capacity > self.model.config.sequence_len:
                 raise ValueError(f"request of {capacity} tokens; this server holds {self.model.config.sequence_len} per row")
         elif not self._graph_applies(rows, capacity):

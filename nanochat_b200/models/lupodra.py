@@ -14,8 +14,6 @@ Everything that reads h (query and key-value down-projections, both gates, a den
 matrix (`w_in`) and one product. Router logits and logits keep the accumulator's precision.
 """
 
-import json
-import os
 from dataclasses import dataclass, field
 from typing import Optional
 
@@ -23,7 +21,9 @@ import torch
 import torch.nn as nn
 
 from nanochat_b200 import common, ops
+from nanochat_b200.models import served
 from nanochat_b200.models.sampling import NaiveSampler
+from nanochat_b200.models.served import ServedModel, Weights, fit, padded, under
 
 
 # ------------------------------------------------------------------------------ config
@@ -137,27 +137,7 @@ class LupodraConfig:
 
 # ------------------------------------------------------------------------------ weights
 
-def _up(n, m=8):
-    return -(-n // m) * m
-
-
-def _fit(w, *shape):
-    """w at the origin of a zero tensor of `shape`."""
-    if tuple(w.shape) == shape:
-        return w
-    out = w.new_zeros(shape)
-    out[tuple(slice(0, s) for s in w.shape)] = w
-    return out
-
-
-class _Weights(nn.Module):
-    """Frozen tensors by attribute name, stored in the compute type unless said otherwise."""
-
-    def put(self, name, value, dtype, device):
-        self.register_parameter(name, nn.Parameter(value.to(dtype).to(device).contiguous(), requires_grad=False))
-
-
-class LatentAttention(_Weights):
+class LatentAttention(Weights):
     """Padded sizes: dp / vp head dimensions, qp query latent, kvp + rp one store entry."""
 
     def __init__(self, spec, eps):
@@ -167,8 +147,8 @@ class LatentAttention(_Weights):
         self.window, self.scale, self.eps = s.window, s.scale, eps
         if s.rot_dims > s.rot_dim or s.rot_dims % 2:
             raise ValueError(f"{s.rot_dims} rotated dimensions do not fit a rotated part of {s.rot_dim}")
-        self.dp, self.vp, self.qp = _up(s.dim), _up(s.vdim), _up(s.q_rank)
-        self.kvp, self.rp = _up(s.kv_rank, 16), _up(s.rot_dim, 16)
+        self.dp, self.vp, self.qp = padded(s.dim), padded(s.vdim), padded(s.q_rank)
+        self.kvp, self.rp = padded(s.kv_rank, 16), padded(s.rot_dim, 16)
         self.c_off, self.rot_off = self.qp, self.qp + self.kvp          # segments of w_in's output
 
     @property
@@ -180,19 +160,19 @@ class LatentAttention(_Weights):
         s, H = self.spec, self.heads
         put = lambda name, w, dt=dtype: self.put(name, w, dt, device)
         dq, dkv = take("dq", s.q_rank, C), take("dkv", s.kv_rank + s.rot_dim, C)
-        put("q_norm", _fit(take("dq.norm", s.q_rank).float(), self.qp), torch.float32)
-        put("kv_norm", _fit(take("dkv.norm", s.kv_rank).float(), self.kvp), torch.float32)
+        put("q_norm", fit(take("dq.norm", s.q_rank).float(), self.qp), torch.float32)
+        put("kv_norm", fit(take("dkv.norm", s.kv_rank).float(), self.kvp), torch.float32)
         uq = take("uq", H * (s.dim + s.rot_dim), s.q_rank).view(H, s.dim + s.rot_dim, s.q_rank)
-        w_q = torch.cat([_fit(uq[:, :s.dim], H, self.dp, self.qp), _fit(uq[:, s.dim:], H, self.rp, self.qp)], 1)
+        w_q = torch.cat([fit(uq[:, :s.dim], H, self.dp, self.qp), fit(uq[:, s.dim:], H, self.rp, self.qp)], 1)
         put("w_q", w_q.reshape(-1, self.qp))
-        uk = _fit(take("uk", H * s.dim, s.kv_rank).view(H, s.dim, s.kv_rank), H, self.dp, self.kvp).reshape(-1, self.kvp)
-        uv = _fit(take("uv", H * s.vdim, s.kv_rank).view(H, s.vdim, s.kv_rank), H, self.vp, self.kvp).reshape(-1, self.kvp)
+        uk = fit(take("uk", H * s.dim, s.kv_rank).view(H, s.dim, s.kv_rank), H, self.dp, self.kvp).reshape(-1, self.kvp)
+        uv = fit(take("uv", H * s.vdim, s.kv_rank).view(H, s.vdim, s.kv_rank), H, self.vp, self.kvp).reshape(-1, self.kvp)
         put("w_kv", torch.cat([uk, uv]))
         o = take("o", C, H * s.vdim).view(C, H, s.vdim)
-        put("w_o", _fit(o, _up(C), H, self.vp).reshape(_up(C), -1))
+        put("w_o", fit(o, padded(C), H, self.vp).reshape(padded(C), -1))
         i = torch.arange(s.rot_dims // 2, dtype=torch.float64)
         self.register_buffer("freq", (s.rot_base ** (-2.0 * i / s.rot_dims)).float().to(device), persistent=False)
-        return [_fit(dq, self.qp, C), _fit(dkv[:s.kv_rank], self.kvp, C), _fit(dkv[s.kv_rank:], self.rp, C)]
+        return [fit(dq, self.qp, C), fit(dkv[:s.kv_rank], self.kvp, C), fit(dkv[s.kv_rank:], self.rp, C)]
 
     @property
     def w_uk(self):
@@ -206,29 +186,29 @@ class LatentAttention(_Weights):
         return ops.latent_attention(self, z, cache, run, T)
 
 
-class DenseFF(_Weights):
+class DenseFF(Weights):
     """W_down act(z), z = W_up h being a segment of the layer's fused input product."""
 
     def __init__(self, spec, eps):
         super().__init__()
-        self.spec, self.eps, self.ff, self.fp = spec, eps, spec.ff, _up(spec.ff)
+        self.spec, self.eps, self.ff, self.fp = spec, eps, spec.ff, padded(spec.ff)
 
     def load(self, take, C, dtype, device):
         up, down = take("up", self.ff, C), take("down", C, self.ff)
-        self.put("w_down", _fit(down, _up(C), self.fp), dtype, device)
+        self.put("w_down", fit(down, padded(C), self.fp), dtype, device)
         self.put("act", take("act", 4).float(), torch.float32, device)
-        return [_fit(up, self.fp, C)], []
+        return [fit(up, self.fp, C)], []
 
     def forward(self, h, z):
         return (ops.linear_rows(ops.poly_norm(z, self.act, self.eps, self.ff), self.w_down),)
 
 
-class MixtureFF(_Weights):
+class MixtureFF(Weights):
     """Expert matrices stacked: w_gate_up (experts, gate rows then up rows, width), w_down (experts, width, fp)."""
 
     def __init__(self, spec, eps):
         super().__init__()
-        self.spec, self.ff, self.fp = spec, spec.ff, _up(spec.ff)
+        self.spec, self.ff, self.fp = spec, spec.ff, padded(spec.ff)
         self.experts, self.top = spec.experts, spec.top
         if not 1 <= self.top <= self.experts:
             raise ValueError(f"top {self.top} of {self.experts} experts")
@@ -237,17 +217,17 @@ class MixtureFF(_Weights):
         gu, down = [], []
         for e in range(self.experts):
             gate, up = take(f"e{e}.gate", self.ff, C), take(f"e{e}.up", self.ff, C)
-            gu.append(torch.cat([_fit(gate, self.fp, _up(C)), _fit(up, self.fp, _up(C))]))
-            down.append(_fit(take(f"e{e}.down", C, self.ff), _up(C), self.fp))
+            gu.append(torch.cat([fit(gate, self.fp, padded(C)), fit(up, self.fp, padded(C))]))
+            down.append(fit(take(f"e{e}.down", C, self.ff), padded(C), self.fp))
         self.put("w_gate_up", torch.stack(gu), dtype, device)
         self.put("w_down", torch.stack(down), dtype, device)
-        return [], [_fit(take("router", self.experts, C), _up(self.experts), C)]
+        return [], [fit(take("router", self.experts, C), padded(self.experts), C)]
 
     def forward(self, h, z):
         return ops.mixture(h, self)
 
 
-class Layer(_Weights):
+class Layer(Weights):
     def __init__(self, spec, eps):
         super().__init__()
         self.spec = spec
@@ -255,20 +235,19 @@ class Layer(_Weights):
         self.mlp = None if spec.mlp is None else (DenseFF if isinstance(spec.mlp, DenseSpec) else MixtureFF)(spec.mlp, eps)
 
     def load(self, take, C, dtype, device):
-        Cp = _up(C)
-        sub = lambda prefix: lambda name, *shape: take(prefix + name, *shape)
-        self.put("norm", _fit(1 + take("norm1", C).float(), Cp), torch.float32, device)
-        rows = self.attn.load(sub("mix."), C, dtype, device)
+        Cp = padded(C)
+        self.put("norm", fit(1 + take("norm1", C).float(), Cp), torch.float32, device)
+        rows = self.attn.load(under(take, "mix."), C, dtype, device)
         self.gates = []                                       # where the gates' segments of w_in's output begin
         for name in ("rg1", "rg2") if self.mlp is not None else ("rg1",):
             self.gates.append(sum(r.shape[0] for r in rows))
-            rows.append(_fit(take(name, C, C), Cp, C))
-            self.put(name + "_bias", _fit(take(name + ".b", C).float(), Cp), torch.float32, device)
-        extra, router = self.mlp.load(sub("mlp."), C, dtype, device) if self.mlp is not None else ([], [])
+            rows.append(fit(take(name, C, C), Cp, C))
+            self.put(name + "_bias", fit(take(name + ".b", C).float(), Cp), torch.float32, device)
+        extra, router = self.mlp.load(under(take, "mlp."), C, dtype, device) if self.mlp is not None else ([], [])
         self.up_off = sum(r.shape[0] for r in rows)
         rows += extra
         self.n_in = sum(r.shape[0] for r in rows)
-        self.put("w_all", _fit(torch.cat(rows + router), self.n_in + sum(r.shape[0] for r in router), Cp), dtype, device)
+        self.put("w_all", fit(torch.cat(rows + router), self.n_in + sum(r.shape[0] for r in router), Cp), dtype, device)
         if router:
             self.mlp.router = self.w_all[self.n_in:]
 
@@ -277,41 +256,28 @@ class Layer(_Weights):
         return self.w_all[:self.n_in]
 
 
-class Lupodra(nn.Module, NaiveSampler):
+class Lupodra(ServedModel, NaiveSampler):
+    step_graph = "LatentDecodeGraph"
+
     def __init__(self, config, dtype=None):
         super().__init__()
         self.config = config
         self.dtype = dtype or common.COMPUTE_DTYPE
-        self.width = _up(config.n_embd)
+        self.width = padded(config.n_embd)
         self.layers = nn.ModuleList([Layer(x, config.eps) for x in config.layers])
         self.runs = [(self.layers[i], again) for i, again in config.runs()]
         self.keep_x0 = any(again for _, again in self.runs)
         self.embed = self.final_norm = None
 
     # ------------------------------------------------------------------------- weights
-    @torch.no_grad()
-    def load_tensors(self, tensors, device):
-        """Take the named tensors (any float type) into the layouts of the kernels."""
-        C, left = self.config.n_embd, set(tensors)
-
-        def take(name, *shape):
-            if name not in tensors:
-                raise KeyError(f"tensor {name!r} is missing")
-            t = tensors[name]
-            if tuple(t.shape) != shape:
-                raise ValueError(f"tensor {name!r} has shape {tuple(t.shape)}, the configuration says {shape}")
-            left.discard(name)
-            return t
-
+    def pack(self, take, device):
+        C = self.config.n_embd
         for i, layer in enumerate(self.layers):
-            layer.load(lambda name, *shape, i=i: take(f"l{i}.{name}", *shape), C, self.dtype, device)
-        embed = _fit(take("embed", self.config.vocab_size, C), _up(self.config.vocab_size), self.width)
+            layer.load(under(take, f"l{i}."), C, self.dtype, device)
+        embed = fit(take("embed", self.config.vocab_size, C), padded(self.config.vocab_size), self.width)
         self.embed = nn.Parameter(embed.to(self.dtype).to(device), requires_grad=False)
-        norm = _fit(1 + take("final.norm", C).float(), self.width)
+        norm = fit(1 + take("final.norm", C).float(), self.width)
         self.final_norm = nn.Parameter(norm.to(device), requires_grad=False)
-        if left:
-            raise ValueError(f"tensors the configuration has no place for: {sorted(left)[:8]}")
-        return self
 
     def tensor_shapes(self):
         """Names and shapes of the stored tensors."""
@@ -332,22 +298,12 @@ class Lupodra(nn.Module, NaiveSampler):
                     out.update({f"{l}mlp.e{e}.gate": (f.ff, C), f"{l}mlp.e{e}.up": (f.ff, C), f"{l}mlp.e{e}.down": (C, f.ff)})
         return out
 
-    def init_weights(self, device, seed=0):
-        """Random weights of a plausible scale (benchmarks, demonstrations)."""
-        g = torch.Generator(device=device).manual_seed(seed)
-        tensors = {}
-        for name, shape in self.tensor_shapes().items():
-            if len(shape) == 2:
-                t = torch.randn(shape, generator=g, device=device) * (1.0 if name == "embed" else shape[1] ** -0.5)
-            else:
-                t = (torch.ones if name.endswith((".dq.norm", ".dkv.norm")) else torch.zeros)(shape, device=device)
-                if name.endswith(".act"):
-                    t = torch.tensor([0.7, 0.3, 0.1, 0.0], device=device)
-            tensors[name] = t.to(torch.bfloat16)
-        return self.load_tensors(tensors, device)
-
-    def get_device(self):
-        return self.embed.device
+    def init_tensor(self, name, shape, normal):
+        if name.endswith((".dq.norm", ".dkv.norm")):
+            return torch.ones(shape)
+        if name.endswith(".act"):
+            return torch.tensor([0.7, 0.3, 0.1, 0.0])
+        return super().init_tensor(name, shape, normal)
 
     # --------------------------------------------------------------------------- cache
     def make_cache(self, rows, sequence_len=None):
@@ -436,8 +392,4 @@ class Lupodra(nn.Module, NaiveSampler):
 
 
 def load_folder(path, device, dtype=None, **serving):
-    """A model from a folder of config.json and model.safetensors."""
-    from nanochat_b200.utils.safetensors import read_safetensors
-    with open(os.path.join(path, "config.json"), "r", encoding="utf-8") as f:
-        config = LupodraConfig.from_dict(json.load(f), **serving)
-    return Lupodra(config, dtype).load_tensors(read_safetensors(os.path.join(path, "model.safetensors")), device)
+    return served.load_folder(path, device, LupodraConfig.from_dict, Lupodra, dtype, **serving)

@@ -48,16 +48,19 @@ def _gpt():
     return Architecture("GPT", config_from_dict, build, load_folder)
 
 
-def _lupodra():
-    from nanochat_b200.models import lupodra as m
+def _served(name):
+    """A model that is served only: module models/<name>, class <Name>, configuration <Name>Config."""
+    import importlib
+    m = importlib.import_module(f"nanochat_b200.models.{name.lower()}")
+    model = getattr(m, name)
 
     def build(config, device, dtype=None):
-        return m.Lupodra(config, dtype).init_weights(device)
+        return model(config, dtype).init_weights(device)
 
-    return Architecture("Lupodra", m.LupodraConfig.from_dict, build, m.load_folder)
+    return Architecture(name, getattr(m, name + "Config").from_dict, build, m.load_folder)
 
 
-_ARCHITECTURES = {"GPT": _gpt, "Lupodra": _lupodra}
+_ARCHITECTURES = {"GPT": _gpt, "Lupodra": lambda: _served("Lupodra"), "Safepel": lambda: _served("Safepel")}
 
 
 def architectures():

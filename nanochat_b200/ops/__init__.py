@@ -8,7 +8,8 @@ Every op has two bodies with one meaning:
                      norm/rope/loss/optimizer kernels).
 
 A third module, `serving.py`, holds the native bodies of the inference-only mechanisms (latent attention, mixtures of
-experts, gated residuals), whose kernels are a library of their own and also run in float32.
+experts, gated residuals, the gated delta rule, window and fixed-decay attention), whose kernels are a library of their own
+and also run in float32.
 
 `use_native(t)` decides per call: CUDA bf16 tensors go to the kernels, everything
 else to the reference body. On a CUDA device a missing extension is an error, not
@@ -166,3 +167,31 @@ def latent_attention(p, z, cache, run, T):
 
 def mixture(h, p):
     return _serve("mixture", h)(h, p)
+
+
+def embed_layer_norm(ids, table, vocab, w_embed, w, eps, n):
+    return _serve("embed_layer_norm", table)(ids, table, vocab, w_embed, w, eps, n)
+
+
+def layer_norm_residual(x, y, w_post, w, eps, n, dtype):
+    return _serve("layer_norm_residual", x)(x, y, w_post, w, eps, n, dtype)
+
+
+def relu_glu(h, w_gate_up):
+    return _serve("relu_glu", h)(h, w_gate_up)
+
+
+def gated_delta(p, z, ba, cache, run, T):
+    return _serve("gated_delta", z)(p, z, ba, cache, run, T)
+
+
+def window_attention(p, z, cache, run, T, y):
+    return _serve("window_attention", z)(p, z, cache, run, T, y)
+
+
+def decay_attention(p, z, cache, run, T, y):
+    return _serve("decay_attention", z)(p, z, cache, run, T, y)
+
+
+def window_and_decay(left, right, z, cache, run, T):
+    return _serve("window_and_decay", z)(left, right, z, cache, run, T)

@@ -1,5 +1,6 @@
-// Flash attention forward for sm_100a (bf16, causal with optional left window): head dim 128, or query / key vectors in
-// two parts (per-head part up to 128, part shared by all key heads up to 64) with values of their own size up to 128.
+// Flash attention forward for sm_100a (bf16, causal with optional left window): head dim 128; query / key vectors in
+// two parts (per-head part up to 128, part shared by all key heads up to 64) with values of their own size up to 128; or
+// head dims up to 128 with an optional soft cap on the scores.
 //
 // One CTA per (256-query block, head, batch): two 128-query tiles share every K/V block that is
 // loaded, and their softmax phases are staggered so the tensor core always has the other tile's
@@ -49,6 +50,8 @@ struct Shape {
   static constexpr int SMEM_BYTES = TILES * K_TILE /*Q*/ + K_STAGES * K_TILE + V_STAGES * V_TILE + 1024 + 256;
   static_assert(SMEM_BYTES <= 227 * 1024, "tiles must fit shared memory");
 };
+// EXACT: every column of the value tile is stored. PARTIAL: the first dv, times out_scale. CAPPED: PARTIAL with soft-capped scores.
+enum Mode : int { EXACT = 0, PARTIAL = 1, CAPPED = 2 };
 }  // namespace attn
 
 struct AttnKernelArgs {
@@ -57,7 +60,9 @@ struct AttnKernelArgs {
   float* amax_o;        // optional max |o|
   long long o_bat, o_tok, o_head;
   int Tq, Tk, H, Hkv;
-  int dv;               // value columns stored (QR > 0 only)
+  int dv;               // value columns stored (not EXACT)
+  float out_scale;      // (not EXACT)
+  float cap_in, cap;    // CAPPED: score -> cap * tanh(score * cap_in / (2 log2 e)), both with the log2 factors of the exponent
   int window;           // < 0: unlimited
   float scale_log2;     // softmax scale * log2(e)
   int* status;
@@ -80,7 +85,7 @@ __device__ __forceinline__ BlockRange tile_blocks(int q0x, const AttnKernelArgs&
   return r;
 }
 
-template <int QU, int QR, int DV>
+template <int QU, int QR, int DV, int MODE>
 __global__ void __launch_bounds__(attn::THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQ2,
@@ -238,7 +243,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const uint32_t t_o = tmem_base + lane_sel + COL_O + x * 128;
     const int hi = qi + off;                        // last visible key
     const int lo = args.window >= 0 ? hi - args.window : -(1 << 30);
-    const float sc = args.scale_log2;
+    const float sc = MODE == CAPPED ? 1.f : args.scale_log2;
     float m_used = NEG_BIG, l_run = 0.f;
     int n = 0;                                      // blocks this tile has processed
     bool ok = true;
@@ -250,6 +255,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
       for (int c = 0; c < BKV / 32; ++c) tmem_ld32(t_s + c * 32, reinterpret_cast<uint32_t(&)[32]>(sv[c * 32]));
       tmem_wait_ld();
+      if constexpr (MODE == CAPPED) {
+        // cap tanh(y) = cap - 2 cap / (1 + e^2y): an absolute error of a few 2^-24 cap, whatever the size of y
+#pragma unroll
+        for (int c = 0; c < BKV; ++c)
+          sv[c] = __float_as_uint(fmaf(-2.f * args.cap, __fdividef(1.f, 1.f + exp2f(__uint_as_float(sv[c]) * args.cap_in)), args.cap));
+      }
       const bool need_mask = (k0 + BKV - 1 > q0x + off) || (k0 + BKV > args.Tk) ||
                              (args.window >= 0 && k0 < q0x + BQ - 1 + off - args.window);
       if (need_mask) {
@@ -314,7 +325,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     // tcgen05.ld is warp-collective: every lane runs the loads, only the stores are predicated
     if (__all_sync(0xffffffffu, ok) && n > 0) {
       const bool row_ok = qi < args.Tq;
-      const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      const float inv_l = (l_run > 0.f ? 1.f / l_run : 0.f) * (MODE == EXACT ? 1.f : args.out_scale);
       float mxo = 0.f;
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(args.o) + (long long)b * args.o_bat +
                             (long long)qi * args.o_tok + (long long)h * args.o_head;
@@ -330,7 +341,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           w.y = pack_bf16(__uint_as_float(v[e + 2]) * inv_l, __uint_as_float(v[e + 3]) * inv_l);
           w.z = pack_bf16(__uint_as_float(v[e + 4]) * inv_l, __uint_as_float(v[e + 5]) * inv_l);
           w.w = pack_bf16(__uint_as_float(v[e + 6]) * inv_l, __uint_as_float(v[e + 7]) * inv_l);
-          if (row_ok && (QR == 0 || c * 32 + e < args.dv)) *reinterpret_cast<uint4*>(orow + c * 32 + e) = w;
+          if (row_ok && (MODE == EXACT || c * 32 + e < args.dv)) *reinterpret_cast<uint4*>(orow + c * 32 + e) = w;
         }
         if (args.amax_o && row_ok) {
 #pragma unroll
@@ -369,12 +380,12 @@ static bool make_part_map(CUtensorMap* m, const void* base, int D, int T, int Hn
   return make_tmap(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, str, box);
 }
 
-template <int QU, int QR, int DV>
+template <int QU, int QR, int DV, int MODE>
 static cudaError_t launch_attn(const SplitAttnDesc& sd, int* status, cudaStream_t stream) {
   using S = attn::Shape<QU, QR, DV>;
   const AttnDesc& d = sd.a;
   static PerDeviceOnce configured;
-  auto kern = attn_fwd_kernel<QU, QR, DV>;
+  auto kern = attn_fwd_kernel<QU, QR, DV, MODE>;
   cudaError_t ce = configured.once([&] {
     return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::SMEM_BYTES);
   });
@@ -392,6 +403,9 @@ static cudaError_t launch_attn(const SplitAttnDesc& sd, int* status, cudaStream_
   a.o = d.o; a.lse = d.lse; a.amax_o = d.amax_o; a.o_bat = d.o_bat; a.o_tok = d.o_tok; a.o_head = d.o_head;
   a.Tq = d.Tq; a.Tk = d.Tk; a.H = d.H; a.Hkv = d.Hkv;
   a.dv = sd.Dv;
+  a.out_scale = sd.out_scale;
+  a.cap = sd.softcap * 1.4426950408889634f;
+  a.cap_in = sd.softcap > 0.f ? 2.f * 1.4426950408889634f * d.scale / sd.softcap : 0.f;
   a.window = d.window;
   a.scale_log2 = d.scale * 1.4426950408889634f;
   a.status = status;
@@ -406,7 +420,7 @@ cudaError_t attention_fwd(const AttnDesc& d, int* status, cudaStream_t stream) {
   SplitAttnDesc sd{};
   sd.a = d;
   sd.Dv = 128;
-  return launch_attn<2, 0, 128>(sd, status, stream);
+  return launch_attn<2, 0, 128, attn::EXACT>(sd, status, stream);
 }
 #endif
 
@@ -414,11 +428,22 @@ bool attention_split_supported(int D, int D2, int Dv) {
   return D > 0 && D <= 128 && D2 > 0 && D2 <= 64 && Dv > 0 && Dv <= 128 && !((D | D2 | Dv) & 7);
 }
 
+bool attention_capped_supported(int D, int Dv) { return D > 0 && D <= 128 && Dv > 0 && Dv <= 128 && !((D | Dv) & 7); }
+
 #ifdef NC_SERVING
 cudaError_t attention_split_fwd(const SplitAttnDesc& d, int* status, cudaStream_t stream) {
   if (!attention_split_supported(d.a.D, d.D2, d.Dv) || d.a.H % d.a.Hkv != 0 || d.a.Tq > d.a.Tk) return cudaErrorInvalidValue;
-  if (d.a.D <= 64) return d.Dv <= 64 ? launch_attn<1, 1, 64>(d, status, stream) : launch_attn<1, 1, 128>(d, status, stream);
-  return d.Dv <= 64 ? launch_attn<2, 1, 64>(d, status, stream) : launch_attn<2, 1, 128>(d, status, stream);
+  using attn::PARTIAL;
+  if (d.a.D <= 64) return d.Dv <= 64 ? launch_attn<1, 1, 64, PARTIAL>(d, status, stream) : launch_attn<1, 1, 128, PARTIAL>(d, status, stream);
+  return d.Dv <= 64 ? launch_attn<2, 1, 64, PARTIAL>(d, status, stream) : launch_attn<2, 1, 128, PARTIAL>(d, status, stream);
+}
+
+cudaError_t attention_capped_fwd(const SplitAttnDesc& d, int* status, cudaStream_t stream) {
+  if (!attention_capped_supported(d.a.D, d.Dv) || d.D2 != 0 || d.a.H % d.a.Hkv != 0 || d.a.Tq > d.a.Tk) return cudaErrorInvalidValue;
+  using namespace attn;
+  if (d.a.D <= 64 && d.Dv <= 64)
+    return d.softcap > 0.f ? launch_attn<1, 0, 64, CAPPED>(d, status, stream) : launch_attn<1, 0, 64, PARTIAL>(d, status, stream);
+  return d.softcap > 0.f ? launch_attn<2, 0, 128, CAPPED>(d, status, stream) : launch_attn<2, 0, 128, PARTIAL>(d, status, stream);
 }
 #endif
 

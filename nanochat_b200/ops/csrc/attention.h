@@ -27,9 +27,15 @@ struct SplitAttnDesc {
   const void *q2, *k2;
   long long q2_bat, q2_tok, q2_head, k2_bat, k2_tok;
   int D2, Dv;
+  float out_scale = 1.f;     // the output is multiplied by it
+  float softcap = 0.f;       // attention_capped_fwd: scores become softcap * tanh(score / softcap); 0: no cap
 };
 bool attention_split_supported(int D, int D2, int Dv);
 cudaError_t attention_split_fwd(const SplitAttnDesc& d, int* status, cudaStream_t stream);
+
+// One part (D2 = 0), D and Dv multiples of 8 up to 128, grouped keys, optional soft cap.
+bool attention_capped_supported(int D, int Dv);
+cudaError_t attention_capped_fwd(const SplitAttnDesc& d, int* status, cudaStream_t stream);
 
 cudaError_t attention_fwd(const AttnDesc& d, int* status, cudaStream_t stream);
 

@@ -74,8 +74,9 @@ NextWeights next_weights(const optional<Tensor>& t) {
 }
 
 // ------------------------------------------------------------------------------------------------- GEMM, attention
-// out (M, N) = A (M, K) B (N, K)^T; grouped: B (groups, N, K), m_group int32, one per 128 rows of A
-void gemm(const Tensor& A, const Tensor& B, Tensor& C, const optional<Tensor>& m_group) {
+// out (M, N) = A (M, K) B (N, K)^T; grouped: B (groups, N, K), m_group int32, one per 128 rows of A. epi: 0 plain, 1 relu,
+// 2 times aux (bf16 like C, may be C itself)
+void gemm(const Tensor& A, const Tensor& B, Tensor& C, const optional<Tensor>& m_group, int64_t epi, const optional<Tensor>& aux) {
   check_rows(A, "A"); check_rows(C, "C");
   const bool grouped = has(m_group);
   TORCH_CHECK(A.scalar_type() == at::kBFloat16 && B.scalar_type() == at::kBFloat16 && B.is_cuda() && B.dim() == (grouped ? 3 : 2) &&
@@ -91,7 +92,35 @@ void gemm(const Tensor& A, const Tensor& B, Tensor& C, const optional<Tensor>& m
                 m_group->numel() * 128 >= A.size(0), "m_group: int32, one per 128 rows");
     d.m_group = m_group->data_ptr<int>(); d.groups = (int)B.size(0); d.bsb = B.stride(0);
   }
+  TORCH_CHECK(epi == 0 || (!grouped && !is_f32(C) && (epi == 1 || (epi == 2 && has(aux)))), "gemm epilogue");
+  d.epi = epi == 1 ? nc::EPI_RELU : epi == 2 ? nc::EPI_MULAUX : nc::EPI_LINEAR;
+  if (has(aux)) {
+    check_rows(*aux, "aux"); same_type(*aux, C, "aux");
+    TORCH_CHECK(aux->sizes() == C.sizes() && epi == 2, "aux like C");
+    d.aux = aux->data_ptr(); d.ldaux = pitch(*aux);
+  }
   NC_CHECK(nc::gemm_bf16(d, status_ptr(A), stream()));
+}
+
+// q (T, H, D), k and v (S, Hkv, D), o (T, H, D): views with dense innermost dims; softcap 0: none
+void attention_capped(const Tensor& q, const Tensor& k, const Tensor& v, Tensor& o, int64_t window_left, double scale, double softcap, double out_scale) {
+  for (const Tensor* t : {&q, &k, &v, (const Tensor*)&o}) {
+    TORCH_CHECK(t->is_cuda() && t->dim() == 3 && t->scalar_type() == at::kBFloat16 && t->stride(-1) == 1 && (reinterpret_cast<uintptr_t>(t->data_ptr()) & 15) == 0,
+                "attention operands: bf16, dense innermost, 16-byte aligned");
+    for (int64_t i = 0; i + 1 < t->dim(); ++i) TORCH_CHECK(t->stride(i) % 8 == 0, "attention operands: pitches must be multiples of 8");
+  }
+  const int64_t T = q.size(0), H = q.size(1), S = k.size(0), Hkv = k.size(1);
+  TORCH_CHECK(k.size(2) == q.size(2) && v.size(0) == S && v.size(1) == Hkv && o.size(0) == T && o.size(1) == H && o.size(2) == v.size(2), "attention shapes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  nc::SplitAttnDesc d{};
+  d.a.q = q.data_ptr(); d.a.q_tok = q.stride(0); d.a.q_head = q.stride(1); d.a.q_bat = q.stride(0) * T;
+  d.a.k = k.data_ptr(); d.a.k_tok = k.stride(0); d.a.k_head = k.stride(1); d.a.k_bat = k.stride(0) * S;
+  d.a.v = v.data_ptr(); d.a.v_tok = v.stride(0); d.a.v_head = v.stride(1); d.a.v_bat = v.stride(0) * S;
+  d.a.o = o.data_ptr(); d.a.o_tok = o.stride(0); d.a.o_head = o.stride(1); d.a.o_bat = o.stride(0) * T;
+  d.a.B = 1; d.a.Tq = (int)T; d.a.Tk = (int)S; d.a.H = (int)H; d.a.Hkv = (int)Hkv; d.a.D = (int)q.size(2);
+  d.Dv = (int)v.size(2);
+  d.a.window = (int)window_left; d.a.scale = (float)scale; d.softcap = (float)softcap; d.out_scale = (float)out_scale;
+  NC_CHECK(nc::attention_capped_fwd(d, status_ptr(q), stream()));
 }
 
 // q (T, H, D), q2 (T, H, D2), k (S, H, D), k2 (S, D2), v (S, H, Dv), o (T, H, Dv): views with dense innermost dims
@@ -158,6 +187,23 @@ void gated_residual_norm_(Tensor& x, const std::vector<std::vector<Tensor>>& ter
   const c10::cuda::CUDAGuard guard(x.device());
   NC_CHECK(gated_residual_norm(is_f32(h), x.data_ptr<float>(), t, (int)terms.size(), (float)mult,
                                has(extra) ? extra->data_ptr<float>() : nullptr, w.data_ptr<float>(), (float)eps, (int)x.size(0), (int)n,
+                               (int)x.size(1), h.data_ptr(), stream()));
+}
+
+// x += LN(y) * wy (ids: x = LN(y[ids]) * wy), h = LN(x) * w
+void layer_norm_residual_(const optional<Tensor>& ids, const Tensor& y, int64_t vocab, const Tensor& wy, Tensor& x, const Tensor& w, double eps,
+                          int64_t n, Tensor& h) {
+  check_rows(y, "y"); check_rows(x, "x"); check_rows(h, "h"); check_vec(wy, x.size(1), "wy"); check_vec(w, x.size(1), "w");
+  TORCH_CHECK(is_f32(x) && x.is_contiguous() && h.is_contiguous() && h.sizes() == x.sizes() && y.size(1) == x.size(1) && n <= x.size(1) &&
+              (is_f32(y) || !is_f32(h)), "layer norm shapes");
+  if (has(ids)) {
+    TORCH_CHECK(ids->is_cuda() && ids->scalar_type() == at::kLong && ids->is_contiguous() && ids->numel() == x.size(0) && vocab <= y.size(0), "ids: int64, one per row");
+  } else {
+    TORCH_CHECK(y.size(0) == x.size(0), "y: one row per row of x");
+  }
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(layer_norm_residual(is_f32(h), is_f32(y), has(ids) ? reinterpret_cast<const long long*>(ids->data_ptr<int64_t>()) : nullptr, y.data_ptr(),
+                               pitch(y), (int)vocab, wy.data_ptr<float>(), x.data_ptr<float>(), w.data_ptr<float>(), (float)eps, (int)x.size(0), (int)n,
                                (int)x.size(1), h.data_ptr(), stream()));
 }
 
@@ -408,6 +454,223 @@ void gemv_residual(const Tensor& y, const Tensor& W, Tensor& x, const Tensor& g,
   NC_CHECK(gemv(d, PRE_PLAIN, GEMV_RESIDUAL, stream()));
 }
 
+// out = x W^T, x bf16 rows
+void gemv_plain(const Tensor& x, const Tensor& W, Tensor& out, const optional<Tensor>& next) {
+  GemvDesc d = gemv_of(x, W, next);
+  TORCH_CHECK(x.scalar_type() == at::kBFloat16, "x: bf16 rows");
+  const int epi = store_kind(d, out);
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(gemv(d, PRE_PLAIN, epi, stream()));
+}
+// out = relu(x Wg^T) * (x Wu^T), W = [Wg; Wu]
+void gemv_relu_glu_(const Tensor& x, const Tensor& W, Tensor& out, const optional<Tensor>& next) {
+  GemvDesc d = gemv_of(x, W, next);
+  TORCH_CHECK(x.scalar_type() == at::kBFloat16 && W.size(0) % 2 == 0, "x: bf16 rows; W: gate rows, then up rows");
+  d.N = (int)(W.size(0) / 2);
+  TORCH_CHECK(store_kind(d, out) == GEMV_STORE_BF16, "out: bf16");
+  const c10::cuda::CUDAGuard guard(x.device());
+  NC_CHECK(gemv_relu_glu(d, stream()));
+}
+
+// ------------------------------------------------------------------------------------------------ recurrences, windows
+// A module's sizes travel as one list: delta [heads, kv_heads, dim, dp, vdim, vp, taps, a_off].
+StateRef state_ref(const Tensor& t, int64_t seqs, int64_t per_seq, const char* name) {
+  TORCH_CHECK(t.is_cuda() && is_f32(t) && t.dim() >= 2 && t.size(0) >= seqs && t.stride(0) % 4 == 0 && (reinterpret_cast<uintptr_t>(t.data_ptr()) & 15) == 0, name,
+              ": float, one row per sequence, 16-byte aligned");
+  int64_t n = 1;
+  for (int64_t i = t.dim() - 1; i >= 1; --i) {
+    TORCH_CHECK(t.stride(i) == n, name, ": dense per sequence");
+    n *= t.size(i);
+  }
+  TORCH_CHECK(n == per_seq && (seqs == 1 || t.stride(0) >= n), name, ": size");
+  return StateRef{t.data_ptr<float>(), (long long)t.stride(0)};
+}
+RowPos row_pos(const Tensor& lens, int64_t per_seq, int64_t rows) {
+  TORCH_CHECK(lens.is_cuda() && lens.scalar_type() == at::kInt && lens.is_contiguous() && per_seq > 0 && rows % per_seq == 0 && rows / per_seq <= lens.numel(),
+              "sequence lengths: int32, one per sequence");
+  return RowPos{lens.data_ptr<int>(), (int)per_seq};
+}
+DeltaInputs delta_inputs(const Tensor& z, const std::vector<int64_t>& size, const Tensor& conv, const optional<Tensor>& ba, const Tensor& neg_a,
+                         const Tensor& dt_bias, const Tensor& ring, const Tensor& lens, int64_t per_seq, bool f32) {
+  check_rows(z, "z");
+  TORCH_CHECK(size.size() == 8, "delta rule: eight sizes");
+  DeltaInputs d{};
+  d.f32 = f32; d.z_f32 = is_f32(z); d.z = z.data_ptr(); d.ldz = pitch(z); d.rows = (int)z.size(0);
+  d.heads = (int)size[0]; d.kv_heads = (int)size[1]; d.dim = (int)size[2]; d.dp = (int)size[3]; d.vdim = (int)size[4]; d.vp = (int)size[5]; d.taps = (int)size[6];
+  d.a_off = (int)size[7];
+  const int64_t channels = 2 * size[1] * size[3] + size[0] * size[5];
+  TORCH_CHECK(size[0] > 0 && size[1] > 0 && size[6] > 0 && channels <= z.size(1), "delta rule: sizes");
+  check_vec(conv, size[6] * channels, "conv"); check_vec(neg_a, size[0], "neg_a"); check_vec(dt_bias, size[0], "dt_bias");
+  d.conv = conv.data_ptr<float>(); d.neg_a = neg_a.data_ptr<float>(); d.dt_bias = dt_bias.data_ptr<float>();
+  if (has(ba)) {
+    TORCH_CHECK(ba->is_cuda() && is_f32(*ba) && ba->dim() == 2 && ba->stride(1) == 1 && ba->size(0) == z.size(0) && size[7] + size[0] <= ba->size(1), "ba: float rows");
+    d.ba = ba->data_ptr<float>(); d.ldba = ba->size(0) == 1 ? ba->size(1) : ba->stride(0);
+  }
+  d.pos = row_pos(lens, per_seq, z.size(0));
+  d.ring = state_ref(ring, z.size(0) / per_seq, size[6] * channels, "ring");
+  return d;
+}
+void delta_prepare_(const Tensor& z, const std::vector<int64_t>& size, const Tensor& conv, const Tensor& ba, const Tensor& neg_a, const Tensor& dt_bias,
+                    const Tensor& ring, const Tensor& lens, int64_t per_seq, Tensor& act, Tensor& norms, Tensor& beta_g) {
+  const DeltaInputs d = delta_inputs(z, size, conv, ba, neg_a, dt_bias, ring, lens, per_seq, is_f32(act));
+  check_rows(act, "act");
+  TORCH_CHECK(act.is_contiguous() && act.size(0) == z.size(0) && act.size(1) == 2 * size[1] * size[3] + size[0] * size[5] && is_f32(norms) && norms.is_contiguous() &&
+              norms.numel() >= z.size(0) * 2 * size[1] && is_f32(beta_g) && beta_g.is_contiguous() && beta_g.numel() >= z.size(0) * 2 * size[0], "delta rule: outputs");
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(delta_prepare(d, act.data_ptr(), norms.data_ptr<float>(), beta_g.data_ptr<float>(), stream()));
+}
+void silu_rows_(const Tensor& z, Tensor& act) {
+  check_rows(z, "z"); check_rows(act, "act"); same_type(z, act, "act");
+  TORCH_CHECK(z.sizes() == act.sizes(), "silu_rows shapes");
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(silu_rows(is_f32(z), z.data_ptr(), pitch(z), (int)z.size(0), (int)z.size(1), act.data_ptr(), pitch(act), stream()));
+}
+// size: [heads, kv_heads, dp, vp]; act: q, k, v side by side. norms and beta_g, or log_decay.
+void recurrence_(const Tensor& act, const std::vector<int64_t>& size, const optional<Tensor>& norms, const optional<Tensor>& beta_g,
+                 const optional<Tensor>& log_decay, const Tensor& state, const Tensor& lens, int64_t per_seq, Tensor& o, const optional<Tensor>& scratch) {
+  check_rows(act, "act"); check_rows(o, "o"); same_type(act, o, "o");
+  TORCH_CHECK(size.size() == 4 && size[0] > 0 && size[1] > 0, "recurrence: four sizes");
+  const int64_t H = size[0], G = size[1], dp = size[2], vp = size[3], rows = act.size(0);
+  TORCH_CHECK(2 * G * dp + H * vp <= act.size(1) && o.size(0) == rows && o.size(1) == H * vp, "recurrence shapes");
+  Recurrence d{};
+  d.f32 = is_f32(act); d.act = act.data_ptr(); d.lda = pitch(act); d.q_off = 0; d.k_off = (int)(G * dp); d.v_off = (int)(2 * G * dp);
+  d.rows = (int)rows; d.heads = (int)H; d.kv_heads = (int)G; d.dp = (int)dp; d.vp = (int)vp;
+  const bool delta = has(beta_g);
+  if (delta) {
+    TORCH_CHECK(has(norms), "delta rule: norms");
+    check_vec(*norms, rows * 2 * G, "norms"); check_vec(*beta_g, rows * 2 * H, "beta_g");
+    d.norms = norms->data_ptr<float>(); d.beta_g = beta_g->data_ptr<float>();
+  } else {
+    TORCH_CHECK(has(log_decay), "fixed decay: log_decay");
+    check_vec(*log_decay, H, "log_decay");
+    d.log_decay = log_decay->data_ptr<float>();
+  }
+  d.pos = row_pos(lens, per_seq, rows);
+  d.state = state_ref(state, rows / per_seq, H * dp * vp, "state");
+  d.o = o.data_ptr(); d.ldo = pitch(o);
+  const c10::cuda::CUDAGuard guard(act.device());
+  if (has(scratch)) {
+    TORCH_CHECK(scratch->is_cuda() && scratch->is_contiguous() && (reinterpret_cast<uintptr_t>(scratch->data_ptr()) & 15) == 0 &&
+                (size_t)(scratch->numel() * scratch->element_size()) >= recurrence_scratch((int)(rows / per_seq), (int)per_seq, (int)H, delta), "scratch: too small");
+    ++g_launches;
+    NC_CHECK(recurrence_chunks(d, scratch->data_ptr(), stream()));
+  } else {
+    NC_CHECK(recurrence_scan(d, stream()));
+  }
+}
+// y = o / rms(o) * w * act(gate) * out_scale in `groups` groups of n real entries
+void norm_gate_(const Tensor& o, const Tensor& gate, const Tensor& w, double eps, int64_t groups, int64_t n, bool sigmoid, double out_scale, Tensor& y) {
+  check_rows(o, "o"); check_rows(gate, "gate"); check_rows(y, "y"); same_type(o, gate, "gate"); same_type(o, y, "y");
+  TORCH_CHECK(groups > 0 && o.size(1) % groups == 0 && gate.sizes() == o.sizes() && y.sizes() == o.sizes(), "norm_gate shapes");
+  check_vec(w, o.size(1) / groups, "w");
+  const c10::cuda::CUDAGuard guard(o.device());
+  NC_CHECK(norm_gate(is_f32(o), o.data_ptr(), pitch(o), gate.data_ptr(), pitch(gate), w.data_ptr<float>(), (float)eps, (int)o.size(0), (int)groups, (int)n,
+                     (int)(o.size(1) / groups), sigmoid ? 1 : 0, (float)out_scale, y.data_ptr(), pitch(y), nullptr, stream()));
+}
+// The same for the delta rule's heads (silu), and the ring keeps the rows' last convolution inputs (z's channels).
+void delta_finish(const Tensor& o, const Tensor& gate, const Tensor& w, double eps, Tensor& y, const Tensor& z, const std::vector<int64_t>& size,
+                  const Tensor& conv, const Tensor& neg_a, const Tensor& dt_bias, const Tensor& ring, const Tensor& lens, int64_t per_seq) {
+  check_rows(o, "o"); check_rows(gate, "gate"); check_rows(y, "y"); same_type(o, gate, "gate"); same_type(o, y, "y"); same_type(o, z, "z");
+  const DeltaInputs d = delta_inputs(z, size, conv, c10::nullopt, neg_a, dt_bias, ring, lens, per_seq, is_f32(o));
+  TORCH_CHECK(o.size(0) == z.size(0) && o.size(1) == size[0] * size[5] && gate.sizes() == o.sizes() && y.sizes() == o.sizes(), "delta_finish shapes");
+  check_vec(w, size[5], "w");
+  const c10::cuda::CUDAGuard guard(o.device());
+  NC_CHECK(norm_gate(is_f32(o), o.data_ptr(), pitch(o), gate.data_ptr(), pitch(gate), w.data_ptr<float>(), (float)eps, (int)o.size(0), (int)size[0], (int)size[4],
+                     (int)size[5], 0, 1.f, y.data_ptr(), pitch(y), &d, stream()));
+}
+// One token per row, z to y.
+void delta_step_(const Tensor& z, const std::vector<int64_t>& size, const Tensor& conv, const Tensor& ba, const Tensor& neg_a, const Tensor& dt_bias,
+                 const Tensor& ring, const Tensor& state, const Tensor& lens, const Tensor& norm, double eps, int64_t gate_off, Tensor& y) {
+  check_rows(y, "y");
+  DeltaStep d{};
+  d.in = delta_inputs(z, size, conv, ba, neg_a, dt_bias, ring, lens, 1, is_f32(y));
+  d.state = state_ref(state, z.size(0), size[0] * size[3] * size[5], "state");
+  check_vec(norm, size[5], "norm");
+  TORCH_CHECK(gate_off >= 0 && gate_off + size[0] * size[5] <= z.size(1) && y.size(0) == z.size(0) && y.size(1) == size[0] * size[5], "delta_step shapes");
+  d.norm = norm.data_ptr<float>(); d.eps = (float)eps; d.gate_off = (int)gate_off; d.y = y.data_ptr(); d.ldy = pitch(y);
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(delta_step(d, stream()));
+}
+
+// size: [heads, kv_heads, dp, q_off, k_off, window]; real: [scale, softcap, out_scale]
+WindowAttn window_of(const Tensor& z, const std::vector<int64_t>& size, const std::vector<double>& real, const Tensor& freq, const Tensor& pool,
+                     const Tensor& table, const Tensor& lens, int64_t per_seq) {
+  check_rows(z, "z");
+  TORCH_CHECK(size.size() == 6 && real.size() == 3 && size[0] > 0 && size[1] > 0 && is_f32(freq) && freq.is_cuda() && freq.is_contiguous() &&
+              freq.numel() % 2 == 0, "window attention: sizes");
+  TORCH_CHECK(size[3] >= 0 && size[3] + size[0] * size[2] <= z.size(1) && size[4] >= 0 && size[4] + size[1] * size[2] <= z.size(1), "window attention: segments of z");
+  WindowAttn d{};
+  d.f32 = is_f32(pool); d.z_f32 = is_f32(z); d.z = z.data_ptr(); d.ldz = pitch(z); d.q_off = (int)size[3]; d.k_off = (int)size[4];
+  d.rows = (int)z.size(0); d.heads = (int)size[0]; d.kv_heads = (int)size[1]; d.dp = (int)size[2]; d.dims = (int)freq.numel(); d.freq = freq.data_ptr<float>();
+  d.pg = pages_of(pool, table); d.pos = positions(lens, table, per_seq, z.size(0)); d.window = (int)size[5];
+  d.scale = (float)real[0]; d.softcap = (float)real[1]; d.out_scale = (float)real[2];
+  return d;
+}
+void window_out(WindowAttn& d, Tensor& y, const Tensor& pool) {
+  check_rows(y, "y"); same_type(y, pool, "y");
+  TORCH_CHECK(y.size(0) == d.rows && y.size(1) == (int64_t)d.heads * d.dp, "window attention: output");
+  d.y = y.data_ptr(); d.ldy = pitch(y);
+}
+void window_post_(Tensor& z, const std::vector<int64_t>& size, const std::vector<double>& real, const Tensor& freq, const Tensor& pool, const Tensor& table,
+                  const Tensor& lens, int64_t per_seq, const optional<Tensor>& dense) {
+  const WindowAttn d = window_of(z, size, real, freq, pool, table, lens, per_seq);
+  same_type(z, pool, "pool");
+  if (has(dense)) {
+    check_rows(*dense, "dense"); same_type(*dense, pool, "dense");
+    TORCH_CHECK(dense->size(0) == z.size(0) && dense->size(1) == pool.size(2), "dense: one entry per row");
+  }
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(window_post(d, has(dense) ? dense->data_ptr() : nullptr, has(dense) ? pitch(*dense) : 0, status_ptr(z), stream()));
+}
+void window_attention_(const Tensor& z, const std::vector<int64_t>& size, const std::vector<double>& real, const Tensor& freq, const Tensor& pool,
+                       const Tensor& table, const Tensor& lens, int64_t per_seq, Tensor& y) {
+  WindowAttn d = window_of(z, size, real, freq, pool, table, lens, per_seq);
+  same_type(z, pool, "pool");
+  window_out(d, y, pool);
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(window_attention(d, stream()));
+}
+// size: [heads, dp, vdim, vp, q_off, k_off, v_off, gate_off]; real: [eps, out_scale]
+DecayStep decay_of(const Tensor& z, const std::vector<int64_t>& size, const std::vector<double>& real, const Tensor& log_decay, const Tensor& state,
+                   const Tensor& lens, const Tensor& norm, Tensor& o, Tensor& done, Tensor& y) {
+  check_rows(z, "z"); check_rows(y, "y");
+  TORCH_CHECK(size.size() == 8 && real.size() == 2 && size[0] > 0, "fixed decay: sizes");
+  const int64_t H = size[0], dp = size[1], vp = size[3], width = H * vp, rows = z.size(0);
+  for (int i = 4; i < 8; ++i) TORCH_CHECK(size[i] >= 0 && size[i] + H * (i < 6 ? dp : vp) <= z.size(1), "fixed decay: segments of z");
+  check_vec(log_decay, H, "log_decay"); check_vec(norm, width, "norm"); check_vec(o, rows * width, "o");
+  TORCH_CHECK(done.is_cuda() && done.scalar_type() == at::kInt && done.is_contiguous() && done.numel() >= rows && y.size(0) == rows && y.size(1) == width, "fixed decay: outputs");
+  DecayStep d{};
+  d.f32 = is_f32(y); d.z_f32 = is_f32(z); d.z = z.data_ptr(); d.ldz = pitch(z);
+  d.heads = (int)H; d.dp = (int)dp; d.vdim = (int)size[2]; d.vp = (int)vp; d.q_off = (int)size[4]; d.k_off = (int)size[5]; d.v_off = (int)size[6]; d.gate_off = (int)size[7];
+  d.rows = (int)rows; d.log_decay = log_decay.data_ptr<float>(); d.state = state_ref(state, rows, H * dp * vp, "state"); d.pos = row_pos(lens, 1, rows);
+  d.norm = norm.data_ptr<float>(); d.eps = (float)real[0]; d.out_scale = (float)real[1]; d.o = o.data_ptr<float>(); d.done = done.data_ptr<int>();
+  d.y = y.data_ptr(); d.ldy = pitch(y);
+  return d;
+}
+void window_step(const Tensor& z, const std::vector<int64_t>& size, const std::vector<double>& real, const Tensor& freq, const Tensor& pool, const Tensor& table,
+                 const Tensor& lens, Tensor& y) {
+  WindowAttn d = window_of(z, size, real, freq, pool, table, lens, 1);
+  window_out(d, y, pool);
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(parallel_step(&d, nullptr, status_ptr(z), stream()));
+}
+void decay_step(const Tensor& z, const std::vector<int64_t>& size, const std::vector<double>& real, const Tensor& log_decay, const Tensor& state,
+                const Tensor& lens, const Tensor& norm, Tensor& o, Tensor& done, Tensor& y) {
+  const DecayStep d = decay_of(z, size, real, log_decay, state, lens, norm, o, done, y);
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(parallel_step(nullptr, &d, status_ptr(z), stream()));
+}
+// Both in one launch: y_left and y_right may be column ranges of one buffer.
+void parallel_step_(const Tensor& z, const std::vector<int64_t>& wsize, const std::vector<double>& wreal, const Tensor& freq, const Tensor& pool,
+                    const Tensor& table, const Tensor& lens, Tensor& y_left, const std::vector<int64_t>& dsize, const std::vector<double>& dreal,
+                    const Tensor& log_decay, const Tensor& state, const Tensor& norm, Tensor& o, Tensor& done, Tensor& y_right) {
+  WindowAttn w = window_of(z, wsize, wreal, freq, pool, table, lens, 1);
+  window_out(w, y_left, pool);
+  const DecayStep d = decay_of(z, dsize, dreal, log_decay, state, lens, norm, o, done, y_right);
+  const c10::cuda::CUDAGuard guard(z.device());
+  NC_CHECK(parallel_step(&w, &d, status_ptr(z), stream()));
+}
+
 std::vector<int64_t> read_status(const Tensor& like) {
   Tensor& t = status_tensor(like.device());
   const Tensor h = t.cpu();
@@ -419,12 +682,34 @@ std::vector<int64_t> read_status(const Tensor& like) {
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
-  m.def("gemm", &gemm, py::arg("A"), py::arg("B"), py::arg("C"), py::arg("m_group") = py::none());
+  m.def("gemm", &gemm, py::arg("A"), py::arg("B"), py::arg("C"), py::arg("m_group") = py::none(), py::arg("epi") = 0,
+        py::arg("aux") = py::none());
+  m.def("attention_capped", &attention_capped);
+  m.def("attention_capped_supported", &nc::attention_capped_supported);
   m.def("attention_split", &attention_split);
   m.def("attention_split_supported", &nc::attention_split_supported);
   m.def("embed_norm", &embed_norm_);
   m.def("gated_residual_norm", &gated_residual_norm_);
   m.def("poly_norm", &poly_norm_);
+  m.def("layer_norm_residual", &layer_norm_residual_);
+  m.def("gemv_plain", &gemv_plain, py::arg("x"), py::arg("W"), py::arg("out"), py::arg("next") = py::none());
+  m.def("gemv_relu_glu", &gemv_relu_glu_, py::arg("x"), py::arg("W"), py::arg("out"), py::arg("next") = py::none());
+  m.def("delta_prepare", &delta_prepare_);
+  m.def("silu_rows", &silu_rows_);
+  m.def("recurrence", &recurrence_);
+  m.def("recurrence_chunks_supported", &recurrence_chunks_supported);
+  m.def("recurrence_scratch", &recurrence_scratch);
+  m.def("norm_gate", &norm_gate_);
+  m.def("delta_finish", &delta_finish);
+  m.def("delta_step", &delta_step_);
+  m.def("delta_step_supported", &delta_step_supported);
+  m.def("window_post", &window_post_);
+  m.def("window_attention", &window_attention_);
+  m.def("window_step", &window_step);
+  m.def("window_step_supported", &window_step_supported);
+  m.def("decay_step", &decay_step);
+  m.def("decay_step_supported", &decay_step_supported);
+  m.def("parallel_step", &parallel_step_);
   m.def("latent_post", &latent_post_);
   m.def("latent_gather", &latent_gather_);
   m.def("rotate_heads", &rotate_heads_);

@@ -128,6 +128,35 @@ __device__ __forceinline__ long long token_offset(const Pages& pg, int s, int t)
   return ((long long)page << pg.shift | (t & ((1 << pg.shift) - 1))) * pg.width;
 }
 
+// (cos, sin) of position * f, f = freq[i] + freq[half + i] (a frequency and what its float leaves over): the product's own
+// rounding error and the left-over enter to first order, so the angle is good to 2^-24 of a turn's size at any position
+__device__ __forceinline__ float2 turn_of(int position, const float* freq, int i, int half) {
+  const float p = (float)position, f = freq[i], a = p * f;
+  const float rest = fmaf(p, f, -a) + p * freq[half + i];
+  float sn, cs;
+  sincosf(a, &sn, &cs);
+  return make_float2(cs - rest * sn, sn + rest * cs);
+}
+
+// ------------------------------------------------------------------- rows, key ranges
+constexpr float NEG_BIG = -1.0e30f;
+__device__ __forceinline__ int row_position(const RowPos& p, int row, int& seq) {
+  seq = row / p.per_seq;
+  return p.lens[seq] + row - seq * p.per_seq;
+}
+
+struct KeyRange { int begin, end; };       // this split's keys
+__device__ __forceinline__ KeyRange split_keys(int pos, int window, int splits, int split, int tile) {
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int n = pos - lo + 1;
+  int chunk = (n + splits - 1) / splits;
+  chunk = (chunk + tile - 1) / tile * tile;
+  KeyRange r;
+  r.begin = lo + split * chunk;
+  r.end = min(pos + 1, r.begin + chunk);
+  return r;
+}
+
 // ---------------------------------------------------------------------------- routing
 // One warp: the entry that follows (last_v, last_i) in the order of falling value, rising index among equals.
 __device__ __forceinline__ void next_best(const float* z, int n, float last_v, int last_i, int lane, float& v, int& i) {

@@ -9,6 +9,7 @@
 //   gemv            one product; input norm (linear once the row statistic is known: the statistic rides along), gated
 //                   residual update of the output, extra CTAs that append the step's entries to the latent store
 //                   Few outputs and a long K: four CTAs of a cluster share K and add up over distributed shared memory
+//   gemv_relu_glu   gate and up product of a dense feed-forward with its activation
 //   expert_*_rows   a step's experts: every chosen expert's weights are read once for all rows that chose it (down: the
 //                   four CTAs of a cluster take every fourth expert)
 #include <cooperative_groups.h>
@@ -245,6 +246,40 @@ __global__ void __cluster_dims__(1, CLUSTER, 1) __launch_bounds__(THREADS) gemv_
   gemv_body<false, 1, CLUSTER>(a);
 }
 
+// Gate and up rows of the same outputs as the two tiles of a CTA; the activation closes the product.
+__global__ void __launch_bounds__(THREADS) gemv_relu_glu_kernel(const GemvArgs a) {
+  constexpr int U = 2;
+  __shared__ float s_acc[WARPS][32][ROWS + 1];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n0 = blockIdx.x * 16, q8 = (lane & 3) * 8, row = lane >> 2;
+  prefetch_l2_slice(a.next, blockIdx.x, a.n_blocks);
+  const TileRows<1> wg = tile_rows<1>(a.W, a.ldw, n0, a.N, lane), wu = tile_rows<1>(a.W + a.N * a.ldw, a.ldw, n0, a.N, lane);
+  const TileRows<2> w = {{wg.lo[0], wu.lo[0]}, {wg.hi[0], wu.hi[0]}};
+  Frag<2, U> f;
+  load_frag(f, w, warp * 32, q8, a.K);
+  pdl_wait();
+  pdl_trigger();
+  float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+  const bf16* xb = (const bf16*)a.x + row * a.ldx;
+  auto x = [&](int k) -> uint4 { return row < a.B ? *reinterpret_cast<const uint4*>(xb + k) : make_uint4(0, 0, 0, 0); };
+  for (int k0 = warp * 32; k0 < a.K;) {
+    mma_frag(acc, f, k0, q8, a.K, x);
+    k0 += U * WARPS * 32;
+    if (k0 < a.K) load_frag(f, w, k0, q8, a.K);
+  }
+  spill_tiles<2>(acc, s_acc, warp, lane);
+  __syncthreads();
+  if (tid < 16 * ROWS) {
+    const int m = tid & 15, b = tid >> 4, n = n0 + m;
+    if (b < a.B && n < a.N) {
+      float g = 0.f, u = 0.f;
+#pragma unroll
+      for (int i = 0; i < WARPS; ++i) { g += s_acc[i][m][b]; u += s_acc[i][m + 16][b]; }
+      ((bf16*)a.out)[b * a.ldo + n] = __float2bfloat16_rn(fmaxf(g, 0.f) * u);
+    }
+  }
+}
+
 // ----------------------------------------------------------------------------- experts
 // The step's choices (rows * top of them) in shared memory, with the position of each expert's first mention and how
 // many distinct experts were mentioned before it.
@@ -405,6 +440,14 @@ cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s) {
   if (pre == PRE_PLAIN && !wide && a.n_blocks < 148 && d.K >= 3072) return launch(d.pdl, gemv_cluster_kernel, dim3(grid, CLUSTER), dim3(THREADS), 0, s, a);
   auto kern = pre == PRE_NORM ? (wide ? gemv_kernel<true, 2> : gemv_kernel<true, 1>) : (wide ? gemv_kernel<false, 2> : gemv_kernel<false, 1>);
   return launch(d.pdl, kern, dim3(grid), dim3(THREADS), 0, s, a);
+}
+
+cudaError_t gemv_relu_glu(const GemvDesc& d, cudaStream_t s) {
+  if (d.rows < 1 || d.rows > ROWS || d.N <= 0 || d.K <= 0 || (d.K & 7) || (d.ldx & 7) || (d.ldw & 7) || d.out == nullptr) return cudaErrorInvalidValue;
+  GemvArgs a{};
+  a.x = d.x; a.ldx = d.ldx; a.W = (const bf16*)d.W; a.ldw = d.ldw; a.B = d.rows; a.N = d.N; a.K = d.K; a.out = d.out; a.ldo = d.ldo; a.next = d.next;
+  a.n_blocks = (d.N + 15) / 16;
+  return launch(d.pdl, gemv_relu_glu_kernel, dim3(a.n_blocks), dim3(THREADS), 0, s, a);
 }
 
 bool expert_rows_supported(int rows, int top) { return rows >= 1 && rows <= ROWS && rows * top <= MAX_CHOICES; }

@@ -11,19 +11,14 @@
 //   latent_values    combines the splits and applies the value projection
 // Scores and weights are float; the exponent base is 2 (scale carries log2 e).
 #include "latent_store.cuh"
+#include "mma.cuh"
 
 namespace nc {
 namespace serve {
 
 namespace {
 
-constexpr float NEG_BIG = -1.0e30f;
 constexpr int MAX_SPLITS = 32;
-
-__device__ __forceinline__ int row_position(const RowPos& p, int row, int& seq) {
-  seq = row / p.per_seq;
-  return p.lens[seq] + row - seq * p.per_seq;
-}
 
 // ---------------------------------------------------------------------- post / gather
 // grid (rows, 1 or 2): y = 0 the store entry, y = 1 the query latent. The norm weights' padding is zero.
@@ -166,18 +161,6 @@ absorb_query_kernel(const T* __restrict__ q, long long ldq, int heads, int head_
 }
 
 // -------------------------------------------------------------------------- attention
-struct KeyRange { int begin, end; };       // this split's keys
-__device__ __forceinline__ KeyRange split_keys(int pos, int window, int splits, int split, int tile) {
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-  const int n = pos - lo + 1;
-  int chunk = (n + splits - 1) / splits;
-  chunk = (chunk + tile - 1) / tile * tile;
-  KeyRange r;
-  r.begin = lo + split * chunk;
-  r.end = min(pos + 1, r.begin + chunk);
-  return r;
-}
-
 // Plain form. grid (splits, heads, rows), 128 threads; dynamic shared memory: W + kvp floats.
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -266,23 +249,6 @@ latent_attention_kernel(const LatentAttn d) {
 // keys, then owns every eighth 16-column unit of the weighted latents.
 constexpr int KT = 64;                       // keys per tile
 constexpr int AW = 8;                        // warps
-__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-
 __host__ __device__ constexpr int padded_width(int W) { return (W + 31) / 32 * 32; }      // scores step through 32 columns
 inline size_t mma_smem_bytes(int W) { return (size_t)(16 + KT) * (padded_width(W) + 8) * 2 + (size_t)16 * (KT + 8) * 2; }
 

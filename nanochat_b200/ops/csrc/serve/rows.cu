@@ -3,6 +3,8 @@
 //   embed_norm            token embedding into the float residual stream, and its norm
 //   gated_residual_norm   residual update by sigmoid-gated sublayer outputs (a mixture of experts' weighted rows are
 //                         summed on the way in), then the next norm: one pass, the row stays in registers / L1
+//   layer_norm_residual   a sublayer's output normed, added to the residual stream, and the next sublayer's norm; the same
+//                         with a token's embedding in place of the sublayer opens the stream
 //   poly_norm             the normed-powers activation
 // One CTA per row.
 #include "common.cuh"
@@ -105,6 +107,85 @@ gated_residual_norm_kernel(float* __restrict__ x, TermsT terms, float mult, cons
   }
 }
 
+// A row of np <= 2048 * NV entries sits in the registers of 256 threads: entry (i * 256 + threadIdx.x) * 8 + j.
+template <int NV, typename TY>
+__device__ __forceinline__ void load_row(float (&v)[NV][8], const TY* src, int np) {
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * 256 + threadIdx.x) * 8;
+    if (c < np) {
+      load8(src + c, v[i]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
+    }
+  }
+}
+// v = (v - mean) / sqrt(variance + eps) * w over the first n entries; w is zero past them
+template <int NV>
+__device__ __forceinline__ void layer_norm_row(float (&v)[NV][8], const float (&w)[NV][8], int n, float eps, float* red) {
+  float s[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[0] += v[i][j];             // padding is zero
+  block_sum<1>(s, red);
+  const float mean = s[0] / n;
+  s[0] = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * 256 + threadIdx.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      v[i][j] -= mean;
+      if (c + j < n) s[0] += v[i][j] * v[i][j];
+    }
+  }
+  block_sum<1>(s, red);
+  const float r = inv_rms(s[0], n, eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[i][j] *= r * w[i][j];
+}
+
+// T: type of h; TY: type of y (an embedding table's rows when ids is given)
+template <typename T, typename TY, int NV>
+__global__ void __launch_bounds__(256)
+layer_norm_residual_kernel(const long long* __restrict__ ids, const TY* __restrict__ y, long long ldy, int vocab, const float* __restrict__ wy,
+                           float* __restrict__ x, const float* __restrict__ w, float eps, int n, int np, T* __restrict__ h) {
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  float wv[NV][8], v[NV][8], xv[NV][8];
+  load_row<NV>(wv, wy, np);
+  pdl_wait();
+  pdl_trigger();
+  long long src = row;
+  if (ids != nullptr) {
+    src = ids[row];
+    src = src < 0 ? 0 : (src >= vocab ? vocab - 1 : src);
+  }
+  load_row<NV>(v, y + src * ldy, np);
+  if (ids == nullptr) load_row<NV>(xv, (const float*)x + row * np, np);
+  layer_norm_row<NV>(v, wv, n, eps, red);
+  load_row<NV>(wv, w, np);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * 256 + threadIdx.x) * 8;
+    if (ids == nullptr) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] += xv[i][j];
+    }
+    if (c < np) store8(x + row * np + c, v[i]);
+  }
+  layer_norm_row<NV>(v, wv, n, eps, red);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * 256 + threadIdx.x) * 8;
+    if (c < np) store8(h + row * np + c, v[i]);
+  }
+}
+
 template <typename T, typename TZ>
 __global__ void __launch_bounds__(256)
 poly_norm_kernel(const TZ* __restrict__ z, long long ldz, const float* __restrict__ coef, float eps, int n, int np,
@@ -157,6 +238,22 @@ cudaError_t gated_residual_norm(bool f32, float* x, const GatedTerm* terms, int 
   if (f32) gated_residual_norm_kernel<float><<<rows, 256, 0, s>>>(x, t, mult, extra, w, eps, n, np, (float*)h);
   else gated_residual_norm_kernel<bf16><<<rows, 256, 0, s>>>(x, t, mult, extra, w, eps, n, np, (bf16*)h);
   return cudaGetLastError();
+}
+
+template <typename T, typename TY>
+static cudaError_t launch_layer_norm(const long long* ids, const TY* y, long long ldy, int vocab, const float* wy, float* x, const float* w,
+                                     float eps, int rows, int n, int np, T* h, cudaStream_t s) {
+  auto k = np <= 2048 ? layer_norm_residual_kernel<T, TY, 1> : np <= 4096 ? layer_norm_residual_kernel<T, TY, 2> : layer_norm_residual_kernel<T, TY, 4>;
+  return launch_pdl(k, dim3(rows), dim3(256), 0, s, ids, y, ldy, vocab, wy, x, w, eps, n, np, h);
+}
+
+cudaError_t layer_norm_residual(bool f32, bool y_f32, const long long* ids, const void* y, long long ldy, int vocab, const float* wy, float* x,
+                                const float* w, float eps, int rows, int n, int np, void* h, cudaStream_t s) {
+  if (rows <= 0 || n <= 0 || n > np || np > 8192 || (np & 7) || (ldy & 7) || ldy < np || (ids && vocab <= 0) || (f32 && !y_f32))
+    return cudaErrorInvalidValue;
+  if (f32) return launch_layer_norm(ids, (const float*)y, ldy, vocab, wy, x, w, eps, rows, n, np, (float*)h, s);
+  if (y_f32) return launch_layer_norm(ids, (const float*)y, ldy, vocab, wy, x, w, eps, rows, n, np, (bf16*)h, s);
+  return launch_layer_norm(ids, (const bf16*)y, ldy, vocab, wy, x, w, eps, rows, n, np, (bf16*)h, s);
 }
 
 cudaError_t poly_norm(bool f32, bool z_f32, const void* z, long long ldz, const float* coef, float eps, int rows, int n, int np,

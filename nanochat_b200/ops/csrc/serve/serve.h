@@ -1,5 +1,7 @@
-// Host interface of the serving kernels: rows.cu (norms, gated residual, activations), gemv.cu (matrix-vector products of
-// a decode step), latent.cu (latent attention over a paged store) and experts.cu (mixture of experts).
+// Host interface of the serving kernels: rows.cu (norms, residual updates, activations), gemv.cu (matrix-vector products of
+// a decode step), latent.cu (latent attention over a paged store), experts.cu (mixture of experts), window.cu (window
+// attention whose values are its unrotated keys), recurrent.cu (gated delta rule, linear attention with a fixed decay) and
+// step.cu (one token of the last two per row).
 //
 // Conventions. "f32" selects float or bf16 for the typed pointers (weights and activations share one type). The
 // residual stream, gates' biases, norm weights, router logits and attention partials are always float. Row sizes and
@@ -48,6 +50,11 @@ struct GatedTerm {
 cudaError_t gated_residual_norm(bool f32, float* x, const GatedTerm* terms, int n_terms, float mult, const float* extra,
                                 const float* w, float eps, int rows, int n, int np, void* h, cudaStream_t s);
 
+// x[r] += N(y[r]) * wy; h[r] = N(x[r]) * w, N the layer norm (mean removed) over the row's n entries. With ids given the
+// stream opens: x[r] = N(y[ids[r]]) * wy, ids clamped to [0, vocab). Rows of up to 8192 entries.
+cudaError_t layer_norm_residual(bool f32, bool y_f32, const long long* ids, const void* y, long long ldy, int vocab, const float* wy, float* x,
+                                const float* w, float eps, int rows, int n, int np, void* h, cudaStream_t s);
+
 // out[r] = c[0] N(z) + c[1] N(z^2) + c[2] N(z^3) + c[3], N(v) = v / rms(v) over the row's n entries.
 cudaError_t poly_norm(bool f32, bool z_f32, const void* z, long long ldz, const float* coef, float eps, int rows, int n, int np,
                       void* out, long long ldo, cudaStream_t s);
@@ -83,6 +90,8 @@ struct GemvDesc {
   bool pdl;
 };
 cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s);
+// out[b, j] = relu(x[b] . W[j]) * (x[b] . W[N + j]), bf16: W holds N gate rows, then N up rows (PRE_PLAIN fields of d)
+cudaError_t gemv_relu_glu(const GemvDesc& d, cudaStream_t s);
 // The experts of a decode step, rows <= 8: out[b] = mult * sigmoid(g + bias) * sum_k wt[b, k] expert(idx[b, k])(h[b]) (+ extra).
 // act: rows * top x fp scratch.
 struct ExpertRows {
@@ -166,6 +175,107 @@ struct ExpertDown {
   void* y; long long ldy;
 };
 cudaError_t expert_down(const ExpertDown& d, cudaStream_t s);
+
+// ---------------------------------------------------------------------------- window.cu
+// Window attention with grouped keys that also serve as values: entry of a token in the store = [kv_heads x dp rotated
+// keys | kv_heads x dp keys as projected]. Rotation pairs entries 2i and 2i + 1 of the first `dims`. Scores are
+// softcap * tanh(scale q.k / softcap) (softcap <= 0: no cap); y is multiplied by out_scale. freq: dims / 2 frequencies,
+// then what their floats leave over.
+struct WindowAttn {
+  bool f32, z_f32;
+  const void* z; long long ldz;           // queries at q_off (heads x dp), keys at k_off (kv_heads x dp)
+  int q_off, k_off;
+  int rows, heads, kv_heads, dp, dims; const float* freq;
+  Pages pg; RowPos pos;
+  int window;                             // keys a query sees, itself included; <= 0: all
+  float scale, softcap, out_scale;
+  void* y; long long ldy;                 // rows x (heads x dp)
+};
+// Queries rotated in place, the rows' entries into the store and (dense) a dense row.
+cudaError_t window_post(const WindowAttn& d, void* dense, long long ldd, int* status, cudaStream_t s);
+// Plain form for any size: rotated queries in z against the store, which holds the rows' own entries already.
+cudaError_t window_attention(const WindowAttn& d, cudaStream_t s);
+
+// ------------------------------------------------------------------------- recurrent.cu
+// Two recurrences over a per-sequence state S (heads x dp x vp floats):
+//   delta    S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q      unit keys and queries, g and beta per token
+//   decay    S <- decay_h S + k v^T;           o = S^T q
+// A sequence at position 0 starts from zeros whatever its state memory holds.
+struct StateRef {
+  float* ptr; long long seq_stride;       // floats between sequences
+};
+// Inputs of the delta rule: q and k of kv_heads heads, v of heads heads, as projected, side by side in z (channels
+// [0, 2 kv_heads dp + heads vp)); a causal convolution of `taps` per channel and silu come first. The ring keeps the inputs
+// of the last taps - 1 tokens per channel: token t in slot t % taps.
+struct DeltaInputs {
+  bool f32, z_f32;
+  const void* z; long long ldz;
+  int rows, heads, kv_heads, dim, dp, vdim, vp, taps;
+  const float* conv;                      // taps x channels, the last row meets the current token
+  const float* ba; long long ldba; int a_off;   // per row: heads logits of beta, at a_off heads inputs of the decay
+  const float* neg_a; const float* dt_bias;     // log g = neg_a * softplus(a + dt_bias)
+  StateRef ring;
+  RowPos pos;
+};
+// Convolution and silu of every channel into act (rows x channels); norms (rows x 2 kv_heads) = 1 / |q| * dim^-1/2, then
+// 1 / |k|; beta_g (rows x 2 heads) = beta, then log g.
+cudaError_t delta_prepare(const DeltaInputs& d, void* act, float* norms, float* beta_g, cudaStream_t s);
+// act = silu(z) over n columns (multiple of 8).
+cudaError_t silu_rows(bool f32, const void* z, long long ldz, int rows, int n, void* act, long long lda, cudaStream_t s);
+
+struct Recurrence {
+  bool f32;
+  const void* act; long long lda;         // rows: q at q_off, k at k_off (kv_heads x dp), v at v_off (heads x vp)
+  int q_off, k_off, v_off;
+  int rows, heads, kv_heads, dp, vp;
+  const float* norms; const float* beta_g;      // delta rule
+  const float* log_decay;                       // fixed decay: natural logarithm per head (beta_g == nullptr)
+  StateRef state;
+  RowPos pos;
+  void* o; long long ldo;                 // rows x (heads x vp)
+};
+// Token by token; any T, float or bf16, dp <= 512.
+cudaError_t recurrence_scan(const Recurrence& d, cudaStream_t s);
+// Chunks of 64 tokens on the tensor cores, bf16, dp <= 128. scratch: recurrence_scratch() bytes.
+bool recurrence_chunks_supported(int dp);
+size_t recurrence_scratch(int seqs, int per_seq, int heads, bool delta);
+cudaError_t recurrence_chunks(const Recurrence& d, void* scratch, cudaStream_t s);
+
+// y = o / rms(o) * w * act(gate) * out_scale; groups of np entries (n real ones) are normed apart, w (np) is shared by the
+// groups. act: 0 silu, 1 sigmoid. ring (optional, delta): also keep the last inputs of the rows' convolution.
+cudaError_t norm_gate(bool f32, const void* o, long long ldo, const void* gate, long long ldg, const float* w, float eps, int rows, int groups,
+                      int n, int np, int act, float out_scale, void* y, long long ldy, const DeltaInputs* ring, cudaStream_t s);
+
+// ------------------------------------------------------------------------------ step.cu
+// One token per row (RowPos::per_seq == 1).
+// Delta rule from z to y (rows x (heads x vp), bf16 or float), state and ring updated, norm and silu gate included.
+struct DeltaStep {
+  DeltaInputs in;
+  StateRef state;
+  const float* norm; float eps;
+  int gate_off;                           // gate logits in z (heads x vp)
+  void* y; long long ldy;
+};
+bool delta_step_supported(int dp, int vp);
+cudaError_t delta_step(const DeltaStep& d, cudaStream_t s);
+// Fixed decay from z to y: q, k, v, gate logits side by side at q_off, k_off, v_off, gate_off of z.
+struct DecayStep {
+  bool f32, z_f32;
+  const void* z; long long ldz;
+  int q_off, k_off, v_off, gate_off;
+  int rows, heads, dp, vp, vdim;
+  const float* log_decay;
+  StateRef state;
+  RowPos pos;
+  const float* norm; float eps, out_scale;
+  float* o;                               // rows x (heads x vp) scratch
+  int* done;                              // rows counters, zero before and after
+  void* y; long long ldy;
+};
+bool decay_step_supported(int dp, int vp);
+// Either mechanism or both side by side in one launch; attention (bf16) appends the token's entry to the store itself.
+bool window_step_supported(bool f32, int dp);
+cudaError_t parallel_step(const WindowAttn* left, const DecayStep* right, int* status, cudaStream_t s);
 
 }  // namespace serve
 }  // namespace nc

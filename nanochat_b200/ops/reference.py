@@ -228,8 +228,9 @@ def muon_update(grads, params, momentum_buf, second_buf, momentum, lr, wd, beta2
 
 # ------------------------------------------------------------------- inference mechanisms
 # Plain bodies of `ops/serving.py`: latent attention over a paged store, gated residual update, normed-powers
-# activation, mixture of experts. Weight holders are the modules of `nanochat_b200.models.lupodra` (sizes padded with
-# zeros). Products run in the weights' type, everything else in float32.
+# activation, mixture of experts, layer-normed residual update, gated delta rule, window attention and fixed-decay linear
+# attention. Weight holders are the modules of `nanochat_b200.models` (sizes padded with zeros). Products run in the
+# weights' type, everything else in float32.
 
 def linear_rows(h, w, out_dtype=None):
     if out_dtype is not None and out_dtype != h.dtype:
@@ -330,3 +331,115 @@ def mixture(h, p):
             out = (g * torch.sigmoid(g) * u).to(h.dtype) @ p.w_down[e].t()
             y.index_add_(0, row, out.float() * wt[row, k, None])
     return (y.to(h.dtype),)
+
+
+def _layer_norm(x, w, eps, n):
+    d = torch.zeros_like(x)
+    d[:, :n] = x[:, :n] - x[:, :n].mean(-1, keepdim=True)
+    return d * _rms(d, eps, n) * w
+
+
+def embed_layer_norm(ids, table, vocab, w_embed, w, eps, n):
+    x = _layer_norm(table[ids.clamp(0, vocab - 1)].float(), w_embed, eps, n)
+    return x, _layer_norm(x, w, eps, n).to(table.dtype)
+
+
+def layer_norm_residual(x, y, w_post, w, eps, n, dtype):
+    x += _layer_norm(y.float(), w_post, eps, n)
+    return _layer_norm(x, w, eps, n).to(dtype)
+
+
+def relu_glu(h, w_gate_up):
+    g, u = (h @ w_gate_up.t()).float().chunk(2, -1)
+    return (torch.relu(g) * u).to(h.dtype)
+
+
+def _silu(x):
+    return x * torch.sigmoid(x)
+
+
+def gated_delta(p, z, ba, cache, run, T):
+    R, H, G, dp, vp, n = z.shape[0], p.heads, p.kv_heads, p.dp, p.vp, p.channels
+    S_all, ring_all = cache.states[run]["S"], cache.states[run]["ring"]
+    x, out = z[:, :n].float(), torch.empty(R, H, vp, device=z.device)
+    for b in range(R // T):
+        start = int(cache.cache_seqlens[b])
+        S = S_all[b].clone() if start else torch.zeros_like(S_all[b])
+        for t in range(T):
+            r, pos = b * T + t, start + t
+            a = p.conv[p.taps - 1] * x[r]
+            for i in range(1, min(p.taps, pos + 1)):
+                a = a + p.conv[p.taps - 1 - i] * ring_all[b, (pos - i) % p.taps]
+            ring_all[b, pos % p.taps] = x[r]
+            a = _silu(a)
+            q, k, v = a[:G * dp].view(G, dp), a[G * dp:2 * G * dp].view(G, dp), a[2 * G * dp:].view(H, vp)
+            unit = lambda u: (u / torch.sqrt(u.square().sum(-1, keepdim=True) + 1e-6)).repeat_interleave(H // G, 0)
+            q, k = unit(q) * p.dim ** -0.5, unit(k)
+            beta = torch.sigmoid(ba[r, :H])
+            g = torch.exp(p.neg_a[:H] * torch.nn.functional.softplus(ba[r, p.hp:p.hp + H] + p.dt_bias[:H]))
+            S = S * g[:, None, None]
+            u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", S, k))
+            S = S + k[:, :, None] * u[:, None, :]
+            out[r] = torch.einsum("hdv,hd->hv", S, q)
+        S_all[b] = S
+    y = out * _rms(out, p.eps, p.vdim) * p.norm
+    return (y.view(R, -1) * _silu(z[:, p.gate_off:p.gate_off + H * vp].float())).to(z.dtype)
+
+
+def _rotate_interleaved(x, positions, freq):
+    """x (R, heads, n): entries 2i and 2i + 1 turn by positions * f[i]; freq: f rounded to float, and the rest of it."""
+    angle = (positions.double()[:, None] * freq.double().sum(0))[:, None]
+    c, s, d = angle.cos().float(), angle.sin().float(), freq.numel()
+    out = x.clone()
+    out[..., 0:d:2] = x[..., 0:d:2] * c - x[..., 1:d:2] * s
+    out[..., 1:d:2] = x[..., 1:d:2] * c + x[..., 0:d:2] * s
+    return out
+
+
+def window_attention(p, z, cache, run, T, y):
+    R, pool, H, G, dp = z.shape[0], cache.pools[run], p.heads, p.kv_heads, p.dp
+    P, flat, table = pool.shape[1], pool.view(-1, pool.shape[2]), cache.table.long()
+    start = cache.cache_seqlens.long()
+    pos = (start[:, None] + torch.arange(T, device=z.device)).reshape(R)
+    seq = torch.arange(R, device=z.device) // T
+    q = _rotate_interleaved(z[:, p.q_off:p.k_off].float().view(R, H, dp), pos, p.freq).to(z.dtype).float()
+    k = z[:, p.k_off:p.end].float().view(R, G, dp)
+    flat[table[seq, pos // P] * P + pos % P] = torch.cat([_rotate_interleaved(k, pos, p.freq), k], 1).reshape(R, -1).to(pool.dtype)
+    for b in range(R // T):
+        rows = slice(b * T, (b + 1) * T)
+        j = torch.arange(int(start[b]) + T, device=z.device)
+        kv = flat[table[b, j // P] * P + j % P].float().view(-1, 2, G, dp).repeat_interleave(H // G, 2)
+        score = torch.einsum("rhd,jhd->hrj", q[rows], kv[:, 0]) * p.scale
+        if p.softcap > 0:
+            score = p.softcap * torch.tanh(score / p.softcap)
+        gap = pos[rows, None] - j
+        hidden = gap < 0
+        if p.window is not None:
+            hidden = hidden | (gap >= p.window)
+        w = torch.softmax(score.masked_fill(hidden, -float("inf")), -1)
+        y[rows] = (torch.einsum("hrj,jhd->rhd", w, kv[:, 1]) * p.out_scale).reshape(T, -1).to(y.dtype)
+    return y
+
+
+def decay_attention(p, z, cache, run, T, y):
+    R, H, S_all = z.shape[0], p.heads, cache.states[run]["S"]
+    q, k = (_silu(z[:, a:a + H * p.dp].float()).to(z.dtype).float().view(R, H, p.dp) for a in (p.q_off, p.k_off))
+    v = _silu(z[:, p.v_off:p.gate_off].float()).to(z.dtype).float().view(R, H, p.vp)
+    out, decay = torch.empty(R, H, p.vp, device=z.device), torch.exp(p.log_decay)[:, None, None]
+    for b in range(R // T):
+        S = S_all[b].clone() if int(cache.cache_seqlens[b]) else torch.zeros_like(S_all[b])
+        for r in range(b * T, (b + 1) * T):
+            S = decay * S + k[r][:, :, None] * v[r][:, None, :]
+            out[r] = torch.einsum("hdv,hd->hv", S, q[r])
+        S_all[b] = S
+    out = out.view(R, -1)
+    gate = torch.sigmoid(z[:, p.gate_off:p.end].float())
+    y[:] = (out * _rms(out, p.eps, H * p.vdim) * p.norm * gate * p.out_scale).to(y.dtype)
+    return y
+
+
+def window_and_decay(left, right, z, cache, run, T):
+    y = torch.empty(z.shape[0], left.y_width + right.y_width, dtype=z.dtype, device=z.device)
+    window_attention(left, z, cache, run, T, y[:, :left.y_width])
+    decay_attention(right, z, cache, run, T, y[:, left.y_width:])
+    return y

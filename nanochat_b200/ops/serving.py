@@ -1,10 +1,11 @@
 """
 Native bodies of the inference mechanisms (`nanochat_b200._S`): latent attention over a paged store, gated residual
-updates, the normed-powers activation, mixtures of experts, and the row linear they share. Every function has a plain
-PyTorch body of the same name in `reference.py`; `ops.__init__` picks one per call.
+updates, the normed-powers activation, mixtures of experts; layer-normed residual updates, the gated delta rule, window
+attention whose values are its keys, linear attention with a fixed decay; and the row linear they share. Every function has
+a plain PyTorch body of the same name in `reference.py`; `ops.__init__` picks one per call.
 
 Rows: a step brings B sequences x T tokens, flattened to B * T rows (row r is token r % T of sequence r // T). Weight
-holders (`p`) are the modules of `nanochat_b200.models.lupodra`: sizes padded to multiples of 8 (16 for what the store
+holders (`p`) are the modules of `nanochat_b200.models` (lupodra, safepel): sizes padded to multiples of 8 (16 for what the store
 holds) with zeros, so that every kernel reads whole 16-byte vectors.
 
 bf16: products on the tcgen05 GEMM. float: the same kernels in float, products by the library in true float32.
@@ -18,6 +19,7 @@ _S = load_serving_extension()
 
 BF16 = torch.bfloat16
 ABSORB_ROWS = 8          # portions up to this many tokens run on absorbed queries (weights dominate), longer ones expand
+CHUNK_ROWS = 16          # portions above this many tokens run their recurrences in chunks, shorter ones token by token
 SPLIT_KEYS = 64          # keys per tile of the tensor-core attention over stored entries
 
 
@@ -168,3 +170,113 @@ def mixture(h, p):
     _S.silu_mul(gu, tile_group, act)
     _S.gemm(act, p.w_down, y, tile_group)
     return (y, slot, wt)
+
+
+# ----------------------------------------------------------- layer-normed residual, feed-forward
+
+def embed_layer_norm(ids, table, vocab, w_embed, w, eps, n):
+    """(x, h): the normed token embeddings as float residual stream, and the first sublayer's norm of it."""
+    x = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
+    h = torch.empty(x.shape, dtype=table.dtype, device=table.device)
+    _S.layer_norm_residual(ids, table, vocab, w_embed, x, w, eps, n, h)
+    return x, h
+
+
+def layer_norm_residual(x, y, w_post, w, eps, n, dtype):
+    """x += norm(y) * w_post in place; returns norm(x) * w."""
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    _S.layer_norm_residual(None, y, 0, w_post, x, w, eps, n, h)
+    return h
+
+
+def relu_glu(h, w_gate_up):
+    """relu(h Wg^T) * (h Wu^T): the activation and the product ride on the two products' epilogues."""
+    fp = w_gate_up.shape[0] // 2
+    if h.dtype == BF16:
+        out = torch.empty(h.shape[0], fp, dtype=BF16, device=h.device)
+        _S.gemm(h, w_gate_up[:fp], out, epi=1)
+        _S.gemm(h, w_gate_up[fp:], out, epi=2, aux=out)
+        return out
+    return torch.relu(linear_rows(h, w_gate_up[:fp])) * linear_rows(h, w_gate_up[fp:])
+
+
+# -------------------------------------------------------------------------------- recurrences
+
+def _recurrence(act, heads, kv_heads, dp, vp, state, cache, T, norms=None, beta_g=None, log_decay=None):
+    o = torch.empty(act.shape[0], heads * vp, dtype=act.dtype, device=act.device)
+    scratch = None
+    if act.dtype == BF16 and T > CHUNK_ROWS and _S.recurrence_chunks_supported(dp):
+        scratch = torch.empty(_S.recurrence_scratch(act.shape[0] // T, T, heads, beta_g is not None), dtype=torch.uint8, device=act.device)
+    _S.recurrence(act, [heads, kv_heads, dp, vp], norms, beta_g, log_decay, state, cache.cache_seqlens, T, o, scratch)
+    return o
+
+
+def gated_delta(p, z, ba, cache, run, T):
+    """What the mixer's output product reads (R, heads * vp); state and convolution inputs move on by T tokens."""
+    R, S, ring = z.shape[0], cache.states[run]["S"], cache.states[run]["ring"]
+    y = torch.empty(R, p.y_width, dtype=z.dtype, device=z.device)
+    if T == 1 and _S.delta_step_supported(p.dp, p.vp):
+        _S.delta_step(z, p.sizes, p.conv, ba, p.neg_a, p.dt_bias, ring, S, cache.cache_seqlens, p.norm, p.eps, p.gate_off, y)
+        return y
+    act = torch.empty(R, p.channels, dtype=z.dtype, device=z.device)
+    norms = torch.empty(R, 2 * p.kv_heads, device=z.device)
+    beta_g = torch.empty(R, 2 * p.heads, device=z.device)
+    _S.delta_prepare(z, p.sizes, p.conv, ba, p.neg_a, p.dt_bias, ring, cache.cache_seqlens, T, act, norms, beta_g)
+    o = _recurrence(act, p.heads, p.kv_heads, p.dp, p.vp, S, cache, T, norms, beta_g)
+    _S.delta_finish(o, z[:, p.gate_off:p.gate_off + p.y_width], p.norm, p.eps, y, z, p.sizes, p.conv, p.neg_a, p.dt_bias, ring, cache.cache_seqlens, T)
+    return y
+
+
+def decay_attention(p, z, cache, run, T, y):
+    """y (R, heads * vp) from p's segments of z; the state moves on by T tokens."""
+    R, S = z.shape[0], cache.states[run]["S"]
+    if T == 1 and _S.decay_step_supported(p.dp, p.vp):
+        o = torch.empty(R, p.y_width, device=z.device)
+        _S.decay_step(z, p.sizes, p.reals, p.log_decay, S, cache.cache_seqlens, p.norm, o, cache.done, y)
+        return y
+    qkv = z[:, p.q_off:p.gate_off]
+    act = torch.empty(qkv.shape, dtype=z.dtype, device=z.device)
+    _S.silu_rows(qkv, act)
+    o = _recurrence(act, p.heads, p.heads, p.dp, p.vp, S, cache, T, log_decay=p.log_decay)
+    _S.norm_gate(o, z[:, p.gate_off:p.end], p.norm, p.eps, 1, p.heads * p.vdim, True, p.out_scale, y)
+    return y
+
+
+# ----------------------------------------------------------------- window attention, keys as values
+
+def window_attention(p, z, cache, run, T, y):
+    """y (R, heads * dp) from p's segments of z (the queries' is overwritten); appends the step's entries to the store."""
+    R, pool, table, lens = z.shape[0], cache.pools[run], cache.table, cache.cache_seqlens
+    if T == 1 and _S.window_step_supported(pool.dtype != BF16, p.dp):
+        _S.window_step(z, p.sizes, p.reals, p.freq, pool, table, lens, y)
+        return y
+    tiles = pool.dtype == BF16 and R == T and _S.attention_capped_supported(p.dp, p.dp)
+    entries = None
+    if tiles:
+        before = cache.get_pos()
+        seen = before if p.window is None else min(before, p.window - 1)
+        entries = torch.empty(seen + T, p.entry, dtype=pool.dtype, device=z.device)
+    _S.window_post(z, p.sizes, p.reals, p.freq, pool, table, lens, T, entries[seen:] if tiles else None)
+    if not tiles:
+        _S.window_attention(z, p.sizes, p.reals, p.freq, pool, table, lens, T, y)
+        return y
+    if seen:
+        _S.latent_gather(pool, table, 0, before - seen, entries[:seen])
+    kv = entries.view(-1, 2, p.kv_heads, p.dp)
+    _S.attention_capped(z[:, p.q_off:p.k_off].unflatten(1, (p.heads, p.dp)), kv[:, 0], kv[:, 1], y.unflatten(1, (p.heads, p.dp)),
+                        -1 if p.window is None else p.window - 1, p.scale, p.softcap, p.out_scale)
+    return y
+
+
+def window_and_decay(left, right, z, cache, run, T):
+    """Both mechanisms on one z into one y: [left | right]."""
+    y = torch.empty(z.shape[0], left.y_width + right.y_width, dtype=z.dtype, device=z.device)
+    y_left, y_right = y[:, :left.y_width], y[:, left.y_width:]
+    if T == 1 and _S.window_step_supported(z.dtype != BF16, left.dp) and _S.decay_step_supported(right.dp, right.vp):
+        o = torch.empty(z.shape[0], right.y_width, device=z.device)
+        _S.parallel_step(z, left.sizes, left.reals, left.freq, cache.pools[run], cache.table, cache.cache_seqlens, y_left,
+                         right.sizes, right.reals, right.log_decay, cache.states[run]["S"], right.norm, o, cache.done, y_right)
+        return y
+    window_attention(left, z, cache, run, T, y_left)
+    decay_attention(right, z, cache, run, T, y_right)
+    return y

@@ -10,7 +10,7 @@ position-dependent quantity is read from device memory (`KVCache.cache_seqlens`)
 step is captured once per (engine, cache) and replayed with a single launch per token.
 
 `StepGraph` is the capture-and-replay shell; `DecodeGraph` is GPT's step, `LatentDecodeGraph` that of models over a
-paged latent store.
+paged latent store, `RecurrentDecodeGraph` that of models with recurrent states. A model names its step in `step_graph`.
 
 `decode_graph_for(engine, kv_cache)` returns the graph of a cache, or None when the
 fast path does not apply (CPU, kernels disabled, more than 64 rows, GPT with a head dim != 128).
@@ -323,6 +323,78 @@ class LatentDecodeGraph(StepGraph):
         K.gemv_norm(x, m.final_norm, eps, C, m.embed, self.all_logits)
 
 
+class RecurrentDecodeGraph(StepGraph):
+    """Decode step of models over a `RecurrentCache`.
+
+    Up to GEMV_ROWS bf16 rows: one chain of kernels, each launched so that it may start while the one before it ends:
+        input product  ->  mixer (delta rule; or window attention and fixed-decay heads side by side)  ->  output product
+        ->  its norm, residual, next norm  ->  gate and up product with the activation  ->  down product  ->  norms
+    Otherwise (more rows, float32, sizes a step kernel does not take): the model's forward over the rows, captured as it is."""
+
+    def __init__(self, model, kv_cache):
+        super().__init__(model, kv_cache)
+        S = ops.serving_module()._S
+        self.S = S
+        cfg, B, dev = model.config, self.B, kv_cache.cache_seqlens.device
+        self.all_logits = torch.empty(B, model.head.shape[0], dtype=torch.float32, device=dev)
+        self.logits = self.all_logits[:, :cfg.vocab_size]
+
+        def fits(mix):
+            if hasattr(mix, "left"):
+                return S.window_step_supported(False, mix.left.dp) and S.decay_step_supported(mix.right.dp, mix.right.vp)
+            return S.delta_step_supported(mix.dp, mix.vp)
+
+        self.fused = B <= GEMV_ROWS and model.dtype == torch.bfloat16 and all(fits(layer.mix) for layer in model.layers)
+        if not self.fused:
+            return
+        f32 = lambda *shape: torch.empty(*shape, dtype=torch.float32, device=dev)
+        b16 = lambda *shape: torch.empty(*shape, dtype=torch.bfloat16, device=dev)
+        most = lambda size: max((size(layer) for layer in model.layers), default=8)
+        self.x, self.h, self.out = f32(B, model.width), b16(B, model.width), f32(B, model.width)
+        self.z = f32(B * most(lambda l: l.mix.w_all.shape[0]))
+        self.y = b16(B * most(lambda l: l.mix.y_width))
+        self.act = b16(B * most(lambda l: 8 if l.mlp is None else l.mlp.fp))
+        self.o = f32(B * most(lambda l: l.mix.right.y_width if hasattr(l.mix, "right") else 8))
+
+    def _forward(self):
+        if self.fused:
+            self._fused_step()
+            self.cache.cache_seqlens.add_(1)
+        else:
+            pos = self.cache._pos
+            self.logits.copy_(self.model.forward(self.ids, kv_cache=self.cache)[:, 0])
+            self.cache._pos = pos                # step() moves the host's mirror, replayed or not
+
+    def _fused_step(self):
+        m, K, B, cache, cfg = self.model, self.S, self.B, self.cache, self.model.config
+        C, eps, lens, table = cfg.n_embd, cfg.eps, cache.cache_seqlens, cache.table
+        ahead = lambda w: w if PREFETCH_NEXT else None
+        view = lambda buf, n: buf[:B * n].view(B, n)
+        subs = m.sublayers()
+        opening = lambda sub: sub.w_gate_up if hasattr(sub, "w_gate_up") else sub.w_all
+        K.layer_norm_residual(self.ids, m.embed, cfg.vocab_size, m.embed_norm, self.x, m.first_norm, eps, C, self.h)
+        for n, (sub, post, after, i) in enumerate(subs):
+            following = opening(subs[n + 1][0]) if n + 1 < len(subs) else m.head[:LM_HEAD_PREFETCH_ROWS]
+            if i is None:
+                act = view(self.act, sub.fp)
+                K.gemv_relu_glu(self.h, sub.w_gate_up, act, ahead(sub.w_down))
+                K.gemv_plain(act, sub.w_down, self.out, ahead(following))
+            else:
+                z, y = view(self.z, sub.w_all.shape[0]), view(self.y, sub.y_width)
+                K.gemv_plain(self.h, sub.w_all, z, ahead(sub.w_o))
+                state = cache.states[i]
+                if hasattr(sub, "left"):
+                    a, b = sub.left, sub.right
+                    K.parallel_step(z, a.sizes, a.reals, a.freq, cache.pools[i], table, lens, y[:, :a.y_width], b.sizes, b.reals, b.log_decay,
+                                    state["S"], b.norm, view(self.o, b.y_width), cache.done, y[:, a.y_width:])
+                else:
+                    K.delta_step(z, sub.sizes, sub.conv, z[:, sub.channels + sub.y_width:], sub.neg_a, sub.dt_bias, state["ring"], state["S"],
+                                 lens, sub.norm, sub.eps, sub.gate_off, y)
+                K.gemv_plain(y, sub.w_o, self.out, ahead(following))
+            K.layer_norm_residual(None, self.out, 0, post, self.x, after, eps, C, self.h)
+        K.gemv_plain(self.h, m.head, self.all_logits)
+
+
 def graph_path_applies(model, rows):
     """True when `rows` sample rows of this model decode through the captured-graph kernels."""
     if ops.get_kernel_mode() != "native":
@@ -347,7 +419,7 @@ def decode_graph_for(engine, kv_cache):
     graphs = engine._decode_graphs
     g = graphs.get(id(kv_cache))
     if g is None or g.cache is not kv_cache or g.pool_version != getattr(kv_cache, "pool_version", 0):
-        kind = LatentDecodeGraph if hasattr(model, "make_cache") else DecodeGraph
+        kind = globals()[getattr(model, "step_graph", "DecodeGraph")]
         g = kind(model, kv_cache)              # first use, or the page pool moved: capture on the new addresses
         graphs[id(kv_cache)] = g
     return g

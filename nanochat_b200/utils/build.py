@@ -89,7 +89,7 @@ def _write_stamp(so_path, digest):
 # Optimizer and collective kernels keep IEEE division / square root and denormals: their state (second moments,
 # running norms) lives for the whole run, and approximate math there shows up as drift, not as noise.
 # The serving kernels also run in float, where angles, exponentials and statistics are held to float accuracy.
-PRECISE_SOURCES = ("optim.cu", "comm.cu", "rows.cu", "latent.cu", "experts.cu")
+PRECISE_SOURCES = ("optim.cu", "comm.cu", "rows.cu", "latent.cu", "experts.cu", "window.cu", "recurrent.cu", "step.cu")
 
 
 def _load(name, so_path):
