@@ -237,12 +237,13 @@ constexpr int LV = VS + 8;
 __host__ __device__ constexpr int up16(int n) { return (n + 15) / 16 * 16; }
 __host__ __device__ constexpr size_t chunk_bytes(bool delta) { return (size_t)(delta ? 4 : 2) * TRI * 2 + SCALARS * 4; }
 
-__device__ __forceinline__ float cumulative_64(float a, float b, int lane, float& first) {
-  // lane l holds entries 2l and 2l + 1; returns the inclusive sums of both
-  float s = a + b;
+// Inclusive sums of 64 entries, lane l holding entries 2l and 2l + 1. Double: a token that forgets nearly everything has a
+// large logarithm, and the tokens after it need the small differences behind it.
+__device__ __forceinline__ double cumulative_64(double a, double b, int lane, double& first) {
+  double s = a + b;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
-    const float t = __shfl_up_sync(0xffffffffu, s, o);
+    const double t = __shfl_up_sync(0xffffffffu, s, o);
     if (lane >= o) s += t;
   }
   first = s - b;
@@ -255,7 +256,8 @@ template <bool DELTA>
 __global__ void __launch_bounds__(128)
 chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  __shared__ float sG[CH], sB[CH], sRk[CH], sRq[CH];
+  __shared__ float sB[CH], sRk[CH], sRq[CH];
+  __shared__ double sG[CH];                                  // log decay from the chunk's start, each token's own included
   const int chunk = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, kvh = h / (r.heads / r.kv_heads);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int t0 = chunk * CH, n = min(CH, r.pos.per_seq - t0);
@@ -290,29 +292,29 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
         sB[i] = i < n ? bg[h] : 0.f;
         lg[e] = i < n ? bg[r.heads + h] : 0.f;
       }
-      float first;
-      const float second = cumulative_64(lg[0], lg[1], lane, first);
+      double first;
+      const double second = cumulative_64(lg[0], lg[1], lane, first);
       sG[lane * 2] = first; sG[lane * 2 + 1] = second;
     } else {
       const float ld = r.log_decay[h];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int i = lane * 2 + e;
-        sG[i] = ld * (i + 1);
+        sG[i] = (double)ld * (i + 1);
         sRq[i] = sRk[i] = i < n ? 1.f : 0.f;
       }
     }
     __syncwarp();
-    const float last = sG[n - 1];
+    const double last = sG[n - 1];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int i = lane * 2 + e;
-      const float g = expf(sG[i]);
+      const float g = expf((float)sG[i]);
       gS[i] = g * sRk[i];
       gS[CH + i] = g * sRq[i];
-      gS[2 * CH + i] = i < n ? sRk[i] * expf(DELTA ? last - sG[i] : r.log_decay[h] * (n - 1 - i)) : 0.f;
+      gS[2 * CH + i] = i < n ? sRk[i] * expf((float)(last - sG[i])) : 0.f;
     }
-    if (lane == 0) gS[3 * CH] = expf(last);
+    if (lane == 0) gS[3 * CH] = expf((float)last);
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -339,7 +341,6 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
     }
   }
   __syncthreads();
-  const float ld = DELTA ? 0.f : r.log_decay[h];
 #pragma unroll
   for (int t = 0; t < 8; ++t) {
     const int j = t * 8 + (lane & 3) * 2;
@@ -350,7 +351,7 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int c = j + e;
-        const float decay = c <= i ? expf(DELTA ? sG[i] - sG[c] : ld * (i - c)) : 0.f;
+        const float decay = c <= i ? expf((float)(sG[i] - sG[c])) : 0.f;
         a[e] = c <= i ? sRq[i] * sRk[c] * decay * qk[t][half * 2 + e] : 0.f;
         if constexpr (DELTA) l[e] = c < i ? sB[i] * sRk[i] * sRk[c] * decay * kk[t][half * 2 + e] : 0.f;
       }
