@@ -50,9 +50,9 @@ def parse_args():
     ap.add_argument("--precision", type=str, default="fp8", choices=["fp8", "bf16", "mxfp8"],
                     help="our arm: fp8 = tensorwise e4m3/e5m2 linear layers (the reference's headline recipe); mxfp8 = "
                          "block-scaled fp8 on the hardware block-scaled GEMM (module path, not the fused layer path)")
-    ap.add_argument("--serve", action="store_true",
-                    help="instead of the headline workload: serving throughput of the latent-attention model beside GPT at "
-                         "equal width and depth (scripts/serve_bench.py), with its kernels' distances from the roofline")
+    ap.add_argument("--serve", nargs="?", const="Lupodra", default=None, choices=["Lupodra", "Safepel"],
+                    help="instead of the headline workload: serving throughput of a served model beside GPT at equal width "
+                         "and depth (scripts/serve_bench.py), with its kernels' distances from the roofline")
     ap.add_argument("--ref-bf16", action="store_true", help="reference arm without --fp8")
     ap.add_argument("--ref-eager", action="store_true", help="reference arm without torch.compile")
     return ap.parse_args()
@@ -487,7 +487,7 @@ if __name__ == "__main__":
         if ROOT not in sys.path:
             sys.path.insert(0, ROOT)
         from scripts.serve_bench import main as serve_main
-        serve_main([])
+        serve_main(["--model", a.serve])
     elif a.impl == "reference":
         run_reference(a)
     else:

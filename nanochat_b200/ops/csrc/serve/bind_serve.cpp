@@ -510,31 +510,47 @@ DeltaInputs delta_inputs(const Tensor& z, const std::vector<int64_t>& size, cons
   d.ring = state_ref(ring, z.size(0) / per_seq, size[6] * channels, "ring");
   return d;
 }
+// Where prepared inputs go: rows x channels in the compute type, or (uint8) tiles.
+bool check_prepared(const Tensor& out, int64_t rows, int64_t per_seq, int64_t H, int64_t G, int64_t dp, int64_t vp, bool f32) {
+  TORCH_CHECK(out.is_cuda() && out.is_contiguous() && (reinterpret_cast<uintptr_t>(out.data_ptr()) & 15) == 0, "prepared inputs: dense, 16-byte aligned");
+  if (out.scalar_type() == at::kByte) {
+    TORCH_CHECK(!f32 && recurrence_chunks_supported((int)dp) && (size_t)out.numel() >= recurrence_tiles((int)(rows / per_seq), (int)per_seq, (int)H, (int)G, (int)dp, (int)vp),
+                "tiles: too small, or sizes the chunk kernels do not take");
+    return true;
+  }
+  TORCH_CHECK(is_f32(out) == f32 && (f32 || out.scalar_type() == at::kBFloat16) && out.dim() == 2 && out.size(0) == rows && out.size(1) == 2 * G * dp + H * vp,
+              "prepared inputs: rows x channels");
+  return false;
+}
 void delta_prepare_(const Tensor& z, const std::vector<int64_t>& size, const Tensor& conv, const Tensor& ba, const Tensor& neg_a, const Tensor& dt_bias,
-                    const Tensor& ring, const Tensor& lens, int64_t per_seq, Tensor& act, Tensor& norms, Tensor& beta_g) {
-  const DeltaInputs d = delta_inputs(z, size, conv, ba, neg_a, dt_bias, ring, lens, per_seq, is_f32(act));
-  check_rows(act, "act");
-  TORCH_CHECK(act.is_contiguous() && act.size(0) == z.size(0) && act.size(1) == 2 * size[1] * size[3] + size[0] * size[5] && is_f32(norms) && norms.is_contiguous() &&
-              norms.numel() >= z.size(0) * 2 * size[1] && is_f32(beta_g) && beta_g.is_contiguous() && beta_g.numel() >= z.size(0) * 2 * size[0], "delta rule: outputs");
+                    const Tensor& ring, const Tensor& lens, int64_t per_seq, Tensor& out, Tensor& norms, Tensor& beta_g) {
+  const DeltaInputs d = delta_inputs(z, size, conv, ba, neg_a, dt_bias, ring, lens, per_seq, is_f32(out));
+  const bool tiles = check_prepared(out, z.size(0), per_seq, size[0], size[1], size[3], size[5], is_f32(out));
+  TORCH_CHECK(is_f32(norms) && norms.is_contiguous() && norms.numel() >= z.size(0) * 2 * size[1] && is_f32(beta_g) && beta_g.is_contiguous() &&
+              beta_g.numel() >= z.size(0) * 2 * size[0], "delta rule: outputs");
   const c10::cuda::CUDAGuard guard(z.device());
-  NC_CHECK(delta_prepare(d, act.data_ptr(), norms.data_ptr<float>(), beta_g.data_ptr<float>(), stream()));
+  NC_CHECK(delta_prepare(d, tiles, out.data_ptr(), norms.data_ptr<float>(), beta_g.data_ptr<float>(), stream()));
 }
-void silu_rows_(const Tensor& z, Tensor& act) {
-  check_rows(z, "z"); check_rows(act, "act"); same_type(z, act, "act");
-  TORCH_CHECK(z.sizes() == act.sizes(), "silu_rows shapes");
+// z: q, k (heads x dp each), v (heads x vp) side by side
+void decay_prepare_(const Tensor& z, int64_t heads, int64_t dp, int64_t vp, int64_t per_seq, Tensor& out) {
+  check_rows(z, "z");
+  TORCH_CHECK(heads > 0 && z.size(1) == heads * (2 * dp + vp) && per_seq > 0 && z.size(0) % per_seq == 0, "decay_prepare shapes");
+  const bool tiles = check_prepared(out, z.size(0), per_seq, heads, heads, dp, vp, is_f32(z));
   const c10::cuda::CUDAGuard guard(z.device());
-  NC_CHECK(silu_rows(is_f32(z), z.data_ptr(), pitch(z), (int)z.size(0), (int)z.size(1), act.data_ptr(), pitch(act), stream()));
+  NC_CHECK(decay_prepare(is_f32(z), z.data_ptr(), pitch(z), (int)z.size(0), (int)per_seq, (int)heads, (int)dp, (int)vp, tiles, out.data_ptr(), stream()));
 }
-// size: [heads, kv_heads, dp, vp]; act: q, k, v side by side. norms and beta_g, or log_decay.
+// size: [heads, kv_heads, dp, vp]; act: what a prepare kernel left; norms and beta_g, or log_decay. Tiles need scratch.
 void recurrence_(const Tensor& act, const std::vector<int64_t>& size, const optional<Tensor>& norms, const optional<Tensor>& beta_g,
                  const optional<Tensor>& log_decay, const Tensor& state, const Tensor& lens, int64_t per_seq, Tensor& o, const optional<Tensor>& scratch) {
-  check_rows(act, "act"); check_rows(o, "o"); same_type(act, o, "o");
+  check_rows(o, "o");
   TORCH_CHECK(size.size() == 4 && size[0] > 0 && size[1] > 0, "recurrence: four sizes");
-  const int64_t H = size[0], G = size[1], dp = size[2], vp = size[3], rows = act.size(0);
-  TORCH_CHECK(2 * G * dp + H * vp <= act.size(1) && o.size(0) == rows && o.size(1) == H * vp, "recurrence shapes");
+  const int64_t H = size[0], G = size[1], dp = size[2], vp = size[3], rows = o.size(0);
+  TORCH_CHECK(o.size(1) == H * vp, "recurrence shapes");
   Recurrence d{};
-  d.f32 = is_f32(act); d.act = act.data_ptr(); d.lda = pitch(act); d.q_off = 0; d.k_off = (int)(G * dp); d.v_off = (int)(2 * G * dp);
+  d.f32 = is_f32(o); d.act = act.data_ptr(); d.lda = 2 * G * dp + H * vp; d.q_off = 0; d.k_off = (int)(G * dp); d.v_off = (int)(2 * G * dp);
   d.rows = (int)rows; d.heads = (int)H; d.kv_heads = (int)G; d.dp = (int)dp; d.vp = (int)vp;
+  d.pos = row_pos(lens, per_seq, rows);
+  const bool tiles = check_prepared(act, rows, per_seq, H, G, dp, vp, d.f32);
   const bool delta = has(beta_g);
   if (delta) {
     TORCH_CHECK(has(norms), "delta rule: norms");
@@ -545,15 +561,14 @@ void recurrence_(const Tensor& act, const std::vector<int64_t>& size, const opti
     check_vec(*log_decay, H, "log_decay");
     d.log_decay = log_decay->data_ptr<float>();
   }
-  d.pos = row_pos(lens, per_seq, rows);
   d.state = state_ref(state, rows / per_seq, H * dp * vp, "state");
   d.o = o.data_ptr(); d.ldo = pitch(o);
-  const c10::cuda::CUDAGuard guard(act.device());
-  if (has(scratch)) {
-    TORCH_CHECK(scratch->is_cuda() && scratch->is_contiguous() && (reinterpret_cast<uintptr_t>(scratch->data_ptr()) & 15) == 0 &&
+  const c10::cuda::CUDAGuard guard(o.device());
+  if (tiles) {
+    TORCH_CHECK(has(scratch) && scratch->is_cuda() && scratch->is_contiguous() && (reinterpret_cast<uintptr_t>(scratch->data_ptr()) & 15) == 0 &&
                 (size_t)(scratch->numel() * scratch->element_size()) >= recurrence_scratch((int)(rows / per_seq), (int)per_seq, (int)H, delta), "scratch: too small");
     ++g_launches;
-    NC_CHECK(recurrence_chunks(d, scratch->data_ptr(), stream()));
+    NC_CHECK(recurrence_chunks(d, scratch->data_ptr(), status_ptr(o), stream()));
   } else {
     NC_CHECK(recurrence_scan(d, stream()));
   }
@@ -695,10 +710,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemv_plain", &gemv_plain, py::arg("x"), py::arg("W"), py::arg("out"), py::arg("next") = py::none());
   m.def("gemv_relu_glu", &gemv_relu_glu_, py::arg("x"), py::arg("W"), py::arg("out"), py::arg("next") = py::none());
   m.def("delta_prepare", &delta_prepare_);
-  m.def("silu_rows", &silu_rows_);
+  m.def("decay_prepare", &decay_prepare_);
   m.def("recurrence", &recurrence_);
   m.def("recurrence_chunks_supported", &recurrence_chunks_supported);
   m.def("recurrence_scratch", &recurrence_scratch);
+  m.def("recurrence_tiles", &recurrence_tiles);
   m.def("norm_gate", &norm_gate_);
   m.def("delta_finish", &delta_finish);
   m.def("delta_step", &delta_step_);

@@ -1,8 +1,8 @@
 // Recurrences over a per-sequence state (dp x vp floats a head): the gated delta rule and linear attention with a fixed
 // decay per head, for portions of several tokens.
 //
-//   delta_prepare     short convolution + silu of queries, keys and values, inverse norms, step sizes, log decays
-//   silu_rows         the activation of the fixed-decay inputs
+//   prepare           short convolution + silu of queries, keys and values (fixed decay: silu alone), inverse norms, step
+//                     sizes, log decays; as rows for the token-by-token kernel or as the chunk kernels' tiles
 //   recurrence_scan   token by token, the state in registers: float, short portions, wide heads
 //   recurrence_chunks chunks of 64 tokens, two kernels:
 //       gram   (parallel over chunks) A = (Q K^T) with decays, causal; for the delta rule also the inverse of the unit
@@ -11,11 +11,15 @@
 //                 R = V - decayed K S,  U = T R        delta rule;   U = V  fixed decay
 //                 O = decayed Q S + A U
 //                 S = decayed S + K^T (decayed U)
+//              One warp copies whole chunks into shared memory, four follow the state from chunk to chunk, four more
+//              read it out behind them.
 //   norm_gate         RMS norm and gate of what a recurrence read out, and the convolution's last inputs
 //
 // Exactness: the products run on bf16 operands, so every operand that is a float (the state, T, A, U, R) enters as the sum
 // of two bf16 values, and what scales rows (inverse norms, decays) is applied to accumulators, not to operands: keys,
 // queries and values are the bf16 activations themselves. The state is float from chunk to chunk.
+#include <type_traits>
+
 #include "mma.cuh"
 
 namespace nc {
@@ -39,23 +43,51 @@ __device__ __forceinline__ void store4(bf16* p, const float (&f)[4]) {
   *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
 }
 
+// ------------------------------------------------------------------------------ tiles
+constexpr int CH = 64;                       // tokens per chunk
+constexpr int LT = CH + 8;                   // pitch of a 64 x 64 operand
+constexpr int MAT = CH * LT;
+constexpr int SCALARS = 200;                 // floats per chunk and head: three vectors of 64, the chunk's total decay, padding
+constexpr int VS = 16;                       // state columns per CTA
+constexpr int LV = VS + 8;
+
+__host__ __device__ constexpr int tile_dim(int dp) { return dp <= 64 ? 64 : 128; }          // columns of a q or k tile
+// Tiles of a portion, bf16: per (sequence, chunk, key head) q then k, 64 x (D + 8); behind them per (sequence, chunk, head,
+// slice of 16 columns) v, 64 x 24. Rows past the portion and columns past a head are zero, the pitch's padding is anything.
+struct Tiles {
+  int chunks, D, slices;
+  long long qk_unit, v_unit, v_base;         // elements
+  __host__ __device__ Tiles(int seqs, int per_seq, int heads, int kv_heads, int dp, int vp) {
+    chunks = (per_seq + CH - 1) / CH;
+    D = tile_dim(dp);
+    slices = (vp + VS - 1) / VS;
+    qk_unit = 2ll * CH * (D + 8);
+    v_unit = (long long)CH * LV;
+    v_base = (long long)seqs * chunks * kv_heads * qk_unit;
+  }
+  __host__ __device__ long long elements(int seqs, int heads) const { return v_base + (long long)seqs * chunks * heads * slices * v_unit; }
+};
+__host__ __device__ constexpr size_t chunk_bytes(bool delta) { return (size_t)(delta ? 4 : 2) * MAT * 2 + SCALARS * 4; }
+
 // ---------------------------------------------------------------------------- prepare
 constexpr int PREP_TOKENS = 8;         // tokens a warp walks through
 
 // grid (token groups of a sequence, ceil(jobs / 4), sequences), a warp per job: query heads, key heads, value heads.
-// TAPS > 0: at most TAPS taps, the inputs slide through registers; 0: any number, re-read
-template <typename T, typename TZ, int TAPS>
+// TAPS > 0: at most TAPS taps, the inputs stay in registers; 0: any number, re-read; -1: no convolution and no norms
+// (fixed decay). TILES: out is laid out as Tiles, otherwise rows x channels.
+template <typename T, typename TZ, int TAPS, bool TILES>
 __global__ void __launch_bounds__(128)
-delta_prepare_kernel(const DeltaInputs d, T* __restrict__ act, float* __restrict__ norms, float* __restrict__ beta_g) {
+prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ norms, float* __restrict__ beta_g) {
   const int lane = threadIdx.x & 31, job = blockIdx.y * 4 + (threadIdx.x >> 5);
   const int G = d.kv_heads, H = d.heads, per_seq = d.pos.per_seq, seq = blockIdx.z;
   if (job >= 2 * G + H) return;
-  const int t0 = blockIdx.x * PREP_TOKENS, n = min(PREP_TOKENS, per_seq - t0);
+  const int t0 = blockIdx.x * PREP_TOKENS, n = min(PREP_TOKENS, per_seq - t0);      // n <= 0: only zeros to write
   const int channels = 2 * G * d.dp + H * d.vp, size = job < 2 * G ? d.dp : d.vp;
   const int ch0 = job < 2 * G ? job * d.dp : 2 * G * d.dp + (job - 2 * G) * d.vp;
-  const int start = d.pos.lens[seq];
+  const int start = TAPS >= 0 ? d.pos.lens[seq] : 0;
   const long long row0 = (long long)seq * per_seq;
-  const float* ring = d.ring.ptr + seq * d.ring.seq_stride;
+  const float* ring = TAPS >= 0 ? d.ring.ptr + seq * d.ring.seq_stride : nullptr;
+  const Tiles tiles(gridDim.z, per_seq, H, G, d.dp, d.vp);
   auto fetch = [&](int t, int ch, float (&x)[4]) {
     if (t >= 0) {
       load4((const TZ*)d.z + (row0 + t) * d.ldz + ch, x);
@@ -65,55 +97,72 @@ delta_prepare_kernel(const DeltaInputs d, T* __restrict__ act, float* __restrict
       x[0] = x[1] = x[2] = x[3] = 0.f;
     }
   };
+  auto place = [&](int t, int c) -> T* {                // c: column of the job's head
+    if (!TILES) return out + (row0 + t0 + t) * channels + ch0 + c;
+    const long long unit = (long long)seq * tiles.chunks + t0 / CH;
+    const int r = t0 % CH + t;
+    if (job < 2 * G) return out + (unit * G + job % G) * tiles.qk_unit + ((job >= G ? CH : 0) + r) * (tiles.D + 8) + c;
+    return out + tiles.v_base + ((unit * H + job - 2 * G) * tiles.slices + c / VS) * tiles.v_unit + r * LV + c % VS;
+  };
   float ss[PREP_TOKENS];
 #pragma unroll
   for (int t = 0; t < PREP_TOKENS; ++t) ss[t] = 0.f;
-  for (int c = lane * 4; c < size; c += 128) {
+  const int columns = !TILES ? size : job < 2 * G ? tiles.D : tiles.slices * VS;
+  for (int c = lane * 4; c < columns; c += 128) {
     const int ch = ch0 + c;
-    constexpr int HELD = TAPS > 0 ? TAPS : 1;
-    float w[HELD][4], x[HELD][4];                       // tap i meets the token i places back
+    constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0;
+    float w[BACK + 1][4], x[PREP_TOKENS + BACK][4];     // x[BACK + t]: token t of the group
+    const bool in = c < size;
+#pragma unroll
+    for (int t = 0; t < PREP_TOKENS + BACK; ++t) {
+      if (in && TAPS != 0 && t - BACK < n && (t >= BACK || BACK - t < d.taps)) {
+        fetch(t0 + t - BACK, ch, x[t]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[t][j] = 0.f;
+      }
+    }
     if (TAPS > 0) {
 #pragma unroll
-      for (int i = 0; i < HELD; ++i) {
-        if (i < d.taps) {
+      for (int i = 0; i <= BACK; ++i) {                 // tap i meets the token i places back
+        if (in && i < d.taps) {
           load4(d.conv + (long long)(d.taps - 1 - i) * channels + ch, w[i]);
-          if (i > 0) fetch(t0 - i, ch, x[i]);
         } else {
 #pragma unroll
-          for (int j = 0; j < 4; ++j) w[i][j] = x[i][j] = 0.f;
+          for (int j = 0; j < 4; ++j) w[i][j] = 0.f;
         }
       }
     }
 #pragma unroll
     for (int t = 0; t < PREP_TOKENS; ++t) {
-      if (t >= n) break;
+      if (!TILES && t >= n) break;
       float a[4] = {0.f, 0.f, 0.f, 0.f};
       if (TAPS > 0) {
-        fetch(t0 + t, ch, x[0]);
 #pragma unroll
-        for (int i = 0; i < HELD; ++i)
+        for (int i = 0; i <= BACK; ++i)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) a[j] += w[i][j] * x[i][j];
+          for (int j = 0; j < 4; ++j) a[j] += w[i][j] * x[BACK + t - i][j];
+      } else if (TAPS == 0) {
+        for (int i = 0; in && t < n && i < d.taps; ++i) {
+          float wi[4], xi[4];
+          load4(d.conv + (long long)(d.taps - 1 - i) * channels + ch, wi);
+          fetch(t0 + t - i, ch, xi);
 #pragma unroll
-        for (int i = HELD - 1; i > 0; --i)
-#pragma unroll
-          for (int j = 0; j < 4; ++j) x[i][j] = i < d.taps ? x[i - 1][j] : 0.f;
-      } else {
-        for (int i = 0; i < d.taps; ++i) {
-          load4(d.conv + (long long)(d.taps - 1 - i) * channels + ch, w[0]);
-          fetch(t0 + t - i, ch, x[0]);
-#pragma unroll
-          for (int j = 0; j < 4; ++j) a[j] += w[0][j] * x[0][j];
+          for (int j = 0; j < 4; ++j) a[j] += wi[j] * xi[j];
         }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) a[j] = x[t][j];
       }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        a[j] = to_f(from_f<T>(silu_of<T>(a[j])));       // the norm is that of the vector that is stored
+        a[j] = t < n ? to_f(from_f<T>(silu_of<T>(a[j]))) : 0.f;     // the norm is that of the vector that is stored
         ss[t] += a[j] * a[j];
       }
-      store4(act + (row0 + t0 + t) * channels + ch, a);
+      store4(place(t, c), a);
     }
   }
+  if (TAPS < 0) return;
   if (job < 2 * G) {
 #pragma unroll
     for (int t = 0; t < PREP_TOKENS; ++t) {
@@ -124,24 +173,10 @@ delta_prepare_kernel(const DeltaInputs d, T* __restrict__ act, float* __restrict
     const int h = job - 2 * G;
     const float* in = d.ba + (row0 + t0 + lane) * d.ldba;
     const float a = in[d.a_off + h] + d.dt_bias[h];
-    float* out = beta_g + (row0 + t0 + lane) * 2 * H;
-    out[h] = sigmoidf(in[h]);
-    out[H + h] = d.neg_a[h] * (a > 20.f ? a : log1pf(expf(a)));
+    float* bg = beta_g + (row0 + t0 + lane) * 2 * H;
+    bg[h] = sigmoidf(in[h]);
+    bg[H + h] = d.neg_a[h] * (a > 20.f ? a : log1pf(expf(a)));
   }
-}
-
-template <typename T>
-__global__ void __launch_bounds__(256)
-silu_rows_kernel(const T* __restrict__ z, long long ldz, int rows, int n, T* __restrict__ act, long long lda) {
-  const int per = n / 8;
-  const long long i = (long long)blockIdx.x * 256 + threadIdx.x, row = i / per;
-  if (row >= rows) return;
-  const int c = (int)(i - row * per) * 8;
-  float v[8];
-  load8(z + row * ldz + c, v);
-#pragma unroll
-  for (int j = 0; j < 8; ++j) v[j] = silu_of<T>(v[j]);
-  store8(act + row * lda + c, v);
 }
 
 // ------------------------------------------------------------------------------- scan
@@ -227,16 +262,6 @@ recurrence_scan_kernel(const Recurrence r) {
 }
 
 // ------------------------------------------------------------------------------ chunks
-constexpr int CH = 64;                       // tokens per chunk
-constexpr int TRI = CH * CH;                 // one 64 x 64 operand
-constexpr int LT = CH + 8;                   // its pitch in shared memory
-constexpr int SCALARS = 200;                 // floats per chunk and head: three vectors of 64, the chunk's total decay, padding
-constexpr int VS = 16;                       // state columns per CTA
-constexpr int LV = VS + 8;
-
-__host__ __device__ constexpr int up16(int n) { return (n + 15) / 16 * 16; }
-__host__ __device__ constexpr size_t chunk_bytes(bool delta) { return (size_t)(delta ? 4 : 2) * TRI * 2 + SCALARS * 4; }
-
 // Inclusive sums of 64 entries, lane l holding entries 2l and 2l + 1. Double: a token that forgets nearly everything has a
 // large logarithm, and the tokens after it need the small differences behind it.
 __device__ __forceinline__ double cumulative_64(double a, double b, int lane, double& first) {
@@ -249,36 +274,92 @@ __device__ __forceinline__ double cumulative_64(double a, double b, int lane, do
   first = s - b;
   return s;
 }
+__device__ __forceinline__ void store_split(bf16* hi_at, bf16* lo_at, float a, float b) {
+  bf16 hi[2], lo[2];
+  split_bf16(a, hi[0], lo[0]);
+  split_bf16(b, hi[1], lo[1]);
+  *reinterpret_cast<__nv_bfloat162*>(hi_at) = __nv_bfloat162(hi[0], hi[1]);
+  *reinterpret_cast<__nv_bfloat162*>(lo_at) = __nv_bfloat162(lo[0], lo[1]);
+}
+
+// Two neighbouring entries (r, c), (r, c + 1) of the product of two 16 x 16 blocks in shared memory.
+constexpr int LL = CH + 4;
+__device__ __forceinline__ void block_dot(const float* a, const float* b, int lda, int ldb, int r, int c, float (&s)[2]) {
+#pragma unroll
+  for (int k = 0; k < 16; k += 4) {
+    const float4 l = *reinterpret_cast<const float4*>(a + r * lda + k);
+    const float lk[4] = {l.x, l.y, l.z, l.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 x = *reinterpret_cast<const float2*>(b + (k + e) * ldb + c);
+      s[0] += lk[e] * x.x;
+      s[1] += lk[e] * x.y;
+    }
+  }
+}
+// X = (1 + L)^-1 for a strictly lower triangular L, both 64 x LL floats; blocks of 16: the diagonal ones by forward
+// substitution, the others below them from the left. All 128 threads call it; L has been written and synchronised.
+__device__ void invert_unit_lower(const float* L, float* X, float (*P)[16][20]) {
+  const int tid = threadIdx.x;
+  if (tid < CH) {
+    const int b = tid & ~15, j = tid & 15;
+    float x[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      float s[2] = {i == j ? 1.f : 0.f, 0.f};
+#pragma unroll
+      for (int m = 0; m < i; ++m) s[m & 1] -= L[(b + i) * LL + b + m] * x[m];
+      x[i] = s[0] + s[1];
+      X[(b + i) * LL + b + j] = x[i];
+    }
+  }
+  __syncthreads();
+  const int r = tid >> 3, c = (tid & 7) * 2;
+#pragma unroll 1
+  for (int d = 1; d < 4; ++d) {
+#pragma unroll 1
+    for (int i = d; i < 4; ++i) {                        // P = sum over the blocks between of L_im X_mj, j = i - d
+      float s[2] = {0.f, 0.f};
+      for (int m = i - d; m < i; ++m) block_dot(L + i * 16 * LL + m * 16, X + m * 16 * LL + (i - d) * 16, LL, LL, r, c, s);
+      *reinterpret_cast<float2*>(&P[i - d][r][c]) = make_float2(s[0], s[1]);
+    }
+    __syncthreads();
+#pragma unroll 1
+    for (int i = d; i < 4; ++i) {
+      float s[2] = {0.f, 0.f};
+      block_dot(X + i * 16 * LL + i * 16, &P[i - d][0][0], LL, 20, r, c, s);
+      *reinterpret_cast<float2*>(X + (i * 16 + r) * LL + (i - d) * 16 + c) = make_float2(-s[0], -s[1]);
+    }
+    __syncthreads();
+  }
+}
 
 // grid (chunks, heads, sequences), 128 threads. Row i of a chunk: scalars [0, 64) decayed 1/|k|, [64, 128) decayed 1/|q|,
 // [128, 192) 1/|k| times the decay from the token to the chunk's end, [192] the decay over the whole chunk.
-template <bool DELTA>
+template <bool DELTA, int D>
 __global__ void __launch_bounds__(128)
 chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
-  extern __shared__ __align__(16) uint8_t smem_raw[];
-  __shared__ float sB[CH], sRk[CH], sRq[CH];
+  constexpr int LD = D + 8, TILE = CH * LD, SYSTEM = 2 * CH * LL * 4;
+  constexpr int BYTES = 2 * TILE * 2 > SYSTEM || !DELTA ? 2 * TILE * 2 : SYSTEM;
+  __shared__ __align__(16) uint8_t smem[BYTES];
+  __shared__ float sB[CH], sRk[CH], sRq[CH], sP[DELTA ? 3 : 1][16][20];
   __shared__ double sG[CH];                                  // log decay from the chunk's start, each token's own included
   const int chunk = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, kvh = h / (r.heads / r.kv_heads);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int t0 = chunk * CH, n = min(CH, r.pos.per_seq - t0);
-  const long long row0 = (long long)seq * r.pos.per_seq + t0;
-  const int D = up16(r.dp), LD = D + 8;
-  bf16* sK = reinterpret_cast<bf16*>(smem_raw);
-  bf16* sQ = sK + CH * LD;
-  float* sL = reinterpret_cast<float*>(smem_raw);            // takes the place of the tiles once they have been used
-  constexpr int LL = CH + 4;
-  const bf16* act = (const bf16*)r.act + row0 * r.lda;
-  for (int i = tid; i < CH * (D / 8); i += 128) {
-    const int row = i / (D / 8), c = (i - row * (D / 8)) * 8;
-    const bool in = row < n && c < r.dp;
-    const long long at = in ? row * r.lda + kvh * r.dp + c : 0;
-    cp_async16_or_zero(sK + row * LD + c, act + (in ? r.k_off : 0) + at, in);
-    cp_async16_or_zero(sQ + row * LD + c, act + (in ? r.q_off : 0) + at, in);
-  }
+  const int n = min(CH, r.pos.per_seq - chunk * CH);
+  const long long row0 = (long long)seq * r.pos.per_seq + chunk * CH;
+  const bf16* sQ = reinterpret_cast<const bf16*>(smem);
+  const bf16* sK = sQ + TILE;
+  float* sL = reinterpret_cast<float*>(smem);                // take the place of the tiles once they have been used
+  float* sX = sL + CH * LL;
+  const Tiles tiles(gridDim.z, r.pos.per_seq, r.heads, r.kv_heads, r.dp, r.vp);
+  const uint8_t* src = reinterpret_cast<const uint8_t*>((const bf16*)r.act + (((long long)seq * tiles.chunks + chunk) * r.kv_heads + kvh) * tiles.qk_unit);
+#pragma unroll
+  for (int i = tid * 16; i < 2 * TILE * 2; i += 128 * 16) cp_async16(smem + i, src + i);
   cp_async_commit();
   uint8_t* unit = scratch + ((long long)(seq * gridDim.x + chunk) * r.heads + h) * chunk_bytes(DELTA);
   bf16* gA = reinterpret_cast<bf16*>(unit);
-  float* gS = reinterpret_cast<float*>(unit + (DELTA ? 4 : 2) * TRI * 2);
+  float* gS = reinterpret_cast<float*>(unit + (DELTA ? 4 : 2) * MAT * 2);
   if (warp == 0) {
     if (DELTA) {
       float lg[2];
@@ -323,6 +404,7 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
   for (int t = 0; t < 8; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) { qk[t][e] = 0.f; if (DELTA) kk[t][e] = 0.f; }
+#pragma unroll
   for (int k = 0; k < D; k += 16) {
     uint32_t aq[4], ak[4];
     ldmatrix4(aq, sQ + (warp * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
@@ -343,6 +425,7 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
   __syncthreads();
 #pragma unroll
   for (int t = 0; t < 8; ++t) {
+    if (t > 2 * warp + 1) break;                                // blocks above the diagonal are never read
     const int j = t * 8 + (lane & 3) * 2;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
@@ -355,248 +438,217 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
         a[e] = c <= i ? sRq[i] * sRk[c] * decay * qk[t][half * 2 + e] : 0.f;
         if constexpr (DELTA) l[e] = c < i ? sB[i] * sRk[i] * sRk[c] * decay * kk[t][half * 2 + e] : 0.f;
       }
-      if (t <= 2 * warp + 1) {
-        bf16 hi[2], lo[2];
-        split_bf16(a[0], hi[0], lo[0]);
-        split_bf16(a[1], hi[1], lo[1]);
-        *reinterpret_cast<__nv_bfloat162*>(gA + i * CH + j) = __nv_bfloat162(hi[0], hi[1]);
-        *reinterpret_cast<__nv_bfloat162*>(gA + TRI + i * CH + j) = __nv_bfloat162(lo[0], lo[1]);
-      }
+      store_split(gA + i * LT + j, gA + MAT + i * LT + j, a[0], a[1]);
       if constexpr (DELTA) *reinterpret_cast<float2*>(sL + i * LL + j) = make_float2(l[0], l[1]);
     }
   }
   if constexpr (DELTA) {
     __syncthreads();
-    if (tid < CH) {                              // column tid of (1 + L)^-1 by forward substitution
-      float x[CH];
-#pragma unroll
-      for (int i = 0; i < CH; ++i) x[i] = 0.f;
-#pragma unroll
-      for (int i = 0; i < CH; ++i) {
-        float s[4] = {i == tid ? 1.f : 0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-        for (int m = 0; m < i; m += 4) {         // L is zero on and above the diagonal
-          const float4 l = *reinterpret_cast<const float4*>(sL + i * LL + m);
-          s[0] -= l.x * x[m]; s[1] -= l.y * x[m + 1]; s[2] -= l.z * x[m + 2]; s[3] -= l.w * x[m + 3];
-        }
-        x[i] = (s[0] + s[1]) + (s[2] + s[3]);
-      }
-      const float beta = sB[tid];
-#pragma unroll
-      for (int i = 0; i < CH; ++i) {
-        bf16 hi, lo;
-        split_bf16(x[i] * beta, hi, lo);
-        gA[2 * TRI + i * CH + tid] = hi;
-        gA[3 * TRI + i * CH + tid] = lo;
-      }
+    invert_unit_lower(sL, sX, sP);
+    for (int e = tid; e < CH * CH / 2; e += 128) {
+      const int i = e / (CH / 2), j = (e % (CH / 2)) * 2;
+      if (j > (i | 15)) continue;
+      const bool diagonal = (i >> 4) == (j >> 4);               // the substitution leaves zeros above the diagonal
+      const float2 x = *reinterpret_cast<const float2*>(sX + i * LL + j);
+      store_split(gA + 2 * MAT + i * LT + j, gA + 3 * MAT + i * LT + j, diagonal && j > i ? 0.f : x.x * sB[j], diagonal && j + 1 > i ? 0.f : x.y * sB[j + 1]);
     }
   }
 }
 
-struct ChunkSmem {
-  int D, LD, k, q, a, v, s, stage, state, u, w, r, total;      // byte offsets inside a stage, then of the shared parts
+// Shared memory of the scan: two stages of a chunk's operands, then what the warps hand each other.
+template <bool DELTA, int D>
+struct ScanSmem {
+  static constexpr int LD = D + 8, MATS = DELTA ? 4 : 2;
+  static constexpr int QK_BYTES = 2 * CH * LD * 2, UNIT_BYTES = MATS * MAT * 2 + SCALARS * 4, V_BYTES = CH * LV * 2;
+  static constexpr int Q = 0, K = CH * LD * 2, A = QK_BYTES, SC = A + MATS * MAT * 2, V = A + UNIT_BYTES;
+  static constexpr int STAGE = QK_BYTES + UNIT_BYTES + V_BYTES;
+  static constexpr int PART = CH * LV, S_PART = D * LV;         // elements of one part (high or low) of a 64 x 16 operand, of the state
+  static constexpr int S = 2 * STAGE;                           // state, two buffers of two parts
+  static constexpr int W = S + 4 * S_PART * 2;                  // U with the decay to the chunk's end
+  static constexpr int R = W + 2 * PART * 2;                    // delta rule: R, then U in two buffers
+  static constexpr int U = R + (DELTA ? 2 * PART * 2 : 0);
+  static constexpr int BAR = U + (DELTA ? 4 * PART * 2 : 0);
+  static constexpr int TOTAL = BAR + 128;
+  static_assert(STAGE % 16 == 0 && TOTAL <= 227 * 1024, "stages must fit shared memory");
 };
-__host__ __device__ inline ChunkSmem chunk_smem(int dp, bool delta) {
-  ChunkSmem m;
-  m.D = up16(dp); m.LD = m.D + 8;
-  m.k = 0;
-  m.q = m.k + CH * m.LD * 2;
-  m.a = m.q + CH * m.LD * 2;
-  m.v = m.a + (delta ? 4 : 2) * CH * LT * 2;
-  m.s = m.v + CH * LV * 2;
-  m.stage = m.s + SCALARS * 4;
-  m.state = 2 * m.stage;                        // state, two parts
-  m.w = m.state + 2 * m.D * LV * 2;             // U with the decay to the chunk's end, two parts
-  m.u = m.w + 2 * CH * LV * 2;                  // U, two parts (delta rule)
-  m.r = m.u + (delta ? 2 * CH * LV * 2 : 0);    // R, two parts (delta rule)
-  m.total = m.r + (delta ? 2 * CH * LV * 2 : 0);
-  return m;
-}
 
-__device__ __forceinline__ void store_split(bf16* hi_at, bf16* lo_at, float a, float b) {
-  bf16 hi[2], lo[2];
-  split_bf16(a, hi[0], lo[0]);
-  split_bf16(b, hi[1], lo[1]);
-  *reinterpret_cast<__nv_bfloat162*>(hi_at) = __nv_bfloat162(hi[0], hi[1]);
-  *reinterpret_cast<__nv_bfloat162*>(lo_at) = __nv_bfloat162(lo[0], lo[1]);
-}
-
-// grid (ceil(vp / 16), heads, sequences), 256 threads: warps 0..3 own the state (16 MT rows each), warps 4..7 the output
-template <bool DELTA, int MT>
-__global__ void __launch_bounds__(256)
-chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int chunks) {
-  extern __shared__ __align__(16) uint8_t smem[];
-  const ChunkSmem m = chunk_smem(r.dp, DELTA);
-  const int v0 = blockIdx.x * VS, h = blockIdx.y, seq = blockIdx.z, kvh = h / (r.heads / r.kv_heads);
+// grid (ceil(vp / 16), heads, sequences), 288 threads: warps 0..3 own the state (16 D / 64 rows each), 4..7 the output, 8 copies.
+// A wait that runs out raises the status and the kernel runs on without waiting, so that no barrier is left short.
+template <bool DELTA, int D>
+__global__ void __launch_bounds__(288)
+chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* status) {
+  using M = ScanSmem<DELTA, D>;
+  constexpr int LD = M::LD, MT = D / 64;
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, kvh = h / (r.heads / r.kv_heads), v0 = slice * VS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int T = r.pos.per_seq, D = m.D, LD = m.LD;
-  const long long row0 = (long long)seq * T;
-  bf16* sS = reinterpret_cast<bf16*>(smem + m.state);
-  bf16* sW = reinterpret_cast<bf16*>(smem + m.w);
-  bf16* sU = reinterpret_cast<bf16*>(smem + m.u);
-  bf16* sR = reinterpret_cast<bf16*>(smem + m.r);
-  const int S_LO = D * LV, T_LO = CH * LV;                       // offset of the low parts
-  const bf16* act = (const bf16*)r.act;
-  auto load_chunk = [&](int c) {
-    uint8_t* st = smem + (c & 1) * m.stage;
-    const int t0 = c * CH, n = min(CH, T - t0);
-    const bf16* rows = act + (row0 + t0) * r.lda;
-    bf16 *sk = reinterpret_cast<bf16*>(st + m.k), *sq = reinterpret_cast<bf16*>(st + m.q), *sa = reinterpret_cast<bf16*>(st + m.a);
-    bf16* sv = reinterpret_cast<bf16*>(st + m.v);
-    for (int i = tid; i < CH * (D / 8); i += 256) {
-      const int row = i / (D / 8), col = (i - row * (D / 8)) * 8;
-      const bool in = row < n && col < r.dp;
-      const long long at = in ? row * r.lda + kvh * r.dp + col : 0;
-      cp_async16_or_zero(sk + row * LD + col, rows + (in ? r.k_off : 0) + at, in);
-      cp_async16_or_zero(sq + row * LD + col, rows + (in ? r.q_off : 0) + at, in);
-    }
-    if (tid < CH * 2) {
-      const int row = tid >> 1, col = (tid & 1) * 8;
-      const bool in = row < n && v0 + col < r.vp;
-      cp_async16_or_zero(sv + row * LV + col, rows + (in ? row * r.lda + r.v_off + (long long)h * r.vp + v0 + col : 0), in);
-    }
-    const uint8_t* unit = scratch + ((long long)(seq * chunks + c) * r.heads + h) * chunk_bytes(DELTA);
-    const bf16* ga = reinterpret_cast<const bf16*>(unit);
-    constexpr int MATS = DELTA ? 4 : 2;
-    for (int i = tid; i < CH * 8; i += 256) {
-      const int row = i >> 3, col = (i & 7) * 8;
-      if (col <= (row | 15)) {                                   // blocks on and below the diagonal
+  const int T = r.pos.per_seq;
+  const Tiles tiles(gridDim.z, T, r.heads, r.kv_heads, r.dp, r.vp);
+  const int chunks = tiles.chunks;
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + M::BAR);       // [2] each, by chunk parity
+  uint64_t *empty = full + 2, *s_ready = full + 4, *u_ready = full + 6, *o_done = full + 8;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(full + 10);
+  if (tid == 0) {
+    for (int i = 0; i < 2; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); mbar_init(&s_ready[i], 4); mbar_init(&u_ready[i], 4); mbar_init(&o_done[i], 4); }
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  __syncthreads();
+  auto wait = [&](uint64_t* bar, int n, int code) { mbar_wait(bar, n & 1, abort_flag, status, code, 0x5c0); };    // its n-th completion
+  auto arrive = [&](uint64_t* bar) { __syncwarp(); if (lane == 0) mbar_arrive(bar); };
+  auto state_sync = [] { asm volatile("bar.sync 1, 128;" ::: "memory"); };
+  const int mrow = (warp & 3) * 16;                              // this warp's 16 tokens of a chunk
+  const int ri = mrow + (lane >> 2), ci = (lane & 3) * 2;        // first row and column of its accumulators
+  auto a_frag = [&](uint32_t (&a)[4], const bf16* tile, int ld, int k) { ldmatrix4(a, tile + (mrow + (lane & 15)) * ld + k + (lane >> 4) * 8); };
+  auto b_frag = [&](uint32_t (&b)[4], const bf16* rows, int k) { ldmatrix4_trans(b, rows + (k + (lane & 15)) * LV + (lane >> 4) * 8); };
+  auto zero = [](float (&a)[2][4]) {
 #pragma unroll
-        for (int a = 0; a < MATS; ++a) cp_async16(sa + a * CH * LT + row * LT + col, ga + a * TRI + row * CH + col);
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) a[t][e] = 0.f;
+  };
+  // 16 tokens x 16 columns of X S, X the chunk's queries or keys
+  auto times_state = [&](float (&o)[2][4], const bf16* rows, const bf16* s) {
+    float lo[2][4];
+    zero(o);
+    zero(lo);
+#pragma unroll
+    for (int k = 0; k < D; k += 16) {
+      uint32_t a[4], bh[4], bl[4];
+      a_frag(a, rows, LD, k);
+      b_frag(bh, s, k);
+      b_frag(bl, s + M::S_PART, k);
+      mma_16816(o[0], a, bh[0], bh[1]);
+      mma_16816(o[1], a, bh[2], bh[3]);
+      mma_16816(lo[0], a, bl[0], bl[1]);
+      mma_16816(lo[1], a, bl[2], bl[3]);
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[t][e] += lo[t][e];
+  };
+  // o += M X for a lower triangular 64 x 64 M in two parts and a 64 x 16 X in XP parts
+  auto times_lower = [&](float (&o)[2][4], const bf16* m, const bf16* x, auto two_parts) {
+    float p[2][4], q[2][4];
+    zero(p);
+    zero(q);
+#pragma unroll
+    for (int k = 0; k < CH; k += 16) {
+      if (k > mrow) break;
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      a_frag(ah, m, LT, k);
+      a_frag(al, m + MAT, LT, k);
+      b_frag(bh, x, k);
+      if constexpr (decltype(two_parts)::value) b_frag(bl, x + M::PART, k);
+      mma_16816(o[0], ah, bh[0], bh[1]);
+      mma_16816(o[1], ah, bh[2], bh[3]);
+      mma_16816(p[0], al, bh[0], bh[1]);
+      mma_16816(p[1], al, bh[2], bh[3]);
+      if constexpr (decltype(two_parts)::value) {
+        mma_16816(q[0], ah, bl[0], bl[1]);
+        mma_16816(q[1], ah, bl[2], bl[3]);
       }
     }
-    if (tid < SCALARS / 4) cp_async16(st + m.s + tid * 16, unit + MATS * TRI * 2 + tid * 16);
-    cp_async_commit();
-  };
-  load_chunk(0);
-  float* state = r.state.ptr + seq * r.state.seq_stride + (long long)h * r.dp * r.vp + v0;
-  const bool fresh = r.pos.lens[seq] == 0;
-  float st[MT][2][4] = {};
-  auto each_state = [&](auto f) {                                // f(row of the state, column, tile, column tile, first element)
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
+    for (int t = 0; t < 2; ++t)
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
+      for (int e = 0; e < 4; ++e) o[t][e] += p[t][e] + q[t][e];
+  };
+  using Two = std::true_type;
+  using One = std::false_type;
+
+  if (warp == 8) {                                               // ---- copies
+    if (lane == 0) {
+      const bf16* qk = (const bf16*)r.act + ((long long)seq * chunks * r.kv_heads + kvh) * tiles.qk_unit;
+      const bf16* v = (const bf16*)r.act + tiles.v_base + (((long long)seq * chunks * r.heads + h) * tiles.slices + slice) * tiles.v_unit;
+      const uint8_t* unit = scratch + ((long long)seq * chunks * r.heads + h) * chunk_bytes(DELTA);
+      for (int c = 0; c < chunks && !*abort_flag; ++c) {
+        const int b = c & 1;
+        uint8_t* st = smem + b * M::STAGE;
+        if (c >= 2) wait(&empty[b], (c >> 1) - 1, ST_WAIT_EMPTY);
+        if (*abort_flag) break;
+        mbar_arrive_expect_tx(&full[b], M::STAGE);
+        bulk_load_1d(st + M::Q, qk + (long long)c * r.kv_heads * tiles.qk_unit, M::QK_BYTES, &full[b]);
+        bulk_load_1d(st + M::A, unit + (long long)c * r.heads * chunk_bytes(DELTA), M::UNIT_BYTES, &full[b]);
+        bulk_load_1d(st + M::V, v + (long long)c * r.heads * tiles.slices * tiles.v_unit, M::V_BYTES, &full[b]);
+      }
+    }
+  } else if (warp < 4) {                                         // ---- state
+    bf16* sW = reinterpret_cast<bf16*>(smem + M::W);
+    bf16* sR = reinterpret_cast<bf16*>(smem + M::R);
+    float* state = r.state.ptr + seq * r.state.seq_stride + (long long)h * r.dp * r.vp + v0;
+    const bool fresh = r.pos.lens[seq] == 0;
+    float st[MT][2][4] = {};
+    auto each_state = [&](auto f) {                              // f(row of the state, column, tile, column tile, first element)
 #pragma unroll
-        for (int half = 0; half < 2; ++half)
-          f((warp + 4 * i) * 16 + (lane >> 2) + half * 8, t * 8 + (lane & 3) * 2, i, t, half * 2);
-  };
-  auto publish_state = [&] {
-    each_state([&](int d, int v, int i, int t, int e) {
-      if (d < D) store_split(sS + d * LV + v, sS + S_LO + d * LV + v, st[i][t][e], st[i][t][e + 1]);
-    });
-  };
-  if (warp < 4) {
+      for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int half = 0; half < 2; ++half)
+            f((warp + 4 * i) * 16 + (lane >> 2) + half * 8, t * 8 + (lane & 3) * 2, i, t, half * 2);
+    };
+    auto publish_state = [&](int buffer) {
+      bf16* s = reinterpret_cast<bf16*>(smem + M::S) + buffer * 2 * M::S_PART;
+      each_state([&](int d, int v, int i, int t, int e) { store_split(s + d * LV + v, s + M::S_PART + d * LV + v, st[i][t][e], st[i][t][e + 1]); });
+      arrive(&s_ready[buffer]);
+    };
     each_state([&](int d, int v, int i, int t, int e) {
       const bool in = !fresh && d < r.dp && v0 + v < r.vp;
       const float2 x = in ? *reinterpret_cast<const float2*>(state + (long long)d * r.vp + v) : make_float2(0.f, 0.f);
       st[i][t][e] = x.x; st[i][t][e + 1] = x.y;
     });
-    publish_state();
-  }
-  const int mrow = (warp & 3) * 16;                              // this warp's 16 tokens of a chunk
-  const int ri = mrow + (lane >> 2), ci = (lane & 3) * 2;        // first row and column of its accumulators
-  auto a_frag = [&](uint32_t (&a)[4], const bf16* tile, int ld, int k) { ldmatrix4(a, tile + (mrow + (lane & 15)) * ld + k + (lane >> 4) * 8); };
-  auto b_frag = [&](uint32_t (&b)[4], const bf16* rows, int k) { ldmatrix4_trans(b, rows + (k + (lane & 15)) * LV + (lane >> 4) * 8); };
-  for (int c = 0; c < chunks; ++c) {
-    cp_async_wait<0>();
-    __syncthreads();                                             // the chunk has arrived; the state is published; the other stage is free
-    if (c + 1 < chunks) load_chunk(c + 1);
-    const uint8_t* stg = smem + (c & 1) * m.stage;
-    const bf16 *sk = reinterpret_cast<const bf16*>(stg + m.k), *sq = reinterpret_cast<const bf16*>(stg + m.q);
-    const bf16 *sA = reinterpret_cast<const bf16*>(stg + m.a), *sT = sA + 2 * CH * LT, *sv = reinterpret_cast<const bf16*>(stg + m.v);
-    const float* sc = reinterpret_cast<const float*>(stg + m.s);
-    float o[2][4];
+    publish_state(0);
+    state_sync();
+    for (int c = 0; c < chunks; ++c) {
+      const int b = c & 1;
+      const uint8_t* stg = smem + b * M::STAGE;
+      const bf16 *sk = reinterpret_cast<const bf16*>(stg + M::K), *sv = reinterpret_cast<const bf16*>(stg + M::V);
+      const float* sc = reinterpret_cast<const float*>(stg + M::SC);
+      wait(&full[b], c >> 1, ST_WAIT_FULL);
+      const float g = sc[3 * CH], w0 = sc[2 * CH + ri], w1 = sc[2 * CH + ri + 8];
+      if constexpr (DELTA) {
+        bf16* sU = reinterpret_cast<bf16*>(smem + M::U) + b * 2 * M::PART;
+        const float k0 = sc[ri], k1 = sc[ri + 8];
+        float x[2][4];
+        times_state(x, sk, reinterpret_cast<const bf16*>(smem + M::S) + b * 2 * M::S_PART);
 #pragma unroll
-    for (int t = 0; t < 2; ++t)
+        for (int t = 0; t < 2; ++t)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
-    // K S (warps 0..3, delta rule) and Q S (warps 4..7)
-    if (DELTA || warp >= 4) {
-      const bf16* rows = warp < 4 ? sk : sq;
-      for (int k = 0; k < D; k += 16) {
-        uint32_t a[4], hi[4], lo[4];
-        a_frag(a, rows, LD, k);
-        b_frag(hi, sS, k);
-        b_frag(lo, sS + S_LO, k);
-        mma_16816(o[0], a, hi[0], hi[1]);
-        mma_16816(o[1], a, hi[2], hi[3]);
-        mma_16816(o[0], a, lo[0], lo[1]);
-        mma_16816(o[1], a, lo[2], lo[3]);
-      }
-#pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) o[t][e] *= sc[(warp < 4 ? 0 : CH) + ri + (e >> 1) * 8];
-    }
-    if (warp < 4) {
-#pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int i = ri + half * 8, j = t * 8 + ci;
-          const float2 v = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + i * LV + j));
-          if (DELTA) {
-            store_split(sR + i * LV + j, sR + T_LO + i * LV + j, v.x - o[t][half * 2], v.y - o[t][half * 2 + 1]);
-          } else {
-            const float w = sc[2 * CH + i];
-            store_split(sW + i * LV + j, sW + T_LO + i * LV + j, v.x * w, v.y * w);
+          for (int half = 0; half < 2; ++half) {
+            const int i = ri + half * 8, j = t * 8 + ci;
+            const float2 v = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + i * LV + j));
+            const float f = half ? k1 : k0;
+            store_split(sR + i * LV + j, sR + M::PART + i * LV + j, v.x - f * x[t][half * 2], v.y - f * x[t][half * 2 + 1]);
           }
-        }
-    }
-    __syncthreads();
-    if constexpr (DELTA) {                                       // U = T R: warp = 16 tokens x 8 columns
-      const int t = warp >> 2;
-      float u[4] = {0.f, 0.f, 0.f, 0.f};
-      for (int k = 0; k <= mrow; k += 16) {
-        uint32_t th[4], tl[4], hi[4], lo[4];
-        a_frag(th, sT, LT, k);
-        a_frag(tl, sT + CH * LT, LT, k);
-        b_frag(hi, sR, k);
-        b_frag(lo, sR + T_LO, k);
-        const uint32_t h0 = t ? hi[2] : hi[0], h1 = t ? hi[3] : hi[1], l0 = t ? lo[2] : lo[0], l1 = t ? lo[3] : lo[1];
-        mma_16816(u, th, h0, h1);
-        mma_16816(u, tl, h0, h1);
-        mma_16816(u, th, l0, l1);
+        state_sync();
+        zero(x);
+        times_lower(x, reinterpret_cast<const bf16*>(stg + M::A) + 2 * MAT, sR, Two{});
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int i = ri + half * 8, j = t * 8 + ci;
+            const float w = half ? w1 : w0;
+            store_split(sW + i * LV + j, sW + M::PART + i * LV + j, x[t][half * 2] * w, x[t][half * 2 + 1] * w);
+            store_split(sU + i * LV + j, sU + M::PART + i * LV + j, x[t][half * 2], x[t][half * 2 + 1]);
+          }
+        arrive(&u_ready[b]);
+      } else {
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int i = ri + half * 8, j = t * 8 + ci;
+            const float2 v = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + i * LV + j));
+            const float w = half ? w1 : w0;
+            store_split(sW + i * LV + j, sW + M::PART + i * LV + j, v.x * w, v.y * w);
+          }
       }
+      state_sync();
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int i = ri + half * 8, j = t * 8 + ci;
-        const float w = sc[2 * CH + i];
-        store_split(sU + i * LV + j, sU + T_LO + i * LV + j, u[half * 2], u[half * 2 + 1]);
-        store_split(sW + i * LV + j, sW + T_LO + i * LV + j, u[half * 2] * w, u[half * 2 + 1] * w);
-      }
-      __syncthreads();
-    }
-    if (warp >= 4) {                                             // O = decayed Q S + A U
-      for (int k = 0; k <= mrow; k += 16) {
-        uint32_t ah[4], al[4], hi[4];
-        a_frag(ah, sA, LT, k);
-        a_frag(al, sA + CH * LT, LT, k);
-        b_frag(hi, DELTA ? sU : sv, k);
-        mma_16816(o[0], ah, hi[0], hi[1]);
-        mma_16816(o[1], ah, hi[2], hi[3]);
-        mma_16816(o[0], al, hi[0], hi[1]);
-        mma_16816(o[1], al, hi[2], hi[3]);
-        if constexpr (DELTA) {
-          uint32_t lo[4];
-          b_frag(lo, sU + T_LO, k);
-          mma_16816(o[0], ah, lo[0], lo[1]);
-          mma_16816(o[1], ah, lo[2], lo[3]);
-        }
-      }
-      bf16* out = (bf16*)r.o + (row0 + c * CH) * r.ldo + (long long)h * r.vp + v0;
-#pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int i = ri + half * 8, j = t * 8 + ci;
-          if (c * CH + i < T && v0 + j < r.vp) *reinterpret_cast<uint32_t*>(out + i * r.ldo + j) = pack_bf16(o[t][half * 2], o[t][half * 2 + 1]);
-        }
-    } else {                                                     // S = decayed S + K^T W
-      const float g = sc[3 * CH];
-#pragma unroll
-      for (int i = 0; i < MT; ++i)
+      for (int i = 0; i < MT; ++i)                               // S = decayed S + K^T W
 #pragma unroll
         for (int t = 0; t < 2; ++t)
 #pragma unroll
@@ -605,27 +657,64 @@ chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int c
       for (int k = 0; k < CH; k += 16) {
         uint32_t hi[4], lo[4];
         b_frag(hi, sW, k);
-        b_frag(lo, sW + T_LO, k);
+        b_frag(lo, sW + M::PART, k);
 #pragma unroll
         for (int i = 0; i < MT; ++i) {
-          const int d0 = (warp + 4 * i) * 16;
-          if (d0 < D) {
-            uint32_t a[4];                                       // K^T: rows are the head's dimensions, k the tokens
-            ldmatrix4_trans(a, sk + (k + (lane & 7) + (lane >> 4) * 8) * LD + d0 + ((lane >> 3) & 1) * 8);
-            mma_16816(st[i][0], a, hi[0], hi[1]);
-            mma_16816(st[i][1], a, hi[2], hi[3]);
-            mma_16816(st[i][0], a, lo[0], lo[1]);
-            mma_16816(st[i][1], a, lo[2], lo[3]);
-          }
+          uint32_t a[4];                                         // K^T: rows are the head's dimensions, k the tokens
+          ldmatrix4_trans(a, sk + (k + (lane & 7) + (lane >> 4) * 8) * LD + (warp + 4 * i) * 16 + ((lane >> 3) & 1) * 8);
+          mma_16816(st[i][0], a, hi[0], hi[1]);
+          mma_16816(st[i][1], a, hi[2], hi[3]);
+          mma_16816(st[i][0], a, lo[0], lo[1]);
+          mma_16816(st[i][1], a, lo[2], lo[3]);
         }
       }
-      publish_state();                                           // Q S and K S of this chunk have been read
+      arrive(&empty[b]);
+      if (c + 1 < chunks) {
+        if (c >= 1) wait(&o_done[b ^ 1], (c - 1) >> 1, ST_WAIT_PEER);      // chunk c - 1 has been read out of that buffer
+        publish_state(b ^ 1);
+        state_sync();
+      }
     }
-  }
-  if (warp < 4)
     each_state([&](int d, int v, int i, int t, int e) {
       if (d < r.dp && v0 + v < r.vp) *reinterpret_cast<float2*>(state + (long long)d * r.vp + v) = make_float2(st[i][t][e], st[i][t][e + 1]);
     });
+  } else {                                                       // ---- output
+    for (int c = 0; c < chunks; ++c) {
+      const int b = c & 1;
+      const uint8_t* stg = smem + b * M::STAGE;
+      const float* sc = reinterpret_cast<const float*>(stg + M::SC);
+      wait(&full[b], c >> 1, ST_WAIT_FULL);
+      wait(&s_ready[b], c >> 1, ST_WAIT_PEER);
+      float o[2][4];
+      times_state(o, reinterpret_cast<const bf16*>(stg + M::Q), reinterpret_cast<const bf16*>(smem + M::S) + b * 2 * M::S_PART);
+      const float q0 = sc[CH + ri], q1 = sc[CH + ri + 8];
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[t][e] *= e < 2 ? q0 : q1;
+      if constexpr (DELTA) {
+        wait(&u_ready[b], c >> 1, ST_WAIT_PEER);
+        times_lower(o, reinterpret_cast<const bf16*>(stg + M::A), reinterpret_cast<const bf16*>(smem + M::U) + b * 2 * M::PART, Two{});
+      } else {
+        times_lower(o, reinterpret_cast<const bf16*>(stg + M::A), reinterpret_cast<const bf16*>(stg + M::V), One{});
+      }
+      arrive(&empty[b]);
+      arrive(&o_done[b]);
+      bf16* out = (bf16*)r.o + ((long long)seq * T + c * CH) * r.ldo + (long long)h * r.vp + v0;
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int i = ri + half * 8, j = t * 8 + ci;
+          if (c * CH + i < T && v0 + j < r.vp) *reinterpret_cast<uint32_t*>(out + i * r.ldo + j) = pack_bf16(o[t][half * 2], o[t][half * 2 + 1]);
+        }
+    }
+  }
+  __syncthreads();
+  if (*abort_flag) {                                             // copies still in flight
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+  }
 }
 
 // ------------------------------------------------------------------------- norm, gate
@@ -662,27 +751,35 @@ __device__ void keep_inputs(const DeltaInputs& d, int job) {
   }
 }
 
-// a warp per group
-template <typename T>
+// LANES lanes per group
+template <typename T, int LANES>
 __global__ void __launch_bounds__(256)
 norm_gate_warp_kernel(const NormGate d, const DeltaInputs ring, int main_blocks) {
   if ((int)blockIdx.x >= main_blocks) return keep_inputs<T>(ring, blockIdx.x - main_blocks);
-  const int lane = threadIdx.x & 31;
-  const long long i = (long long)blockIdx.x * 8 + (threadIdx.x >> 5), row = i / d.groups;
-  if (row >= d.rows) return;
-  const int g0 = (int)(i - row * d.groups) * d.np;
-  const T* o = (const T*)d.o + row * d.ldo + g0;
-  float ss = 0.f;
-  for (int c = lane * 8; c < d.np; c += 256) {
+  const int lane = threadIdx.x % LANES;
+  const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) / LANES, row = i / d.groups;
+  const bool on = row < d.rows;
+  const int g0 = on ? (int)(i - row * d.groups) * d.np : 0;
+  const T* o = (const T*)d.o + (on ? row * d.ldo + g0 : 0);
+  float ss = 0.f, first[8];
+  for (int c = lane * 8; on && c < d.np; c += LANES * 8) {
     float v[8];
     load8(o + c, v);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+    for (int j = 0; j < 8; ++j) { ss += v[j] * v[j]; if (c < LANES * 8) first[j] = v[j]; }
   }
-  const float r = inv_rms(warp_sum(ss), d.n, d.eps) * d.out_scale;
-  for (int c = lane * 8; c < d.np; c += 256) {
+#pragma unroll
+  for (int s = LANES / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if (!on) return;
+  const float r = inv_rms(ss, d.n, d.eps) * d.out_scale;
+  for (int c = lane * 8; c < d.np; c += LANES * 8) {
     float v[8];
-    load8(o + c, v);
+    if (c < LANES * 8) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] = first[j];
+    } else {
+      load8(o + c, v);
+    }
     gate8<T>(d, v, row, g0 + c, c, r);
   }
 }
@@ -709,10 +806,12 @@ norm_gate_row_kernel(const NormGate d) {
   }
 }
 
+bool sizes_ok(const DeltaInputs& d) {
+  return d.rows > 0 && d.pos.per_seq > 0 && d.rows % d.pos.per_seq == 0 && d.rows / d.pos.per_seq <= 65535 && d.heads > 0 && d.kv_heads > 0 &&
+         d.heads % d.kv_heads == 0 && d.dp > 0 && d.vp > 0 && !(d.dp & 7) && !(d.vp & 7) && !(d.ldz & 7) && d.z && !(d.f32 && !d.z_f32);
+}
 bool inputs_ok(const DeltaInputs& d) {
-  return d.rows > 0 && d.pos.lens && d.pos.per_seq > 0 && d.rows % d.pos.per_seq == 0 && d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 &&
-         d.dim > 0 && d.dim <= d.dp && d.vdim > 0 && d.vdim <= d.vp && !(d.dp & 7) && !(d.vp & 7) && d.taps > 0 && !(d.ldz & 7) && d.z && d.conv &&
-         d.ring.ptr && !(d.ring.seq_stride & 3) && !(d.f32 && !d.z_f32);
+  return sizes_ok(d) && d.pos.lens && d.dim > 0 && d.dim <= d.dp && d.vdim > 0 && d.vdim <= d.vp && d.taps > 0 && d.conv && d.ring.ptr && !(d.ring.seq_stride & 3);
 }
 bool recurrence_ok(const Recurrence& d) {
   return d.rows > 0 && d.pos.lens && d.pos.per_seq > 0 && d.rows % d.pos.per_seq == 0 && d.rows / d.pos.per_seq <= 65535 && d.heads > 0 && d.heads <= 65535 &&
@@ -720,31 +819,34 @@ bool recurrence_ok(const Recurrence& d) {
          !(d.lda & 7) && !(d.ldo & 7) && d.act && d.o && d.state.ptr && !(d.state.seq_stride & 3) && (d.beta_g ? d.norms != nullptr : d.log_decay != nullptr);
 }
 
-}  // namespace
-
-cudaError_t delta_prepare(const DeltaInputs& d, void* act, float* norms, float* beta_g, cudaStream_t s) {
-  if (!inputs_ok(d) || !d.ba || d.rows / d.pos.per_seq > 65535) return cudaErrorInvalidValue;
-  const dim3 grid((d.pos.per_seq + PREP_TOKENS - 1) / PREP_TOKENS, (2 * d.kv_heads + d.heads + 3) / 4, d.rows / d.pos.per_seq);
-  const bool held = d.taps <= 4;
-  if (d.f32) {
-    auto k = held ? delta_prepare_kernel<float, float, 4> : delta_prepare_kernel<float, float, 0>;
-    k<<<grid, 128, 0, s>>>(d, (float*)act, norms, beta_g);
-  } else if (d.z_f32) {
-    auto k = held ? delta_prepare_kernel<bf16, float, 4> : delta_prepare_kernel<bf16, float, 0>;
-    k<<<grid, 128, 0, s>>>(d, (bf16*)act, norms, beta_g);
-  } else {
-    auto k = held ? delta_prepare_kernel<bf16, bf16, 4> : delta_prepare_kernel<bf16, bf16, 0>;
-    k<<<grid, 128, 0, s>>>(d, (bf16*)act, norms, beta_g);
-  }
+template <typename T, typename TZ, bool TILES>
+cudaError_t launch_prepare(const DeltaInputs& d, void* out, float* norms, float* beta_g, cudaStream_t s) {
+  const int tokens = TILES ? (d.pos.per_seq + CH - 1) / CH * CH : d.pos.per_seq;
+  const dim3 grid((tokens + PREP_TOKENS - 1) / PREP_TOKENS, (2 * d.kv_heads + d.heads + 3) / 4, d.rows / d.pos.per_seq);
+  auto k = !d.conv ? prepare_kernel<T, TZ, -1, TILES> : d.taps <= 4 ? prepare_kernel<T, TZ, 4, TILES> : prepare_kernel<T, TZ, 0, TILES>;
+  k<<<grid, 128, 0, s>>>(d, (T*)out, norms, beta_g);
   return cudaGetLastError();
 }
+cudaError_t launch_prepare(const DeltaInputs& d, bool tiles, void* out, float* norms, float* beta_g, cudaStream_t s) {
+  if (tiles && (d.f32 || !recurrence_chunks_supported(d.dp))) return cudaErrorInvalidValue;
+  if (d.f32 != d.z_f32) return cudaErrorInvalidValue;
+  if (d.f32) return launch_prepare<float, float, false>(d, out, norms, beta_g, s);
+  return tiles ? launch_prepare<bf16, bf16, true>(d, out, norms, beta_g, s) : launch_prepare<bf16, bf16, false>(d, out, norms, beta_g, s);
+}
 
-cudaError_t silu_rows(bool f32, const void* z, long long ldz, int rows, int n, void* act, long long lda, cudaStream_t s) {
-  if (rows <= 0 || n <= 0 || (n & 7) || (ldz & 7) || (lda & 7)) return cudaErrorInvalidValue;
-  const unsigned blocks = (unsigned)(((long long)rows * (n / 8) + 255) / 256);
-  if (f32) silu_rows_kernel<float><<<blocks, 256, 0, s>>>((const float*)z, ldz, rows, n, (float*)act, lda);
-  else silu_rows_kernel<bf16><<<blocks, 256, 0, s>>>((const bf16*)z, ldz, rows, n, (bf16*)act, lda);
-  return cudaGetLastError();
+}  // namespace
+
+cudaError_t delta_prepare(const DeltaInputs& d, bool tiles, void* out, float* norms, float* beta_g, cudaStream_t s) {
+  if (!inputs_ok(d) || !d.ba || !norms || !beta_g) return cudaErrorInvalidValue;
+  return launch_prepare(d, tiles, out, norms, beta_g, s);
+}
+
+cudaError_t decay_prepare(bool f32, const void* z, long long ldz, int rows, int per_seq, int heads, int dp, int vp, bool tiles, void* out, cudaStream_t s) {
+  DeltaInputs d{};
+  d.f32 = d.z_f32 = f32; d.z = z; d.ldz = ldz; d.rows = rows; d.heads = d.kv_heads = heads; d.dp = dp; d.vp = vp; d.taps = 1;
+  d.pos.per_seq = per_seq;
+  if (!sizes_ok(d)) return cudaErrorInvalidValue;
+  return launch_prepare(d, tiles, out, nullptr, nullptr, s);
 }
 
 template <typename T, bool DELTA>
@@ -764,34 +866,31 @@ cudaError_t recurrence_scan(const Recurrence& d, cudaStream_t s) {
 }
 
 bool recurrence_chunks_supported(int dp) { return dp > 0 && dp <= 128 && !(dp & 7); }
+size_t recurrence_tiles(int seqs, int per_seq, int heads, int kv_heads, int dp, int vp) {
+  return (size_t)Tiles(seqs, per_seq, heads, kv_heads, dp, vp).elements(seqs, heads) * 2;
+}
 size_t recurrence_scratch(int seqs, int per_seq, int heads, bool delta) {
   return (size_t)seqs * ((per_seq + CH - 1) / CH) * heads * chunk_bytes(delta);
 }
 
-template <bool DELTA>
-static cudaError_t launch_chunks(const Recurrence& d, uint8_t* scratch, cudaStream_t s) {
+template <bool DELTA, int D>
+static cudaError_t launch_chunks(const Recurrence& d, uint8_t* scratch, int* status, cudaStream_t s) {
   static PerDeviceOnce configured;
-  constexpr int MAX_SMEM = 200 * 1024;
-  cudaError_t e = configured.once([] {
-    cudaError_t r = cudaFuncSetAttribute(chunk_scan_kernel<DELTA, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM);
-    return r != cudaSuccess ? r : cudaFuncSetAttribute(chunk_scan_kernel<DELTA, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM);
-  });
+  constexpr int SMEM = ScanSmem<DELTA, D>::TOTAL;
+  cudaError_t e = configured.once([] { return cudaFuncSetAttribute(chunk_scan_kernel<DELTA, D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); });
   if (e != cudaSuccess) return e;
-  const int seqs = d.rows / d.pos.per_seq, chunks = (d.pos.per_seq + CH - 1) / CH, LD = up16(d.dp) + 8;
-  const ChunkSmem m = chunk_smem(d.dp, DELTA);
-  if (m.total > MAX_SMEM) return cudaErrorInvalidValue;
-  const int tiles = 2 * CH * LD * 2, system = CH * (CH + 4) * 4;
-  chunk_gram_kernel<DELTA><<<dim3(chunks, d.heads, seqs), 128, tiles > system ? tiles : system, s>>>(d, scratch);
+  const int seqs = d.rows / d.pos.per_seq, chunks = (d.pos.per_seq + CH - 1) / CH;
+  chunk_gram_kernel<DELTA, D><<<dim3(chunks, d.heads, seqs), 128, 0, s>>>(d, scratch);
   e = cudaGetLastError();
   if (e != cudaSuccess) return e;
-  const dim3 grid((d.vp + VS - 1) / VS, d.heads, seqs);
-  if (m.D <= 64) chunk_scan_kernel<DELTA, 1><<<grid, 256, m.total, s>>>(d, scratch, chunks);
-  else chunk_scan_kernel<DELTA, 2><<<grid, 256, m.total, s>>>(d, scratch, chunks);
+  chunk_scan_kernel<DELTA, D><<<dim3((d.vp + VS - 1) / VS, d.heads, seqs), 288, SMEM, s>>>(d, scratch, status);
   return cudaGetLastError();
 }
-cudaError_t recurrence_chunks(const Recurrence& d, void* scratch, cudaStream_t s) {
+cudaError_t recurrence_chunks(const Recurrence& d, void* scratch, int* status, cudaStream_t s) {
   if (!recurrence_ok(d) || d.f32 || !recurrence_chunks_supported(d.dp) || !scratch) return cudaErrorInvalidValue;
-  return d.beta_g ? launch_chunks<true>(d, (uint8_t*)scratch, s) : launch_chunks<false>(d, (uint8_t*)scratch, s);
+  uint8_t* p = (uint8_t*)scratch;
+  if (tile_dim(d.dp) == 64) return d.beta_g ? launch_chunks<true, 64>(d, p, status, s) : launch_chunks<false, 64>(d, p, status, s);
+  return d.beta_g ? launch_chunks<true, 128>(d, p, status, s) : launch_chunks<false, 128>(d, p, status, s);
 }
 
 cudaError_t norm_gate(bool f32, const void* o, long long ldo, const void* gate, long long ldg, const float* w, float eps, int rows, int groups,
@@ -804,12 +903,16 @@ cudaError_t norm_gate(bool f32, const void* o, long long ldo, const void* gate, 
     else norm_gate_row_kernel<bf16><<<rows, 256, 0, s>>>(d);
     return cudaGetLastError();
   }
-  const int blocks = (int)(((long long)rows * groups + 7) / 8);
+  const int lanes = np <= 64 ? 8 : np <= 128 ? 16 : 32;
+  const int blocks = (int)(((long long)rows * groups * lanes + 255) / 256);
   const int extra = ring ? (ring->taps - 1) * (ring->rows / ring->pos.per_seq) : 0;
   const DeltaInputs in = ring ? *ring : DeltaInputs{};
-  if (f32) norm_gate_warp_kernel<float><<<blocks + extra, 256, 0, s>>>(d, in, blocks);
-  else norm_gate_warp_kernel<bf16><<<blocks + extra, 256, 0, s>>>(d, in, blocks);
-  return cudaGetLastError();
+  auto go = [&](auto k8, auto k16, auto k32) {
+    (lanes == 8 ? k8 : lanes == 16 ? k16 : k32)<<<blocks + extra, 256, 0, s>>>(d, in, blocks);
+    return cudaGetLastError();
+  };
+  if (f32) return go(norm_gate_warp_kernel<float, 8>, norm_gate_warp_kernel<float, 16>, norm_gate_warp_kernel<float, 32>);
+  return go(norm_gate_warp_kernel<bf16, 8>, norm_gate_warp_kernel<bf16, 16>, norm_gate_warp_kernel<bf16, 32>);
 }
 
 }  // namespace serve

@@ -217,11 +217,11 @@ struct DeltaInputs {
   StateRef ring;
   RowPos pos;
 };
-// Convolution and silu of every channel into act (rows x channels); norms (rows x 2 kv_heads) = 1 / |q| * dim^-1/2, then
-// 1 / |k|; beta_g (rows x 2 heads) = beta, then log g.
-cudaError_t delta_prepare(const DeltaInputs& d, void* act, float* norms, float* beta_g, cudaStream_t s);
-// act = silu(z) over n columns (multiple of 8).
-cudaError_t silu_rows(bool f32, const void* z, long long ldz, int rows, int n, void* act, long long lda, cudaStream_t s);
+// Convolution and silu of every channel into out: rows x channels, or (tiles, bf16) recurrence_tiles() bytes for
+// recurrence_chunks; norms (rows x 2 kv_heads) = 1 / |q| * dim^-1/2, then 1 / |k|; beta_g (rows x 2 heads) = beta, then log g.
+cudaError_t delta_prepare(const DeltaInputs& d, bool tiles, void* out, float* norms, float* beta_g, cudaStream_t s);
+// silu of q, k (heads x dp each) and v (heads x vp), side by side in z, into out likewise.
+cudaError_t decay_prepare(bool f32, const void* z, long long ldz, int rows, int per_seq, int heads, int dp, int vp, bool tiles, void* out, cudaStream_t s);
 
 struct Recurrence {
   bool f32;
@@ -236,10 +236,12 @@ struct Recurrence {
 };
 // Token by token; any T, float or bf16, dp <= 512.
 cudaError_t recurrence_scan(const Recurrence& d, cudaStream_t s);
-// Chunks of 64 tokens on the tensor cores, bf16, dp <= 128. scratch: recurrence_scratch() bytes.
+// Chunks of 64 tokens on the tensor cores, bf16, dp <= 128: act holds tiles (lda and offsets unused), scratch
+// recurrence_scratch() bytes.
 bool recurrence_chunks_supported(int dp);
+size_t recurrence_tiles(int seqs, int per_seq, int heads, int kv_heads, int dp, int vp);
 size_t recurrence_scratch(int seqs, int per_seq, int heads, bool delta);
-cudaError_t recurrence_chunks(const Recurrence& d, void* scratch, cudaStream_t s);
+cudaError_t recurrence_chunks(const Recurrence& d, void* scratch, int* status, cudaStream_t s);
 
 // y = o / rms(o) * w * act(gate) * out_scale; groups of np entries (n real ones) are normed apart, w (np) is shared by the
 // groups. act: 0 silu, 1 sigmoid. ring (optional, delta): also keep the last inputs of the rows' convolution.

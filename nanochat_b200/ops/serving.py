@@ -202,11 +202,19 @@ def relu_glu(h, w_gate_up):
 
 # -------------------------------------------------------------------------------- recurrences
 
-def _recurrence(act, heads, kv_heads, dp, vp, state, cache, T, norms=None, beta_g=None, log_decay=None):
-    o = torch.empty(act.shape[0], heads * vp, dtype=act.dtype, device=act.device)
-    scratch = None
-    if act.dtype == BF16 and T > CHUNK_ROWS and _S.recurrence_chunks_supported(dp):
-        scratch = torch.empty(_S.recurrence_scratch(act.shape[0] // T, T, heads, beta_g is not None), dtype=torch.uint8, device=act.device)
+def _prepared(z, T, heads, kv_heads, dp, vp):
+    """Where a prepare kernel puts its outputs: tiles of the chunk kernels, or rows for the token-by-token kernel."""
+    R = z.shape[0]
+    if z.dtype == BF16 and T > CHUNK_ROWS and _S.recurrence_chunks_supported(dp):
+        return torch.empty(_S.recurrence_tiles(R // T, T, heads, kv_heads, dp, vp), dtype=torch.uint8, device=z.device)
+    return torch.empty(R, 2 * kv_heads * dp + heads * vp, dtype=z.dtype, device=z.device)
+
+
+def _recurrence(act, z, heads, kv_heads, dp, vp, state, cache, T, norms=None, beta_g=None, log_decay=None):
+    R = z.shape[0]
+    o, scratch = torch.empty(R, heads * vp, dtype=z.dtype, device=z.device), None
+    if act.dtype == torch.uint8:
+        scratch = torch.empty(_S.recurrence_scratch(R // T, T, heads, beta_g is not None), dtype=torch.uint8, device=z.device)
     _S.recurrence(act, [heads, kv_heads, dp, vp], norms, beta_g, log_decay, state, cache.cache_seqlens, T, o, scratch)
     return o
 
@@ -218,11 +226,11 @@ def gated_delta(p, z, ba, cache, run, T):
     if T == 1 and _S.delta_step_supported(p.dp, p.vp):
         _S.delta_step(z, p.sizes, p.conv, ba, p.neg_a, p.dt_bias, ring, S, cache.cache_seqlens, p.norm, p.eps, p.gate_off, y)
         return y
-    act = torch.empty(R, p.channels, dtype=z.dtype, device=z.device)
+    act = _prepared(z, T, p.heads, p.kv_heads, p.dp, p.vp)
     norms = torch.empty(R, 2 * p.kv_heads, device=z.device)
     beta_g = torch.empty(R, 2 * p.heads, device=z.device)
     _S.delta_prepare(z, p.sizes, p.conv, ba, p.neg_a, p.dt_bias, ring, cache.cache_seqlens, T, act, norms, beta_g)
-    o = _recurrence(act, p.heads, p.kv_heads, p.dp, p.vp, S, cache, T, norms, beta_g)
+    o = _recurrence(act, z, p.heads, p.kv_heads, p.dp, p.vp, S, cache, T, norms, beta_g)
     _S.delta_finish(o, z[:, p.gate_off:p.gate_off + p.y_width], p.norm, p.eps, y, z, p.sizes, p.conv, p.neg_a, p.dt_bias, ring, cache.cache_seqlens, T)
     return y
 
@@ -234,10 +242,9 @@ def decay_attention(p, z, cache, run, T, y):
         o = torch.empty(R, p.y_width, device=z.device)
         _S.decay_step(z, p.sizes, p.reals, p.log_decay, S, cache.cache_seqlens, p.norm, o, cache.done, y)
         return y
-    qkv = z[:, p.q_off:p.gate_off]
-    act = torch.empty(qkv.shape, dtype=z.dtype, device=z.device)
-    _S.silu_rows(qkv, act)
-    o = _recurrence(act, p.heads, p.heads, p.dp, p.vp, S, cache, T, log_decay=p.log_decay)
+    act = _prepared(z, T, p.heads, p.heads, p.dp, p.vp)
+    _S.decay_prepare(z[:, p.q_off:p.gate_off], p.heads, p.dp, p.vp, T, act)
+    o = _recurrence(act, z, p.heads, p.heads, p.dp, p.vp, S, cache, T, log_decay=p.log_decay)
     _S.norm_gate(o, z[:, p.gate_off:p.end], p.norm, p.eps, 1, p.heads * p.vdim, True, p.out_scale, y)
     return y
 

@@ -1,9 +1,9 @@
 """
-Serving benchmark of the latent-attention model (Lupodra) beside GPT at equal width and depth, random weights:
+Serving benchmark of a model that is served only (Lupodra, Safepel) beside GPT at equal width and depth, random weights:
 
-    python -m scripts.serve_bench                        # every size below
-    python -m scripts.serve_bench --sizes d12 --batch-sizes 1,8
-    python bench.py --serve                              # the same
+    python -m scripts.serve_bench                        # Lupodra, every size below
+    python -m scripts.serve_bench --model Safepel --sizes d12 --batch-sizes 1,8
+    python bench.py --serve Safepel                      # the same, every size
 
 Per size and model: prefill tokens/s of a prompt (device time of the prompt pass: CUDA events around it, median of
 several, a write larger than L2 before each) and tokens/s of decoding through `Engine.generate` at several batch
@@ -37,6 +37,25 @@ def lupodra_config(width, layers, window=512):
             "layers": [{"type": "latent_attention", "mixer": mixer, "mlp": moe if i % 2 else dense} for i in range(layers)]}
 
 
+def safepel_config(width, layers, window=512):
+    """Delta layers (as many 128-dim value heads as GPT has heads, half as many key heads) and parallel ones (half the heads
+    attend to a window, half decay) in turn, gated feed-forwards of 8/3 width: 12 width^2 weights a layer, as GPT has."""
+    heads = width // 128
+    keys = max(k for k in range(1, heads // 2 + 1) if heads % k == 0)
+    ff = -(-width * 8 // 3 // 64) * 64
+    delta = {"heads": heads, "kv_heads": keys, "dim": 128, "vdim": 128, "conv": 4}
+    a, b = heads - heads // 2, heads // 2
+    left = {"heads": a, "kv_heads": 1, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 20.0, "rot": {"base": 10000.0, "dims": 128}, "mask": {"size": window}}
+    right = {"heads": b, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** -(2 + 6 * i / b) for i in range(b)]}
+    parallel = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7}
+    kinds = [("delta", delta), ("parallel", parallel)]
+    return {"architecture": "Safepel", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "layers": [{"type": kinds[i % 2][0], "mixer": kinds[i % 2][1], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+CONFIGS = {"Lupodra": lupodra_config, "Safepel": safepel_config}
+
+
 def build(kind, width, layers, device):
     from nanochat_b200.models.registry import get_architecture
     arch = get_architecture(kind)
@@ -44,7 +63,7 @@ def build(kind, width, layers, device):
         config = arch.config_from_dict(dict(sequence_len=4096, vocab_size=VOCAB, n_layer=layers, n_head=width // 128, n_kv_head=width // 128,
                                             n_embd=width, window_pattern="SSSL"))
         return arch.build(config, device)
-    return arch.build(arch.config_from_dict(lupodra_config(width, layers), sequence_len=4096), device)
+    return arch.build(arch.config_from_dict(CONFIGS[kind](width, layers), sequence_len=4096), device)
 
 
 def prefill_ms(engine, prompt, iters=7):
@@ -69,7 +88,7 @@ def prefill_ms(engine, prompt, iters=7):
     return statistics.median(times)
 
 
-def run(sizes, batch_sizes, prompts, decode_tokens, kinds=("Lupodra", "GPT")):
+def run(sizes, batch_sizes, prompts, decode_tokens, kinds):
     _, _, _, _, device = compute_init("cuda")
     tok = _SyntheticTokenizer(VOCAB)
     out = []
@@ -99,7 +118,9 @@ def run(sizes, batch_sizes, prompts, decode_tokens, kinds=("Lupodra", "GPT")):
 
 
 def main(argv=None):
-    ap = argparse.ArgumentParser(description="Serving benchmark of the latent-attention model beside GPT")
+    ap = argparse.ArgumentParser(description="Serving benchmark of a served model beside GPT")
+    ap.add_argument("--model", default="Lupodra", choices=sorted(CONFIGS))
+    ap.add_argument("--alone", action="store_true", help="skip GPT")
     ap.add_argument("--sizes", default=",".join(SIZES))
     ap.add_argument("--batch-sizes", default="1,8,32")
     ap.add_argument("--prompts", default="512,2048")
@@ -107,11 +128,12 @@ def main(argv=None):
     ap.add_argument("--no-kernels", action="store_true", help="skip the per-kernel comparison")
     args = ap.parse_args(argv)
     ints = lambda s: [int(x) for x in s.split(",") if x]
-    rec = {"metric": "serving throughput, Lupodra beside GPT", "data": "synthetic, random weights", "dtype": "bf16",
-           "rows": run(args.sizes.split(","), ints(args.batch_sizes), ints(args.prompts), args.decode_tokens)}
+    kinds = (args.model,) if args.alone else (args.model, "GPT")
+    rec = {"metric": f"serving throughput, {args.model} beside GPT", "data": "synthetic, random weights", "dtype": "bf16",
+           "rows": run(args.sizes.split(","), ints(args.batch_sizes), ints(args.prompts), args.decode_tokens, kinds)}
     if not args.no_kernels:
-        from nanochat_b200.ops.microbench import bench_serve
-        rec["kernels"] = bench_serve()
+        from nanochat_b200.ops.microbench import SERVE
+        rec["kernels"] = SERVE[args.model]()
     if os.path.exists("MEASURED_PEAKS.json"):
         with open("MEASURED_PEAKS.json") as f:
             rec["measured_peaks"] = {k: v for k, v in json.load(f).items() if k in ("hbm_gbs", "bf16_tflops")}

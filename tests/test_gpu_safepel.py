@@ -36,7 +36,7 @@ def test_every_cut_of_a_prompt_gives_the_oracles_logits(name, dtype):
 
 @DTYPES
 @pytest.mark.parametrize("spec", [dict(heads=4, kv_heads=2, dim=24, vdim=40, conv=4), dict(heads=2, kv_heads=1, dim=128, vdim=72, conv=2),
-                                  dict(heads=3, kv_heads=3, dim=13, vdim=3, conv=1), dict(heads=6, kv_heads=1, dim=64, vdim=64, conv=9),
+                                  dict(heads=3, kv_heads=3, dim=13, vdim=19, conv=1), dict(heads=6, kv_heads=1, dim=64, vdim=64, conv=9),
                                   dict(heads=1, kv_heads=1, dim=200, vdim=264, conv=4)])
 def test_delta_rule(spec, dtype):
     """Chunk borders at multiples of 64 from a portion's start, short portions below the chunked path, single tokens."""
@@ -164,6 +164,27 @@ def recurrence_inputs(seqs, T, H, G, dp, vp, seed=0):
     return act, norms, beta_g, torch.randn(seqs, H, dp, vp, generator=g)
 
 
+def as_tiles(act, seqs, H, G, dp, vp):
+    """Rows of q, k, v as the chunk kernels' tiles: 64 tokens of a head, heads padded to 64 or 128 columns, pitch 8 more;
+    then v in slices of 16 columns, pitch 24. Padding that no one may read is NaN."""
+    K = kernels()._S
+    T = act.shape[0] // seqs
+    chunks, D, slices = -(-T // 64), 64 if dp <= 64 else 128, -(-vp // 16)
+    full = torch.zeros(seqs, chunks * 64, act.shape[1], dtype=BF16)
+    full[:, :T] = act.view(seqs, T, -1)
+    full = full.view(seqs, chunks, 64, -1)
+    qk = torch.full((seqs, chunks, G, 2, 64, D + 8), float("nan"), dtype=BF16)
+    qk[..., :D] = 0
+    qk[..., :dp] = full[..., :2 * G * dp].view(seqs, chunks, 64, 2, G, dp).permute(0, 1, 4, 3, 2, 5)
+    wide = torch.zeros(seqs, chunks, 64, H, slices * 16, dtype=BF16)
+    wide[..., :vp] = full[..., 2 * G * dp:].view(seqs, chunks, 64, H, vp)
+    v = torch.full((seqs, chunks, H, slices, 64, 24), float("nan"), dtype=BF16)
+    v[..., :16] = wide.view(seqs, chunks, 64, H, slices, 16).permute(0, 1, 3, 4, 2, 5)
+    out = torch.cat([qk.flatten(), v.flatten()]).view(torch.uint8).cuda()
+    assert out.numel() == K.recurrence_tiles(seqs, T, H, G, dp, vp)
+    return out
+
+
 def recurrence_expected(act, seqs, H, G, dp, vp, state, norms=None, beta_g=None, log_decay=None):
     R = act.shape[0]
     T, out, states = R // seqs, [], []
@@ -210,7 +231,8 @@ def test_recurrence_in_chunks_and_token_by_token(seqs, T, H, G, dp, vp, delta, f
         S.copy_(state if not fresh else torch.full_like(state, float("nan")))
         o = torch.full((seqs * T, H * vp), float("nan"), dtype=BF16, device="cuda")
         scratch = torch.empty(K.recurrence_scratch(seqs, T, H, delta), dtype=torch.uint8, device="cuda") if chunks else None
-        K.recurrence(act.cuda(), [H, G, dp, vp], dev.get("norms"), dev.get("beta_g"), dev.get("log_decay"), S, lens, T, o, scratch)
+        put = as_tiles(act, seqs, H, G, dp, vp) if chunks else act.cuda()
+        K.recurrence(put, [H, G, dp, vp], dev.get("norms"), dev.get("beta_g"), dev.get("log_decay"), S, lens, T, o, scratch)
         assert cases.row_errors(o, want).max() < 8e-3, chunks
         assert cases.row_errors(S.flatten(2), want_state.flatten(2)).max() < 2e-5, chunks
     kernels().check_status()
@@ -228,7 +250,7 @@ def test_state_is_kept_in_floats_over_many_chunks():
     S = torch.empty(1, 1, dp, vp, device="cuda")
     o = torch.empty(T, vp, dtype=BF16, device="cuda")
     scratch = torch.empty(K.recurrence_scratch(1, T, 1, False), dtype=torch.uint8, device="cuda")
-    K.recurrence(act.cuda(), [1, 1, dp, vp], None, None, log_decay.cuda(), S, torch.zeros(1, dtype=torch.int32, device="cuda"), T, o, scratch)
+    K.recurrence(as_tiles(act, 1, 1, 1, dp, vp), [1, 1, dp, vp], None, None, log_decay.cuda(), S, torch.zeros(1, dtype=torch.int32, device="cuda"), T, o, scratch)
     assert ((S.cpu().double() - want).abs() / want.abs()).max() < 2e-5
 
 
