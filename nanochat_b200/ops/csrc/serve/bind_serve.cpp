@@ -390,10 +390,10 @@ void expert_rows_(const Tensor& h, const Tensor& Wgu, const Tensor& Wdown, const
 }
 
 // ------------------------------------------------------------------------------------------------------------ gemv
-GemvDesc gemv_of(const Tensor& x, const Tensor& W, const optional<Tensor>& next) {
+GemvDesc gemv_of(const Tensor& x, const Tensor& W, const optional<Tensor>& next, bool any_rows = false) {
   TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1 && W.is_cuda() && W.scalar_type() == at::kBFloat16, "gemv operands");
   check_rows(x, "x"); check_rows(W, "W");
-  TORCH_CHECK(x.size(1) == W.size(1) && x.size(0) <= 8, "gemv shapes");
+  TORCH_CHECK(x.size(1) == W.size(1) && (any_rows || x.size(0) <= 8), "gemv shapes");
   GemvDesc d{};
   d.x = x.data_ptr(); d.ldx = pitch(x); d.W = W.data_ptr(); d.ldw = pitch(W); d.rows = (int)x.size(0); d.N = (int)W.size(0); d.K = (int)x.size(1);
   d.next = next_weights(next); d.pdl = true; d.accumulate = true;
@@ -456,7 +456,7 @@ void gemv_residual(const Tensor& y, const Tensor& W, Tensor& x, const Tensor& g,
 
 // out = x W^T, x bf16 rows
 void gemv_plain(const Tensor& x, const Tensor& W, Tensor& out, const optional<Tensor>& next) {
-  GemvDesc d = gemv_of(x, W, next);
+  GemvDesc d = gemv_of(x, W, next, true);
   TORCH_CHECK(x.scalar_type() == at::kBFloat16, "x: bf16 rows");
   const int epi = store_kind(d, out);
   const c10::cuda::CUDAGuard guard(x.device());

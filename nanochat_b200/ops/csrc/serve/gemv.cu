@@ -158,7 +158,9 @@ __device__ __forceinline__ void gemv_body(const GemvArgs& a) {
     return;
   }
   const int n0 = blockIdx.x * (MT * 16), q8 = (lane & 3) * 8, row = lane >> 2;
-  if (SPLIT == 1 || blockIdx.y == 0) prefetch_l2_slice(a.next, blockIdx.x, a.n_blocks);
+  // grid y without a split: groups of eight rows (plain stores only)
+  const int group = SPLIT == 1 ? (int)blockIdx.y : 0, B = SPLIT == 1 ? min(ROWS, a.B - group * ROWS) : a.B;
+  if (blockIdx.y == 0) prefetch_l2_slice(a.next, blockIdx.x, a.n_blocks);
   const TileRows<MT> w = tile_rows<MT>(a.W, a.ldw, n0, a.N, lane);
   Frag<MT, U> f;
   const int k_first = warp * 32 + (SPLIT > 1 ? (int)blockIdx.y * STEP : 0);
@@ -171,9 +173,9 @@ __device__ __forceinline__ void gemv_body(const GemvArgs& a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
   const float* xf = (const float*)a.x + row * a.ldx;
-  const bf16* xb = (const bf16*)a.x + row * a.ldx;
+  const bf16* xb = (const bf16*)a.x + (group * ROWS + row) * a.ldx;
   auto x = [&](int k) -> uint4 {
-    if (row >= a.B) return make_uint4(0, 0, 0, 0);
+    if (row >= B) return make_uint4(0, 0, 0, 0);
     if (!NORM) return *reinterpret_cast<const uint4*>(xb + k);
     float v[8], nw[8];
     load8(xf + k, v);
@@ -220,16 +222,16 @@ __device__ __forceinline__ void gemv_body(const GemvArgs& a) {
     if (blockIdx.y != 0) return;
   }
   if (tid < MT * 16 * ROWS) {
-    if (b < a.B && n < a.N) {
+    if (b < B && n < a.N) {
       if constexpr (SPLIT == 1) {
 #pragma unroll
         for (int i = 0; i < WARPS; ++i) v += s_acc[i][m][b];
       }
       if (NORM) v *= scale(b);
       if (a.epi == GEMV_STORE_F32) {
-        ((float*)a.out)[b * a.ldo + n] = v;
+        ((float*)a.out)[(group * ROWS + b) * a.ldo + n] = v;
       } else if (a.epi == GEMV_STORE_BF16) {
-        ((bf16*)a.out)[b * a.ldo + n] = __float2bfloat16_rn(v);
+        ((bf16*)a.out)[(group * ROWS + b) * a.ldo + n] = __float2bfloat16_rn(v);
       } else {
         float r = a.mult * sigmoidf(a.g[b * a.ldg + n] + a.bias[n]) * v;
         if (a.extra) r += a.extra[b * a.ldr + n];
@@ -423,8 +425,8 @@ expert_down_rows_kernel(const ExpertArgs a) {
 }  // namespace
 
 cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s) {
-  if (d.rows < 1 || d.rows > ROWS || d.N <= 0 || d.K <= 0 || (d.K & 7) || (d.ldx & 7) || (d.ldw & 7) || d.n_real > d.K)
-    return cudaErrorInvalidValue;
+  if (d.rows < 1 || d.N <= 0 || d.K <= 0 || (d.K & 7) || (d.ldx & 7) || (d.ldw & 7) || d.n_real > d.K) return cudaErrorInvalidValue;
+  if (d.rows > ROWS && (pre != PRE_PLAIN || epi == GEMV_RESIDUAL || d.rows > 65535 * ROWS)) return cudaErrorInvalidValue;
   if (pre == PRE_NORM ? (d.w == nullptr || d.n_real <= 0) : (pre != PRE_PLAIN || d.store != nullptr || d.h_out != nullptr)) return cudaErrorInvalidValue;
   if (epi == GEMV_RESIDUAL ? (d.resid == nullptr || d.g == nullptr || d.bias == nullptr) : d.out == nullptr) return cudaErrorInvalidValue;
   if (d.h_out != nullptr && (d.ldh & 7)) return cudaErrorInvalidValue;
@@ -437,9 +439,9 @@ cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s) {
   a.n_blocks = (d.N + (wide ? 31 : 15)) / (wide ? 32 : 16);
   int grid = a.n_blocks;
   if (d.store) { a.store = *d.store; grid += d.rows; }
-  if (pre == PRE_PLAIN && !wide && a.n_blocks < 148 && d.K >= 3072) return launch(d.pdl, gemv_cluster_kernel, dim3(grid, CLUSTER), dim3(THREADS), 0, s, a);
+  if (pre == PRE_PLAIN && !wide && a.n_blocks < 148 && d.K >= 3072 && d.rows <= ROWS) return launch(d.pdl, gemv_cluster_kernel, dim3(grid, CLUSTER), dim3(THREADS), 0, s, a);
   auto kern = pre == PRE_NORM ? (wide ? gemv_kernel<true, 2> : gemv_kernel<true, 1>) : (wide ? gemv_kernel<false, 2> : gemv_kernel<false, 1>);
-  return launch(d.pdl, kern, dim3(grid), dim3(THREADS), 0, s, a);
+  return launch(d.pdl, kern, dim3(grid, (d.rows + ROWS - 1) / ROWS), dim3(THREADS), 0, s, a);
 }
 
 cudaError_t gemv_relu_glu(const GemvDesc& d, cudaStream_t s) {

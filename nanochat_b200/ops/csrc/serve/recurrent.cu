@@ -11,15 +11,13 @@
 //                 R = V - decayed K S,  U = T R        delta rule;   U = V  fixed decay
 //                 O = decayed Q S + A U
 //                 S = decayed S + K^T (decayed U)
-//              One warp copies whole chunks into shared memory, four follow the state from chunk to chunk, four more
+//              One warp copies whole chunks into shared memory, eight follow the state from chunk to chunk, four more
 //              read it out behind them.
 //   norm_gate         RMS norm and gate of what a recurrence read out, and the convolution's last inputs
 //
 // Exactness: the products run on bf16 operands, so every operand that is a float (the state, T, A, U, R) enters as the sum
 // of two bf16 values, and what scales rows (inverse norms, decays) is applied to accumulators, not to operands: keys,
 // queries and values are the bf16 activations themselves. The state is float from chunk to chunk.
-#include <type_traits>
-
 #include "mma.cuh"
 
 namespace nc {
@@ -45,8 +43,11 @@ __device__ __forceinline__ void store4(bf16* p, const float (&f)[4]) {
 
 // ------------------------------------------------------------------------------ tiles
 constexpr int CH = 64;                       // tokens per chunk
-constexpr int LT = CH + 8;                   // pitch of a 64 x 64 operand
-constexpr int MAT = CH * LT;
+// A lower triangular 64 x 64 operand: four bands of 16 rows, band b with its first 16 (b + 1) columns and a pitch of 8 more.
+__host__ __device__ constexpr int band_pitch(int b) { return 16 * (b + 1) + 8; }
+__host__ __device__ constexpr int band_at(int b) { return 16 * (8 * b * (b + 1) + 8 * b); }
+constexpr int MAT = band_at(4);
+__device__ __forceinline__ int band_index(int i, int j) { return band_at(i >> 4) + (i & 15) * band_pitch(i >> 4) + j; }
 constexpr int SCALARS = 200;                 // floats per chunk and head: three vectors of 64, the chunk's total decay, padding
 constexpr int VS = 16;                       // state columns per CTA
 constexpr int LV = VS + 8;
@@ -70,7 +71,7 @@ struct Tiles {
 __host__ __device__ constexpr size_t chunk_bytes(bool delta) { return (size_t)(delta ? 4 : 2) * MAT * 2 + SCALARS * 4; }
 
 // ---------------------------------------------------------------------------- prepare
-constexpr int PREP_TOKENS = 8;         // tokens a warp walks through
+constexpr int PREP_TOKENS = 4;         // tokens a warp walks through
 
 // grid (token groups of a sequence, ceil(jobs / 4), sequences), a warp per job: query heads, key heads, value heads.
 // TAPS > 0: at most TAPS taps, the inputs stay in registers; 0: any number, re-read; -1: no convolution and no norms
@@ -97,29 +98,36 @@ prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ nor
       x[0] = x[1] = x[2] = x[3] = 0.f;
     }
   };
-  auto place = [&](int t, int c) -> T* {                // c: column of the job's head
-    if (!TILES) return out + (row0 + t0 + t) * channels + ch0 + c;
-    const long long unit = (long long)seq * tiles.chunks + t0 / CH;
-    const int r = t0 % CH + t;
-    if (job < 2 * G) return out + (unit * G + job % G) * tiles.qk_unit + ((job >= G ? CH : 0) + r) * (tiles.D + 8) + c;
-    return out + tiles.v_base + ((unit * H + job - 2 * G) * tiles.slices + c / VS) * tiles.v_unit + r * LV + c % VS;
-  };
+  // where the head's columns of the group's first token go, and from one token to the next
+  const long long unit = (long long)seq * tiles.chunks + t0 / CH;
+  const int r0 = t0 % CH;
+  T* dst = !TILES ? out + (row0 + t0) * channels + ch0
+           : job < 2 * G ? out + (unit * G + job % G) * tiles.qk_unit + ((job >= G ? CH : 0) + r0) * (tiles.D + 8)
+                         : out + tiles.v_base + (unit * H + job - 2 * G) * tiles.slices * tiles.v_unit + r0 * LV;
+  const int step = !TILES ? channels : job < 2 * G ? tiles.D + 8 : LV;
   float ss[PREP_TOKENS];
 #pragma unroll
   for (int t = 0; t < PREP_TOKENS; ++t) ss[t] = 0.f;
   const int columns = !TILES ? size : job < 2 * G ? tiles.D : tiles.slices * VS;
+  constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0;
+  const bool inside = t0 >= BACK && n == PREP_TOKENS;   // every input is a row of this portion
   for (int c = lane * 4; c < columns; c += 128) {
     const int ch = ch0 + c;
-    constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0;
     float w[BACK + 1][4], x[PREP_TOKENS + BACK][4];     // x[BACK + t]: token t of the group
     const bool in = c < size;
+    if (TAPS != 0 && inside && in) {
+      const TZ* src = (const TZ*)d.z + (row0 + t0 - BACK) * d.ldz + ch;
 #pragma unroll
-    for (int t = 0; t < PREP_TOKENS + BACK; ++t) {
-      if (in && TAPS != 0 && t - BACK < n && (t >= BACK || BACK - t < d.taps)) {
-        fetch(t0 + t - BACK, ch, x[t]);
-      } else {
+      for (int t = 0; t < PREP_TOKENS + BACK; ++t) load4(src + t * d.ldz, x[t]);
+    } else {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) x[t][j] = 0.f;
+      for (int t = 0; t < PREP_TOKENS + BACK; ++t) {
+        if (in && TAPS != 0 && t - BACK < n && (t >= BACK || BACK - t < d.taps)) {
+          fetch(t0 + t - BACK, ch, x[t]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) x[t][j] = 0.f;
+        }
       }
     }
     if (TAPS > 0) {
@@ -133,6 +141,7 @@ prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ nor
         }
       }
     }
+    T* at = TILES && job >= 2 * G ? dst + (c / VS) * tiles.v_unit + c % VS : dst + c;
 #pragma unroll
     for (int t = 0; t < PREP_TOKENS; ++t) {
       if (!TILES && t >= n) break;
@@ -159,7 +168,7 @@ prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ nor
         a[j] = t < n ? to_f(from_f<T>(silu_of<T>(a[j]))) : 0.f;     // the norm is that of the vector that is stored
         ss[t] += a[j] * a[j];
       }
-      store4(place(t, c), a);
+      store4(at + t * step, a);
     }
   }
   if (TAPS < 0) return;
@@ -298,7 +307,7 @@ __device__ __forceinline__ void block_dot(const float* a, const float* b, int ld
   }
 }
 // X = (1 + L)^-1 for a strictly lower triangular L, both 64 x LL floats; blocks of 16: the diagonal ones by forward
-// substitution, the others below them from the left. All 128 threads call it; L has been written and synchronised.
+// substitution, the others below them from the left. All 256 threads call it; L has been written and synchronised.
 __device__ void invert_unit_lower(const float* L, float* X, float (*P)[16][20]) {
   const int tid = threadIdx.x;
   if (tid < CH) {
@@ -314,18 +323,18 @@ __device__ void invert_unit_lower(const float* L, float* X, float (*P)[16][20]) 
     }
   }
   __syncthreads();
-  const int r = tid >> 3, c = (tid & 7) * 2;
+  const int half = tid >> 7, r = (tid & 127) >> 3, c = (tid & 7) * 2;      // each half takes every other block
 #pragma unroll 1
   for (int d = 1; d < 4; ++d) {
 #pragma unroll 1
-    for (int i = d; i < 4; ++i) {                        // P = sum over the blocks between of L_im X_mj, j = i - d
+    for (int i = d + half; i < 4; i += 2) {              // P = sum over the blocks between of L_im X_mj, j = i - d
       float s[2] = {0.f, 0.f};
       for (int m = i - d; m < i; ++m) block_dot(L + i * 16 * LL + m * 16, X + m * 16 * LL + (i - d) * 16, LL, LL, r, c, s);
       *reinterpret_cast<float2*>(&P[i - d][r][c]) = make_float2(s[0], s[1]);
     }
     __syncthreads();
 #pragma unroll 1
-    for (int i = d; i < 4; ++i) {
+    for (int i = d + half; i < 4; i += 2) {
       float s[2] = {0.f, 0.f};
       block_dot(X + i * 16 * LL + i * 16, &P[i - d][0][0], LL, 20, r, c, s);
       *reinterpret_cast<float2*>(X + (i * 16 + r) * LL + (i - d) * 16 + c) = make_float2(-s[0], -s[1]);
@@ -334,10 +343,10 @@ __device__ void invert_unit_lower(const float* L, float* X, float (*P)[16][20]) 
   }
 }
 
-// grid (chunks, heads, sequences), 128 threads. Row i of a chunk: scalars [0, 64) decayed 1/|k|, [64, 128) decayed 1/|q|,
+// grid (chunks, heads, sequences), 256 threads: warp w has 16 tokens and every other pair of 8-key tiles. Row i of a chunk: scalars [0, 64) decayed 1/|k|, [64, 128) decayed 1/|q|,
 // [128, 192) 1/|k| times the decay from the token to the chunk's end, [192] the decay over the whole chunk.
 template <bool DELTA, int D>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
   constexpr int LD = D + 8, TILE = CH * LD, SYSTEM = 2 * CH * LL * 4;
   constexpr int BYTES = 2 * TILE * 2 > SYSTEM || !DELTA ? 2 * TILE * 2 : SYSTEM;
@@ -355,7 +364,7 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
   const Tiles tiles(gridDim.z, r.pos.per_seq, r.heads, r.kv_heads, r.dp, r.vp);
   const uint8_t* src = reinterpret_cast<const uint8_t*>((const bf16*)r.act + (((long long)seq * tiles.chunks + chunk) * r.kv_heads + kvh) * tiles.qk_unit);
 #pragma unroll
-  for (int i = tid * 16; i < 2 * TILE * 2; i += 128 * 16) cp_async16(smem + i, src + i);
+  for (int i = tid * 16; i < 2 * TILE * 2; i += 256 * 16) cp_async16(smem + i, src + i);
   cp_async_commit();
   uint8_t* unit = scratch + ((long long)(seq * gridDim.x + chunk) * r.heads + h) * chunk_bytes(DELTA);
   bf16* gA = reinterpret_cast<bf16*>(unit);
@@ -399,63 +408,67 @@ chunk_gram_kernel(const Recurrence r, uint8_t* __restrict__ scratch) {
   }
   cp_async_wait<0>();
   __syncthreads();
-  float qk[8][4], kk[DELTA ? 8 : 1][4];
+  const int mt = warp & 3, odd = warp >> 2;
+  float qk[4][4], kk[DELTA ? 4 : 1][4];                         // tile u: keys (2 (u / 2) + odd) * 16 + (u % 2) * 8 ...
 #pragma unroll
-  for (int t = 0; t < 8; ++t)
+  for (int t = 0; t < 4; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) { qk[t][e] = 0.f; if (DELTA) kk[t][e] = 0.f; }
 #pragma unroll
   for (int k = 0; k < D; k += 16) {
     uint32_t aq[4], ak[4];
-    ldmatrix4(aq, sQ + (warp * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
-    if (DELTA) ldmatrix4(ak, sK + (warp * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+    ldmatrix4(aq, sQ + (mt * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+    if (DELTA) ldmatrix4(ak, sK + (mt * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
 #pragma unroll
-    for (int t = 0; t < 8; t += 2) {
-      if (t > 2 * warp + 1) break;
-      uint32_t b[4];                                            // keys t * 8 .. t * 8 + 15, both halves of k
-      ldmatrix4(b, sK + (t * 8 + (lane & 7) + (lane >> 4) * 8) * LD + k + ((lane >> 3) & 1) * 8);
-      mma_16816(qk[t], aq, b[0], b[1]);
-      mma_16816(qk[t + 1], aq, b[2], b[3]);
+    for (int u = 0; u < 2; ++u) {
+      const int j0 = (2 * u + odd) * 16;
+      if (j0 > mt * 16) break;                                  // blocks above the diagonal are never read
+      uint32_t b[4];                                            // 16 keys, both halves of k
+      ldmatrix4(b, sK + (j0 + (lane & 7) + (lane >> 4) * 8) * LD + k + ((lane >> 3) & 1) * 8);
+      mma_16816(qk[2 * u], aq, b[0], b[1]);
+      mma_16816(qk[2 * u + 1], aq, b[2], b[3]);
       if constexpr (DELTA) {
-        mma_16816(kk[t], ak, b[0], b[1]);
-        mma_16816(kk[t + 1], ak, b[2], b[3]);
+        mma_16816(kk[2 * u], ak, b[0], b[1]);
+        mma_16816(kk[2 * u + 1], ak, b[2], b[3]);
       }
     }
   }
   __syncthreads();
 #pragma unroll
-  for (int t = 0; t < 8; ++t) {
-    if (t > 2 * warp + 1) break;                                // blocks above the diagonal are never read
-    const int j = t * 8 + (lane & 3) * 2;
+  for (int u = 0; u < 4; ++u) {
+    const int j0 = (2 * (u >> 1) + odd) * 16;
+    if (j0 > mt * 16) break;
+    const int j = j0 + (u & 1) * 8 + (lane & 3) * 2;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int i = warp * 16 + (lane >> 2) + half * 8;
+      const int i = mt * 16 + (lane >> 2) + half * 8;
       float a[2], l[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int c = j + e;
         const float decay = c <= i ? expf((float)(sG[i] - sG[c])) : 0.f;
-        a[e] = c <= i ? sRq[i] * sRk[c] * decay * qk[t][half * 2 + e] : 0.f;
-        if constexpr (DELTA) l[e] = c < i ? sB[i] * sRk[i] * sRk[c] * decay * kk[t][half * 2 + e] : 0.f;
+        a[e] = c <= i ? sRq[i] * sRk[c] * decay * qk[u][half * 2 + e] : 0.f;
+        if constexpr (DELTA) l[e] = c < i ? sB[i] * sRk[i] * sRk[c] * decay * kk[u][half * 2 + e] : 0.f;
       }
-      store_split(gA + i * LT + j, gA + MAT + i * LT + j, a[0], a[1]);
+      store_split(gA + band_index(i, j), gA + MAT + band_index(i, j), a[0], a[1]);
       if constexpr (DELTA) *reinterpret_cast<float2*>(sL + i * LL + j) = make_float2(l[0], l[1]);
     }
   }
   if constexpr (DELTA) {
     __syncthreads();
     invert_unit_lower(sL, sX, sP);
-    for (int e = tid; e < CH * CH / 2; e += 128) {
+    for (int e = tid; e < CH * CH / 2; e += 256) {
       const int i = e / (CH / 2), j = (e % (CH / 2)) * 2;
       if (j > (i | 15)) continue;
       const bool diagonal = (i >> 4) == (j >> 4);               // the substitution leaves zeros above the diagonal
       const float2 x = *reinterpret_cast<const float2*>(sX + i * LL + j);
-      store_split(gA + 2 * MAT + i * LT + j, gA + 3 * MAT + i * LT + j, diagonal && j > i ? 0.f : x.x * sB[j], diagonal && j + 1 > i ? 0.f : x.y * sB[j + 1]);
+      store_split(gA + 2 * MAT + band_index(i, j), gA + 3 * MAT + band_index(i, j), diagonal && j > i ? 0.f : x.x * sB[j], diagonal && j + 1 > i ? 0.f : x.y * sB[j + 1]);
     }
   }
 }
 
-// Shared memory of the scan: two stages of a chunk's operands, then what the warps hand each other.
+// Shared memory of the scan: three stages of a chunk's operands, then what the warps hand each other.
+constexpr int STAGES = 3;
 template <bool DELTA, int D>
 struct ScanSmem {
   static constexpr int LD = D + 8, MATS = DELTA ? 4 : 2;
@@ -463,8 +476,8 @@ struct ScanSmem {
   static constexpr int Q = 0, K = CH * LD * 2, A = QK_BYTES, SC = A + MATS * MAT * 2, V = A + UNIT_BYTES;
   static constexpr int STAGE = QK_BYTES + UNIT_BYTES + V_BYTES;
   static constexpr int PART = CH * LV, S_PART = D * LV;         // elements of one part (high or low) of a 64 x 16 operand, of the state
-  static constexpr int S = 2 * STAGE;                           // state, two buffers of two parts
-  static constexpr int W = S + 4 * S_PART * 2;                  // U with the decay to the chunk's end
+  static constexpr int S = STAGES * STAGE;                      // state
+  static constexpr int W = S + 2 * S_PART * 2;                  // U with the decay to the chunk's end
   static constexpr int R = W + 2 * PART * 2;                    // delta rule: R, then U in two buffers
   static constexpr int U = R + (DELTA ? 2 * PART * 2 : 0);
   static constexpr int BAR = U + (DELTA ? 4 * PART * 2 : 0);
@@ -472,101 +485,60 @@ struct ScanSmem {
   static_assert(STAGE % 16 == 0 && TOTAL <= 227 * 1024, "stages must fit shared memory");
 };
 
-// grid (ceil(vp / 16), heads, sequences), 288 threads: warps 0..3 own the state (16 D / 64 rows each), 4..7 the output, 8 copies.
+constexpr int SCAN_THREADS = 13 * 32;
+// grid (ceil(vp / 16), heads, sequences): warps 0..7 own the state, 8..11 the output, 12 copies. The state warps split tokens as
+// 16 tokens x 8 columns (warp & 3, warp >> 2), the state as 16 rows x 16 columns (D = 128) or 16 x 8 (D = 64).
 // A wait that runs out raises the status and the kernel runs on without waiting, so that no barrier is left short.
 template <bool DELTA, int D>
-__global__ void __launch_bounds__(288)
+__global__ void __launch_bounds__(SCAN_THREADS)
 chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* status) {
   using M = ScanSmem<DELTA, D>;
-  constexpr int LD = M::LD, MT = D / 64;
+  constexpr int LD = M::LD, NT = D / 64;                         // NT: 8-column tiles of the state a warp holds
   extern __shared__ __align__(128) uint8_t smem[];
   const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, kvh = h / (r.heads / r.kv_heads), v0 = slice * VS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int T = r.pos.per_seq;
   const Tiles tiles(gridDim.z, T, r.heads, r.kv_heads, r.dp, r.vp);
   const int chunks = tiles.chunks;
-  uint64_t* full = reinterpret_cast<uint64_t*>(smem + M::BAR);       // [2] each, by chunk parity
-  uint64_t *empty = full + 2, *s_ready = full + 4, *u_ready = full + 6, *o_done = full + 8;
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(full + 10);
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + M::BAR);       // per stage: a chunk has arrived, has been used
+  uint64_t* empty = full + STAGES;
+  uint64_t *s_ready = empty + STAGES, *s_read = s_ready + 1;         // the state is published, has been read by the output warps
+  uint64_t *u_ready = s_read + 1, *u_read = u_ready + 2;             // [2] U is there, has been read, by chunk parity
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(u_read + 2);
   if (tid == 0) {
-    for (int i = 0; i < 2; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); mbar_init(&s_ready[i], 4); mbar_init(&u_ready[i], 4); mbar_init(&o_done[i], 4); }
+    for (int i = 0; i < STAGES; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 12); }
+    mbar_init(s_ready, 8); mbar_init(s_read, 4);
+    for (int i = 0; i < 2; ++i) { mbar_init(&u_ready[i], 8); mbar_init(&u_read[i], 4); }
     *abort_flag = 0;
     fence_mbar_init();
   }
   __syncthreads();
   auto wait = [&](uint64_t* bar, int n, int code) { mbar_wait(bar, n & 1, abort_flag, status, code, 0x5c0); };    // its n-th completion
   auto arrive = [&](uint64_t* bar) { __syncwarp(); if (lane == 0) mbar_arrive(bar); };
-  auto state_sync = [] { asm volatile("bar.sync 1, 128;" ::: "memory"); };
-  const int mrow = (warp & 3) * 16;                              // this warp's 16 tokens of a chunk
+  auto state_sync = [] { asm volatile("bar.sync 1, 256;" ::: "memory"); };
+  const int band = warp & 3, mrow = band * 16;                   // this warp's 16 tokens of a chunk
   const int ri = mrow + (lane >> 2), ci = (lane & 3) * 2;        // first row and column of its accumulators
-  auto a_frag = [&](uint32_t (&a)[4], const bf16* tile, int ld, int k) { ldmatrix4(a, tile + (mrow + (lane & 15)) * ld + k + (lane >> 4) * 8); };
+  auto a_frag = [&](uint32_t (&a)[4], const bf16* tile, int k) { ldmatrix4(a, tile + (mrow + (lane & 15)) * LD + k + (lane >> 4) * 8); };
+  auto tri_frag = [&](uint32_t (&a)[4], const bf16* mat, int k) { ldmatrix4(a, mat + band_at(band) + (lane & 15) * band_pitch(band) + k + (lane >> 4) * 8); };
+  // 16 rows of a 16-column operand: both column tiles of one part, or one column tile of both parts (high in b[0..1])
   auto b_frag = [&](uint32_t (&b)[4], const bf16* rows, int k) { ldmatrix4_trans(b, rows + (k + (lane & 15)) * LV + (lane >> 4) * 8); };
-  auto zero = [](float (&a)[2][4]) {
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) a[t][e] = 0.f;
+  auto b_parts = [&](uint32_t (&b)[4], const bf16* rows, int low, int column, int k) {
+    ldmatrix4_trans(b, rows + (lane >> 4) * low + (k + (lane & 15)) * LV + column);
   };
-  // 16 tokens x 16 columns of X S, X the chunk's queries or keys
-  auto times_state = [&](float (&o)[2][4], const bf16* rows, const bf16* s) {
-    float lo[2][4];
-    zero(o);
-    zero(lo);
+  auto add = [](float (&a)[4], const float (&b)[4]) {
 #pragma unroll
-    for (int k = 0; k < D; k += 16) {
-      uint32_t a[4], bh[4], bl[4];
-      a_frag(a, rows, LD, k);
-      b_frag(bh, s, k);
-      b_frag(bl, s + M::S_PART, k);
-      mma_16816(o[0], a, bh[0], bh[1]);
-      mma_16816(o[1], a, bh[2], bh[3]);
-      mma_16816(lo[0], a, bl[0], bl[1]);
-      mma_16816(lo[1], a, bl[2], bl[3]);
-    }
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[t][e] += lo[t][e];
+    for (int e = 0; e < 4; ++e) a[e] += b[e];
   };
-  // o += M X for a lower triangular 64 x 64 M in two parts and a 64 x 16 X in XP parts
-  auto times_lower = [&](float (&o)[2][4], const bf16* m, const bf16* x, auto two_parts) {
-    float p[2][4], q[2][4];
-    zero(p);
-    zero(q);
-#pragma unroll
-    for (int k = 0; k < CH; k += 16) {
-      if (k > mrow) break;
-      uint32_t ah[4], al[4], bh[4], bl[4];
-      a_frag(ah, m, LT, k);
-      a_frag(al, m + MAT, LT, k);
-      b_frag(bh, x, k);
-      if constexpr (decltype(two_parts)::value) b_frag(bl, x + M::PART, k);
-      mma_16816(o[0], ah, bh[0], bh[1]);
-      mma_16816(o[1], ah, bh[2], bh[3]);
-      mma_16816(p[0], al, bh[0], bh[1]);
-      mma_16816(p[1], al, bh[2], bh[3]);
-      if constexpr (decltype(two_parts)::value) {
-        mma_16816(q[0], ah, bl[0], bl[1]);
-        mma_16816(q[1], ah, bl[2], bl[3]);
-      }
-    }
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[t][e] += p[t][e] + q[t][e];
-  };
-  using Two = std::true_type;
-  using One = std::false_type;
 
-  if (warp == 8) {                                               // ---- copies
+  if (warp == 12) {                                              // ---- copies
     if (lane == 0) {
       const bf16* qk = (const bf16*)r.act + ((long long)seq * chunks * r.kv_heads + kvh) * tiles.qk_unit;
       const bf16* v = (const bf16*)r.act + tiles.v_base + (((long long)seq * chunks * r.heads + h) * tiles.slices + slice) * tiles.v_unit;
       const uint8_t* unit = scratch + ((long long)seq * chunks * r.heads + h) * chunk_bytes(DELTA);
       for (int c = 0; c < chunks && !*abort_flag; ++c) {
-        const int b = c & 1;
+        const int b = c % STAGES;
         uint8_t* st = smem + b * M::STAGE;
-        if (c >= 2) wait(&empty[b], (c >> 1) - 1, ST_WAIT_EMPTY);
+        if (c >= STAGES) wait(&empty[b], c / STAGES - 1, ST_WAIT_EMPTY);
         if (*abort_flag) break;
         mbar_arrive_expect_tx(&full[b], M::STAGE);
         bulk_load_1d(st + M::Q, qk + (long long)c * r.kv_heads * tiles.qk_unit, M::QK_BYTES, &full[b]);
@@ -574,140 +546,182 @@ chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* 
         bulk_load_1d(st + M::V, v + (long long)c * r.heads * tiles.slices * tiles.v_unit, M::V_BYTES, &full[b]);
       }
     }
-  } else if (warp < 4) {                                         // ---- state
+  } else if (warp < 8) {                                         // ---- state
+    const int nt = warp >> 2, j = nt * 8 + ci;                   // this warp's columns of the tokens' operands
+    const int d0 = (NT == 2 ? warp : warp & 3) * 16, c0 = NT == 2 ? 0 : nt * 8;      // its part of the state
     bf16* sW = reinterpret_cast<bf16*>(smem + M::W);
     bf16* sR = reinterpret_cast<bf16*>(smem + M::R);
     float* state = r.state.ptr + seq * r.state.seq_stride + (long long)h * r.dp * r.vp + v0;
     const bool fresh = r.pos.lens[seq] == 0;
-    float st[MT][2][4] = {};
-    auto each_state = [&](auto f) {                              // f(row of the state, column, tile, column tile, first element)
+    float st[NT][4] = {};
+    auto each_state = [&](auto f) {                              // f(row of the state, column, tile, first element)
 #pragma unroll
-      for (int i = 0; i < MT; ++i)
+      for (int t = 0; t < NT; ++t)
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
-#pragma unroll
-          for (int half = 0; half < 2; ++half)
-            f((warp + 4 * i) * 16 + (lane >> 2) + half * 8, t * 8 + (lane & 3) * 2, i, t, half * 2);
+        for (int half = 0; half < 2; ++half) f(d0 + (lane >> 2) + half * 8, c0 + t * 8 + ci, t, half * 2);
     };
-    auto publish_state = [&](int buffer) {
-      bf16* s = reinterpret_cast<bf16*>(smem + M::S) + buffer * 2 * M::S_PART;
-      each_state([&](int d, int v, int i, int t, int e) { store_split(s + d * LV + v, s + M::S_PART + d * LV + v, st[i][t][e], st[i][t][e + 1]); });
-      arrive(&s_ready[buffer]);
+    bf16* sS = reinterpret_cast<bf16*>(smem + M::S);
+    auto publish_state = [&] {
+      each_state([&](int d, int v, int t, int e) { store_split(sS + d * LV + v, sS + M::S_PART + d * LV + v, st[t][e], st[t][e + 1]); });
+      arrive(s_ready);
     };
-    each_state([&](int d, int v, int i, int t, int e) {
+    each_state([&](int d, int v, int t, int e) {
       const bool in = !fresh && d < r.dp && v0 + v < r.vp;
       const float2 x = in ? *reinterpret_cast<const float2*>(state + (long long)d * r.vp + v) : make_float2(0.f, 0.f);
-      st[i][t][e] = x.x; st[i][t][e + 1] = x.y;
+      st[t][e] = x.x; st[t][e + 1] = x.y;
     });
-    publish_state(0);
+    publish_state();
     state_sync();
     for (int c = 0; c < chunks; ++c) {
-      const int b = c & 1;
-      const uint8_t* stg = smem + b * M::STAGE;
+      const int stage = c % STAGES;
+      const uint8_t* stg = smem + stage * M::STAGE;
       const bf16 *sk = reinterpret_cast<const bf16*>(stg + M::K), *sv = reinterpret_cast<const bf16*>(stg + M::V);
       const float* sc = reinterpret_cast<const float*>(stg + M::SC);
-      wait(&full[b], c >> 1, ST_WAIT_FULL);
-      const float g = sc[3 * CH], w0 = sc[2 * CH + ri], w1 = sc[2 * CH + ri + 8];
+      wait(&full[stage], c / STAGES, ST_WAIT_FULL);
+      const float g = sc[3 * CH], w[2] = {sc[2 * CH + ri], sc[2 * CH + ri + 8]};
+      float2 v[2];
+#pragma unroll
+      for (int half = 0; half < 2; ++half) v[half] = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + (ri + half * 8) * LV + j));
       if constexpr (DELTA) {
-        bf16* sU = reinterpret_cast<bf16*>(smem + M::U) + b * 2 * M::PART;
-        const float k0 = sc[ri], k1 = sc[ri + 8];
-        float x[2][4];
-        times_state(x, sk, reinterpret_cast<const bf16*>(smem + M::S) + b * 2 * M::S_PART);
+        bf16* sU = reinterpret_cast<bf16*>(smem + M::U) + (c & 1) * 2 * M::PART;
+        const bf16* sT = reinterpret_cast<const bf16*>(stg + M::A) + 2 * MAT;
+        const float f[2] = {sc[ri], sc[ri + 8]};
+        float x[2][4] = {}, y[2][4] = {};                        // even and odd steps: shorter chains
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
+        for (int k = 0; k < D; k += 16) {                        // K S
+          uint32_t a[4], p[4];
+          a_frag(a, sk, k);
+          b_parts(p, sS, M::S_PART, nt * 8, k);
+          mma_16816(x[(k >> 4) & 1], a, p[0], p[1]);
+          mma_16816(y[(k >> 4) & 1], a, p[2], p[3]);
+        }
+        add(x[0], x[1]);
+        add(y[0], y[1]);
+        add(x[0], y[0]);
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int i = ri + half * 8, j = t * 8 + ci;
-            const float2 v = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + i * LV + j));
-            const float f = half ? k1 : k0;
-            store_split(sR + i * LV + j, sR + M::PART + i * LV + j, v.x - f * x[t][half * 2], v.y - f * x[t][half * 2 + 1]);
-          }
+        for (int half = 0; half < 2; ++half) {
+          const int i = ri + half * 8;
+          store_split(sR + i * LV + j, sR + M::PART + i * LV + j, v[half].x - f[half] * x[0][half * 2], v[half].y - f[half] * x[0][half * 2 + 1]);
+        }
         state_sync();
-        zero(x);
-        times_lower(x, reinterpret_cast<const bf16*>(stg + M::A) + 2 * MAT, sR, Two{});
+        float u[3][4] = {};
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
+        for (int k = 0; k < CH; k += 16) {                       // U = T R
+          if (k > mrow) break;
+          uint32_t th[4], tl[4], p[4];
+          tri_frag(th, sT, k);
+          tri_frag(tl, sT + MAT, k);
+          b_parts(p, sR, M::PART, nt * 8, k);
+          mma_16816(u[0], th, p[0], p[1]);
+          mma_16816(u[1], tl, p[0], p[1]);
+          mma_16816(u[2], th, p[2], p[3]);
+        }
+        add(u[0], u[1]);
+        add(u[0], u[2]);
+        if (c >= 2) wait(&u_read[c & 1], (c >> 1) - 1, ST_WAIT_PEER);      // chunk c - 2 has been read out of this buffer
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int i = ri + half * 8, j = t * 8 + ci;
-            const float w = half ? w1 : w0;
-            store_split(sW + i * LV + j, sW + M::PART + i * LV + j, x[t][half * 2] * w, x[t][half * 2 + 1] * w);
-            store_split(sU + i * LV + j, sU + M::PART + i * LV + j, x[t][half * 2], x[t][half * 2 + 1]);
-          }
-        arrive(&u_ready[b]);
+        for (int half = 0; half < 2; ++half) {
+          const int i = ri + half * 8;
+          store_split(sW + i * LV + j, sW + M::PART + i * LV + j, u[0][half * 2] * w[half], u[0][half * 2 + 1] * w[half]);
+          store_split(sU + i * LV + j, sU + M::PART + i * LV + j, u[0][half * 2], u[0][half * 2 + 1]);
+        }
+        arrive(&u_ready[c & 1]);
       } else {
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
-#pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int i = ri + half * 8, j = t * 8 + ci;
-            const float2 v = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + i * LV + j));
-            const float w = half ? w1 : w0;
-            store_split(sW + i * LV + j, sW + M::PART + i * LV + j, v.x * w, v.y * w);
-          }
-      }
-      state_sync();
-#pragma unroll
-      for (int i = 0; i < MT; ++i)                               // S = decayed S + K^T W
-#pragma unroll
-        for (int t = 0; t < 2; ++t)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) st[i][t][e] *= g;
-#pragma unroll
-      for (int k = 0; k < CH; k += 16) {
-        uint32_t hi[4], lo[4];
-        b_frag(hi, sW, k);
-        b_frag(lo, sW + M::PART, k);
-#pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          uint32_t a[4];                                         // K^T: rows are the head's dimensions, k the tokens
-          ldmatrix4_trans(a, sk + (k + (lane & 7) + (lane >> 4) * 8) * LD + (warp + 4 * i) * 16 + ((lane >> 3) & 1) * 8);
-          mma_16816(st[i][0], a, hi[0], hi[1]);
-          mma_16816(st[i][1], a, hi[2], hi[3]);
-          mma_16816(st[i][0], a, lo[0], lo[1]);
-          mma_16816(st[i][1], a, lo[2], lo[3]);
+        for (int half = 0; half < 2; ++half) {
+          const int i = ri + half * 8;
+          store_split(sW + i * LV + j, sW + M::PART + i * LV + j, v[half].x * w[half], v[half].y * w[half]);
         }
       }
-      arrive(&empty[b]);
+      state_sync();
+      float lo[NT][4] = {};
+#pragma unroll
+      for (int t = 0; t < NT; ++t)                               // S = decayed S + K^T W
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[t][e] *= g;
+#pragma unroll
+      for (int k = 0; k < CH; k += 16) {
+        uint32_t a[4];                                           // K^T: rows are the head's dimensions, k the tokens
+        ldmatrix4_trans(a, sk + (k + (lane & 7) + (lane >> 4) * 8) * LD + d0 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+          uint32_t p[4];
+          b_parts(p, sW, M::PART, c0 + t * 8, k);
+          mma_16816(st[t], a, p[0], p[1]);
+          mma_16816(lo[t], a, p[2], p[3]);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < NT; ++t) add(st[t], lo[t]);
+      arrive(&empty[stage]);
       if (c + 1 < chunks) {
-        if (c >= 1) wait(&o_done[b ^ 1], (c - 1) >> 1, ST_WAIT_PEER);      // chunk c - 1 has been read out of that buffer
-        publish_state(b ^ 1);
+        wait(s_read, c, ST_WAIT_PEER);
+        publish_state();
         state_sync();
       }
     }
-    each_state([&](int d, int v, int i, int t, int e) {
-      if (d < r.dp && v0 + v < r.vp) *reinterpret_cast<float2*>(state + (long long)d * r.vp + v) = make_float2(st[i][t][e], st[i][t][e + 1]);
+    each_state([&](int d, int v, int t, int e) {
+      if (d < r.dp && v0 + v < r.vp) *reinterpret_cast<float2*>(state + (long long)d * r.vp + v) = make_float2(st[t][e], st[t][e + 1]);
     });
   } else {                                                       // ---- output
     for (int c = 0; c < chunks; ++c) {
-      const int b = c & 1;
-      const uint8_t* stg = smem + b * M::STAGE;
+      const int stage = c % STAGES;
+      const uint8_t* stg = smem + stage * M::STAGE;
       const float* sc = reinterpret_cast<const float*>(stg + M::SC);
-      wait(&full[b], c >> 1, ST_WAIT_FULL);
-      wait(&s_ready[b], c >> 1, ST_WAIT_PEER);
-      float o[2][4];
-      times_state(o, reinterpret_cast<const bf16*>(stg + M::Q), reinterpret_cast<const bf16*>(smem + M::S) + b * 2 * M::S_PART);
+      const bf16 *sq = reinterpret_cast<const bf16*>(stg + M::Q), *sA = reinterpret_cast<const bf16*>(stg + M::A);
+      const bf16* sS = reinterpret_cast<const bf16*>(smem + M::S);
+      const bf16* sU = DELTA ? reinterpret_cast<const bf16*>(smem + M::U) + (c & 1) * 2 * M::PART : reinterpret_cast<const bf16*>(stg + M::V);
+      wait(&full[stage], c / STAGES, ST_WAIT_FULL);
+      wait(s_ready, c, ST_WAIT_PEER);
+      float o[2][4] = {}, p[2][4] = {};
+#pragma unroll
+      for (int k = 0; k < D; k += 16) {                          // Q S
+        uint32_t a[4], bh[4], bl[4];
+        a_frag(a, sq, k);
+        b_frag(bh, sS, k);
+        b_frag(bl, sS + M::S_PART, k);
+        mma_16816(o[0], a, bh[0], bh[1]);
+        mma_16816(o[1], a, bh[2], bh[3]);
+        mma_16816(p[0], a, bl[0], bl[1]);
+        mma_16816(p[1], a, bl[2], bl[3]);
+      }
+      arrive(s_read);
       const float q0 = sc[CH + ri], q1 = sc[CH + ri + 8];
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[t][e] *= e < 2 ? q0 : q1;
-      if constexpr (DELTA) {
-        wait(&u_ready[b], c >> 1, ST_WAIT_PEER);
-        times_lower(o, reinterpret_cast<const bf16*>(stg + M::A), reinterpret_cast<const bf16*>(smem + M::U) + b * 2 * M::PART, Two{});
-      } else {
-        times_lower(o, reinterpret_cast<const bf16*>(stg + M::A), reinterpret_cast<const bf16*>(stg + M::V), One{});
+        for (int e = 0; e < 4; ++e) { o[t][e] = (o[t][e] + p[t][e]) * (e < 2 ? q0 : q1); p[t][e] = 0.f; }
+      if (DELTA) wait(&u_ready[c & 1], c >> 1, ST_WAIT_PEER);
+#pragma unroll
+      for (int k = 0; k < CH; k += 16) {                         // + A U
+        if (k > mrow) break;
+        uint32_t ah[4], al[4], uh[4];
+        tri_frag(ah, sA, k);
+        tri_frag(al, sA + MAT, k);
+        b_frag(uh, sU, k);
+        mma_16816(o[0], ah, uh[0], uh[1]);
+        mma_16816(o[1], ah, uh[2], uh[3]);
+        mma_16816(p[0], al, uh[0], uh[1]);
+        mma_16816(p[1], al, uh[2], uh[3]);
+        if constexpr (DELTA) {
+          uint32_t ul[4];
+          b_frag(ul, sU + M::PART, k);
+          mma_16816(o[0], ah, ul[0], ul[1]);
+          mma_16816(o[1], ah, ul[2], ul[3]);
+        }
       }
-      arrive(&empty[b]);
-      arrive(&o_done[b]);
+      arrive(&empty[stage]);
+      if (DELTA) arrive(&u_read[c & 1]);
       bf16* out = (bf16*)r.o + ((long long)seq * T + c * CH) * r.ldo + (long long)h * r.vp + v0;
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
+      for (int t = 0; t < 2; ++t) {
+        add(o[t], p[t]);
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int i = ri + half * 8, j = t * 8 + ci;
           if (c * CH + i < T && v0 + j < r.vp) *reinterpret_cast<uint32_t*>(out + i * r.ldo + j) = pack_bf16(o[t][half * 2], o[t][half * 2 + 1]);
         }
+      }
     }
   }
   __syncthreads();
@@ -880,10 +894,10 @@ static cudaError_t launch_chunks(const Recurrence& d, uint8_t* scratch, int* sta
   cudaError_t e = configured.once([] { return cudaFuncSetAttribute(chunk_scan_kernel<DELTA, D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); });
   if (e != cudaSuccess) return e;
   const int seqs = d.rows / d.pos.per_seq, chunks = (d.pos.per_seq + CH - 1) / CH;
-  chunk_gram_kernel<DELTA, D><<<dim3(chunks, d.heads, seqs), 128, 0, s>>>(d, scratch);
+  chunk_gram_kernel<DELTA, D><<<dim3(chunks, d.heads, seqs), 256, 0, s>>>(d, scratch);
   e = cudaGetLastError();
   if (e != cudaSuccess) return e;
-  chunk_scan_kernel<DELTA, D><<<dim3((d.vp + VS - 1) / VS, d.heads, seqs), 288, SMEM, s>>>(d, scratch, status);
+  chunk_scan_kernel<DELTA, D><<<dim3((d.vp + VS - 1) / VS, d.heads, seqs), SCAN_THREADS, SMEM, s>>>(d, scratch, status);
   return cudaGetLastError();
 }
 cudaError_t recurrence_chunks(const Recurrence& d, void* scratch, int* status, cudaStream_t s) {

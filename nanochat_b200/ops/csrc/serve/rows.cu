@@ -107,12 +107,12 @@ gated_residual_norm_kernel(float* __restrict__ x, TermsT terms, float mult, cons
   }
 }
 
-// A row of np <= 2048 * NV entries sits in the registers of 256 threads: entry (i * 256 + threadIdx.x) * 8 + j.
-template <int NV, typename TY>
+// A row of np <= 8 * THREADS * NV entries sits in the registers of a block: entry (i * THREADS + threadIdx.x) * 8 + j.
+template <int THREADS, int NV, typename TY>
 __device__ __forceinline__ void load_row(float (&v)[NV][8], const TY* src, int np) {
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = (i * 256 + threadIdx.x) * 8;
+    const int c = (i * THREADS + threadIdx.x) * 8;
     if (c < np) {
       load8(src + c, v[i]);
     } else {
@@ -121,28 +121,42 @@ __device__ __forceinline__ void load_row(float (&v)[NV][8], const TY* src, int n
     }
   }
 }
-// v = (v - mean) / sqrt(variance + eps) * w over the first n entries; w is zero past them
-template <int NV>
+// Sum over the block with one barrier; `red` (THREADS / 32 floats) is used by this call alone.
+template <int THREADS>
+__device__ __forceinline__ float row_sum(float s, float* red) {
+  constexpr int WARPS = THREADS / 32;
+  s = warp_sum(s);
+  const int lane = threadIdx.x & 31;
+  if (lane == 0) red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  s = 0.f;
+#pragma unroll
+  for (int w = 0; w < WARPS; w += 4) {
+    const float4 t = *reinterpret_cast<const float4*>(red + w);
+    s += (t.x + t.y) + (t.z + t.w);
+  }
+  return s;
+}
+// v = (v - mean) / sqrt(variance + eps) * w over the first n entries; v and w are zero past them. red: two sums' memory.
+template <int THREADS, int NV>
 __device__ __forceinline__ void layer_norm_row(float (&v)[NV][8], const float (&w)[NV][8], int n, float eps, float* red) {
-  float s[1] = {0.f};
+  float s = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i)
 #pragma unroll
-    for (int j = 0; j < 8; ++j) s[0] += v[i][j];             // padding is zero
-  block_sum<1>(s, red);
-  const float mean = s[0] / n;
-  s[0] = 0.f;
+    for (int j = 0; j < 8; ++j) s += v[i][j];
+  const float mean = row_sum<THREADS>(s, red) / n;
+  s = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = (i * 256 + threadIdx.x) * 8;
+    const int left = n - (i * THREADS + (int)threadIdx.x) * 8;      // entries of this vector that count
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       v[i][j] -= mean;
-      if (c + j < n) s[0] += v[i][j] * v[i][j];
+      if (j < left) s += v[i][j] * v[i][j];
     }
   }
-  block_sum<1>(s, red);
-  const float r = inv_rms(s[0], n, eps);
+  const float r = inv_rms(row_sum<THREADS>(s, red + 8), n, eps);
 #pragma unroll
   for (int i = 0; i < NV; ++i)
 #pragma unroll
@@ -150,14 +164,14 @@ __device__ __forceinline__ void layer_norm_row(float (&v)[NV][8], const float (&
 }
 
 // T: type of h; TY: type of y (an embedding table's rows when ids is given)
-template <typename T, typename TY, int NV>
-__global__ void __launch_bounds__(256)
+template <typename T, typename TY, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS)
 layer_norm_residual_kernel(const long long* __restrict__ ids, const TY* __restrict__ y, long long ldy, int vocab, const float* __restrict__ wy,
                            float* __restrict__ x, const float* __restrict__ w, float eps, int n, int np, T* __restrict__ h) {
-  __shared__ float red[32];
+  __shared__ __align__(16) float red[4][8];
   const long long row = blockIdx.x;
   float wv[NV][8], v[NV][8], xv[NV][8];
-  load_row<NV>(wv, wy, np);
+  load_row<THREADS, NV>(wv, wy, np);
   pdl_wait();
   pdl_trigger();
   long long src = row;
@@ -165,23 +179,23 @@ layer_norm_residual_kernel(const long long* __restrict__ ids, const TY* __restri
     src = ids[row];
     src = src < 0 ? 0 : (src >= vocab ? vocab - 1 : src);
   }
-  load_row<NV>(v, y + src * ldy, np);
-  if (ids == nullptr) load_row<NV>(xv, (const float*)x + row * np, np);
-  layer_norm_row<NV>(v, wv, n, eps, red);
-  load_row<NV>(wv, w, np);
+  load_row<THREADS, NV>(v, y + src * ldy, np);
+  if (ids == nullptr) load_row<THREADS, NV>(xv, (const float*)x + row * np, np);
+  layer_norm_row<THREADS, NV>(v, wv, n, eps, red[0]);
+  load_row<THREADS, NV>(wv, w, np);
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = (i * 256 + threadIdx.x) * 8;
+    const int c = (i * THREADS + threadIdx.x) * 8;
     if (ids == nullptr) {
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[i][j] += xv[i][j];
     }
     if (c < np) store8(x + row * np + c, v[i]);
   }
-  layer_norm_row<NV>(v, wv, n, eps, red);
+  layer_norm_row<THREADS, NV>(v, wv, n, eps, red[2]);
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = (i * 256 + threadIdx.x) * 8;
+    const int c = (i * THREADS + threadIdx.x) * 8;
     if (c < np) store8(h + row * np + c, v[i]);
   }
 }
@@ -243,8 +257,11 @@ cudaError_t gated_residual_norm(bool f32, float* x, const GatedTerm* terms, int 
 template <typename T, typename TY>
 static cudaError_t launch_layer_norm(const long long* ids, const TY* y, long long ldy, int vocab, const float* wy, float* x, const float* w,
                                      float eps, int rows, int n, int np, T* h, cudaStream_t s) {
-  auto k = np <= 2048 ? layer_norm_residual_kernel<T, TY, 1> : np <= 4096 ? layer_norm_residual_kernel<T, TY, 2> : layer_norm_residual_kernel<T, TY, 4>;
-  return launch_pdl(k, dim3(rows), dim3(256), 0, s, ids, y, ldy, vocab, wy, x, w, eps, n, np, h);
+  auto go = [&](auto k, int threads) { return launch_pdl(k, dim3(rows), dim3(threads), 0, s, ids, y, ldy, vocab, wy, x, w, eps, n, np, h); };
+  if (np <= 1024) return go(layer_norm_residual_kernel<T, TY, 128, 1>, 128);
+  if (np <= 2048) return go(layer_norm_residual_kernel<T, TY, 128, 2>, 128);
+  if (np <= 4096) return go(layer_norm_residual_kernel<T, TY, 256, 2>, 256);
+  return go(layer_norm_residual_kernel<T, TY, 256, 4>, 256);
 }
 
 cudaError_t layer_norm_residual(bool f32, bool y_f32, const long long* ids, const void* y, long long ldy, int vocab, const float* wy, float* x,

@@ -60,7 +60,7 @@ cudaError_t poly_norm(bool f32, bool z_f32, const void* z, long long ldz, const 
                       void* out, long long ldo, cudaStream_t s);
 
 // ------------------------------------------------------------------------------ gemv.cu
-// Matrix-vector products of a decode step, bf16 weights, rows <= 8: out[b, j] = epilogue(sum_k pre(x)[b, k] W[j, k]).
+// Matrix-vector products of a decode step, bf16 weights, rows <= 8 (plain stores: any number, eight at a time; for few outputs): out[b, j] = epilogue(sum_k pre(x)[b, k] W[j, k]).
 enum GemvPre : int {
   PRE_NORM = 0,     // x float, x / rms(x) * w
   PRE_PLAIN = 1,    // x bf16

@@ -8,7 +8,9 @@
 //                   distributed shared memory
 //       decay       a CTA per (head, row) updates its state; the row's last CTA to finish norms and gates the row
 //
-// The state is read before the wait on the kernel in front: nothing but the step before has written it.
+// What the step before has left (states, convolution inputs, stored keys, lengths) and the weights are read before the wait on
+// the kernel in front, the layer's input product. Both recurrences read out what they write without a second pass over the
+// state: (g S + k u^T)^T q = g S^T q + (k . q) u.
 #include <cooperative_groups.h>
 
 #include "mma.cuh"
@@ -50,17 +52,20 @@ struct StateTile {
 #pragma unroll
     for (int i = 0; i < NR; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
   }
-  // this thread's part of S^T x, left in part[grp][columns]
-  __device__ void dot(const float* x, int dp, int vp, float* part) const {
-    float p[4] = {0.f, 0.f, 0.f, 0.f};
+  // this thread's part of S^T x, left in part[grp][columns]; with y, returns the row group's part of x . y
+  __device__ float dot(const float* x, int dp, int vp, float* part, const float* y = nullptr) const {
+    float p[4] = {0.f, 0.f, 0.f, 0.f}, xy = 0.f;
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int d = grp + i * groups;
-      const float xd = on && d < dp ? x[d] : 0.f;
+      const bool in = on && d < dp;
+      const float xd = in ? x[d] : 0.f;
+      if (y) xy += in ? xd * y[d] : 0.f;
 #pragma unroll
       for (int j = 0; j < 4; ++j) p[j] += s[i][j] * xd;
     }
     if (on) *reinterpret_cast<float4*>(part + grp * vp + vi * 4) = make_float4(p[0], p[1], p[2], p[3]);
+    return xy;
   }
   // S <- g S + k u^T
   __device__ void update(float g, const float* k, const float (&u)[4], int dp) {
@@ -87,8 +92,9 @@ __device__ __forceinline__ void sum_parts(const float* part, int groups, int vp,
     t[0] += a.x; t[1] += a.y; t[2] += a.z; t[3] += a.w;
   }
 }
-// floats of dynamic shared memory: q, k (dp), v (vp), partial sums (1024: groups * vp <= THREADS * 4)
-__host__ __device__ constexpr int step_floats(int dp, int vp) { return 2 * dp + vp + THREADS * 4; }
+// floats of dynamic shared memory: q, k (dp), v (vp), two partial sums of up to THREADS * 4 each, the row groups' k . q
+__host__ __device__ constexpr int step_floats(int dp, int vp) { return 2 * dp + vp + 2 * THREADS * 4 + THREADS; }
+constexpr int MAX_CHANNELS = 6 * THREADS;      // q, k and v of one head
 
 template <typename T, typename TZ, int NR>
 __global__ void __launch_bounds__(THREADS)
@@ -96,36 +102,57 @@ delta_step_kernel(const DeltaStep d) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[2][32];
   __shared__ float s_beta, s_g;
+  constexpr int PER = MAX_CHANNELS / THREADS;
   const DeltaInputs& in = d.in;
   const int h = blockIdx.x, row = blockIdx.y, rep = in.heads / in.kv_heads, kvh = h / rep;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int dp = in.dp, vp = in.vp, channels = 2 * in.kv_heads * dp + in.heads * vp;
-  float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part = sm + 2 * dp + vp;
+  const int dp = in.dp, vp = in.vp, channels = 2 * in.kv_heads * dp + in.heads * vp, mine = 2 * dp + vp;
+  float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part_k = sv + vp, *part_q = part_k + THREADS * 4, *part_kq = part_q + THREADS * 4;
   float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * vp;
+  float* ring = in.ring.ptr + row * in.ring.seq_stride;
+  const int pos = in.pos.lens[row];
   StateTile<NR> S;
   S.load(state, dp, vp);
+  auto channel = [&](int c) { return c < dp ? kvh * dp + c : c < 2 * dp ? in.kv_heads * dp + kvh * dp + c - dp : 2 * in.kv_heads * dp + h * vp + c - 2 * dp; };
+  float past[PER], w_now[PER];                     // the convolution without the current token, and its weight
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = tid + i * THREADS;
+    if (c >= mine) break;
+    const int ch = channel(c);
+    w_now[i] = in.conv[(long long)(in.taps - 1) * channels + ch];
+    past[i] = 0.f;
+    for (int t = 1; t < in.taps && t <= pos; ++t)
+      past[i] += in.conv[(long long)(in.taps - 1 - t) * channels + ch] * ring[(long long)((pos - t) % in.taps) * channels + ch];
+  }
+  const float bias = in.dt_bias[h], neg_a = in.neg_a[h];
+  if (pos == 0) S.clear();
   pdl_wait();
   pdl_trigger();
-  const int pos = in.pos.lens[row];
-  if (pos == 0) S.clear();
-  float* ring = in.ring.ptr + row * in.ring.seq_stride;
+  const int col = S.vi * 4;
+  float gate[4], beta_in = 0.f, decay_in = 0.f;
+  if (tid == THREADS - 1) {
+    beta_in = in.ba[row * in.ldba + h];
+    decay_in = in.ba[row * in.ldba + in.a_off + h] + bias;
+  }
   float ss[2] = {0.f, 0.f};
-  for (int c = tid; c < 2 * dp + vp; c += THREADS) {
-    const int ch = c < dp ? kvh * dp + c : c < 2 * dp ? in.kv_heads * dp + kvh * dp + c - dp : 2 * in.kv_heads * dp + h * vp + c - 2 * dp;
-    const float x = zf<TZ>(in.z, row * in.ldz + ch);
-    float a = in.conv[(long long)(in.taps - 1) * channels + ch] * x;
-    for (int i = 1; i < in.taps && i <= pos; ++i)
-      a += in.conv[(long long)(in.taps - 1 - i) * channels + ch] * ring[(long long)((pos - i) % in.taps) * channels + ch];
-    a = silu_exact(a);
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = tid + i * THREADS;
+    if (c >= mine) break;
+    const int ch = channel(c);
+    const float x = zf<TZ>(in.z, row * in.ldz + ch), a = silu_exact(past[i] + w_now[i] * x);
     sm[c] = a;
     if (c < 2 * dp) ss[c >= dp] += a * a;
     if (c >= 2 * dp || h % rep == 0) ring[(long long)(pos % in.taps) * channels + ch] = x;      // one writer per channel
   }
+  if (S.grp == 0) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) gate[j] = zf<TZ>(in.z, row * in.ldz + d.gate_off + (long long)h * vp + col + j);
+  }
   if (tid == THREADS - 1) {
-    const float* ba = in.ba + row * in.ldba;
-    const float a = ba[in.a_off + h] + in.dt_bias[h];
-    s_beta = sigmoidf(ba[h]);
-    s_g = expf(in.neg_a[h] * (a > 20.f ? a : log1pf(expf(a))));
+    s_beta = sigmoidf(beta_in);
+    s_g = expf(neg_a * (decay_in > 20.f ? decay_in : log1pf(expf(decay_in))));
   }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
@@ -133,38 +160,36 @@ delta_step_kernel(const DeltaStep d) {
     if (lane == 0) red[i][warp] = ss[i];
   }
   __syncthreads();
+  S.dot(sk, dp, vp, part_k);
+  const float kq_part = S.dot(sq, dp, vp, part_q, sk);
+  if (S.on && S.vi == 0) part_kq[S.grp] = kq_part;
 #pragma unroll
   for (int i = 0; i < 2; ++i) ss[i] = warp_sum(lane < THREADS / 32 ? red[i][lane] : 0.f);
   const float rq = 1.f / sqrtf(ss[0] + 1e-6f) / sqrtf((float)in.dim), rk = 1.f / sqrtf(ss[1] + 1e-6f), g = s_g;
-  S.dot(sk, dp, vp, part);
   __syncthreads();
+  float u[4] = {0.f, 0.f, 0.f, 0.f}, o[4] = {0.f, 0.f, 0.f, 0.f}, so[1] = {0.f};
   if (S.on) {
-    float t[4], u[4];
-    sum_parts(part, S.groups, vp, S.vi * 4, t);
+    float t[4];
+    sum_parts(part_k, S.groups, vp, col, t);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) u[j] = rk * s_beta * (sv[S.vi * 4 + j] - g * rk * t[j]);
-    S.update(g, sk, u, dp);
-    S.store(state, dp, vp);
+    for (int j = 0; j < 4; ++j) u[j] = rk * s_beta * (sv[col + j] - g * rk * t[j]);
   }
-  __syncthreads();
-  S.dot(sq, dp, vp, part);
-  __syncthreads();
-  float o[4] = {0.f, 0.f, 0.f, 0.f}, so[1] = {0.f};
-  const int col = tid * 4;
-  if (col < vp) {
-    sum_parts(part, S.groups, vp, col, o);
+  if (S.grp == 0) {                                // the first threads read out
+    float t[4], kq = 0.f;
+    sum_parts(part_q, S.groups, vp, col, t);
+    for (int i = 0; i < S.groups; ++i) kq += part_kq[i];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) { o[j] *= rq; so[0] += o[j] * o[j]; }
+    for (int j = 0; j < 4; ++j) { o[j] = rq * (g * t[j] + kq * u[j]); so[0] += o[j] * o[j]; }
   }
-  block_sum<1>(so, red[0]);
-  if (col < vp) {
+  if (vp <= 128) so[0] = warp_sum(so[0]);          // they are lanes of one warp
+  else block_sum<1>(so, red[0]);
+  if (S.grp == 0) {
     const float r = inv_rms(so[0], in.vdim, d.eps);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float gate = zf<TZ>(in.z, row * in.ldz + d.gate_off + (long long)h * vp + col + j);
-      ((T*)d.y)[row * d.ldy + (long long)h * vp + col + j] = from_f<T>(o[j] * r * d.norm[col + j] * silu_exact(gate));
-    }
+    for (int j = 0; j < 4; ++j) ((T*)d.y)[row * d.ldy + (long long)h * vp + col + j] = from_f<T>(o[j] * r * d.norm[col + j] * silu_exact(gate[j]));
   }
+  S.update(g, sk, u, dp);
+  S.store(state, dp, vp);
 }
 
 // ------------------------------------------------------------------------- fixed decay
@@ -173,35 +198,39 @@ __device__ void decay_head(const DecayStep& d, int h, int row, float* sm) {
   __shared__ float red[32];
   __shared__ int s_last;
   const int tid = threadIdx.x, dp = d.dp, vp = d.vp, width = d.heads * vp;
-  float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part = sm + 2 * dp + vp;
+  float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part = sv + vp, *part_kq = part + 2 * THREADS * 4;
   float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * vp;
   StateTile<NR> S;
   S.load(state, dp, vp);
+  if (d.pos.lens[row] == 0) S.clear();
+  const float g = expf(d.log_decay[h]);
   pdl_wait();
   pdl_trigger();
-  if (d.pos.lens[row] == 0) S.clear();
   for (int c = tid; c < 2 * dp + vp; c += THREADS) {
     const int at = c < dp ? d.q_off + h * dp + c : c < 2 * dp ? d.k_off + h * dp + c - dp : d.v_off + h * vp + c - 2 * dp;
     sm[c] = silu_exact(zf<TZ>(d.z, row * d.ldz + at));
   }
   __syncthreads();
-  if (S.on) {
-    const float u[4] = {sv[S.vi * 4], sv[S.vi * 4 + 1], sv[S.vi * 4 + 2], sv[S.vi * 4 + 3]};
-    S.update(expf(d.log_decay[h]), sk, u, dp);
-    S.store(state, dp, vp);
-  }
-  S.dot(sq, dp, vp, part);
+  const float kq_part = S.dot(sq, dp, vp, part, sk);
+  if (S.on && S.vi == 0) part_kq[S.grp] = kq_part;
   __syncthreads();
   float* o = d.o + (long long)row * width;
-  const int col = tid * 4;
-  if (col < vp) {
-    float t[4];
+  const int col = S.vi * 4;
+  if (S.grp == 0) {
+    float t[4], kq = 0.f;
     sum_parts(part, S.groups, vp, col, t);
-    *reinterpret_cast<float4*>(o + h * vp + col) = make_float4(t[0], t[1], t[2], t[3]);
+    for (int i = 0; i < S.groups; ++i) kq += part_kq[i];
+    *reinterpret_cast<float4*>(o + h * vp + col) =
+        make_float4(g * t[0] + kq * sv[col], g * t[1] + kq * sv[col + 1], g * t[2] + kq * sv[col + 2], g * t[3] + kq * sv[col + 3]);
+    __threadfence();
   }
-  __threadfence();
   __syncthreads();
   if (tid == 0) s_last = atomicAdd(d.done + row, 1) == d.heads - 1;
+  if (S.on) {
+    const float u[4] = {sv[col], sv[col + 1], sv[col + 2], sv[col + 3]};
+    S.update(g, sk, u, dp);
+    S.store(state, dp, vp);
+  }
   __syncthreads();
   if (!s_last) return;
   if (tid == 0) d.done[row] = 0;
@@ -245,8 +274,6 @@ __device__ void window_group(const WindowAttn& d, int group, int row, uint8_t* s
     const int per = (DP - d.dp) / 8, r = i / per;
     *reinterpret_cast<uint4*>(sQ + r * LD + d.dp + (i - r * per) * 8) = make_uint4(0, 0, 0, 0);
   }
-  pdl_wait();
-  pdl_trigger();
   const int pos = d.pos.lens[row];
   const KeyRange kr = split_keys(pos, d.window, splits, split, KT);
   const bool any = kr.begin < kr.end;
@@ -278,6 +305,10 @@ __device__ void window_group(const WindowAttn& d, int group, int row, uint8_t* s
   if (any) {
     load_tile(kr.begin);
     for (int i = tid; i < d.dims / 2; i += THREADS) s_cs[i] = turn_of(pos, d.freq, i, d.dims / 2);
+  }
+  pdl_wait();
+  pdl_trigger();
+  if (any) {
     __syncthreads();
     const TZ* z = (const TZ*)d.z + row * d.ldz;
     const int pairs = d.dp / 2;
@@ -513,7 +544,7 @@ cudaError_t launch_parallel_rows(const WindowAttn& left, const DecayStep& right,
 
 }  // namespace
 
-bool delta_step_supported(int dp, int vp) { return !(dp & 7) && !(vp & 7) && state_rows(dp, vp) > 0 && dp <= 2048; }
+bool delta_step_supported(int dp, int vp) { return !(dp & 7) && !(vp & 7) && state_rows(dp, vp) > 0 && 2 * dp + vp <= MAX_CHANNELS; }
 bool decay_step_supported(int dp, int vp) { return delta_step_supported(dp, vp); }
 bool window_step_supported(bool f32, int dp) { return !f32 && dp > 0 && dp <= 256 && !(dp & 7); }
 

@@ -20,6 +20,7 @@ _S = load_serving_extension()
 BF16 = torch.bfloat16
 ABSORB_ROWS = 8          # portions up to this many tokens run on absorbed queries (weights dominate), longer ones expand
 CHUNK_ROWS = 16          # portions above this many tokens run their recurrences in chunks, shorter ones token by token
+FEW_OUTPUTS = 64         # products with up to this many outputs leave most SMs without a GEMM tile: eight rows at a time instead
 SPLIT_KEYS = 64          # keys per tile of the tensor-core attention over stored entries
 
 
@@ -41,7 +42,10 @@ def linear_rows(h, w, out_dtype=None):
     """h (R, K) @ w (N, K)^T; `out_dtype` float32 keeps the accumulator's precision."""
     if h.dtype == BF16:
         out = torch.empty(h.shape[0], w.shape[0], dtype=out_dtype or BF16, device=h.device)
-        _S.gemm(h, w, out)
+        if w.shape[0] <= FEW_OUTPUTS:
+            _S.gemv_plain(h, w, out)
+        else:
+            _S.gemm(h, w, out)
         return out
     before = torch.get_float32_matmul_precision()
     if before == "highest":
