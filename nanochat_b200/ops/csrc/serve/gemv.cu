@@ -435,7 +435,8 @@ cudaError_t gemv(const GemvDesc& d, int pre, int epi, cudaStream_t s) {
   a.W = (const bf16*)d.W; a.ldw = d.ldw; a.B = d.rows; a.N = d.N; a.K = d.K; a.epi = epi; a.accumulate = d.accumulate;
   a.out = d.out; a.ldo = d.ldo; a.resid = d.resid; a.ldr = d.ldr; a.g = d.g; a.ldg = d.ldg; a.bias = d.bias;
   a.mult = d.mult; a.extra = d.extra; a.h_out = (bf16*)d.h_out; a.ldh = d.ldh; a.next = d.next;
-  const bool wide = d.N >= 148 * 32;               // enough outputs for two tiles per CTA: the rows are read half as often
+  // enough outputs, or groups of rows, for two tiles per CTA: the rows are read half as often
+  const bool wide = d.N >= 148 * 32 || (d.rows > ROWS && d.N > 16);
   a.n_blocks = (d.N + (wide ? 31 : 15)) / (wide ? 32 : 16);
   int grid = a.n_blocks;
   if (d.store) { a.store = *d.store; grid += d.rows; }

@@ -11,13 +11,15 @@
 //                 R = V - decayed K S,  U = T R        delta rule;   U = V  fixed decay
 //                 O = decayed Q S + A U
 //                 S = decayed S + K^T (decayed U)
-//              One warp copies whole chunks into shared memory, eight follow the state from chunk to chunk, four more
+//              One warp copies whole chunks into shared memory, four follow the state from chunk to chunk, four more
 //              read it out behind them.
 //   norm_gate         RMS norm and gate of what a recurrence read out, and the convolution's last inputs
 //
-// Exactness: the products run on bf16 operands, so every operand that is a float (the state, T, A, U, R) enters as the sum
-// of two bf16 values, and what scales rows (inverse norms, decays) is applied to accumulators, not to operands: keys,
-// queries and values are the bf16 activations themselves. The state is float from chunk to chunk.
+// Exactness: the products run on bf16 operands, so every operand that is a float (S, T, A, U, R) enters as the sum of two bf16
+// values, and what scales rows (inverse norms, decays) is applied to accumulators, not to operands: keys, queries and values are
+// the bf16 activations themselves. The state is float from chunk to chunk, and a read-out that nearly cancels keeps its digits.
+#include <type_traits>
+
 #include "mma.cuh"
 
 namespace nc {
@@ -26,6 +28,24 @@ namespace serve {
 namespace {
 
 template <typename T> __device__ __forceinline__ float silu_of(float v) { return v * sigmoid_of<T>(v); }
+
+// four neighbouring values as they lie in memory
+template <typename T> struct Raw4;
+template <> struct Raw4<float> {
+  float4 a;
+  __device__ void load(const float* p) { a = *reinterpret_cast<const float4*>(p); }
+  __device__ void set(const float (&f)[4]) { a = make_float4(f[0], f[1], f[2], f[3]); }
+  __device__ void get(float (&f)[4]) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; }
+};
+template <> struct Raw4<bf16> {
+  uint2 u;
+  __device__ void load(const bf16* p) { u = *reinterpret_cast<const uint2*>(p); }
+  __device__ void set(const float (&f)[4]) { u = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3])); }
+  __device__ void get(float (&f)[4]) const {
+    const float2 a = unpack_bf16(u.x), b = unpack_bf16(u.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+};
 
 __device__ __forceinline__ void load4(const float* p, float (&f)[4]) {
   const float4 a = *reinterpret_cast<const float4*>(p);
@@ -71,13 +91,13 @@ struct Tiles {
 __host__ __device__ constexpr size_t chunk_bytes(bool delta) { return (size_t)(delta ? 4 : 2) * MAT * 2 + SCALARS * 4; }
 
 // ---------------------------------------------------------------------------- prepare
-constexpr int PREP_TOKENS = 4;         // tokens a warp walks through
+constexpr int PREP_TOKENS = 8;         // tokens a warp walks through
 
 // grid (token groups of a sequence, ceil(jobs / 4), sequences), a warp per job: query heads, key heads, value heads.
 // TAPS > 0: at most TAPS taps, the inputs stay in registers; 0: any number, re-read; -1: no convolution and no norms
 // (fixed decay). TILES: out is laid out as Tiles, otherwise rows x channels.
 template <typename T, typename TZ, int TAPS, bool TILES>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, sizeof(TZ) == 2 ? 6 : 4)
 prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ norms, float* __restrict__ beta_g) {
   const int lane = threadIdx.x & 31, job = blockIdx.y * 4 + (threadIdx.x >> 5);
   const int G = d.kv_heads, H = d.heads, per_seq = d.pos.per_seq, seq = blockIdx.z;
@@ -113,21 +133,19 @@ prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ nor
   const bool inside = t0 >= BACK && n == PREP_TOKENS;   // every input is a row of this portion
   for (int c = lane * 4; c < columns; c += 128) {
     const int ch = ch0 + c;
-    float w[BACK + 1][4], x[PREP_TOKENS + BACK][4];     // x[BACK + t]: token t of the group
+    float w[BACK + 1][4];
+    Raw4<TZ> x[PREP_TOKENS + BACK];                     // x[BACK + t]: token t of the group (the ring holds what z held)
     const bool in = c < size;
     if (TAPS != 0 && inside && in) {
       const TZ* src = (const TZ*)d.z + (row0 + t0 - BACK) * d.ldz + ch;
 #pragma unroll
-      for (int t = 0; t < PREP_TOKENS + BACK; ++t) load4(src + t * d.ldz, x[t]);
+      for (int t = 0; t < PREP_TOKENS + BACK; ++t) x[t].load(src + t * d.ldz);
     } else {
 #pragma unroll
       for (int t = 0; t < PREP_TOKENS + BACK; ++t) {
-        if (in && TAPS != 0 && t - BACK < n && (t >= BACK || BACK - t < d.taps)) {
-          fetch(t0 + t - BACK, ch, x[t]);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 4; ++j) x[t][j] = 0.f;
-        }
+        float f[4] = {0.f, 0.f, 0.f, 0.f};
+        if (in && TAPS != 0 && t - BACK < n && (t >= BACK || BACK - t < d.taps)) fetch(t0 + t - BACK, ch, f);
+        x[t].set(f);
       }
     }
     if (TAPS > 0) {
@@ -148,9 +166,12 @@ prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ nor
       float a[4] = {0.f, 0.f, 0.f, 0.f};
       if (TAPS > 0) {
 #pragma unroll
-        for (int i = 0; i <= BACK; ++i)
+        for (int i = 0; i <= BACK; ++i) {
+          float f[4];
+          x[BACK + t - i].get(f);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) a[j] += w[i][j] * x[BACK + t - i][j];
+          for (int j = 0; j < 4; ++j) a[j] += w[i][j] * f[j];
+        }
       } else if (TAPS == 0) {
         for (int i = 0; in && t < n && i < d.taps; ++i) {
           float wi[4], xi[4];
@@ -160,8 +181,7 @@ prepare_kernel(const DeltaInputs d, T* __restrict__ out, float* __restrict__ nor
           for (int j = 0; j < 4; ++j) a[j] += wi[j] * xi[j];
         }
       } else {
-#pragma unroll
-        for (int j = 0; j < 4; ++j) a[j] = x[t][j];
+        x[t].get(a);
       }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
@@ -485,15 +505,15 @@ struct ScanSmem {
   static_assert(STAGE % 16 == 0 && TOTAL <= 227 * 1024, "stages must fit shared memory");
 };
 
-constexpr int SCAN_THREADS = 13 * 32;
-// grid (ceil(vp / 16), heads, sequences): warps 0..7 own the state, 8..11 the output, 12 copies. The state warps split tokens as
-// 16 tokens x 8 columns (warp & 3, warp >> 2), the state as 16 rows x 16 columns (D = 128) or 16 x 8 (D = 64).
+constexpr int SCAN_THREADS = 9 * 32;
+// grid (ceil(vp / 16), heads, sequences): warps 0..3 own the state (16 D / 64 rows each), 4..7 the output, 8 copies. Shared
+// memory bandwidth and the latency of its loads set the pace, so a product requests all its fragments before the first use.
 // A wait that runs out raises the status and the kernel runs on without waiting, so that no barrier is left short.
 template <bool DELTA, int D>
 __global__ void __launch_bounds__(SCAN_THREADS)
 chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* status) {
   using M = ScanSmem<DELTA, D>;
-  constexpr int LD = M::LD, NT = D / 64;                         // NT: 8-column tiles of the state a warp holds
+  constexpr int LD = M::LD, MT = D / 64;                         // MT: 16-row tiles of the state a warp holds
   extern __shared__ __align__(128) uint8_t smem[];
   const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, kvh = h / (r.heads / r.kv_heads), v0 = slice * VS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -506,31 +526,82 @@ chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* 
   uint64_t *u_ready = s_read + 1, *u_read = u_ready + 2;             // [2] U is there, has been read, by chunk parity
   volatile int* abort_flag = reinterpret_cast<volatile int*>(u_read + 2);
   if (tid == 0) {
-    for (int i = 0; i < STAGES; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 12); }
-    mbar_init(s_ready, 8); mbar_init(s_read, 4);
-    for (int i = 0; i < 2; ++i) { mbar_init(&u_ready[i], 8); mbar_init(&u_read[i], 4); }
+    for (int i = 0; i < STAGES; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); }
+    mbar_init(s_ready, 4); mbar_init(s_read, 4);
+    for (int i = 0; i < 2; ++i) { mbar_init(&u_ready[i], 4); mbar_init(&u_read[i], 4); }
     *abort_flag = 0;
     fence_mbar_init();
   }
   __syncthreads();
   auto wait = [&](uint64_t* bar, int n, int code) { mbar_wait(bar, n & 1, abort_flag, status, code, 0x5c0); };    // its n-th completion
   auto arrive = [&](uint64_t* bar) { __syncwarp(); if (lane == 0) mbar_arrive(bar); };
-  auto state_sync = [] { asm volatile("bar.sync 1, 256;" ::: "memory"); };
+  auto state_sync = [] { asm volatile("bar.sync 1, 128;" ::: "memory"); };
   const int band = warp & 3, mrow = band * 16;                   // this warp's 16 tokens of a chunk
   const int ri = mrow + (lane >> 2), ci = (lane & 3) * 2;        // first row and column of its accumulators
   auto a_frag = [&](uint32_t (&a)[4], const bf16* tile, int k) { ldmatrix4(a, tile + (mrow + (lane & 15)) * LD + k + (lane >> 4) * 8); };
   auto tri_frag = [&](uint32_t (&a)[4], const bf16* mat, int k) { ldmatrix4(a, mat + band_at(band) + (lane & 15) * band_pitch(band) + k + (lane >> 4) * 8); };
-  // 16 rows of a 16-column operand: both column tiles of one part, or one column tile of both parts (high in b[0..1])
   auto b_frag = [&](uint32_t (&b)[4], const bf16* rows, int k) { ldmatrix4_trans(b, rows + (k + (lane & 15)) * LV + (lane >> 4) * 8); };
-  auto b_parts = [&](uint32_t (&b)[4], const bf16* rows, int low, int column, int k) {
-    ldmatrix4_trans(b, rows + (lane >> 4) * low + (k + (lane & 15)) * LV + column);
-  };
   auto add = [](float (&a)[4], const float (&b)[4]) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) a[e] += b[e];
   };
+  // 16 tokens x 16 columns of X S, X the chunk's queries or keys
+  auto times_state = [&](float (&o)[2][4], const bf16* rows, const bf16* s) {
+    constexpr int HALF = D / 32;                                 // k-steps in flight
+    float lo[2][4] = {};
+#pragma unroll
+    for (int k0 = 0; k0 < D; k0 += HALF * 16) {
+      uint32_t a[HALF][4], bh[HALF][4], bl[HALF][4];
+#pragma unroll
+      for (int k = 0; k < HALF; ++k) {
+        a_frag(a[k], rows, k0 + k * 16);
+        b_frag(bh[k], s, k0 + k * 16);
+        b_frag(bl[k], s + M::S_PART, k0 + k * 16);
+      }
+#pragma unroll
+      for (int k = 0; k < HALF; ++k) {
+        mma_16816(o[0], a[k], bh[k][0], bh[k][1]);
+        mma_16816(o[1], a[k], bh[k][2], bh[k][3]);
+        mma_16816(lo[0], a[k], bl[k][0], bl[k][1]);
+        mma_16816(lo[1], a[k], bl[k][2], bl[k][3]);
+      }
+    }
+    add(o[0], lo[0]);
+    add(o[1], lo[1]);
+  };
+  // o += M X for a lower triangular M in two parts and a 64 x 16 X in one or two
+  auto times_lower = [&](float (&o)[2][4], const bf16* m, const bf16* x, auto two_parts) {
+    constexpr bool TWO = decltype(two_parts)::value;
+    uint32_t ah[4][4], al[4][4], bh[4][4], bl[TWO ? 4 : 1][4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (k > band) break;
+      tri_frag(ah[k], m, k * 16);
+      b_frag(bh[k], x, k * 16);
+      tri_frag(al[k], m + MAT, k * 16);
+      if constexpr (TWO) b_frag(bl[k], x + M::PART, k * 16);
+    }
+    float p[2][4] = {}, q[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (k > band) break;
+      mma_16816(o[0], ah[k], bh[k][0], bh[k][1]);
+      mma_16816(o[1], ah[k], bh[k][2], bh[k][3]);
+      mma_16816(p[0], al[k], bh[k][0], bh[k][1]);
+      mma_16816(p[1], al[k], bh[k][2], bh[k][3]);
+      if constexpr (TWO) {
+        mma_16816(q[0], ah[k], bl[k][0], bl[k][1]);
+        mma_16816(q[1], ah[k], bl[k][2], bl[k][3]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t) {
+      add(o[t], p[t]);
+      if constexpr (TWO) add(o[t], q[t]);
+    }
+  };
 
-  if (warp == 12) {                                              // ---- copies
+  if (warp == 8) {                                               // ---- copies
     if (lane == 0) {
       const bf16* qk = (const bf16*)r.act + ((long long)seq * chunks * r.kv_heads + kvh) * tiles.qk_unit;
       const bf16* v = (const bf16*)r.act + tiles.v_base + (((long long)seq * chunks * r.heads + h) * tiles.slices + slice) * tiles.v_unit;
@@ -546,29 +617,29 @@ chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* 
         bulk_load_1d(st + M::V, v + (long long)c * r.heads * tiles.slices * tiles.v_unit, M::V_BYTES, &full[b]);
       }
     }
-  } else if (warp < 8) {                                         // ---- state
-    const int nt = warp >> 2, j = nt * 8 + ci;                   // this warp's columns of the tokens' operands
-    const int d0 = (NT == 2 ? warp : warp & 3) * 16, c0 = NT == 2 ? 0 : nt * 8;      // its part of the state
+  } else if (warp < 4) {                                         // ---- state
     bf16* sW = reinterpret_cast<bf16*>(smem + M::W);
     bf16* sR = reinterpret_cast<bf16*>(smem + M::R);
+    bf16* sS = reinterpret_cast<bf16*>(smem + M::S);
     float* state = r.state.ptr + seq * r.state.seq_stride + (long long)h * r.dp * r.vp + v0;
     const bool fresh = r.pos.lens[seq] == 0;
-    float st[NT][4] = {};
-    auto each_state = [&](auto f) {                              // f(row of the state, column, tile, first element)
+    float st[MT][2][4] = {};
+    auto each_state = [&](auto f) {                              // f(row of the state, column, tile, column tile, first element)
 #pragma unroll
-      for (int t = 0; t < NT; ++t)
+      for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int half = 0; half < 2; ++half) f(d0 + (lane >> 2) + half * 8, c0 + t * 8 + ci, t, half * 2);
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) f((warp + 4 * i) * 16 + (lane >> 2) + half * 8, t * 8 + ci, i, t, half * 2);
     };
-    bf16* sS = reinterpret_cast<bf16*>(smem + M::S);
     auto publish_state = [&] {
-      each_state([&](int d, int v, int t, int e) { store_split(sS + d * LV + v, sS + M::S_PART + d * LV + v, st[t][e], st[t][e + 1]); });
+      each_state([&](int d, int v, int i, int t, int e) { store_split(sS + d * LV + v, sS + M::S_PART + d * LV + v, st[i][t][e], st[i][t][e + 1]); });
       arrive(s_ready);
     };
-    each_state([&](int d, int v, int t, int e) {
+    each_state([&](int d, int v, int i, int t, int e) {
       const bool in = !fresh && d < r.dp && v0 + v < r.vp;
       const float2 x = in ? *reinterpret_cast<const float2*>(state + (long long)d * r.vp + v) : make_float2(0.f, 0.f);
-      st[t][e] = x.x; st[t][e + 1] = x.y;
+      st[i][t][e] = x.x; st[i][t][e + 1] = x.y;
     });
     publish_state();
     state_sync();
@@ -578,150 +649,119 @@ chunk_scan_kernel(const Recurrence r, const uint8_t* __restrict__ scratch, int* 
       const bf16 *sk = reinterpret_cast<const bf16*>(stg + M::K), *sv = reinterpret_cast<const bf16*>(stg + M::V);
       const float* sc = reinterpret_cast<const float*>(stg + M::SC);
       wait(&full[stage], c / STAGES, ST_WAIT_FULL);
-      const float g = sc[3 * CH], w[2] = {sc[2 * CH + ri], sc[2 * CH + ri + 8]};
-      float2 v[2];
+      uint32_t kt[MT][4][4];                                     // K^T: rows are the head's dimensions, k the tokens
 #pragma unroll
-      for (int half = 0; half < 2; ++half) v[half] = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + (ri + half * 8) * LV + j));
+      for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          ldmatrix4_trans(kt[i][k], sk + (k * 16 + (lane & 7) + (lane >> 4) * 8) * LD + (warp + 4 * i) * 16 + ((lane >> 3) & 1) * 8);
+      const float g = sc[3 * CH], w[2] = {sc[2 * CH + ri], sc[2 * CH + ri + 8]};
+      float2 v[2][2];
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) v[t][half] = unpack_bf16(*reinterpret_cast<const uint32_t*>(sv + (ri + half * 8) * LV + t * 8 + ci));
       if constexpr (DELTA) {
         bf16* sU = reinterpret_cast<bf16*>(smem + M::U) + (c & 1) * 2 * M::PART;
-        const bf16* sT = reinterpret_cast<const bf16*>(stg + M::A) + 2 * MAT;
         const float f[2] = {sc[ri], sc[ri + 8]};
-        float x[2][4] = {}, y[2][4] = {};                        // even and odd steps: shorter chains
+        float x[2][4] = {};
+        times_state(x, sk, sS);
 #pragma unroll
-        for (int k = 0; k < D; k += 16) {                        // K S
-          uint32_t a[4], p[4];
-          a_frag(a, sk, k);
-          b_parts(p, sS, M::S_PART, nt * 8, k);
-          mma_16816(x[(k >> 4) & 1], a, p[0], p[1]);
-          mma_16816(y[(k >> 4) & 1], a, p[2], p[3]);
-        }
-        add(x[0], x[1]);
-        add(y[0], y[1]);
-        add(x[0], y[0]);
+        for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int i = ri + half * 8;
-          store_split(sR + i * LV + j, sR + M::PART + i * LV + j, v[half].x - f[half] * x[0][half * 2], v[half].y - f[half] * x[0][half * 2 + 1]);
-        }
+          for (int half = 0; half < 2; ++half) {
+            const int at = (ri + half * 8) * LV + t * 8 + ci;
+            store_split(sR + at, sR + M::PART + at, v[t][half].x - f[half] * x[t][half * 2], v[t][half].y - f[half] * x[t][half * 2 + 1]);
+          }
         state_sync();
-        float u[3][4] = {};
-#pragma unroll
-        for (int k = 0; k < CH; k += 16) {                       // U = T R
-          if (k > mrow) break;
-          uint32_t th[4], tl[4], p[4];
-          tri_frag(th, sT, k);
-          tri_frag(tl, sT + MAT, k);
-          b_parts(p, sR, M::PART, nt * 8, k);
-          mma_16816(u[0], th, p[0], p[1]);
-          mma_16816(u[1], tl, p[0], p[1]);
-          mma_16816(u[2], th, p[2], p[3]);
-        }
-        add(u[0], u[1]);
-        add(u[0], u[2]);
+        float u[2][4] = {};
+        times_lower(u, reinterpret_cast<const bf16*>(stg + M::A) + 2 * MAT, sR, std::true_type{});
         if (c >= 2) wait(&u_read[c & 1], (c >> 1) - 1, ST_WAIT_PEER);      // chunk c - 2 has been read out of this buffer
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int i = ri + half * 8;
-          store_split(sW + i * LV + j, sW + M::PART + i * LV + j, u[0][half * 2] * w[half], u[0][half * 2 + 1] * w[half]);
-          store_split(sU + i * LV + j, sU + M::PART + i * LV + j, u[0][half * 2], u[0][half * 2 + 1]);
-        }
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int at = (ri + half * 8) * LV + t * 8 + ci;
+            store_split(sW + at, sW + M::PART + at, u[t][half * 2] * w[half], u[t][half * 2 + 1] * w[half]);
+            store_split(sU + at, sU + M::PART + at, u[t][half * 2], u[t][half * 2 + 1]);
+          }
         arrive(&u_ready[c & 1]);
       } else {
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int i = ri + half * 8;
-          store_split(sW + i * LV + j, sW + M::PART + i * LV + j, v[half].x * w[half], v[half].y * w[half]);
-        }
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int at = (ri + half * 8) * LV + t * 8 + ci;
+            store_split(sW + at, sW + M::PART + at, v[t][half].x * w[half], v[t][half].y * w[half]);
+          }
       }
       state_sync();
-      float lo[NT][4] = {};
+      uint32_t wh[4][4], wl[4][4];
 #pragma unroll
-      for (int t = 0; t < NT; ++t)                               // S = decayed S + K^T W
-#pragma unroll
-        for (int e = 0; e < 4; ++e) st[t][e] *= g;
-#pragma unroll
-      for (int k = 0; k < CH; k += 16) {
-        uint32_t a[4];                                           // K^T: rows are the head's dimensions, k the tokens
-        ldmatrix4_trans(a, sk + (k + (lane & 7) + (lane >> 4) * 8) * LD + d0 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-        for (int t = 0; t < NT; ++t) {
-          uint32_t p[4];
-          b_parts(p, sW, M::PART, c0 + t * 8, k);
-          mma_16816(st[t], a, p[0], p[1]);
-          mma_16816(lo[t], a, p[2], p[3]);
-        }
+      for (int k = 0; k < 4; ++k) {
+        b_frag(wh[k], sW, k * 16);
+        b_frag(wl[k], sW + M::PART, k * 16);
       }
-#pragma unroll
-      for (int t = 0; t < NT; ++t) add(st[t], lo[t]);
       arrive(&empty[stage]);
+      float lo[MT][2][4] = {};
+#pragma unroll
+      for (int i = 0; i < MT; ++i)                               // S = decayed S + K^T W
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) st[i][t][e] *= g;
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          mma_16816(st[i][0], kt[i][k], wh[k][0], wh[k][1]);
+          mma_16816(st[i][1], kt[i][k], wh[k][2], wh[k][3]);
+          mma_16816(lo[i][0], kt[i][k], wl[k][0], wl[k][1]);
+          mma_16816(lo[i][1], kt[i][k], wl[k][2], wl[k][3]);
+        }
+#pragma unroll
+      for (int i = 0; i < MT; ++i) { add(st[i][0], lo[i][0]); add(st[i][1], lo[i][1]); }
       if (c + 1 < chunks) {
         wait(s_read, c, ST_WAIT_PEER);
         publish_state();
         state_sync();
       }
     }
-    each_state([&](int d, int v, int t, int e) {
-      if (d < r.dp && v0 + v < r.vp) *reinterpret_cast<float2*>(state + (long long)d * r.vp + v) = make_float2(st[t][e], st[t][e + 1]);
+    each_state([&](int d, int v, int i, int t, int e) {
+      if (d < r.dp && v0 + v < r.vp) *reinterpret_cast<float2*>(state + (long long)d * r.vp + v) = make_float2(st[i][t][e], st[i][t][e + 1]);
     });
   } else {                                                       // ---- output
     for (int c = 0; c < chunks; ++c) {
       const int stage = c % STAGES;
       const uint8_t* stg = smem + stage * M::STAGE;
       const float* sc = reinterpret_cast<const float*>(stg + M::SC);
-      const bf16 *sq = reinterpret_cast<const bf16*>(stg + M::Q), *sA = reinterpret_cast<const bf16*>(stg + M::A);
-      const bf16* sS = reinterpret_cast<const bf16*>(smem + M::S);
-      const bf16* sU = DELTA ? reinterpret_cast<const bf16*>(smem + M::U) + (c & 1) * 2 * M::PART : reinterpret_cast<const bf16*>(stg + M::V);
       wait(&full[stage], c / STAGES, ST_WAIT_FULL);
       wait(s_ready, c, ST_WAIT_PEER);
-      float o[2][4] = {}, p[2][4] = {};
-#pragma unroll
-      for (int k = 0; k < D; k += 16) {                          // Q S
-        uint32_t a[4], bh[4], bl[4];
-        a_frag(a, sq, k);
-        b_frag(bh, sS, k);
-        b_frag(bl, sS + M::S_PART, k);
-        mma_16816(o[0], a, bh[0], bh[1]);
-        mma_16816(o[1], a, bh[2], bh[3]);
-        mma_16816(p[0], a, bl[0], bl[1]);
-        mma_16816(p[1], a, bl[2], bl[3]);
-      }
+      float o[2][4] = {};
+      times_state(o, reinterpret_cast<const bf16*>(stg + M::Q), reinterpret_cast<const bf16*>(smem + M::S));
       arrive(s_read);
-      const float q0 = sc[CH + ri], q1 = sc[CH + ri + 8];
+      const float q[2] = {sc[CH + ri], sc[CH + ri + 8]};
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { o[t][e] = (o[t][e] + p[t][e]) * (e < 2 ? q0 : q1); p[t][e] = 0.f; }
-      if (DELTA) wait(&u_ready[c & 1], c >> 1, ST_WAIT_PEER);
-#pragma unroll
-      for (int k = 0; k < CH; k += 16) {                         // + A U
-        if (k > mrow) break;
-        uint32_t ah[4], al[4], uh[4];
-        tri_frag(ah, sA, k);
-        tri_frag(al, sA + MAT, k);
-        b_frag(uh, sU, k);
-        mma_16816(o[0], ah, uh[0], uh[1]);
-        mma_16816(o[1], ah, uh[2], uh[3]);
-        mma_16816(p[0], al, uh[0], uh[1]);
-        mma_16816(p[1], al, uh[2], uh[3]);
-        if constexpr (DELTA) {
-          uint32_t ul[4];
-          b_frag(ul, sU + M::PART, k);
-          mma_16816(o[0], ah, ul[0], ul[1]);
-          mma_16816(o[1], ah, ul[2], ul[3]);
-        }
+        for (int e = 0; e < 4; ++e) o[t][e] *= q[e >> 1];
+      const bf16* sA = reinterpret_cast<const bf16*>(stg + M::A);
+      if constexpr (DELTA) {
+        wait(&u_ready[c & 1], c >> 1, ST_WAIT_PEER);
+        times_lower(o, sA, reinterpret_cast<const bf16*>(smem + M::U) + (c & 1) * 2 * M::PART, std::true_type{});
+        arrive(&u_read[c & 1]);
+      } else {
+        times_lower(o, sA, reinterpret_cast<const bf16*>(stg + M::V), std::false_type{});
       }
       arrive(&empty[stage]);
-      if (DELTA) arrive(&u_read[c & 1]);
       bf16* out = (bf16*)r.o + ((long long)seq * T + c * CH) * r.ldo + (long long)h * r.vp + v0;
 #pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        add(o[t], p[t]);
+      for (int t = 0; t < 2; ++t)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int i = ri + half * 8, j = t * 8 + ci;
           if (c * CH + i < T && v0 + j < r.vp) *reinterpret_cast<uint32_t*>(out + i * r.ldo + j) = pack_bf16(o[t][half * 2], o[t][half * 2 + 1]);
         }
-      }
     }
   }
   __syncthreads();

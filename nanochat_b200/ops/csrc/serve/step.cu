@@ -1,7 +1,8 @@
 // One token per row through the mixers of recurrent.cu and window.cu, from the projections to what the output product
 // reads.
 //
-//   delta_step      a CTA per (head, row): convolution, unit norms, step size and decay, state, norm and gate
+//   delta_step      a cluster per (head, row), each CTA with a part of the value columns: convolution, unit norms, step size and
+//                   decay, state, norm and gate
 //   parallel_step   window attention and fixed-decay heads side by side in one grid of clusters
 //       attention   a cluster per (16 query heads of a key head, row) splits the window's keys; the CTA that covers the
 //                   newest key takes it from the projection and appends it to the store; the partial results meet in
@@ -28,14 +29,14 @@ constexpr int MAX_NR = 32;               // state rows a thread holds, four colu
 __device__ __forceinline__ float silu_exact(float v) { return v * sigmoidf(v); }
 template <typename TZ> __device__ __forceinline__ float zf(const void* z, long long i) { return to_f(((const TZ*)z)[i]); }
 
-// A state of dp x vp floats over the block: thread (column group vi, row group grp) holds rows grp, grp + groups, ... of
-// four columns.
+// A state of dp x vp floats (rows `pitch` apart in memory) over the block: thread (column group vi, row group grp) holds rows
+// grp, grp + groups, ... of four columns.
 template <int NR>
 struct StateTile {
   float s[NR][4];
   int vi, grp, groups;
   bool on;
-  __device__ void load(const float* st, int dp, int vp) {
+  __device__ void load(const float* st, int dp, int vp, int pitch) {
     const int vt = vp / 4;
     groups = THREADS / vt;
     vi = threadIdx.x % vt;
@@ -44,7 +45,7 @@ struct StateTile {
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int d = grp + i * groups;
-      const float4 v = on && d < dp ? *reinterpret_cast<const float4*>(st + (long long)d * vp + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 v = on && d < dp ? *reinterpret_cast<const float4*>(st + (long long)d * pitch + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
       s[i][0] = v.x; s[i][1] = v.y; s[i][2] = v.z; s[i][3] = v.w;
     }
   }
@@ -77,11 +78,11 @@ struct StateTile {
       for (int j = 0; j < 4; ++j) s[i][j] = g * s[i][j] + kd * u[j];
     }
   }
-  __device__ void store(float* st, int dp, int vp) const {
+  __device__ void store(float* st, int dp, int pitch) const {
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int d = grp + i * groups;
-      if (on && d < dp) *reinterpret_cast<float4*>(st + (long long)d * vp + vi * 4) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
+      if (on && d < dp) *reinterpret_cast<float4*>(st + (long long)d * pitch + vi * 4) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
     }
   }
 };
@@ -96,24 +97,26 @@ __device__ __forceinline__ void sum_parts(const float* part, int groups, int vp,
 __host__ __device__ constexpr int step_floats(int dp, int vp) { return 2 * dp + vp + 2 * THREADS * 4 + THREADS; }
 constexpr int MAX_CHANNELS = 6 * THREADS;      // q, k and v of one head
 
+// grid (ranks, heads, rows) in clusters of `ranks` CTAs: each has vp / ranks of the head's value columns
 template <typename T, typename TZ, int NR>
 __global__ void __launch_bounds__(THREADS)
 delta_step_kernel(const DeltaStep d) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[2][32];
-  __shared__ float s_beta, s_g;
+  __shared__ float s_beta, s_g, s_sum;
   constexpr int PER = MAX_CHANNELS / THREADS;
   const DeltaInputs& in = d.in;
-  const int h = blockIdx.x, row = blockIdx.y, rep = in.heads / in.kv_heads, kvh = h / rep;
+  const int rank = blockIdx.x, ranks = gridDim.x, h = blockIdx.y, row = blockIdx.z, rep = in.heads / in.kv_heads, kvh = h / rep;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int dp = in.dp, vp = in.vp, channels = 2 * in.kv_heads * dp + in.heads * vp, mine = 2 * dp + vp;
+  const int dp = in.dp, vp = in.vp / ranks, channels = 2 * in.kv_heads * dp + in.heads * in.vp, mine = 2 * dp + vp;
+  const int v_at = h * in.vp + rank * vp;          // this CTA's first value column among all heads'
   float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part_k = sv + vp, *part_q = part_k + THREADS * 4, *part_kq = part_q + THREADS * 4;
-  float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * vp;
+  float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * in.vp + rank * vp;
   float* ring = in.ring.ptr + row * in.ring.seq_stride;
   const int pos = in.pos.lens[row];
   StateTile<NR> S;
-  S.load(state, dp, vp);
-  auto channel = [&](int c) { return c < dp ? kvh * dp + c : c < 2 * dp ? in.kv_heads * dp + kvh * dp + c - dp : 2 * in.kv_heads * dp + h * vp + c - 2 * dp; };
+  S.load(state, dp, vp, in.vp);
+  auto channel = [&](int c) { return c < dp ? kvh * dp + c : c < 2 * dp ? in.kv_heads * dp + kvh * dp + c - dp : 2 * in.kv_heads * dp + v_at + c - 2 * dp; };
   float past[PER], w_now[PER];                     // the convolution without the current token, and its weight
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
@@ -127,9 +130,12 @@ delta_step_kernel(const DeltaStep d) {
   }
   const float bias = in.dt_bias[h], neg_a = in.neg_a[h];
   if (pos == 0) S.clear();
+  const int col = S.vi * 4;
+  float norm[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) norm[j] = S.grp == 0 ? d.norm[rank * vp + col + j] : 0.f;
   pdl_wait();
   pdl_trigger();
-  const int col = S.vi * 4;
   float gate[4], beta_in = 0.f, decay_in = 0.f;
   if (tid == THREADS - 1) {
     beta_in = in.ba[row * in.ldba + h];
@@ -144,11 +150,11 @@ delta_step_kernel(const DeltaStep d) {
     const float x = zf<TZ>(in.z, row * in.ldz + ch), a = silu_exact(past[i] + w_now[i] * x);
     sm[c] = a;
     if (c < 2 * dp) ss[c >= dp] += a * a;
-    if (c >= 2 * dp || h % rep == 0) ring[(long long)(pos % in.taps) * channels + ch] = x;      // one writer per channel
+    if (c >= 2 * dp || (rank == 0 && h % rep == 0)) ring[(long long)(pos % in.taps) * channels + ch] = x;      // one writer per channel
   }
   if (S.grp == 0) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) gate[j] = zf<TZ>(in.z, row * in.ldz + d.gate_off + (long long)h * vp + col + j);
+    for (int j = 0; j < 4; ++j) gate[j] = zf<TZ>(in.z, row * in.ldz + d.gate_off + v_at + col + j);
   }
   if (tid == THREADS - 1) {
     s_beta = sigmoidf(beta_in);
@@ -183,13 +189,21 @@ delta_step_kernel(const DeltaStep d) {
   }
   if (vp <= 128) so[0] = warp_sum(so[0]);          // they are lanes of one warp
   else block_sum<1>(so, red[0]);
+  if (ranks > 1) {                                 // the head's norm is over all columns
+    cg::cluster_group cluster = cg::this_cluster();
+    if (tid == 0) s_sum = so[0];
+    cluster.sync();
+    so[0] = 0.f;
+    for (int i = 0; i < ranks; ++i) so[0] += *cluster.map_shared_rank(&s_sum, i);
+  }
   if (S.grp == 0) {
     const float r = inv_rms(so[0], in.vdim, d.eps);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) ((T*)d.y)[row * d.ldy + (long long)h * vp + col + j] = from_f<T>(o[j] * r * d.norm[col + j] * silu_exact(gate[j]));
+    for (int j = 0; j < 4; ++j) ((T*)d.y)[row * d.ldy + v_at + col + j] = from_f<T>(o[j] * r * norm[j] * silu_exact(gate[j]));
   }
   S.update(g, sk, u, dp);
-  S.store(state, dp, vp);
+  S.store(state, dp, in.vp);
+  if (ranks > 1) cg::this_cluster().sync();        // the others' shared memory stays until it has been read
 }
 
 // ------------------------------------------------------------------------- fixed decay
@@ -201,7 +215,7 @@ __device__ void decay_head(const DecayStep& d, int h, int row, float* sm) {
   float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part = sv + vp, *part_kq = part + 2 * THREADS * 4;
   float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * vp;
   StateTile<NR> S;
-  S.load(state, dp, vp);
+  S.load(state, dp, vp, vp);
   if (d.pos.lens[row] == 0) S.clear();
   const float g = expf(d.log_decay[h]);
   pdl_wait();
@@ -487,15 +501,31 @@ int state_rows(int dp, int vp) {           // state rows per thread, 0: the stat
   return n <= 4 ? 4 : n <= 8 ? 8 : n <= 16 ? 16 : n <= MAX_NR ? MAX_NR : 0;
 }
 
+// CTAs of a head: enough to fill the SMs, whole groups of eight columns each
+int delta_ranks(int heads, int rows, int vp) {
+  for (int r = 4; r > 1; r /= 2)
+    if (vp % (8 * r) == 0 && heads * rows * r <= 592) return r;
+  return 1;
+}
 template <typename T, typename TZ>
 cudaError_t launch_delta(const DeltaStep& d, cudaStream_t s) {
-  const dim3 grid(d.in.heads, d.in.rows);
-  const size_t smem = step_floats(d.in.dp, d.in.vp) * sizeof(float);
-  switch (state_rows(d.in.dp, d.in.vp)) {
-    case 4: return launch_pdl(delta_step_kernel<T, TZ, 4>, grid, dim3(THREADS), smem, s, d);
-    case 8: return launch_pdl(delta_step_kernel<T, TZ, 8>, grid, dim3(THREADS), smem, s, d);
-    case 16: return launch_pdl(delta_step_kernel<T, TZ, 16>, grid, dim3(THREADS), smem, s, d);
-    case 32: return launch_pdl(delta_step_kernel<T, TZ, 32>, grid, dim3(THREADS), smem, s, d);
+  const int ranks = delta_ranks(d.in.heads, d.in.rows, d.in.vp), vp = d.in.vp / ranks;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(ranks, d.in.heads, d.in.rows);
+  cfg.blockDim = dim3(THREADS);
+  cfg.dynamicSmemBytes = step_floats(d.in.dp, vp) * sizeof(float);
+  cfg.stream = s;
+  cudaLaunchAttribute at[2];
+  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  at[0].val.programmaticStreamSerializationAllowed = 1;
+  at[1].id = cudaLaunchAttributeClusterDimension;
+  at[1].val.clusterDim.x = ranks; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
+  cfg.attrs = at; cfg.numAttrs = 2;
+  switch (state_rows(d.in.dp, vp)) {
+    case 4: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 4>, d);
+    case 8: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 8>, d);
+    case 16: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 16>, d);
+    case 32: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 32>, d);
   }
   return cudaErrorInvalidValue;
 }
@@ -550,7 +580,7 @@ bool window_step_supported(bool f32, int dp) { return !f32 && dp > 0 && dp <= 25
 
 cudaError_t delta_step(const DeltaStep& d, cudaStream_t s) {
   const DeltaInputs& in = d.in;
-  if (in.rows <= 0 || in.rows > 65535 || in.pos.per_seq != 1 || !in.pos.lens || in.heads <= 0 || in.kv_heads <= 0 || in.heads % in.kv_heads || in.taps <= 0 ||
+  if (in.rows <= 0 || in.rows > 65535 || in.heads > 65535 || in.pos.per_seq != 1 || !in.pos.lens || in.heads <= 0 || in.kv_heads <= 0 || in.heads % in.kv_heads || in.taps <= 0 ||
       !delta_step_supported(in.dp, in.vp) || in.dim > in.dp || in.vdim > in.vp || !in.z || !in.ba || !in.ring.ptr || !d.state.ptr || (d.state.seq_stride & 3) ||
       !d.y || (in.f32 && !in.z_f32))
     return cudaErrorInvalidValue;

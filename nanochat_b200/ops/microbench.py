@@ -374,9 +374,137 @@ def bench_serve(T=2048, C=1664, window=512, ctx=1024):
     return rows
 
 
+def bench_recurrent(T=2048, C=1664, window=512, ctx=1024):
+    """Every kernel of the model with recurrent layers (Safepel) at the d26 width beside the like kernel of GPT, as
+    `bench_serve` does: heads of 128 dimensions, as many as GPT's in every mixer, one key head per value head in the delta
+    rule and one for all in the window attention. A recurrence's roofline counts its inputs, outputs and state once and
+    6 (delta) or 4 (fixed decay) operations per state entry and token, whatever the kernels do internally."""
+    from nanochat_b200.ops import native as nat
+    from nanochat_b200.ops import serving as sv
+    K, N = sv._S, nat._C
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    if os.path.exists("MEASURED_PEAKS.json"):
+        with open("MEASURED_PEAKS.json") as f:
+            peaks.update({k: v for k, v in json.load(f).items() if k in peaks})
+    dev, bf16, f32 = "cuda", torch.bfloat16, torch.float32
+    r = lambda *s, dtype=bf16: torch.randn(*s, device=dev).to(dtype)
+    e = lambda *s, dtype=bf16: torch.empty(*s, device=dev, dtype=dtype)
+    H, D, ff, taps, P = C // 128, 128, -(-C * 8 // 3 // 64) * 64, 4, 64
+    rows, base = [], {}
+
+    def add(name, us, flops=0.0, nbytes=0.0, like=None, key=None):
+        roof = max(flops / peaks["bf16_tflops"] / 1e6, nbytes / peaks["hbm_gbs"] / 1e3)
+        row = {"kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "distance": round(us / roof, 2)}
+        if like is not None:
+            row["like"] = like
+            row["relative_distance"] = round(us / roof / base[like], 2)
+        if key is not None:
+            base[key] = us / roof
+        rows.append(row)
+
+    us = lambda fn: 1e3 * _time(fn, 10, 3)
+    # ------------------------------------------------------------------ prompts
+    x, w, y = r(T, C), r(4 * C, C), e(T, 4 * C)
+    add("gpt gemm (MLP up)", us(lambda: nat.gemm(x, w, y)), 2.0 * T * C * 4 * C, key="gemm")
+    w_in, z = r(4 * H * D, C), e(T, 4 * H * D)
+    add("gemm (delta input projection)", us(lambda: K.gemm(x, w_in, z)), 2.0 * T * C * 4 * H * D, like="gemm")
+    gu, act = r(2 * ff, C), e(T, ff)
+    add("gemm pair (gate with relu, up times gate)", us(lambda: (K.gemm(x, gu[:ff], act, epi=1), K.gemm(x, gu[ff:], act, epi=2, aux=act))),
+        2.0 * T * C * 2 * ff, like="gemm")
+    xr, lam = r(T, C), torch.ones(1, device=dev)
+    xm, xn = e(T, C), e(T, C)
+    add("gpt mix + norm", us(lambda: N.mixnorm_fwd(xr, x, lam, lam, 0, xm, xn, None)), nbytes=2.0 * T * C * 4, key="rows")
+    xf, wn, h = r(T, C, dtype=f32), r(C, dtype=f32), e(T, C)
+    add("norm + residual + norm", us(lambda: K.layer_norm_residual(None, x, 0, wn, xf, wn, 1e-6, C, h)), nbytes=T * C * (8 + 2 + 2.0), like="rows")
+    hp = -(-H // 8) * 8
+    wba, ba = r(2 * hp, C), e(T, 2 * hp, dtype=f32)
+    add("beta and decay inputs (product of few outputs)", _time_chain([lambda: K.gemv_plain(x, wba, ba)] * 8), nbytes=2.0 * (T + 2 * hp) * C, like="rows")
+    for win, tag in ((window, f"window {window}"),):
+        q, k, v, o = (r(1, T, H, 128) for _ in range(4))
+        lse = e(1, H, T, dtype=f32)
+        pairs = _attn_pairs(T, win)
+        add(f"gpt attention, {tag}", us(lambda: N.attn_fwd(q, k, v, o, lse, win, 0.088)), 4.0 * H * 128 * pairs, key="attn")
+        q3, kv, o3 = r(T, H, D), r(T, 2, 1, D), e(T, H, D)
+        for cap, what in ((0.0, "no cap"), (20.0, "soft cap")):
+            add(f"grouped attention, {tag}, {what}", us(lambda: K.attention_capped(q3, kv[:, 0], kv[:, 1], o3, win - 1, 0.088, cap, 0.7)), 4.0 * H * 128 * pairs, like="attn")
+    qkv, cs, rstd = r(1, T, 3 * H * 128), torch.full((1, T, 64), 0.7, device=dev, dtype=bf16), e(T, 2 * H, dtype=f32)
+    add("gpt rotary + QK norm", us(lambda: N.qkv_post_fwd(qkv, H, H, cs.view(T, 64), cs.view(T, 64), T, rstd, None, None, None, None)),
+        nbytes=2.0 * T * 2 * H * 128 * 2, key="post")
+    size, ch = [H, H, D, D, D, D, taps, hp], 3 * H * D
+    conv, one, lens = r(taps * ch, dtype=f32), torch.ones(hp, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+    ring, state = torch.zeros(1, taps, ch, device=dev), torch.zeros(1, H, D, D, device=dev)
+    norms, bg = e(T, 2 * H, dtype=f32), e(T, 2 * H, dtype=f32)
+    tiles = torch.empty(K.recurrence_tiles(1, T, H, H, D, D), dtype=torch.uint8, device=dev)
+    add("convolutions, unit norms, step sizes", us(lambda: K.delta_prepare(z, size, conv, ba, -one, one, ring, lens, T, tiles, norms, bg)), nbytes=2.0 * T * 2 * ch, like="post")
+    o2, y2, scratch = e(T, H * D), e(T, H * D), torch.empty(K.recurrence_scratch(1, T, H, True), dtype=torch.uint8, device=dev)
+    add("delta rule in chunks (two kernels)", us(lambda: K.recurrence(tiles, [H, H, D, D], norms, bg, None, state, lens, T, o2, scratch)),
+        6.0 * T * H * D * D, nbytes=2.0 * T * 4 * H * D + 8.0 * H * D * D, like="attn")
+    gate, wd = z[:, ch:], r(D, dtype=f32)
+    add("head norm + gate", us(lambda: K.delta_finish(o2, gate, wd, 1e-6, y2, z, size, conv, -one, one, ring, lens, T)), nbytes=2.0 * T * 3 * H * D, like="post")
+    add("silu of the fixed-decay inputs", us(lambda: K.decay_prepare(z[:, :ch], H, D, D, T, tiles)), nbytes=2.0 * T * 2 * ch, like="post")
+    ld, wr = torch.full((hp,), -0.01, device=dev), r(H * D, dtype=f32)
+    add("fixed decay in chunks (two kernels)", us(lambda: K.recurrence(tiles, [H, H, D, D], None, None, ld, state, lens, T, o2, scratch)),
+        4.0 * T * H * D * D, nbytes=2.0 * T * 4 * H * D + 8.0 * H * D * D, like="attn")
+    add("row norm + gate", us(lambda: K.norm_gate(o2, gate, wr, 1e-6, 1, H * D, True, 0.7, y2)), nbytes=2.0 * T * 3 * H * D, like="post")
+    pages = -(-(T + 1) // P)
+    pool, table = torch.zeros(pages, P, 2 * D, dtype=bf16, device=dev), torch.arange(pages, dtype=torch.int32, device=dev)[None].contiguous()
+    freq, dense = torch.stack([10000.0 ** (-torch.arange(D // 2, device=dev, dtype=f32) * 2 / D), torch.zeros(D // 2, device=dev)]), e(T, 2 * D)
+    wsize, wreal = [H, 1, D, 0, H * D, window], [0.088, 20.0, 0.7]
+    add("rotate queries, keys into the store", us(lambda: K.window_post(z, wsize, wreal, freq, pool, table, lens, T, dense)), nbytes=2.0 * T * (2 * H * D + D + 4 * D), like="post")
+    # ------------------------------------------------------------------- decode
+    L = 12                                          # chain length: weights of several layers, more than L2 holds
+    for B in (1, 8):
+        lens = torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
+        xb, wq, ob = r(B, C), [r(3 * C, C) for _ in range(L)], e(B, 3 * C)
+        add(f"gpt gemv (QKV), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, ob, None, 0, True, None) for a in wq]), nbytes=2.0 * 3 * C * C, key=f"gemv{B}")
+        wp, op, aux = [r(C, C) for _ in range(L)], e(B, C), r(B, C)
+        add(f"gpt gemv (attention out), {B} rows", _time_chain([lambda a=a: N.gemv_rows(xb, a, op, aux, 0, False, None) for a in wp]), nbytes=2.0 * C * C, key=f"gemvo{B}")
+        lam, xs = torch.ones(1, device=dev), [r(B, C) for _ in range(L)]
+        add(f"gpt mix + norm, {B} rows", _time_chain([lambda a=a: N.mixnorm_fwd(a, xb, lam, lam, 0, e1, e2, None) for e1, e2 in ((e(B, C), e(B, C)),) for a in xs]),
+            nbytes=2.0 * B * C * 4, key=f"row{B}")
+        n_in = 4 * H * D + 2 * hp
+        wa, zb = [r(n_in, C) for _ in range(L)], e(B, n_in, dtype=f32)
+        add(f"delta input projection, {B} rows", _time_chain([lambda a=a: K.gemv_plain(xb, a, zb) for a in wa]), nbytes=2.0 * n_in * C, like=f"gemv{B}")
+        zb.normal_()
+        pg = -(-ctx // P)
+        table = torch.arange(B * pg, dtype=torch.int32, device=dev).view(B, pg).contiguous()
+        k4 = [torch.randn(B * pg, P, H, 128, device=dev).to(bf16) for _ in range(L)]
+        scr, yg, qg = torch.zeros(N.decode_attn_scratch(B, H), device=dev), e(B, H * 128), r(B, H * 128)
+        add(f"gpt decode attention, {window} keys, {B} rows", _time_chain([lambda a=a: N.decode_attn(qg, a, a, lens, H, H, window - 1, 0.088, scr, yg, table) for a in k4]),
+            nbytes=2.0 * B * window * H * 256, flops=4.0 * B * window * H * 128, key=f"dattn{B}")
+        del k4
+        states, rings, yb = [torch.zeros(B, H, D, D, device=dev) for _ in range(L)], torch.zeros(B, taps, ch, device=dev), e(B, H * D)
+        add(f"delta step, {B} rows", _time_chain([lambda s=s: K.delta_step(zb, size, conv, zb[:, 4 * H * D:], -one, one, rings, s, lens, wd, 1e-6, ch, yb) for s in states]),
+            nbytes=8.0 * B * H * D * D, flops=6.0 * B * H * D * D, like=f"dattn{B}")
+        pools = [torch.randn(B * pg, P, 2 * D, device=dev).to(bf16) for _ in range(L)]
+        zp, wsz = r(B, H * D + D + 4 * H * D, dtype=f32), [H, 1, D, 0, H * D, window]
+        dsz = [H, D, D, D, H * D + D, 2 * H * D + D, 3 * H * D + D, 4 * H * D + D]
+        o4, done, y4 = e(B, H * D, dtype=f32), torch.zeros(B, dtype=torch.int32, device=dev), e(B, 2 * H * D)
+        add(f"window attention beside fixed decay, {B} rows",
+            _time_chain([lambda p=p, s=s: K.parallel_step(zp, wsz, wreal, freq, p, table, lens, y4[:, :H * D], dsz, [1e-6, 0.7], ld, s, wr, o4, done, y4[:, H * D:])
+                         for p, s in zip(pools, states)]),
+            nbytes=8.0 * B * H * D * D + 2.0 * B * window * 2 * D, flops=4.0 * B * H * D * (D + window), like=f"dattn{B}")
+        wo, out = [r(C, H * D) for _ in range(L)], e(B, C, dtype=f32)
+        add(f"output projection, {B} rows", _time_chain([lambda a=a: K.gemv_plain(yb, a, out) for a in wo]), nbytes=2.0 * C * H * D, like=f"gemvo{B}")
+        xf, hb = r(B, C, dtype=f32), e(B, C)
+        add(f"norm + residual + norm, {B} rows", _time_chain([lambda: K.layer_norm_residual(None, out, 0, wn, xf, wn, 1e-6, C, hb) for _ in range(L)]),
+            nbytes=B * C * (8 + 4 + 2.0), like=f"row{B}")
+        wg, ab = [r(2 * ff, C) for _ in range(L)], e(B, ff)
+        add(f"gate and up with activation, {B} rows", _time_chain([lambda a=a: K.gemv_relu_glu(xb, a, ab) for a in wg]), nbytes=2.0 * 2 * ff * C, like=f"gemv{B}")
+        wdn = [r(C, ff) for _ in range(L)]
+        add(f"down projection, {B} rows", _time_chain([lambda a=a: K.gemv_plain(ab, a, out) for a in wdn]), nbytes=2.0 * ff * C, like=f"gemv{B}")
+    sv.check_status()
+    nat.check_status()
+    return rows
+
+
+SERVE = {"Lupodra": bench_serve, "Safepel": bench_recurrent}
+
+
 def main():
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("op", choices=["gemm", "attn_fwd", "attn_bwd", "sweep", "serve"])
+    ap.add_argument("--model", default="Lupodra", choices=sorted(SERVE), help="serve: whose kernels")
     ap.add_argument("--m", type=int, default=32768)
     ap.add_argument("--n", type=int, default=4992)
     ap.add_argument("--k", type=int, default=1664)
@@ -396,7 +524,7 @@ def main():
     from nanochat_b200.ops import native as nat
     torch.manual_seed(0)
     if args.op == "serve":
-        for row in bench_serve():
+        for row in SERVE[args.model]():
             print(json.dumps(row))
         return
     res = {"gemm": bench_gemm, "attn_fwd": bench_attn_fwd, "attn_bwd": bench_attn_bwd, "sweep": bench_sweep}[args.op](args, nat)
