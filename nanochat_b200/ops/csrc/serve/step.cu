@@ -1,8 +1,7 @@
 // One token per row through the mixers of recurrent.cu and window.cu, from the projections to what the output product
 // reads.
 //
-//   delta_step      a cluster per (head, row), each CTA with a part of the value columns: convolution, unit norms, step size and
-//                   decay, state, norm and gate
+//   delta_step      a CTA per (head, row): convolution, unit norms, step size and decay, state, norm and gate
 //   parallel_step   window attention and fixed-decay heads side by side in one grid of clusters
 //       attention   a cluster per (16 query heads of a key head, row) splits the window's keys; the CTA that covers the
 //                   newest key takes it from the projection and appends it to the store; the partial results meet in
@@ -26,26 +25,26 @@ namespace cg = cooperative_groups;
 constexpr int THREADS = 256;
 constexpr int MAX_NR = 32;               // state rows a thread holds, four columns each
 
-__device__ __forceinline__ float silu_exact(float v) { return v * sigmoidf(v); }
+template <typename T> __device__ __forceinline__ float silu_of(float v) { return v * sigmoid_of<T>(v); }
 template <typename TZ> __device__ __forceinline__ float zf(const void* z, long long i) { return to_f(((const TZ*)z)[i]); }
 
-// A state of dp x vp floats (rows `pitch` apart in memory) over the block: thread (column group vi, row group grp) holds rows
-// grp, grp + groups, ... of four columns.
+// A state of dp x vp floats over the block: thread (column group vi, row group grp) holds NR neighbouring rows, from grp * NR
+// on, of four columns. dp is a multiple of 8, NR of 4: rows come and go in fours.
 template <int NR>
 struct StateTile {
   float s[NR][4];
-  int vi, grp, groups;
+  int vi, grp, d0, groups;
   bool on;
-  __device__ void load(const float* st, int dp, int vp, int pitch) {
+  __device__ void load(const float* st, int dp, int vp) {
     const int vt = vp / 4;
-    groups = THREADS / vt;
+    groups = (dp + NR - 1) / NR;
     vi = threadIdx.x % vt;
     grp = threadIdx.x / vt;
+    d0 = grp * NR;
     on = grp < groups;
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
-      const int d = grp + i * groups;
-      const float4 v = on && d < dp ? *reinterpret_cast<const float4*>(st + (long long)d * pitch + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 v = d0 + i < dp ? *reinterpret_cast<const float4*>(st + (long long)(d0 + i) * vp + vi * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
       s[i][0] = v.x; s[i][1] = v.y; s[i][2] = v.z; s[i][3] = v.w;
     }
   }
@@ -53,17 +52,24 @@ struct StateTile {
 #pragma unroll
     for (int i = 0; i < NR; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
   }
+  __device__ static void four(const float* x, int d, int dp, float (&f)[4]) {
+    const float4 v = d < dp ? *reinterpret_cast<const float4*>(x + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  }
   // this thread's part of S^T x, left in part[grp][columns]; with y, returns the row group's part of x . y
   __device__ float dot(const float* x, int dp, int vp, float* part, const float* y = nullptr) const {
     float p[4] = {0.f, 0.f, 0.f, 0.f}, xy = 0.f;
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int d = grp + i * groups;
-      const bool in = on && d < dp;
-      const float xd = in ? x[d] : 0.f;
-      if (y) xy += in ? xd * y[d] : 0.f;
+    for (int i = 0; i < NR; i += 4) {
+      float xv[4], yv[4];
+      four(x, d0 + i, dp, xv);
+      if (y) four(y, d0 + i, dp, yv);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) p[j] += s[i][j] * xd;
+      for (int r = 0; r < 4; ++r) {
+        if (y) xy += xv[r] * yv[r];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) p[j] += s[i + r][j] * xv[r];
+      }
     }
     if (on) *reinterpret_cast<float4*>(part + grp * vp + vi * 4) = make_float4(p[0], p[1], p[2], p[3]);
     return xy;
@@ -71,23 +77,24 @@ struct StateTile {
   // S <- g S + k u^T
   __device__ void update(float g, const float* k, const float (&u)[4], int dp) {
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int d = grp + i * groups;
-      const float kd = on && d < dp ? k[d] : 0.f;
+    for (int i = 0; i < NR; i += 4) {
+      float kv[4];
+      four(k, d0 + i, dp, kv);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) s[i][j] = g * s[i][j] + kd * u[j];
+      for (int r = 0; r < 4; ++r)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[i + r][j] = g * s[i + r][j] + kv[r] * u[j];
     }
   }
-  __device__ void store(float* st, int dp, int pitch) const {
+  __device__ void store(float* st, int dp, int vp) const {
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int d = grp + i * groups;
-      if (on && d < dp) *reinterpret_cast<float4*>(st + (long long)d * pitch + vi * 4) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
-    }
+    for (int i = 0; i < NR; ++i)
+      if (d0 + i < dp) *reinterpret_cast<float4*>(st + (long long)(d0 + i) * vp + vi * 4) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
   }
 };
 __device__ __forceinline__ void sum_parts(const float* part, int groups, int vp, int col, float (&t)[4]) {
   t[0] = t[1] = t[2] = t[3] = 0.f;
+#pragma unroll 8
   for (int g = 0; g < groups; ++g) {
     const float4 a = *reinterpret_cast<const float4*>(part + g * vp + col);
     t[0] += a.x; t[1] += a.y; t[2] += a.z; t[3] += a.w;
@@ -97,64 +104,67 @@ __device__ __forceinline__ void sum_parts(const float* part, int groups, int vp,
 __host__ __device__ constexpr int step_floats(int dp, int vp) { return 2 * dp + vp + 2 * THREADS * 4 + THREADS; }
 constexpr int MAX_CHANNELS = 6 * THREADS;      // q, k and v of one head
 
-// grid (ranks, heads, rows) in clusters of `ranks` CTAs: each has vp / ranks of the head's value columns
 template <typename T, typename TZ, int NR>
 __global__ void __launch_bounds__(THREADS)
 delta_step_kernel(const DeltaStep d) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[2][32];
-  __shared__ float s_beta, s_g, s_sum;
+  __shared__ float s_beta, s_g;
   constexpr int PER = MAX_CHANNELS / THREADS;
   const DeltaInputs& in = d.in;
-  const int rank = blockIdx.x, ranks = gridDim.x, h = blockIdx.y, row = blockIdx.z, rep = in.heads / in.kv_heads, kvh = h / rep;
+  const int h = blockIdx.x, row = blockIdx.y, rep = in.heads / in.kv_heads, kvh = h / rep;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int dp = in.dp, vp = in.vp / ranks, channels = 2 * in.kv_heads * dp + in.heads * in.vp, mine = 2 * dp + vp;
-  const int v_at = h * in.vp + rank * vp;          // this CTA's first value column among all heads'
+  const int dp = in.dp, vp = in.vp, channels = 2 * in.kv_heads * dp + in.heads * vp, mine = 2 * dp + vp;
   float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part_k = sv + vp, *part_q = part_k + THREADS * 4, *part_kq = part_q + THREADS * 4;
-  float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * in.vp + rank * vp;
+  float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * vp;
   float* ring = in.ring.ptr + row * in.ring.seq_stride;
-  const int pos = in.pos.lens[row];
+  const int pos = in.pos.lens[row], slot = pos % in.taps;
   StateTile<NR> S;
-  S.load(state, dp, vp, in.vp);
-  auto channel = [&](int c) { return c < dp ? kvh * dp + c : c < 2 * dp ? in.kv_heads * dp + kvh * dp + c - dp : 2 * in.kv_heads * dp + v_at + c - 2 * dp; };
+  S.load(state, dp, vp);
+  auto channel = [&](int c) { return c < dp ? kvh * dp + c : c < 2 * dp ? in.kv_heads * dp + kvh * dp + c - dp : 2 * in.kv_heads * dp + h * vp + c - 2 * dp; };
   float past[PER], w_now[PER];                     // the convolution without the current token, and its weight
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int c = tid + i * THREADS;
-    if (c >= mine) break;
-    const int ch = channel(c);
-    w_now[i] = in.conv[(long long)(in.taps - 1) * channels + ch];
-    past[i] = 0.f;
-    for (int t = 1; t < in.taps && t <= pos; ++t)
-      past[i] += in.conv[(long long)(in.taps - 1 - t) * channels + ch] * ring[(long long)((pos - t) % in.taps) * channels + ch];
+    past[i] = w_now[i] = 0.f;
+    if (c < mine) {
+      const int ch = channel(c);
+      w_now[i] = in.conv[(long long)(in.taps - 1) * channels + ch];
+      for (int t = 1; t < in.taps && t <= pos; ++t) {
+        const int at = slot - t < 0 ? slot - t + in.taps : slot - t;
+        past[i] += in.conv[(long long)(in.taps - 1 - t) * channels + ch] * ring[(long long)at * channels + ch];
+      }
+    }
   }
   const float bias = in.dt_bias[h], neg_a = in.neg_a[h];
   if (pos == 0) S.clear();
   const int col = S.vi * 4;
-  float norm[4];
+  float norm[4], gate[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) norm[j] = S.grp == 0 ? d.norm[rank * vp + col + j] : 0.f;
+  for (int j = 0; j < 4; ++j) norm[j] = S.grp == 0 ? d.norm[col + j] : 0.f;
   pdl_wait();
   pdl_trigger();
-  float gate[4], beta_in = 0.f, decay_in = 0.f;
+  float x[PER], beta_in = 0.f, decay_in = 0.f;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = tid + i * THREADS;
+    x[i] = c < mine ? zf<TZ>(in.z, row * in.ldz + channel(c)) : 0.f;
+  }
   if (tid == THREADS - 1) {
     beta_in = in.ba[row * in.ldba + h];
     decay_in = in.ba[row * in.ldba + in.a_off + h] + bias;
   }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) gate[j] = S.grp == 0 ? zf<TZ>(in.z, row * in.ldz + d.gate_off + (long long)h * vp + col + j) : 0.f;
   float ss[2] = {0.f, 0.f};
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int c = tid + i * THREADS;
-    if (c >= mine) break;
-    const int ch = channel(c);
-    const float x = zf<TZ>(in.z, row * in.ldz + ch), a = silu_exact(past[i] + w_now[i] * x);
+    if (c >= mine) continue;
+    const float a = silu_of<T>(past[i] + w_now[i] * x[i]);
     sm[c] = a;
     if (c < 2 * dp) ss[c >= dp] += a * a;
-    if (c >= 2 * dp || (rank == 0 && h % rep == 0)) ring[(long long)(pos % in.taps) * channels + ch] = x;      // one writer per channel
-  }
-  if (S.grp == 0) {
-#pragma unroll
-    for (int j = 0; j < 4; ++j) gate[j] = zf<TZ>(in.z, row * in.ldz + d.gate_off + v_at + col + j);
+    if (c >= 2 * dp || h % rep == 0) ring[(long long)slot * channels + channel(c)] = x[i];      // one writer per channel
   }
   if (tid == THREADS - 1) {
     s_beta = sigmoidf(beta_in);
@@ -169,9 +179,10 @@ delta_step_kernel(const DeltaStep d) {
   S.dot(sk, dp, vp, part_k);
   const float kq_part = S.dot(sq, dp, vp, part_q, sk);
   if (S.on && S.vi == 0) part_kq[S.grp] = kq_part;
+  ss[0] = ss[1] = 0.f;
 #pragma unroll
-  for (int i = 0; i < 2; ++i) ss[i] = warp_sum(lane < THREADS / 32 ? red[i][lane] : 0.f);
-  const float rq = 1.f / sqrtf(ss[0] + 1e-6f) / sqrtf((float)in.dim), rk = 1.f / sqrtf(ss[1] + 1e-6f), g = s_g;
+  for (int w = 0; w < THREADS / 32; ++w) { ss[0] += red[0][w]; ss[1] += red[1][w]; }
+  const float rq = 1.f / sqrtf((ss[0] + 1e-6f) * in.dim), rk = 1.f / sqrtf(ss[1] + 1e-6f), g = s_g;
   __syncthreads();
   float u[4] = {0.f, 0.f, 0.f, 0.f}, o[4] = {0.f, 0.f, 0.f, 0.f}, so[1] = {0.f};
   if (S.on) {
@@ -183,27 +194,20 @@ delta_step_kernel(const DeltaStep d) {
   if (S.grp == 0) {                                // the first threads read out
     float t[4], kq = 0.f;
     sum_parts(part_q, S.groups, vp, col, t);
+#pragma unroll 8
     for (int i = 0; i < S.groups; ++i) kq += part_kq[i];
 #pragma unroll
     for (int j = 0; j < 4; ++j) { o[j] = rq * (g * t[j] + kq * u[j]); so[0] += o[j] * o[j]; }
   }
   if (vp <= 128) so[0] = warp_sum(so[0]);          // they are lanes of one warp
   else block_sum<1>(so, red[0]);
-  if (ranks > 1) {                                 // the head's norm is over all columns
-    cg::cluster_group cluster = cg::this_cluster();
-    if (tid == 0) s_sum = so[0];
-    cluster.sync();
-    so[0] = 0.f;
-    for (int i = 0; i < ranks; ++i) so[0] += *cluster.map_shared_rank(&s_sum, i);
-  }
   if (S.grp == 0) {
     const float r = inv_rms(so[0], in.vdim, d.eps);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) ((T*)d.y)[row * d.ldy + v_at + col + j] = from_f<T>(o[j] * r * norm[j] * silu_exact(gate[j]));
+    for (int j = 0; j < 4; ++j) ((T*)d.y)[row * d.ldy + (long long)h * vp + col + j] = from_f<T>(o[j] * r * norm[j] * silu_of<T>(gate[j]));
   }
   S.update(g, sk, u, dp);
-  S.store(state, dp, in.vp);
-  if (ranks > 1) cg::this_cluster().sync();        // the others' shared memory stays until it has been read
+  S.store(state, dp, vp);
 }
 
 // ------------------------------------------------------------------------- fixed decay
@@ -215,14 +219,14 @@ __device__ void decay_head(const DecayStep& d, int h, int row, float* sm) {
   float *sq = sm, *sk = sm + dp, *sv = sm + 2 * dp, *part = sv + vp, *part_kq = part + 2 * THREADS * 4;
   float* state = d.state.ptr + row * d.state.seq_stride + (long long)h * dp * vp;
   StateTile<NR> S;
-  S.load(state, dp, vp, vp);
+  S.load(state, dp, vp);
   if (d.pos.lens[row] == 0) S.clear();
   const float g = expf(d.log_decay[h]);
   pdl_wait();
   pdl_trigger();
   for (int c = tid; c < 2 * dp + vp; c += THREADS) {
     const int at = c < dp ? d.q_off + h * dp + c : c < 2 * dp ? d.k_off + h * dp + c - dp : d.v_off + h * vp + c - 2 * dp;
-    sm[c] = silu_exact(zf<TZ>(d.z, row * d.ldz + at));
+    sm[c] = silu_of<T>(zf<TZ>(d.z, row * d.ldz + at));
   }
   __syncthreads();
   const float kq_part = S.dot(sq, dp, vp, part, sk);
@@ -233,6 +237,7 @@ __device__ void decay_head(const DecayStep& d, int h, int row, float* sm) {
   if (S.grp == 0) {
     float t[4], kq = 0.f;
     sum_parts(part, S.groups, vp, col, t);
+#pragma unroll 8
     for (int i = 0; i < S.groups; ++i) kq += part_kq[i];
     *reinterpret_cast<float4*>(o + h * vp + col) =
         make_float4(g * t[0] + kq * sv[col], g * t[1] + kq * sv[col + 1], g * t[2] + kq * sv[col + 2], g * t[3] + kq * sv[col + 3]);
@@ -257,7 +262,7 @@ __device__ void decay_head(const DecayStep& d, int h, int row, float* sm) {
   block_sum<1>(ss, red);
   const float r = inv_rms(ss[0], d.heads * d.vdim, d.eps) * d.out_scale;
   for (int c = tid; c < width; c += THREADS)
-    ((T*)d.y)[row * d.ldy + c] = from_f<T>(__ldcg(o + c) * r * d.norm[c] * sigmoidf(zf<TZ>(d.z, row * d.ldz + d.gate_off + c)));
+    ((T*)d.y)[row * d.ldy + c] = from_f<T>(__ldcg(o + c) * r * d.norm[c] * sigmoid_of<T>(zf<TZ>(d.z, row * d.ldz + d.gate_off + c)));
 }
 
 // --------------------------------------------------------------------------- attention
@@ -501,31 +506,15 @@ int state_rows(int dp, int vp) {           // state rows per thread, 0: the stat
   return n <= 4 ? 4 : n <= 8 ? 8 : n <= 16 ? 16 : n <= MAX_NR ? MAX_NR : 0;
 }
 
-// CTAs of a head: enough to fill the SMs, whole groups of eight columns each
-int delta_ranks(int heads, int rows, int vp) {
-  for (int r = 4; r > 1; r /= 2)
-    if (vp % (8 * r) == 0 && heads * rows * r <= 592) return r;
-  return 1;
-}
 template <typename T, typename TZ>
 cudaError_t launch_delta(const DeltaStep& d, cudaStream_t s) {
-  const int ranks = delta_ranks(d.in.heads, d.in.rows, d.in.vp), vp = d.in.vp / ranks;
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(ranks, d.in.heads, d.in.rows);
-  cfg.blockDim = dim3(THREADS);
-  cfg.dynamicSmemBytes = step_floats(d.in.dp, vp) * sizeof(float);
-  cfg.stream = s;
-  cudaLaunchAttribute at[2];
-  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  at[0].val.programmaticStreamSerializationAllowed = 1;
-  at[1].id = cudaLaunchAttributeClusterDimension;
-  at[1].val.clusterDim.x = ranks; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
-  cfg.attrs = at; cfg.numAttrs = 2;
-  switch (state_rows(d.in.dp, vp)) {
-    case 4: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 4>, d);
-    case 8: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 8>, d);
-    case 16: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 16>, d);
-    case 32: return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, TZ, 32>, d);
+  const dim3 grid(d.in.heads, d.in.rows);
+  const size_t smem = step_floats(d.in.dp, d.in.vp) * sizeof(float);
+  switch (state_rows(d.in.dp, d.in.vp)) {
+    case 4: return launch_pdl(delta_step_kernel<T, TZ, 4>, grid, dim3(THREADS), smem, s, d);
+    case 8: return launch_pdl(delta_step_kernel<T, TZ, 8>, grid, dim3(THREADS), smem, s, d);
+    case 16: return launch_pdl(delta_step_kernel<T, TZ, 16>, grid, dim3(THREADS), smem, s, d);
+    case 32: return launch_pdl(delta_step_kernel<T, TZ, 32>, grid, dim3(THREADS), smem, s, d);
   }
   return cudaErrorInvalidValue;
 }
